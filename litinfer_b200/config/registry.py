@@ -19,6 +19,7 @@ from .gorulorn import GorulornConfig
 from .pifazen import PifazenConfig
 from .qwen2 import ConfigError, Qwen2Config
 from .spec import ModelSpec
+from .zigolix import ZigolixConfig
 
 _ARCHITECTURES: Dict[str, Type] = {}
 
@@ -87,3 +88,4 @@ register_architecture(FilasunConfig.ARCHITECTURE, FilasunConfig)
 register_architecture(GorulornConfig.ARCHITECTURE, GorulornConfig)
 register_architecture(DemavikConfig.ARCHITECTURE, DemavikConfig)
 register_architecture(PifazenConfig.ARCHITECTURE, PifazenConfig)
+register_architecture(ZigolixConfig.ARCHITECTURE, ZigolixConfig)

@@ -99,11 +99,14 @@ class ScheduleEntry:
     """Run block ``block``.  ``cache_from`` None: this entry owns a cache (or
     state); otherwise it reads what schedule entry ``cache_from`` wrote in
     this step and writes nothing.  ``add``: (name of a table in ``ModelSpec.stream_tables``, row): that row is added to the
-    residual stream right before the block runs (a vector per pass of a span of layers that runs several times)."""
+    residual stream right before the block runs (a vector per pass of a span of layers that runs several times).  ``join``: the name
+    of a map in ``ModelSpec.stream_maps``; before anything of ``add``, the stream x becomes ``M [x; x0]`` with x0 the embedding
+    output (a span that reads the embedding anew at the start of every pass)."""
 
     block: int
     cache_from: Optional[int] = None
     add: Optional[Tuple[str, int]] = None
+    join: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -133,6 +136,9 @@ class ModelSpec:
     streams: Optional[int] = None
     # tables of vectors that schedule entries add to the residual stream (``ScheduleEntry.add``): tensor name -> rows
     stream_tables: Mapping[str, int] = field(default_factory=dict)
+    # maps [hidden, 2 hidden] that schedule entries put the residual stream beside the embedding output through
+    # (``ScheduleEntry.join``; the embedding output is the stream as it enters the first block): tensor names
+    stream_maps: Tuple[str, ...] = ()
     # parts that add something to the residual stream right after the embedding and may keep a state per request for it
     # (an embedding of token pairs): (spec, tensor-name prefix) each, kinds of the registry of stream inputs
     stream_inputs: Tuple[Tuple[PartSpec, str], ...] = ()
@@ -157,6 +163,8 @@ def validate_schedule(spec: ModelSpec) -> None:
             name, row = e.add
             if name not in spec.stream_tables or not 0 <= int(row) < int(spec.stream_tables[name]):
                 raise ValueError(f"schedule entry {i} adds row {row} of '{name}', which the model's stream tables do not have")
+        if e.join is not None and (e.join not in spec.stream_maps or spec.streams is not None):
+            raise ValueError(f"schedule entry {i} puts the stream through '{e.join}', which is not among the model's stream maps (of a single stream)")
         if e.cache_from is not None:
             if not 0 <= e.cache_from < i:
                 raise ValueError(f"schedule entry {i} reads the cache of entry {e.cache_from}, which does not run before it")

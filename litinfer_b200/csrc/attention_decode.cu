@@ -87,12 +87,8 @@ decode_attention_whole_kernel(const bf16* __restrict__ qkv, const bf16* __restri
     const int G = nh / nkv;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
-    const bf16* qrow = qkv + (size_t)tok * (nh + 2 * nkv) * DH + (size_t)kvh * G * DH;
     unsigned qa[DH / 16][4];
-    const bf16* q_lo = g < G ? qrow + (size_t)g * DH : nullptr;
-    const bf16* q_hi = g + 8 < G ? qrow + (size_t)(g + 8) * DH : nullptr;
-    if constexpr (KB == 16) load_q<DH>(qa, q_lo, q_hi, t);
-    else load_q32<DH>(qa, q_lo, q_hi, t);
+    load_query_heads<DH, KB, kMod>(qa, qkv, tok, kvh, nh, nkv, g, t, mod);
     RowState<DH> st;
     st.init();
     const int lo2[2] = {lo, lo}, hi2[2] = {p, p};
@@ -279,13 +275,14 @@ bool li_attention_decode_accepts(int nh, int nkv, int dh, int page_size) {
 int li_attention_decode(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks,
                         const int* ctx_lens, const int* old_lens, const int* q_start, int S, int nh, int nkv, int dh, int page_size, int num_pages,
                         float scale, int window, int max_ctx_len, int expected, float softcap, const float* slopes, const void* gate,
-                        int keep_first, const float* sinks, cudaStream_t stream) {
+                        int keep_first, const float* sinks, int maps, cudaStream_t stream) {
     ScoreMod mod;
     mod.softcap = softcap;
     mod.slopes = slopes;
     mod.gate = (const bf16*)gate;
     mod.keep_first = window > 0 ? keep_first : 0;
     mod.sinks = sinks;
+    mod.maps = maps;
 #define LI_CASE(D)                                                                                                             \
     case D:                                                                                                                    \
         return mod.any() ? launch<D, true>(qkv, out, kcache, vcache, block_table, max_blocks, ctx_lens, old_lens, q_start, S, nh, nkv, page_size, \

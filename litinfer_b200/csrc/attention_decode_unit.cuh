@@ -22,6 +22,28 @@ __host__ __device__ inline void split_range(int ctx, int window, int kSplit, int
     *last = (ctx - 1) / kSplit;
 }
 
+// Query fragments of the heads kvh * G .. kvh * G + G - 1 of row `tok`: rows g and g + 8 of the tile (heads past the last:
+// zeros).  kMod: a query row may stand for several heads (ScoreMod::maps), each with a part of it.
+template <int DH, int KB, bool kMod>
+__device__ __forceinline__ void load_query_heads(unsigned (&qa)[DH / 16][4], const bf16* __restrict__ qkv, int tok, int kvh, int nh, int nkv, int g, int t,
+                                                 const attn::ScoreMod& mod) {
+    const int G = nh / nkv;
+    const int maps = kMod ? mod.maps : 1;
+    const bf16* row = qkv + (size_t)tok * (nh / maps + 2 * nkv) * DH;
+    const int h_lo = kvh * G + g, h_hi = h_lo + 8;
+    const bf16* q_lo = g < G ? row + (size_t)(h_lo / maps) * DH : nullptr;
+    const bf16* q_hi = g + 8 < G ? row + (size_t)(h_hi / maps) * DH : nullptr;
+    if constexpr (KB == 16) load_q<DH>(qa, q_lo, q_hi, t);
+    else load_q32<DH>(qa, q_lo, q_hi, t);
+    if constexpr (kMod) {
+        if (maps > 1) {
+            const int part = DH / maps;
+            const int from[2] = {(h_lo % maps) * part, (h_hi % maps) * part}, to[2] = {from[0] + part, from[1] + part};
+            keep_part_of_q<DH, KB == 32>(qa, from, to, t);
+        }
+    }
+}
+
 // One block of KB keys (16: 8-byte loads; 32: 16-byte loads, half as many requests per byte) from the pages of a
 // sequence into the running softmax of a warp.  All loads of the block are issued before the first use.
 template <int DH, int KB, bool kMod = false>
@@ -114,12 +136,8 @@ __device__ __forceinline__ void decode_attention_unit(int split, int kvh, int s,
     }
     wait_for_queries();
     // query fragments: rows g and g + 8 are heads kvh * G + g (+ 8)
-    const bf16* qrow = qkv + (size_t)tok * (nh + 2 * nkv) * DH + (size_t)kvh * G * DH;
     unsigned qa[DH / 16][4];
-    const bf16* q_lo = g < G ? qrow + (size_t)g * DH : nullptr;
-    const bf16* q_hi = g + 8 < G ? qrow + (size_t)(g + 8) * DH : nullptr;
-    if constexpr (KB == 16) load_q<DH>(qa, q_lo, q_hi, t);
-    else load_q32<DH>(qa, q_lo, q_hi, t);
+    load_query_heads<DH, KB, kMod>(qa, qkv, tok, kvh, nh, nkv, g, t, mod);
     RowState<DH> st;
     st.init();
     const int lo2[2] = {lo, lo}, hi2[2] = {k_end - 1, k_end - 1};

@@ -24,6 +24,7 @@
 // Optional changes of what is seen and of the softmax's denominator:
 //   keep_first > 0 (with a window): keys 0 .. keep_first - 1 stay visible behind the window, at their own positions;
 //   sinks [nh]:   exp(sinks[h]) joins the denominator of head h once; it has no key and no value and is not scaled.
+// maps > 1: a query row of head_dim elements stands for `maps` heads (attention_mma.cuh: ScoreMod); qkv then holds nh / maps of them.
 #include "common.cuh"
 
 namespace {
@@ -37,7 +38,7 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
                          const int* __restrict__ block_table, int max_blocks, const int* __restrict__ seq_of_token,
                          const int* __restrict__ positions, int total, int nh, int nkv, int dh, int page_size, int num_pages,
                          float scale, int window, float softcap, const float* __restrict__ slopes, const T* __restrict__ gate,
-                         int keep_first, const float* __restrict__ sinks) {
+                         int keep_first, const float* __restrict__ sinks, int maps) {
     const int warp = blockIdx.x * kWarpsPerBlock + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     if (warp >= total) return;
@@ -46,15 +47,16 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
     const int s = seq_of_token[t];
     const int p = positions[t];
     const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
-    const int row = (nh + 2 * nkv) * dh;
-    const T* q = qkv + (size_t)t * row + h * dh;
+    const int row = (nh / maps + 2 * nkv) * dh;
+    const T* q = qkv + (size_t)t * row + (h / maps) * dh;
     const int per = (dh + 31) >> 5;
+    const int part = dh / maps, part_lo = (h % maps) * part, part_hi = part_lo + part;
 
     float qr[kMaxPerLane], acc[kMaxPerLane];
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
         const int d = lane + 32 * i;
-        qr[i] = (i < per && d < dh) ? to_float(q[d]) : 0.0f;
+        qr[i] = (i < per && d >= part_lo && d < part_hi) ? to_float(q[d]) : 0.0f;
         acc[i] = 0.0f;
     }
     float m = -INFINITY, l = 0.0f;
@@ -74,7 +76,7 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
 #pragma unroll
         for (int i = 0; i < kMaxPerLane; ++i) {
             const int d = lane + 32 * i;
-            if (i < per && d < dh) dot = fmaf(qr[i], to_float(kcache[base + d]), dot);
+            if (i < per && d >= part_lo && d < part_hi) dot = fmaf(qr[i], to_float(kcache[base + d]), dot);
         }
         float sc = warp_sum(dot) * scale;
         if (softcap > 0.0f) sc = softcap * tanhf(sc / softcap);
@@ -113,7 +115,7 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
 int li_attention_generic(const void* qkv, void* out, const void* kcache, const void* vcache, int dtype, const int* block_table,
                          int max_blocks, const int* seq_of_token, const int* positions, int T, int nh, int nkv, int dh,
                          int page_size, int num_pages, float scale, int window, float softcap, const float* slopes, const void* gate,
-                         int keep_first, const float* sinks, cudaStream_t stream) {
+                         int keep_first, const float* sinks, int maps, cudaStream_t stream) {
     LI_REQUIRE(dh <= 32 * kMaxPerLane, "attention: head_dim %d is larger than %d", dh, 32 * kMaxPerLane);
     const long long total = (long long)T * nh;
     LI_REQUIRE(total < (1LL << 31), "attention: too many (token, head) pairs");
@@ -121,11 +123,11 @@ int li_attention_generic(const void* qkv, void* out, const void* kcache, const v
     if (dtype == LI_F32)
         attention_generic_kernel<float><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
             (const float*)qkv, (float*)out, (const float*)kcache, (const float*)vcache, block_table, max_blocks, seq_of_token, positions,
-            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, softcap, slopes, (const float*)gate, keep_first, sinks);
+            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, softcap, slopes, (const float*)gate, keep_first, sinks, maps);
     else if (dtype == LI_BF16)
         attention_generic_kernel<bf16><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
             (const bf16*)qkv, (bf16*)out, (const bf16*)kcache, (const bf16*)vcache, block_table, max_blocks, seq_of_token, positions,
-            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, softcap, slopes, (const bf16*)gate, keep_first, sinks);
+            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, softcap, slopes, (const bf16*)gate, keep_first, sinks, maps);
     else
         return li_fail("attention: unknown dtype %d", dtype);
     return li_check_launch("attention (generic)");

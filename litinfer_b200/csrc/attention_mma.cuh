@@ -24,22 +24,19 @@ namespace attn {
 // Optional changes of the scores and of the output (see attention_generic.cu): a cap softcap * tanh(s / softcap) after
 // the scale, slopes[h] * (p - key) taken off, and the head's output times sigmoid(gate[token, h]).  And of what is seen
 // and summed: with a window the keys below keep_first stay visible behind it; exp(sinks[h]) joins the denominator of head
-// h once.  All off when zero.
+// h once.  And of what a query head is: with maps > 1 every query row of head_dim elements is cut into `maps` parts of equal
+// length and stands for that many heads (head h is part h % maps of row h / maps); a head's scores take its part of the key
+// against its part of the query only, its values are the whole value row (several maps of attention over the same values,
+// differential attention).  All off when zero (maps: when one).
 struct ScoreMod {
     float softcap = 0.0f;
     const float* slopes = nullptr;
     const bf16* gate = nullptr;
     int keep_first = 0;
     const float* sinks = nullptr;
-    bool any() const { return softcap > 0.0f || slopes != nullptr || gate != nullptr || keep_first > 0 || sinks != nullptr; }
+    int maps = 1;
+    bool any() const { return softcap > 0.0f || slopes != nullptr || gate != nullptr || keep_first > 0 || sinks != nullptr || maps > 1; }
 };
-
-// tanh from the fast exponential and reciprocal (relative error about 1e-6): 1 - 2 / (1 + e^(2x)).
-__device__ __forceinline__ float tanh_fast(float x) {
-    float e;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
-    return 1.0f - __fdividef(2.0f, 1.0f + e);
-}
 
 // The score of a key at `dist` positions behind its query, from the scaled dot product.
 __device__ __forceinline__ float changed_score(float s, float softcap, float slope, int dist) {
@@ -112,6 +109,21 @@ __device__ __forceinline__ void load_q(unsigned (&qa)[DH / 16][4], const bf16* r
         const uint2 r0 = row_lo ? ld8(row_lo + st * 16 + t * 4) : make_uint2(0, 0);
         const uint2 r1 = row_hi ? ld8(row_hi + st * 16 + t * 4) : make_uint2(0, 0);
         qa[st][0] = r0.x; qa[st][1] = r1.x; qa[st][2] = r0.y; qa[st][3] = r1.y;
+    }
+}
+
+// With several maps a row stands for, the fragments outside a row's part are zeros: from, to say which elements of row g
+// (index 0) and of row g + 8 (index 1) are the row's own (multiples of 8, as load_q and load_q32 take their pieces).
+template <int DH, bool kWide>
+__device__ __forceinline__ void keep_part_of_q(unsigned (&qa)[DH / 16][4], const int (&from)[2], const int (&to)[2], int t) {
+    constexpr int F = DH / 32;
+#pragma unroll
+    for (int st = 0; st < DH / 16; ++st) {
+        const bool paired = kWide && st < 2 * F;                 // 8 elements a thread for two k-steps, else 4 for one
+        const int col = paired ? (st >> 1) * 32 + t * 8 : st * 16 + t * 4;
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+            if (col < from[r] || col >= to[r]) qa[st][r] = qa[st][2 + r] = 0u;
     }
 }
 

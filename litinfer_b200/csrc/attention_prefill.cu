@@ -83,7 +83,9 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
     const int g = lane >> 2, t = lane & 3;
     const int ctx = ctx_lens[s];
     const int kvh = h / (nh / nkv);
-    const int row_elems = (nh + 2 * nkv) * DH;
+    const int maps = kMod ? mod.maps : 1;                  // heads that a query row stands for; this head's part of it
+    const int row_elems = (nh / maps + 2 * nkv) * DH;
+    [[maybe_unused]] const int part_lo = kMod ? (h % maps) * (DH / maps) : 0, part_hi = kMod ? part_lo + DH / maps : DH;
     const int i0 = cta_i0 + warp * 16;                     // first token of this warp within the portion
     const bool warp_active = i0 < n;
     const int r_lo = i0 + g, r_hi = i0 + g + 8;
@@ -91,8 +93,8 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
     // query fragments, permuted like the key fragments: group f gives k-steps 2f (elements 0-3 of the thread's 8) and 2f+1
     unsigned qa[KS][4];
     {
-        const bf16* q0 = (warp_active && r_lo < n) ? qkv + (size_t)(tok0 + r_lo) * row_elems + (size_t)h * DH : nullptr;
-        const bf16* q1 = (warp_active && r_hi < n) ? qkv + (size_t)(tok0 + r_hi) * row_elems + (size_t)h * DH : nullptr;
+        const bf16* q0 = (warp_active && r_lo < n) ? qkv + (size_t)(tok0 + r_lo) * row_elems + (size_t)(h / maps) * DH : nullptr;
+        const bf16* q1 = (warp_active && r_hi < n) ? qkv + (size_t)(tok0 + r_hi) * row_elems + (size_t)(h / maps) * DH : nullptr;
 #pragma unroll
         for (int f = 0; f < F; ++f) {
             const uint4 a = q0 ? *reinterpret_cast<const uint4*>(q0 + f * 32 + t * 8) : make_uint4(0, 0, 0, 0);
@@ -104,6 +106,12 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
             const uint2 a = q0 ? ld8(q0 + F * 32 + t * 4) : make_uint2(0, 0);
             const uint2 b = q1 ? ld8(q1 + F * 32 + t * 4) : make_uint2(0, 0);
             qa[KS - 1][0] = a.x; qa[KS - 1][1] = b.x; qa[KS - 1][2] = a.y; qa[KS - 1][3] = b.y;
+        }
+        if constexpr (kMod) {
+            if (maps > 1) {
+                const int from[2] = {part_lo, part_lo}, to[2] = {part_hi, part_hi};
+                keep_part_of_q<DH, true>(qa, from, to, t);
+            }
         }
     }
     RowState<DH> st;
@@ -192,6 +200,8 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
                 const int key = k_row_key(r);
 #pragma unroll
                 for (int f = 0; f < F; ++f) {
+                    if constexpr (kMod)
+                        if (f * 32 + 32 <= part_lo || f * 32 >= part_hi) continue;          // zeros of the query: another map's part
                     const uint4 b = *reinterpret_cast<const uint4*>(krow + swz(f * 4 + t, key, KCH) * 16);
                     mma_bf16(sc[tau], qa[2 * f][0], qa[2 * f][1], qa[2 * f][2], qa[2 * f][3], b.x, b.y);
                     mma_bf16(sc[tau], qa[2 * f + 1][0], qa[2 * f + 1][1], qa[2 * f + 1][2], qa[2 * f + 1][3], b.z, b.w);
@@ -337,7 +347,7 @@ bool li_attention_prefill_accepts(int nh, int nkv, int dh, int page_size) {
 int li_attention_prefill(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks,
                          const int* q_start, const int* ctx_lens, int T, int S, int nh, int nkv, int dh, int page_size,
                          int num_pages, float scale, int window, int max_q_len, int skip_single, float softcap, const float* slopes,
-                         const void* gate, int keep_first, const float* sinks, cudaStream_t stream) {
+                         const void* gate, int keep_first, const float* sinks, int maps, cudaStream_t stream) {
     (void)T;
     attn::ScoreMod mod;
     mod.softcap = softcap;
@@ -345,6 +355,7 @@ int li_attention_prefill(const void* qkv, void* out, const void* kcache, const v
     mod.gate = (const bf16*)gate;
     mod.keep_first = window > 0 ? keep_first : 0;
     mod.sinks = sinks;
+    mod.maps = maps;
     LI_REQUIRE(scale > 0.0f, "attention (prefill): the scale must be positive, got %g", (double)scale);
 #define LI_CASE(D)                                                                                                                  \
     case D:                                                                                                                         \

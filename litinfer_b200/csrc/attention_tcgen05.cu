@@ -66,14 +66,30 @@ __host__ __device__ constexpr size_t smem_pad() {
     return sizeof(Smem<DH>) + 1024 <= 232448 ? 1024 : 232448 - sizeof(Smem<DH>);
 }
 
-template <int DH>
+// tanh(x) for |x| <= 1: x times a polynomial in x^2 fitted to tanh(x) / x at Chebyshev points (absolute error below 6e-7)
+constexpr float kTanhSmall = 1.0f;
+__device__ __forceinline__ float tanh_small(float x) {
+    const float y = x * x;
+    float p = -0.0030804092530161142f;
+    p = fmaf(p, y, 0.01677674594125271f);
+    p = fmaf(p, y, -0.05163545906543732f);
+    p = fmaf(p, y, 0.13282513618469238f);
+    p = fmaf(p, y, -0.33329179883003235f);
+    p = fmaf(p, y, 0.999999463558197f);
+    return x * p;
+}
+
+// kCap: scores are capped, cap * tanh(s / cap), before the mask and the softmax (`softcap` > 0).  maps > 1: a query row of DH elements
+// stands for that many heads, each with a part of it (attention_mma.cuh: ScoreMod): a head's product S takes the k-steps of
+// its own part only, and with head_dim 128 and two maps only that part's panel of the keys is brought in.
+template <int DH, bool kCap>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const int* __restrict__ block_table,
                             int max_blocks, const int* __restrict__ q_start, const int* __restrict__ ctx_lens, int nh, int nkv,
                             int page_size, int num_pages, float scale, int window, int skip_single, int* __restrict__ error_flag, int trace,
                             const int* __restrict__ units, float* __restrict__ partial, unsigned* __restrict__ counters,
-                            const float* __restrict__ sinks, int keep_first) {
+                            const float* __restrict__ sinks, int keep_first, float softcap, int maps) {
     extern __shared__ unsigned char smem_raw[];
     Smem<DH>& sm = *reinterpret_cast<Smem<DH>*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     // the tiles want 1024-byte alignment; with head_dim 128 there is not a whole kilobyte to spare for it
@@ -82,6 +98,9 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
         return;
     }
     constexpr int kPanels = DH / 64;
+    // this head's part of the query row: k-steps of the product S, and the panels of the keys they read
+    const int k_lo = ((int)blockIdx.x % maps) * (DH / 16 / maps), k_hi = k_lo + DH / 16 / maps;
+    const int panel_lo = k_lo >> 2, panel_hi = (k_hi + 3) >> 2;
     constexpr unsigned kTmemCols = 512;              // S of two tiles: 128 columns each; O: up to 128; Q: up to 64
     // What this CTA works on.  With a work list (`units`, made on the host with the step's other metadata: two counts, two
     // unused words, then per entry sequence, tile of tokens, part | parts << 8, unused; heaviest first, the parts of a tile
@@ -193,7 +212,7 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
             if (lane == 0) {
                 stamp(keys ? 0 : 4, 0, j);
                 ok = mbar_wait(keys ? &sm.k_empty[b] : &sm.v_empty[b], free_parity);
-                if (ok) mbar_expect_tx(keys ? &sm.k_full[b] : &sm.v_full[b], kKeys * DH * 2);
+                if (ok) mbar_expect_tx(keys ? &sm.k_full[b] : &sm.v_full[b], keys ? kKeys * 128 * (panel_hi - panel_lo) : kKeys * DH * 2);
                 stamp(keys ? 0 : 4, 1, j);
             }
             ok = __shfl_sync(0xffffffffu, ok, 0);
@@ -202,7 +221,7 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
                 if (keys) {
 #pragma unroll
                     for (int pn = 0; pn < kPanels; ++pn)
-                        tma_load_2d(sm.k[b] + pn * (kKeys * 128) + lane * 2048, &map_k, pn * 64, (page * nkv + kvh) * page_size + off, &sm.k_full[b]);
+                        if (pn >= panel_lo && pn < panel_hi) tma_load_2d(sm.k[b] + pn * (kKeys * 128) + lane * 2048, &map_k, pn * 64, (page * nkv + kvh) * page_size + off, &sm.k_full[b]);
                 } else {
                     tma_load_2d(sm.v[b] + lane * (DH * 32), &map_v, off, (page * nkv + kvh) * DH, &sm.v_full[b]);
                 }
@@ -226,8 +245,9 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
                 for (int k = 0; k < DH / 16; ++k) {
+                    if (k < k_lo || k >= k_hi) continue;
                     const unsigned long long db = umma_desc(sm.k[b] + (k >> 2) * (kKeys * 128)) + (unsigned long long)((k & 3) * 2);
-                    umma_bf16_ta(tmem_s + 128 * (j & 1), tmem_q + 8 * k, db, idesc_s, k ? 1u : 0u);
+                    umma_bf16_ta(tmem_s + 128 * (j & 1), tmem_q + 8 * k, db, idesc_s, k > k_lo ? 1u : 0u);
                 }
                 umma_commit(&sm.s_full[j & 1]);
                 umma_commit(&sm.k_empty[b]);
@@ -269,7 +289,9 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
         const bool valid = cta_i0 + r < n;
         const int p = valid ? p_first + r : -1;                  // its position; no key is visible to an unused row
         const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
-        const float scale_log2 = scale * 1.4426950408889634f;
+        // (capped scores are brought to base-2 units as they are capped, and the factor below is 1)
+        const float scale_log2 = kCap ? 1.0f : scale * 1.4426950408889634f;
+        [[maybe_unused]] const float cap_in = kCap ? scale / softcap : 0.0f, cap_out = softcap * 1.4426950408889634f;
         // m: the maximum the exponentials are taken against.  It follows the true maximum lazily: only when that has grown by
         // more than kLazy (in powers of two) is the output so far, which accumulates in tensor memory, scaled down to the
         // new one.  Until then the probabilities may reach 2^kLazy, which costs bfloat16 and the float sums nothing, and
@@ -282,7 +304,7 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
         if (half * 64 < DH) {                                    // the same for the whole warp
             unsigned qw[32];
             if (valid) {
-                const uint4* src = reinterpret_cast<const uint4*>(qkv + (size_t)(tok0 + cta_i0 + r) * row_elems + (size_t)h * DH + half * 64);
+                const uint4* src = reinterpret_cast<const uint4*>(qkv + (size_t)(tok0 + cta_i0 + r) * row_elems + (size_t)(h / maps) * DH + half * 64);
 #pragma unroll
                 for (int i = 0; i < 8; ++i) {
                     const uint4 t4 = __ldg(src + i);
@@ -307,6 +329,20 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
             // this thread's 64 scores of the tile, read once and kept for both passes; a key the row does not see reads -inf
             float v[HK];
             tmem_ld_32x64(tmem_s + 128 * (j & 1) + lane_addr + half * HK, v);
+            if constexpr (kCap) {
+                // cap * tanh(s scale / cap) in base-2 units: small arguments by a polynomial on the multiply-add pipe, and if
+                // any of the thread's is larger all of them through the exponential
+                float top = 0.0f;
+#pragma unroll
+                for (int i = 0; i < HK; ++i) top = fmaxf(top, fabsf(v[i]));
+                if (top * cap_in <= kTanhSmall) {
+#pragma unroll
+                    for (int i = 0; i < HK; ++i) v[i] = tanh_small(v[i] * cap_in) * cap_out;
+                } else {
+#pragma unroll
+                    for (int i = 0; i < HK; ++i) v[i] = tanh_fast(v[i] * cap_in) * cap_out;
+                }
+            }
             const bool whole = (key0 >= lo || key0 + HK <= keep) && key0 + HK - 1 <= p;
             if (!whole) {
 #pragma unroll
@@ -506,23 +542,23 @@ SplitSpace& split_space() {
     return space;
 }
 
-template <int DH>
+template <int DH, bool kCap>
 int launch(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks, const int* q_start,
            const int* ctx_lens, int T, int S, int nh, int nkv, int page_size, int num_pages, float scale, int window, int max_q_len,
-           int skip_single, const int* units, int unit_slots, const float* sinks, int keep_first, cudaStream_t stream) {
+           int skip_single, const int* units, int unit_slots, const float* sinks, int keep_first, float softcap, int maps, cudaStream_t stream) {
     EncodeTiledFn encode = nullptr;
     int *err_host = nullptr, *err_dev = nullptr;
     if (int rc = setup(&encode, &err_host, &err_dev)) return rc;
     if (*err_host != 0)
         return li_fail("attention (tcgen05): an earlier launch gave up waiting on a barrier (status %d); the results since then are invalid", *err_host);
     CUtensorMap map_k, map_v;
-    const long long row_elems = (long long)(nh + 2 * nkv) * DH;
+    const long long row_elems = (long long)(nh / maps + 2 * nkv) * DH;
     if (int rc = make_map_ex(&map_k, kcache, (unsigned long long)num_pages * nkv * page_size, DH, 64, 16, 128)) return rc;
     if (int rc = make_map_ex(&map_v, vcache, (unsigned long long)num_pages * nkv * DH, (unsigned long long)page_size, 16, DH, 32)) return rc;
     const size_t smem = sizeof(Smem<DH>) + smem_pad<DH>();
     static bool raised = false;
     if (!raised) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<DH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<DH, kCap>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return li_fail("attention (tcgen05): cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
         raised = true;
     }
@@ -542,9 +578,9 @@ int launch(const void* qkv, void* out, const void* kcache, const void* vcache, c
     }
     const dim3 grid = units ? dim3(nh, unit_slots, 1) : dim3(nh, ceil_div(max_q_len, kRows), S);
     static const int trace = getenv("LITINFER_B200_ATTN_TRACE") ? 1 : 0;
-    li_launch_pdl(prefill_attention_tc_kernel<DH>, grid, dim3(kThreads), smem, stream, (const bf16*)qkv, row_elems, map_k, map_v, (bf16*)out, block_table, max_blocks,
+    li_launch_pdl(prefill_attention_tc_kernel<DH, kCap>, grid, dim3(kThreads), smem, stream, (const bf16*)qkv, row_elems, map_k, map_v, (bf16*)out, block_table, max_blocks,
                   q_start, ctx_lens, nh, nkv, page_size, num_pages, scale, window, skip_single, err_dev, trace, units, partial,
-                  space.counters, sinks, keep_first);
+                  space.counters, sinks, keep_first, softcap, maps);
     return li_check_launch("attention (tcgen05)");
 }
 
@@ -558,13 +594,15 @@ bool li_attention_tcgen05_accepts(const void* qkv, const void* kcache, const voi
 int li_attention_tcgen05(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks,
                          const int* q_start, const int* ctx_lens, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages,
                          float scale, int window, int max_q_len, int skip_single, const int* units, int unit_slots, const float* sinks,
-                         int keep_first, cudaStream_t stream) {
+                         int keep_first, float softcap, int maps, cudaStream_t stream) {
+    LI_REQUIRE(maps == 1 || maps == 2, "attention (tcgen05): takes one or two maps a query row, not %d", maps);
     LI_REQUIRE(li_attention_tcgen05_accepts(qkv, kcache, vcache, nh, nkv, dh, page_size),
                "attention (tcgen05): refuses heads=%d/%d head_dim=%d page=%d (head_dim 64 or 128, pages a multiple of 16)", nh, nkv, dh, page_size);
     LI_REQUIRE(scale > 0.0f, "attention (tcgen05): the scale must be positive");
-    if (dh == 64)
-        return launch<64>(qkv, out, kcache, vcache, block_table, max_blocks, q_start, ctx_lens, T, S, nh, nkv, page_size, num_pages, scale,
-                          window, max_q_len, skip_single, units, unit_slots, sinks, keep_first, stream);
-    return launch<128>(qkv, out, kcache, vcache, block_table, max_blocks, q_start, ctx_lens, T, S, nh, nkv, page_size, num_pages, scale,
-                       window, max_q_len, skip_single, units, unit_slots, sinks, keep_first, stream);
+#define LI_CASE(D, CAP)                                                                                                                        \
+    launch<D, CAP>(qkv, out, kcache, vcache, block_table, max_blocks, q_start, ctx_lens, T, S, nh, nkv, page_size, num_pages, scale, window, \
+                   max_q_len, skip_single, units, unit_slots, sinks, keep_first, softcap, maps, stream)
+    if (dh == 64) return softcap > 0.0f ? LI_CASE(64, true) : LI_CASE(64, false);
+    return softcap > 0.0f ? LI_CASE(128, true) : LI_CASE(128, false);
+#undef LI_CASE
 }

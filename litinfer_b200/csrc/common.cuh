@@ -18,11 +18,11 @@
 
 enum LiDtype : int { LI_F32 = 0, LI_BF16 = 1 };
 // What a matrix product does to its result: nothing, or the SwiGLU of interleaved gate and up columns.
-// LI_EPILOGUE_GLU_CLAMPED: the same columns, another activation (glu_of below); the product's `bias` argument then points
-// at its two parameters on the device, {limit, alpha}, since a gated product has no bias.
-enum LiEpilogue : int { LI_EPILOGUE_NONE = 0, LI_EPILOGUE_SWIGLU = 1, LI_EPILOGUE_GLU_CLAMPED = 2 };
-static inline bool li_epilogue_is_gated(int e) { return e == LI_EPILOGUE_SWIGLU || e == LI_EPILOGUE_GLU_CLAMPED; }
-// what a gated epilogue needs of the bias argument: none for SwiGLU, the parameters for the clamped unit
+// LI_EPILOGUE_GLU_CLAMPED, LI_EPILOGUE_GEGLU: the same columns, another activation (glu_of below); for the clamped unit the
+// product's `bias` argument points at its two parameters on the device, {limit, alpha}, since a gated product has no bias.
+enum LiEpilogue : int { LI_EPILOGUE_NONE = 0, LI_EPILOGUE_SWIGLU = 1, LI_EPILOGUE_GLU_CLAMPED = 2, LI_EPILOGUE_GEGLU = 3 };
+static inline bool li_epilogue_is_gated(int e) { return e == LI_EPILOGUE_SWIGLU || e == LI_EPILOGUE_GLU_CLAMPED || e == LI_EPILOGUE_GEGLU; }
+// what a gated epilogue needs of the bias argument: the parameters for the clamped unit, none for the others
 static inline bool li_epilogue_bias_ok(int e, const float* bias) { return (e == LI_EPILOGUE_GLU_CLAMPED) == (bias != nullptr); }
 
 int li_fail(const char* fmt, ...);            // stores the message, returns 1
@@ -92,6 +92,9 @@ __device__ __forceinline__ float poly_exp2(float x) {
     return __int_as_float(__float_as_int(p) + (__float_as_int(t) << 23));
 }
 
+// tanh from the fast exponential and quotient (absolute error about 1e-6): 1 - 2 / (1 + e^(2x)).
+__device__ __forceinline__ float tanh_fast(float x) { return 1.0f - __fdividef(2.0f, 1.0f + fast_exp2(x * 2.8853900817779268f)); }
+
 // up * gate / (1 + exp(-gate)) (src/ops/swiglu/op.cpp:17-23) in float.  For an output that is rounded to 16 bits the
 // exponential and the quotient come from the fast units (errors near 2^-21, far below that rounding): an epilogue in which
 // one warp works through its row alone is bound by the length of this chain of instructions.
@@ -101,13 +104,23 @@ __device__ __forceinline__ float swiglu_of(float gate, float up) {
     else return up * (gate / (1.0f + expf(-gate)));
 }
 
+// up * gelu(gate) with the tanh form of gelu, 0.5 g (1 + tanh(z)), z = sqrt(2 / pi) (g + 0.044715 g^3).  For an output that
+// is rounded to 16 bits as g / (1 + exp(-2 z)), which is the same function, with the fast units.
+template <typename Tout>
+__device__ __forceinline__ float geglu_of(float gate, float up) {
+    const float z = 0.7978845608028654f * fmaf(0.044715f * gate * gate, gate, gate);
+    if constexpr (sizeof(Tout) == 2) return up * __fdividef(gate, 1.0f + fast_exp2(-2.8853900817779268f * z));
+    else return up * (0.5f * gate * (1.0f + tanhf(z)));
+}
+
 // The activation of a gated product's epilogue, chosen when the kernel is compiled (an epilogue in which one warp works
 // through its row alone is bound by the length of this chain of instructions: a choice per element costs SwiGLU 2 % of a
-// decode step).  Not kClamped: SwiGLU.  kClamped, with params = {limit, alpha}: the gated unit with bounded operands,
-// g = min(gate, limit), u = clamp(up, -limit, limit), g / (1 + exp(-alpha g)) * (u + 1).
-template <typename Tout, bool kClamped>
+// decode step).  kKind is the epilogue's number: 1 SwiGLU, 3 the same with gelu (GEGLU), 2, with params = {limit, alpha}, the
+// gated unit with bounded operands, g = min(gate, limit), u = clamp(up, -limit, limit), g / (1 + exp(-alpha g)) * (u + 1).
+template <typename Tout, int kKind>
 __device__ __forceinline__ float glu_of(float gate, float up, const float* __restrict__ params) {
-    if constexpr (!kClamped) return swiglu_of<Tout>(gate, up);
+    if constexpr (kKind == LI_EPILOGUE_SWIGLU) return swiglu_of<Tout>(gate, up);
+    if constexpr (kKind == LI_EPILOGUE_GEGLU) return geglu_of<Tout>(gate, up);
     const float limit = __ldg(params), alpha = __ldg(params + 1);
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     if constexpr (sizeof(Tout) == 2) return __fdividef(g, 1.0f + fast_exp2(-1.4426950408889634f * alpha * g)) * (u + 1.0f);

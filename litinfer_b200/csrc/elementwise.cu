@@ -403,6 +403,34 @@ LI_EXPORT int li_glu_clamped(const void* gate_up, void* out, int dtype, int T, i
     return li_check_launch("glu_clamped");
 }
 
+// up * gelu(gate), the tanh form; gate_up [T, 2 I] as gate | up.  Float arithmetic, one rounding.
+namespace {
+template <typename T>
+__global__ void geglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int I, long long n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const long long stride = (long long)gridDim.x * blockDim.x;
+    for (; i < n; i += stride) {
+        const long long t = i / I;
+        const int j = (int)(i - t * I);
+        out[i] = from_float<T>(geglu_of<T>(to_float(gate_up[t * 2 * I + j]), to_float(gate_up[t * 2 * I + I + j])));
+    }
+}
+}  // namespace
+
+LI_EXPORT int li_geglu(const void* gate_up, void* out, int dtype, int T, int I, cudaStream_t stream) {
+    LI_REQUIRE(T >= 0 && I > 0, "geglu: bad sizes T=%d I=%d", T, I);
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "geglu: unknown dtype %d", dtype);
+    const long long n = (long long)T * I;
+    if (n == 0) return 0;
+    cudaError_t e;
+    if (dtype == LI_F32) e = li_launch_pdl(geglu_kernel<float>, dim3(grid_for(n, 256)), dim3(256), 0, stream, (const float*)gate_up, (float*)out, I, n);
+    else e = li_launch_pdl(geglu_kernel<bf16>, dim3(grid_for(n, 256)), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, I, n);
+    if (e != cudaSuccess) return li_fail("geglu: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("geglu");
+}
+
 // PolyNorm and a sigmoid gate.
 //   li_polynorm: per token row z [n]: out = a N(z) + b N(z^2) + c N(z^3) + e with powers element by element and
 //     N(v) = v / sqrt(mean(v^2) + eps); coef = {a, b, c, e} float on the device.  The three means are taken in one pass (the row

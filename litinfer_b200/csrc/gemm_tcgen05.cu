@@ -623,6 +623,9 @@ int li_linear_tcgen05_grouped(const void* a, const void* w, void* out, int M, in
     if (epilogue == LI_EPILOGUE_GLU_CLAMPED)
         return wide ? launch_tile<128, 256, bf16, 2>(a, w, glu_params, out, M, N, K, stream, 1, RopeEpilogue{}, tile_group, G)
                     : launch_tile<128, 128, bf16, 2>(a, w, glu_params, out, M, N, K, stream, 1, RopeEpilogue{}, tile_group, G);
+    if (epilogue == LI_EPILOGUE_GEGLU)
+        return wide ? launch_tile<128, 256, bf16, 3>(a, w, nullptr, out, M, N, K, stream, 1, RopeEpilogue{}, tile_group, G)
+                    : launch_tile<128, 128, bf16, 3>(a, w, nullptr, out, M, N, K, stream, 1, RopeEpilogue{}, tile_group, G);
     if (gated)
         return wide ? launch_tile<128, 256, bf16, 1>(a, w, nullptr, out, M, N, K, stream, 1, RopeEpilogue{}, tile_group, G)
                     : launch_tile<128, 128, bf16, 1>(a, w, nullptr, out, M, N, K, stream, 1, RopeEpilogue{}, tile_group, G);
@@ -656,6 +659,7 @@ int li_linear_tcgen05(const void* a, const void* w, const float* bias, void* out
         LI_REQUIRE(N % 16 == 0 && li_epilogue_bias_ok(epilogue, bias) && dtype_out == LI_BF16,
                    "linear (tcgen05): the swiglu epilogue needs N a multiple of 16, no bias and bfloat16 output");
         return epilogue == LI_EPILOGUE_GLU_CLAMPED ? launch<bf16, 2>(a, w, bias, out, M, N, K, stream, g_forced_tile)
+               : epilogue == LI_EPILOGUE_GEGLU     ? launch<bf16, 3>(a, w, bias, out, M, N, K, stream, g_forced_tile)
                                                    : launch<bf16, 1>(a, w, bias, out, M, N, K, stream, g_forced_tile);
     }
     if (dtype_out == LI_BF16) return launch<bf16, 0>(a, w, bias, out, M, N, K, stream, g_forced_tile);

@@ -201,7 +201,9 @@ int li_linear_tcgen05_persistent(const void* a, const void* w, const float* bias
     if (li_epilogue_is_gated(epilogue)) {
         LI_REQUIRE(N % 16 == 0 && li_epilogue_bias_ok(epilogue, bias) && dtype_out == LI_BF16,
                    "linear (tcgen05, persistent): the swiglu epilogue needs N a multiple of 16, no bias and bfloat16 output");
-        return epilogue == LI_EPILOGUE_GLU_CLAMPED ? launch<bf16, 2>(a, w, bias, out, M, N, K, stream) : launch<bf16, 1>(a, w, bias, out, M, N, K, stream);
+        return epilogue == LI_EPILOGUE_GLU_CLAMPED ? launch<bf16, 2>(a, w, bias, out, M, N, K, stream)
+               : epilogue == LI_EPILOGUE_GEGLU     ? launch<bf16, 3>(a, w, bias, out, M, N, K, stream)
+                                                   : launch<bf16, 1>(a, w, bias, out, M, N, K, stream);
     }
     if (dtype_out == LI_BF16) return launch<bf16, 0>(a, w, bias, out, M, N, K, stream);
     if (dtype_out == LI_F32) return launch<float, 0>(a, w, bias, out, M, N, K, stream);

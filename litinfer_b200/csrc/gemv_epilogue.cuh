@@ -102,7 +102,7 @@ __device__ __forceinline__ void store_elements(Get get, const float* __restrict_
                 gate *= rs_sm[tok];
                 up *= rs_sm[tok];
             }
-            if (col < half_n && tok < M) out[(size_t)tok * half_n + col] = from_float<Tout>(glu_of<Tout, kSwiglu == 2>(gate, up, bias));
+            if (col < half_n && tok < M) out[(size_t)tok * half_n + col] = from_float<Tout>(glu_of<Tout, kSwiglu>(gate, up, bias));
         }
     }
 }

@@ -82,7 +82,7 @@ __device__ __forceinline__ void tmem_ld<64>(unsigned taddr, float (&v)[64]) {
     }
 }
 
-enum { kEpiNone = 0, kEpiSwiglu = 1, kEpiAddScaled = 2, kEpiGluClamped = 3 };     // (the last: SwiGLU's layout, another activation)
+enum { kEpiNone = 0, kEpiSwiglu = 1, kEpiAddScaled = 2, kEpiGluClamped = 3, kEpiGeglu = 4 };     // (the last two: SwiGLU's layout, another activation)
 
 template <int BT, typename Tout, int kEpi>
 __global__ void __launch_bounds__(kThreads)
@@ -90,7 +90,8 @@ gemv_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     const float* __restrict__ bias, Tout* __restrict__ out, float* __restrict__ partial,
                     unsigned* __restrict__ counters, int M, int N, int K, int ksplit, int* __restrict__ error_flag, const RowScale rs,
                     const AddScaled add) {
-    constexpr bool kSwiglu = kEpi == kEpiSwiglu || kEpi == kEpiGluClamped, kAdd = kEpi == kEpiAddScaled;
+    constexpr int kSwiglu = kEpi == kEpiSwiglu ? LI_EPILOGUE_SWIGLU : kEpi == kEpiGluClamped ? LI_EPILOGUE_GLU_CLAMPED : kEpi == kEpiGeglu ? LI_EPILOGUE_GEGLU : 0;
+    constexpr bool kAdd = kEpi == kEpiAddScaled;
     extern __shared__ unsigned char smem_raw[];
     Smem<BT>& sm = *reinterpret_cast<Smem<BT>*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -256,7 +257,7 @@ gemv_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     const int tid = (int)threadIdx.x - 64;
                     if (tid < M)
                         add.ssq_out[(size_t)tid * gridDim.x + tile] = ((sm.squares[0][tid] + sm.squares[1][tid]) + sm.squares[2][tid]) + sm.squares[3][tid];
-                } else if constexpr (!kSwiglu) {
+                } else if constexpr (kSwiglu == 0) {
                     const float b = (bias && row < N) ? bias[row] : 0.0f;
 #pragma unroll
                     for (int j = 0; j < BT; ++j)
@@ -270,7 +271,7 @@ gemv_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         const float up = __shfl_down_sync(0xffffffffu, v[j], 8);
                         if (j < M && (lane & 8) == 0 && row + 8 < N) {
                             const float gate = v[j];
-                            out[(size_t)j * half_n + col] = from_float<Tout>(glu_of<Tout, kEpi == kEpiGluClamped>(gate, up, bias));
+                            out[(size_t)j * half_n + col] = from_float<Tout>(glu_of<Tout, kSwiglu>(gate, up, bias));
                         }
                     }
                 }
@@ -377,6 +378,7 @@ int li_linear_gemv_tcgen05(const void* a, const void* w, const float* bias, void
         LI_REQUIRE(N % 16 == 0 && li_epilogue_bias_ok(epilogue, bias) && dtype_out == LI_BF16,
                    "linear (tcgen05 gemv): the swiglu epilogue needs N a multiple of 16, no bias and bfloat16 output");
         return epilogue == LI_EPILOGUE_GLU_CLAMPED ? launch_bt<bf16, kEpiGluClamped>(a, w, bias, out, M, N, K, stream, rs)
+               : epilogue == LI_EPILOGUE_GEGLU     ? launch_bt<bf16, kEpiGeglu>(a, w, bias, out, M, N, K, stream, rs)
                                                    : launch_bt<bf16, kEpiSwiglu>(a, w, bias, out, M, N, K, stream, rs);
     }
     if (dtype_out == LI_BF16) return launch_bt<bf16, kEpiNone>(a, w, bias, out, M, N, K, stream, rs);

@@ -126,7 +126,7 @@ __device__ __forceinline__ void mma16816(float (&c)[4], unsigned a0, unsigned a1
 // TM 64: many rows a group (portions of prompts); a warp takes 16 rows and all 64 columns.  TM 16: few rows a group
 // (single tokens: the weights are what is read): a warp takes all 16 rows and 16 of the columns, and four stages of
 // 64 elements keep more of the weights on their way.
-// kSwiglu (1, or 2: the gated unit with bounded operands, glu_params = {limit, alpha} on the device): the columns come as 8 gate,
+// kSwiglu (1, 3: GEGLU, or 2: the gated unit with bounded operands, glu_params = {limit, alpha} on the device): the columns come as 8 gate,
 // 8 up, 8 gate, 8 up, ... (the rows of every group's matrix interleaved in eights), and out [M, N / 2] takes
 // up * gate / (1 + exp(-gate)) (or the bounded unit): a thread holds a gate column and its up column in neighbouring tiles of 8.
 template <int TM, int TK, int ST, int kSwiglu>
@@ -215,8 +215,8 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 if (gate_col + i + 8 < N) {
-                    if (r_lo < m_end) c[(size_t)r_lo * ldc + n + i] = __float2bfloat16_rn(glu_of<bf16, kSwiglu == 2>(acc[j][i], acc[j + 1][i], glu_params));
-                    if (r_hi < m_end) c[(size_t)r_hi * ldc + n + i] = __float2bfloat16_rn(glu_of<bf16, kSwiglu == 2>(acc[j][2 + i], acc[j + 1][2 + i], glu_params));
+                    if (r_lo < m_end) c[(size_t)r_lo * ldc + n + i] = __float2bfloat16_rn(glu_of<bf16, kSwiglu>(acc[j][i], acc[j + 1][i], glu_params));
+                    if (r_hi < m_end) c[(size_t)r_hi * ldc + n + i] = __float2bfloat16_rn(glu_of<bf16, kSwiglu>(acc[j][2 + i], acc[j + 1][2 + i], glu_params));
                 }
             }
         }
@@ -472,7 +472,7 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, const int* __restrict
 
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __restrict__ place_of, const float* __restrict__ weights, int top, int H,
-                                   T* __restrict__ y) {
+                                   const T* __restrict__ extra, T* __restrict__ y) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -482,6 +482,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
             const float v = to_float(rows[(size_t)place_of[(size_t)t * top + k] * H + i]);
             acc += weights ? weights[(size_t)t * top + k] * v : v;
         }
+        if (extra) acc += to_float(extra[(size_t)t * H + i]);
         y[(size_t)t * H + i] = from_float<T>(acc);
     }
 }
@@ -505,7 +506,7 @@ LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* 
     LI_REQUIRE(epilogue == LI_EPILOGUE_NONE || li_epilogue_is_gated(epilogue), "grouped_linear: unknown epilogue %d", epilogue);
     LI_REQUIRE(li_epilogue_bias_ok(epilogue, glu_params) || epilogue == LI_EPILOGUE_NONE, "grouped_linear: the bounded unit needs its parameters, the others take none");
     const bool swiglu = li_epilogue_is_gated(epilogue);
-    const bool clamped = epilogue == LI_EPILOGUE_GLU_CLAMPED;
+    const bool clamped = epilogue == LI_EPILOGUE_GLU_CLAMPED, geglu = epilogue == LI_EPILOGUE_GEGLU;
     const int out_cols = swiglu ? N / 2 : N;
     LI_REQUIRE(lda >= K && ldc >= out_cols, "grouped_linear: rows of %d and %d elements cannot hold K=%d and %d outputs", lda, ldc, K, out_cols);
     LI_REQUIRE(row_offsets == nullptr || (a_gcol == 0 && c_gcol == 0), "grouped_linear: groups are rows or columns, not both");
@@ -529,9 +530,9 @@ LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* 
 #define LI_GROUPED_MMA(TM_, TK_, ST_, EPI_, GRID_)                                                                                          \
     li_launch_pdl(grouped_mma_kernel<TM_, TK_, ST_, EPI_>, GRID_, dim3(128), 0, stream, (const bf16*)a, lda, a_gcol, (const bf16*)w, (bf16*)out, ldc, \
                   c_gcol, row_offsets, M, N, K, G, glu_params)
-        e = clamped ? LI_GROUPED_MMA(16, 64, 4, 2, grid16) : swiglu ? LI_GROUPED_MMA(16, 64, 4, 1, grid16) : LI_GROUPED_MMA(16, 64, 4, 0, grid16);
+        e = clamped ? LI_GROUPED_MMA(16, 64, 4, 2, grid16) : geglu ? LI_GROUPED_MMA(16, 64, 4, 3, grid16) : swiglu ? LI_GROUPED_MMA(16, 64, 4, 1, grid16) : LI_GROUPED_MMA(16, 64, 4, 0, grid16);
     } else if (dtype == LI_BF16 && aligned)
-        e = clamped ? LI_GROUPED_MMA(64, 32, 3, 2, grid) : swiglu ? LI_GROUPED_MMA(64, 32, 3, 1, grid) : LI_GROUPED_MMA(64, 32, 3, 0, grid);
+        e = clamped ? LI_GROUPED_MMA(64, 32, 3, 2, grid) : geglu ? LI_GROUPED_MMA(64, 32, 3, 3, grid) : swiglu ? LI_GROUPED_MMA(64, 32, 3, 1, grid) : LI_GROUPED_MMA(64, 32, 3, 0, grid);
 #undef LI_GROUPED_MMA
     else if (dtype == LI_F32)
         e = li_launch_pdl(grouped_linear_kernel<float, float>, grid, dim3(256), 0, stream, (const float*)a, lda, a_gcol, (const float*)w, (float*)out,
@@ -597,18 +598,18 @@ LI_EXPORT int li_moe_gather(const void* h, int dtype, const int* pair_at, const 
     return li_check_launch("moe_gather");
 }
 
-// y [T, H]: y[t] = sum_k rows[place_of[t * top + k]] (times weights[t * top + k] if weights is given).
-LI_EXPORT int li_moe_combine(const void* rows, int dtype, const int* place_of, const float* weights, int T, int top, int H, void* y,
-                             cudaStream_t stream) {
+// y [T, H]: y[t] = sum_k rows[place_of[t * top + k]] (times weights[t * top + k] if weights is given), plus extra[t] if given.
+LI_EXPORT int li_moe_combine(const void* rows, int dtype, const int* place_of, const float* weights, const void* extra, int T, int top, int H,
+                             void* y, cudaStream_t stream) {
     LI_REQUIRE(T >= 0 && top > 0 && H > 0, "moe_combine: bad sizes");
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "moe_combine: unknown dtype %d", dtype);
     if (T == 0) return 0;
     const int threads = H >= 1024 ? 256 : 128;
     cudaError_t e;
     if (dtype == LI_F32)
-        e = li_launch_pdl(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)rows, place_of, weights, top, H, (float*)y);
+        e = li_launch_pdl(moe_combine_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)rows, place_of, weights, top, H, (const float*)extra, (float*)y);
     else
-        e = li_launch_pdl(moe_combine_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16*)rows, place_of, weights, top, H, (bf16*)y);
+        e = li_launch_pdl(moe_combine_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16*)rows, place_of, weights, top, H, (const bf16*)extra, (bf16*)y);
     if (e != cudaSuccess) return li_fail("moe_combine: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("moe_combine");
 }

@@ -45,7 +45,7 @@ int li_paged_attention(const void* qkv, void* out, const void* kcache, const voi
     block_table, int max_blocks, const int* q_start, const int* ctx_lens, const int* seq_of_token, const int*
     positions, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages, float scale, int window, int
     max_q_len, int max_ctx_len, const int* old_lens, int singles, const int* units, int slots_portions, int slots_all,
-    float softcap, const float* slopes, const void* gate, int keep_first, const float* sinks, cudaStream_t stream);
+    float softcap, const float* slopes, const void* gate, int keep_first, const float* sinks, int maps, cudaStream_t stream);
 
 /* The same through one implementation: 0 general, 1 decode, 2 mma.sync tiles, 3 tcgen05 tiles (tests and
  * measurements). */
@@ -53,7 +53,7 @@ int li_paged_attention_with(int which, const void* qkv, void* out, const void* k
     const int* block_table, int max_blocks, const int* q_start, const int* ctx_lens, const int* seq_of_token, const
     int* positions, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages, float scale, int window, int
     max_q_len, int max_ctx_len, const int* old_lens, int singles, const int* units, int slots_portions, int slots_all,
-    float softcap, const float* slopes, const void* gate, int keep_first, const float* sinks, cudaStream_t stream);
+    float softcap, const float* slopes, const void* gate, int keep_first, const float* sinks, int maps, cudaStream_t stream);
 
 /* ---- decode_step.cu: a decode step as one persistent kernel (decode_step.h has the structures) ---- */
 struct LiDecodeStep;
@@ -108,6 +108,9 @@ int li_apply_row_scale(const void* hprime, const float* ssq, int nparts, int wid
 /* out[t, i] = g / (1 + exp(-alpha g)) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); gate_up
  * [T, 2 I] as gate | up. */
 int li_glu_clamped(const void* gate_up, void* out, int dtype, int T, int I, float limit, float alpha, cudaStream_t stream);
+
+/* out[t, i] = up * gelu(gate), the tanh form of gelu; gate_up [T, 2 I] as gate | up. */
+int li_geglu(const void* gate_up, void* out, int dtype, int T, int I, cudaStream_t stream);
 
 /* out = a N(z) + b N(z^2) + c N(z^3) + e per row of z [T, n], powers element by element, N(v) = v / sqrt(mean(v^2) + eps),
  * coef = {a, b, c, e} float on the device. */
@@ -224,7 +227,7 @@ int li_linear_gemv_static(const void* a, const void* w, const float* bias, void*
 void li_gemv_tcgen05_force_ksplit(int n);
 
 /* ---- linear.cu ---- */
-/* out[M, N] = a[M, K] w[N, K]^T (+ bias), epilogue 0 none / 1 SwiGLU over interleaved gate|up rows; float32 in
+/* out[M, N] = a[M, K] w[N, K]^T (+ bias), epilogue 0 none / 1 SwiGLU, 2 bounded unit, 3 GEGLU over interleaved gate|up rows; float32 in
  * float32 out, or bfloat16 in, bfloat16 or float out. */
 int li_linear(const void* a, const void* w, const float* bias, void* out, int dtype_in, int dtype_out, int M, int N,
     int K, int epilogue, cudaStream_t stream);
@@ -268,10 +271,14 @@ int li_linear_rope_kv(const void* a, const void* w, const float* bias, void* qkv
 /* Per row: x += post(y) (post: a norm of y [R, H] with the weight w_post; NULL: x += y; y NULL: nothing is added), then
  * out = next(x) if w_next is given (without it, out, if given, takes x as it is in the run dtype).  A norm is centered (mean taken off, variance as the mean of squared deviations:
  * layer norm without bias) or not (RMS norm).  rows (may be NULL; only without y): out[r] = next(x[rows[r]]).
- * y_places (may be NULL): token r's y is the sum over j < y_top of y[y_places[r y_top + j]] (times y_weights[...] if given). */
+ * y_places (may be NULL): token r's y is the sum over j < y_top of y[y_places[r y_top + j]] (times y_weights[...] if given), plus
+ * y_extra[r] if that is given. */
 int li_norm_add_norm(float* x, const void* y, int dtype, const float* w_post, int post_centered, float eps_post, const float* w_next,
     int next_centered, float eps_next, void* out, const int* rows, int R, int n_src, int H, const int* y_places,
-    int y_top, const float* y_weights, cudaStream_t stream);
+    int y_top, const float* y_weights, const void* y_extra, cudaStream_t stream);
+
+/* out [T, 2 H] in the run dtype: x [T, H] (plus delta [T, H] if given) beside x0 [T, H], both float. */
+int li_join_rows(const float* x, const void* delta, const float* x0, void* out, int dtype, int T, int H, cudaStream_t stream);
 
 /* x[t] += row for every token. */
 int li_add_row(float* x, const float* row, int T, int H, cudaStream_t stream);
@@ -309,6 +316,22 @@ int li_latent_rope_post(const void* low, int dtype, int ld_low, int col_c, int c
 int li_row_rinv(const void* x, int dtype, int ld, int col0, int n0, int width0, int col1, int n1, int width1, float eps, float* out,
     int T, cudaStream_t stream);
 
+/* Rotation of the first rotary_dim elements of the query and key heads of proj [T, ld] (pair i by float(pos) / denom[i];
+ * interleaved: pair (2i, 2i + 1), else (i, i + rotary_dim / 2); cosine and sine times magnitude), then (norm != 0) each head
+ * divided by sqrt(sum x^2 / norm_width + eps), times q_norm / k_norm [dh] if given; queries to out [T, (nh + 2 nkv) dh], keys
+ * and values into the paged cache, or with to_cache 0 to their columns of out.  keys_are_values: proj holds q | k only, and
+ * a key head as projected, before rotation and norm, is the value. */
+int li_rope_norm_kv(const void* proj, int ld, void* out, int dtype, const int* positions, const float* denom, float magnitude, int interleaved,
+    int rotary_dim, const float* q_norm, const float* k_norm, int norm, float eps, int norm_width,
+    const int* slot_mapping, void* kcache, void* vcache, int T, int nh, int nkv, int dh, int page_size,
+    int num_pages, int write, int to_cache, int keys_are_values, cudaStream_t stream);
+
+/* Two maps of attention over the same values, att [T, 2 H dl] (head h's maps at columns 2 h dl and (2 h + 1) dl, dv real
+ * elements each): out[t, h] = (a1 - lambda a2) / sqrt(mean(.^2) + eps) * gain, times sigmoid(gate [T, gate_ld] at gate_col + h dv
+ * + i) if a gate is given; out [T, H dv]. */
+int li_map_difference(const void* att, int dtype, int dl, const void* gate, int gate_ld, int gate_col, float lambda, float eps, float gain,
+    void* out, int T, int H, int dv, cudaStream_t stream);
+
 /* ---- grouped.cu: products in groups, routing of a mixture of experts ---- */
 /* out_g = a_g w_g^T, w [G, N, K].  row_offsets [G + 1] (device): group g owns those rows of a [M, lda] and out [M, ldc].
  * row_offsets NULL: every group takes all M rows, inputs at column g * a_gcol, outputs at column g * c_gcol.
@@ -339,9 +362,9 @@ int li_moe_sort(const int* ids, int n, int E, int matrices, int pad, int* offset
 /* out [n, H]: row r is h[pair_at[r] / top], times weights[pair_at[r]] if weights is given; zeros where pair_at[r] < 0. */
 int li_moe_gather(const void* h, int dtype, const int* pair_at, const float* weights, int n, int top, int H, void* out, cudaStream_t stream);
 
-/* y [T, H]: y[t] = sum_k rows[place_of[t * top + k]] (times weights[t * top + k] if weights is given). */
-int li_moe_combine(const void* rows, int dtype, const int* place_of, const float* weights, int T, int top, int H, void* y,
-    cudaStream_t stream);
+/* y [T, H]: y[t] = sum_k rows[place_of[t * top + k]] (times weights[t * top + k] if weights is given), plus extra[t] if given. */
+int li_moe_combine(const void* rows, int dtype, const int* place_of, const float* weights, const void* extra, int T, int top, int H,
+    void* y, cudaStream_t stream);
 
 /* ---- sampling.cu ---- */
 /* out[r] = the first maximum of logits[r]. */

@@ -9,6 +9,7 @@
 //     deviations),  v / sqrt(mean(v^2) + eps) * w  (centered 0: RMS norm)  or just  v * w  (centered 2: a factor per channel).  Rows may be gathered (rows[r]) when
 //     there is no y: the model's last norm on the wanted rows only.
 //   li_add_row: x[t] += table[row] for every token (a vector per pass of a looped span of layers).
+//   li_join_rows: [x | x0] side by side in the run dtype: the input of a map that reads the stream beside the embedding output.
 //   li_rmsnorm_cols: RMS norm of n columns of a run-dtype matrix, written to (up to) two places of another matrix.
 //
 // All sums, means and the residual stream are float; y and out are in the run dtype.  One block per row.  The variance
@@ -209,7 +210,8 @@ template <typename T, bool kVec>
 __global__ void norm_add_norm_regs_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w_post, int post_centered,
                                           float eps_post, const float* __restrict__ w_next, int next_centered, float eps_next,
                                           T* __restrict__ out, const int* __restrict__ rows, int n_src, int H,
-                                          const int* __restrict__ y_places, int y_top, const float* __restrict__ y_weights) {
+                                          const int* __restrict__ y_places, int y_top, const float* __restrict__ y_weights,
+                                          const T* __restrict__ y_extra) {
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -235,6 +237,13 @@ __global__ void norm_add_norm_regs_kernel(float* __restrict__ x, const T* __rest
                 const float f = y_weights ? y_weights[(size_t)r * y_top + j] : 1.0f;
 #pragma unroll
                 for (int k = 0; k < kRegs; ++k) yv[k] = fmaf(f, part[k], yv[k]);
+            }
+            if (y_extra) {
+                // and one row of the token's own (a shared expert)
+                float part[kRegs];
+                load_row<kVec>(part, y_extra + (size_t)r * H, H);
+#pragma unroll
+                for (int k = 0; k < kRegs; ++k) yv[k] += part[k];
             }
         } else {
             load_row<kVec>(yv, y + (size_t)r * H, H);
@@ -266,6 +275,37 @@ __global__ void add_row_kernel(float* __restrict__ x, const float* __restrict__ 
     if (i < n) x[i] += row[i % H];
 }
 
+// out[t] = (x[t] + delta[t] | x0[t]), four elements a thread where rows are multiples of four, else one
+template <typename T, int V>
+__global__ void join_rows_kernel(const float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ x0, T* __restrict__ out, long long n, int H) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= n) return;
+    const long long t = i / (2 * H);
+    const int c = (int)(i - t * 2 * H);
+    const bool first = c < H;
+    const size_t src = (size_t)t * H + (first ? c : c - H);
+    float v[V];
+    if constexpr (V == 4) {
+        const float4 a = *reinterpret_cast<const float4*>((first ? x : x0) + src);
+        v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
+    } else {
+        v[0] = (first ? x : x0)[src];
+    }
+    if (first && delta) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] += to_float(delta[src + k]);
+    }
+    if constexpr (V == 4 && sizeof(T) == 2) {
+        __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3])};
+        *reinterpret_cast<uint2*>(out + i) = *reinterpret_cast<uint2*>(h);
+    } else {
+#pragma unroll
+        for (int k = 0; k < V; ++k) out[i + k] = from_float<T>(v[k]);
+    }
+}
+
 template <typename T>
 __global__ void rmsnorm_cols_kernel(const T* __restrict__ in, int ld_in, int col, int n, int width, const float* __restrict__ w, float eps,
                                     T* __restrict__ out, int ld_out, int col_a, int col_b) {
@@ -295,9 +335,11 @@ __global__ void rmsnorm_cols_kernel(const T* __restrict__ in, int ld_in, int col
 // be NULL; only without y): out[r] = next(x[rows[r]]).  x is [n_src, H] float and is changed in place when y is given.
 // y_places (may be NULL; H up to 8,192): token r's y is the sum over j < y_top of y[y_places[r y_top + j]] (times
 // y_weights[r y_top + j] if given), summed in float in that order: the combine of a mixture of experts, not written out.
+// y_extra (may be NULL; with y_places): one more row per token that joins the sum, y_extra [R, H] (a shared expert's output).
 LI_EXPORT int li_norm_add_norm(float* x, const void* y, int dtype, const float* w_post, int post_centered, float eps_post, const float* w_next,
                                int next_centered, float eps_next, void* out, const int* rows, int R, int n_src, int H, const int* y_places,
-                               int y_top, const float* y_weights, cudaStream_t stream) {
+                               int y_top, const float* y_weights, const void* y_extra, cudaStream_t stream) {
+    LI_REQUIRE(y_extra == nullptr || y_places != nullptr, "norm_add_norm: a further row goes with a sum of rows");
     LI_REQUIRE(y_places == nullptr || (y != nullptr && y_top > 0 && H <= 8 * 1024), "norm_add_norm: a sum of rows needs the rows, a count and at most 8192 columns");
     LI_REQUIRE(R >= 0 && H > 0 && n_src >= 0, "norm_add_norm: bad sizes R=%d H=%d", R, H);
     LI_REQUIRE(y == nullptr || rows == nullptr, "norm_add_norm: gathered rows cannot take a sublayer's output");
@@ -310,11 +352,11 @@ LI_EXPORT int li_norm_add_norm(float* x, const void* y, int dtype, const float* 
         int threads = ((ceil_div(H, kRegs) + 31) / 32) * 32;
         if (threads < 64) threads = 64;
         // 16-byte moves where every row starts on such a boundary
-        const bool vec = H % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
+        const bool vec = H % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)y_extra % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
                          ((uintptr_t)w_post % 16) == 0 && ((uintptr_t)w_next % 16) == 0;
 #define LI_NORM_LAUNCH(TT, VEC)                                                                                                                  \
     e = li_launch_pdl(norm_add_norm_regs_kernel<TT, VEC>, dim3(R), dim3(threads), 0, stream, x, (const TT*)y, w_post, post_centered, eps_post, w_next, \
-                      next_centered, eps_next, (TT*)out, rows, n_src, H, y_places, y_top, y_weights)
+                      next_centered, eps_next, (TT*)out, rows, n_src, H, y_places, y_top, y_weights, (const TT*)y_extra)
         if (dtype == LI_F32) {
             if (vec) LI_NORM_LAUNCH(float, true);
             else LI_NORM_LAUNCH(float, false);
@@ -344,6 +386,26 @@ LI_EXPORT int li_add_row(float* x, const float* row, int T, int H, cudaStream_t 
     const cudaError_t e = li_launch_pdl(add_row_kernel, dim3((unsigned)ceil_div_ll(n, 256)), dim3(256), 0, stream, x, row, n, H);
     if (e != cudaSuccess) return li_fail("add_row: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("add_row");
+}
+
+// out [T, 2 H] in the run dtype: x [T, H] (plus delta [T, H] if given: an output still to be added to the stream) beside x0
+// [T, H], both float.
+LI_EXPORT int li_join_rows(const float* x, const void* delta, const float* x0, void* out, int dtype, int T, int H, cudaStream_t stream) {
+    LI_REQUIRE(T >= 0 && H > 0, "join_rows: bad sizes");
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "join_rows: unknown dtype %d", dtype);
+    if (T == 0) return 0;
+    const long long n = 2LL * T * H;
+    const bool vec = H % 4 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)x0 % 16) == 0 && ((uintptr_t)out % 16) == 0;
+    const dim3 grid((unsigned)ceil_div_ll(vec ? n / 4 : n, 256));
+    cudaError_t e;
+    if (dtype == LI_F32)
+        e = vec ? li_launch_pdl(join_rows_kernel<float, 4>, grid, dim3(256), 0, stream, x, (const float*)delta, x0, (float*)out, n, H)
+                : li_launch_pdl(join_rows_kernel<float, 1>, grid, dim3(256), 0, stream, x, (const float*)delta, x0, (float*)out, n, H);
+    else
+        e = vec ? li_launch_pdl(join_rows_kernel<bf16, 4>, grid, dim3(256), 0, stream, x, (const bf16*)delta, x0, (bf16*)out, n, H)
+                : li_launch_pdl(join_rows_kernel<bf16, 1>, grid, dim3(256), 0, stream, x, (const bf16*)delta, x0, (bf16*)out, n, H);
+    if (e != cudaSuccess) return li_fail("join_rows: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("join_rows");
 }
 
 // in [T, ld_in]: columns col .. col + n - 1 are normalised (the mean of squares taken over `width` elements: n, or fewer

@@ -395,3 +395,297 @@ LI_EXPORT int li_latent_rope_post(const void* low, int dtype, int ld_low, int co
     if (e != cudaSuccess) return li_fail("latent_rope_post: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("latent_rope_post");
 }
+
+// Rotation first, norm behind it, and the projected keys as values: what stands between a q|k (or q|k|v) product and attention
+// in a layer whose queries and keys are rotated and then divided by their root mean square, head by head.
+//   * `keys_are_values`: the row holds no values; a key head's projection, before rotation and norm, is also its value;
+//   * rotation of the first rotary_dim elements: pair i turns by float(pos) / denom[i]; `interleaved`: the pair is
+//     (2i, 2i + 1), else (i, i + rotary_dim / 2); cosine and sine are multiplied by `magnitude`;
+//   * norm != 0: x / sqrt(sum x^2 / norm_width + eps) per query and key head, times a weight of head size if given;
+//   * queries to `out` [T, (nh + 2 nkv) dh], keys and values into the paged cache (values transposed), or with to_cache 0 to
+//     their columns of `out`.
+// A block takes one token and some of its heads, a warp a head at a time; a lane holds V neighbouring elements of every 32 V,
+// so that the pairs of neighbours never leave a lane.  All arithmetic in float from run-dtype inputs, one rounding.
+namespace {
+constexpr int kRopeNormWarps = 4;
+
+template <typename T, int V>
+__device__ __forceinline__ void load_elements(float (&v)[V], const T* __restrict__ p, int left) {
+    if constexpr (V == 4 && sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        v[0] = __uint_as_float(u.x << 16), v[1] = __uint_as_float(u.x & 0xffff0000u);
+        v[2] = __uint_as_float(u.y << 16), v[3] = __uint_as_float(u.y & 0xffff0000u);
+    } else if constexpr (V == 4) {
+        const float4 u = *reinterpret_cast<const float4*>(p);
+        v[0] = u.x, v[1] = u.y, v[2] = u.z, v[3] = u.w;
+    } else {
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = k < left ? to_float(p[k]) : 0.0f;
+    }
+}
+
+template <typename T, int V>
+__device__ __forceinline__ void store_elements_of(T* __restrict__ p, const float (&v)[V], int left) {
+    if constexpr (V == 4 && sizeof(T) == 2) {
+        __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3])};
+        *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(h);
+    } else if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+#pragma unroll
+        for (int k = 0; k < V; ++k)
+            if (k < left) p[k] = from_float<T>(v[k]);
+    }
+}
+
+// STEPS: how many times 32 V elements a head takes at most
+template <typename T, int V, int STEPS>
+__global__ void __launch_bounds__(kRopeNormWarps * 32)
+rope_norm_kv_kernel(const T* __restrict__ proj, int ld, T* __restrict__ out, const int* __restrict__ positions, const float* __restrict__ denom,
+                    float magnitude, int interleaved, int rotary_dim, const float* __restrict__ q_norm, const float* __restrict__ k_norm, int norm,
+                    float eps, int norm_width, const int* __restrict__ slot_mapping, T* __restrict__ kcache, T* __restrict__ vcache, int nh, int nkv,
+                    int dh, int page_size, int num_pages, int write, int to_cache, int keys_are_values, int heads_per_block) {
+    extern __shared__ float sm[];                                 // cosines and sines of the token's pairs, then a head's elements per warp
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int half = rotary_dim >> 1;
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, c;
+        sincosf(pos / denom[i], &sn, &c);
+        sm[2 * i] = c * magnitude;
+        sm[2 * i + 1] = sn * magnitude;
+    }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* sh = sm + rotary_dim + (size_t)warp * dh;
+    const int heads_in = nh + (keys_are_values ? 1 : 2) * nkv;
+    const int head_end = min(heads_in, ((int)blockIdx.y + 1) * heads_per_block);
+    int page = 0, off = 0;
+    bool slot_ok = false;
+    if (write && to_cache) {
+        const int slot = slot_mapping[t];
+        page = slot / page_size;
+        off = slot - page * page_size;
+        slot_ok = slot >= 0 && page < num_pages;                  // validated on the host; never write outside the cache
+    }
+    const T* row = proj + (size_t)t * ld;
+    T* orow = out + (size_t)t * (nh + 2 * nkv) * dh;
+    for (int head = (int)blockIdx.y * heads_per_block + warp; head < head_end; head += kRopeNormWarps) {
+        const bool is_q = head < nh, is_k = !is_q && head < nh + nkv;
+        if (!is_q && !write) continue;
+        float v[STEPS][V];
+#pragma unroll
+        for (int i = 0; i < STEPS; ++i) {
+            const int d = V * (lane + 32 * i);
+            if (d < dh) {
+                load_elements<T, V>(v[i], row + (size_t)head * dh + d, dh - d);
+            } else {
+#pragma unroll
+                for (int k = 0; k < V; ++k) v[i][k] = 0.0f;
+            }
+        }
+        const bool is_v = !is_q && !is_k;
+        const int kvh = is_q ? 0 : (is_k ? head - nh : head - nh - nkv);
+        if (is_v || (is_k && keys_are_values)) {
+            // the value: as projected
+            if (!to_cache) {
+                T* o = orow + (size_t)(nh + nkv + kvh) * dh;
+#pragma unroll
+                for (int i = 0; i < STEPS; ++i) {
+                    const int d = V * (lane + 32 * i);
+                    if (d < dh) store_elements_of<T, V>(o + d, v[i], dh - d);
+                }
+            } else if (slot_ok) {
+                T* dst = vcache + ((size_t)page * nkv + kvh) * dh * page_size + off;
+#pragma unroll
+                for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                    for (int k = 0; k < V; ++k) {
+                        const int d = V * (lane + 32 * i) + k;
+                        if (d < dh) dst[(size_t)d * page_size] = from_float<T>(v[i][k]);
+                    }
+            }
+            if (is_v) continue;
+        }
+        if (rotary_dim > 0) {
+            if (interleaved) {
+#pragma unroll
+                for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                    for (int k = 0; k < V; k += 2) {
+                        const int d = V * (lane + 32 * i) + k;
+                        if (d < rotary_dim) {
+                            const float a = v[i][k], b = v[i][k + 1], c = sm[d], sn = sm[d + 1];
+                            v[i][k] = a * c - b * sn;
+                            v[i][k + 1] = b * c + a * sn;
+                        }
+                    }
+            } else {
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                    for (int k = 0; k < V; ++k) {
+                        const int d = V * (lane + 32 * i) + k;
+                        if (d < rotary_dim) sh[d] = v[i][k];
+                    }
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                    for (int k = 0; k < V; ++k) {
+                        const int d = V * (lane + 32 * i) + k;
+                        if (d < rotary_dim) {
+                            const int j = d < half ? d : d - half;
+                            const float a = sh[j], b = sh[j + half], c = sm[2 * j], sn = sm[2 * j + 1];
+                            v[i][k] = d < half ? a * c - b * sn : b * c + a * sn;
+                        }
+                    }
+            }
+        }
+        if (norm) {
+            float q = 0.0f;
+#pragma unroll
+            for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                for (int k = 0; k < V; ++k) q = fmaf(v[i][k], v[i][k], q);
+            q = warp_sum(q);
+            const float rinv = 1.0f / sqrtf(q / (float)norm_width + eps);
+            const float* w = is_q ? q_norm : k_norm;
+#pragma unroll
+            for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                for (int k = 0; k < V; ++k) {
+                    const int d = V * (lane + 32 * i) + k;
+                    v[i][k] *= (w && d < dh) ? rinv * w[d] : rinv;
+                }
+        }
+        T* dst;
+        if (is_q || !to_cache) dst = orow + (size_t)head * dh;
+        else if (slot_ok) dst = kcache + (((size_t)page * nkv + kvh) * page_size + off) * dh;
+        else continue;
+#pragma unroll
+        for (int i = 0; i < STEPS; ++i) {
+            const int d = V * (lane + 32 * i);
+            if (d < dh) store_elements_of<T, V>(dst + d, v[i], dh - d);
+        }
+    }
+}
+
+// Two maps of attention over the same values: out[t, h] = (a1 - lambda a2) / sqrt(mean(.^2) + eps) * gain, times
+// sigmoid(gate) element by element if a gate is given.  att [T, 2 H dl]: head h's maps at columns 2 h dl and (2 h + 1) dl, dv of
+// their dl elements are real; a warp per (token, head).
+template <typename T, int V, int STEPS>
+__global__ void __launch_bounds__(256)
+map_difference_kernel(const T* __restrict__ att, int dl, const T* __restrict__ gate, int gate_ld, int gate_col, float lambda, float eps, float gain,
+                      T* __restrict__ out, int total, int H, int dv) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit >= total) return;
+    const int t = unit / H, h = unit - t * H;
+    const T* a = att + ((size_t)t * 2 * H + 2 * h) * dl;
+    const T* g = gate ? gate + (size_t)t * gate_ld + gate_col + (size_t)h * dv : nullptr;
+    float v[STEPS][V], gv[STEPS][V];
+    float q = 0.0f;
+#pragma unroll
+    for (int i = 0; i < STEPS; ++i) {
+        const int d = V * (lane + 32 * i);
+        float b[V];
+        if (d < dv) {
+            load_elements<T, V>(v[i], a + d, dv - d);
+            load_elements<T, V>(b, a + dl + d, dv - d);
+            if (g) load_elements<T, V>(gv[i], g + d, dv - d);
+        } else {
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[i][k] = b[k] = gv[i][k] = 0.0f;
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            v[i][k] = fmaf(-lambda, b[k], v[i][k]);
+            q = fmaf(v[i][k], v[i][k], q);
+        }
+    }
+    const float f = gain / sqrtf(warp_sum(q) / (float)dv + eps);
+    T* o = out + ((size_t)t * H + h) * dv;
+#pragma unroll
+    for (int i = 0; i < STEPS; ++i) {
+        const int d = V * (lane + 32 * i);
+        if (d < dv) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[i][k] = g ? v[i][k] * f / (1.0f + expf(-gv[i][k])) : v[i][k] * f;
+            store_elements_of<T, V>(o + d, v[i], dv - d);
+        }
+    }
+}
+}  // namespace
+
+LI_EXPORT int li_rope_norm_kv(const void* proj, int ld, void* out, int dtype, const int* positions, const float* denom, float magnitude, int interleaved,
+                              int rotary_dim, const float* q_norm, const float* k_norm, int norm, float eps, int norm_width,
+                              const int* slot_mapping, void* kcache, void* vcache, int T, int nh, int nkv, int dh, int page_size,
+                              int num_pages, int write, int to_cache, int keys_are_values, cudaStream_t stream) {
+    LI_REQUIRE(T >= 0 && nh > 0 && nkv > 0 && dh > 0 && page_size > 0, "rope_norm_kv: bad sizes");
+    LI_REQUIRE(ld >= (nh + (keys_are_values ? 1 : 2) * nkv) * dh, "rope_norm_kv: rows of %d elements are too short", ld);
+    LI_REQUIRE(dh <= 512, "rope_norm_kv: head_dim %d is larger than 512", dh);
+    LI_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= dh, "rope_norm_kv: rotary_dim %d must be even and at most head_dim %d", rotary_dim, dh);
+    LI_REQUIRE(rotary_dim == 0 || denom != nullptr, "rope_norm_kv: rotary_dim %d without denominators", rotary_dim);
+    LI_REQUIRE(!norm || (norm_width > 0 && norm_width <= dh), "rope_norm_kv: bad norm width %d", norm_width);
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "rope_norm_kv: unknown dtype %d", dtype);
+    LI_REQUIRE(proj != out, "rope_norm_kv: the output needs rows of its own");
+    if (T == 0) return 0;
+    const int heads = nh + (keys_are_values ? 1 : 2) * nkv;
+    // many tokens: four heads a warp (fewer, fuller blocks); few: one
+    const int per_block = T >= 64 ? 4 * kRopeNormWarps : kRopeNormWarps;
+    const dim3 grid(T, ceil_div(heads, per_block));
+    LI_REQUIRE(grid.y <= 65535, "rope_norm_kv: too many heads for one launch");
+    const size_t smem = ((size_t)rotary_dim + (interleaved ? 0 : (size_t)kRopeNormWarps * dh)) * sizeof(float);
+    const bool vec = dh % 4 == 0 && ld % 4 == 0 && ((uintptr_t)proj % 16) == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)kcache % 16) == 0;
+    cudaError_t e;
+#define LI_ROPE_NORM(TT, V_, S_)                                                                                                                      \
+    e = li_launch_pdl(rope_norm_kv_kernel<TT, V_, S_>, grid, dim3(kRopeNormWarps * 32), smem, stream, (const TT*)proj, ld, (TT*)out, positions, denom, magnitude, \
+                      interleaved, rotary_dim, q_norm, k_norm, norm, eps, norm_width, slot_mapping, (TT*)kcache, (TT*)vcache, nh, nkv, dh, page_size,   \
+                      num_pages, write, to_cache, keys_are_values, per_block)
+    if (dtype == LI_F32) {
+        if (vec && dh <= 128) LI_ROPE_NORM(float, 4, 1);
+        else if (vec) LI_ROPE_NORM(float, 4, 4);
+        else LI_ROPE_NORM(float, 2, 8);
+    } else {
+        if (vec && dh <= 128) LI_ROPE_NORM(bf16, 4, 1);
+        else if (vec) LI_ROPE_NORM(bf16, 4, 4);
+        else LI_ROPE_NORM(bf16, 2, 8);
+    }
+#undef LI_ROPE_NORM
+    if (e != cudaSuccess) return li_fail("rope_norm_kv: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("rope_norm_kv");
+}
+
+LI_EXPORT int li_map_difference(const void* att, int dtype, int dl, const void* gate, int gate_ld, int gate_col, float lambda, float eps, float gain,
+                                void* out, int T, int H, int dv, cudaStream_t stream) {
+    LI_REQUIRE(T >= 0 && H > 0 && dv > 0 && dl >= dv && dv <= 512, "map_difference: bad sizes H=%d dv=%d of %d", H, dv, dl);
+    LI_REQUIRE(gate == nullptr || (gate_col >= 0 && gate_col + H * dv <= gate_ld), "map_difference: gate columns from %d do not fit rows of %d", gate_col, gate_ld);
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "map_difference: unknown dtype %d", dtype);
+    if (T == 0) return 0;
+    const long long total = (long long)T * H;
+    LI_REQUIRE(total < (1LL << 31) - 8, "map_difference: too many (token, head) pairs");
+    const dim3 grid((unsigned)ceil_div_ll(total, 8));
+    const bool vec = dl % 4 == 0 && dv % 4 == 0 && gate_ld % 4 == 0 && gate_col % 4 == 0 && ((uintptr_t)att % 16) == 0 && ((uintptr_t)gate % 16) == 0 &&
+                     ((uintptr_t)out % 16) == 0;
+    cudaError_t e;
+#define LI_MAP_DIFF(TT, V_, S_)                                                                                                                   \
+    e = li_launch_pdl(map_difference_kernel<TT, V_, S_>, grid, dim3(256), 0, stream, (const TT*)att, dl, (const TT*)gate, gate_ld, gate_col, lambda, eps, \
+                      gain, (TT*)out, (int)total, H, dv)
+    if (dtype == LI_F32) {
+        if (vec && dv <= 128) LI_MAP_DIFF(float, 4, 1);
+        else if (vec) LI_MAP_DIFF(float, 4, 4);
+        else LI_MAP_DIFF(float, 2, 8);
+    } else {
+        if (vec && dv <= 128) LI_MAP_DIFF(bf16, 4, 1);
+        else if (vec) LI_MAP_DIFF(bf16, 4, 4);
+        else LI_MAP_DIFF(bf16, 2, 8);
+    }
+#undef LI_MAP_DIFF
+    if (e != cudaSuccess) return li_fail("map_difference: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("map_difference");
+}

@@ -227,8 +227,8 @@ def logit_cap(logits: torch.Tensor, cap: float) -> None:
     _check(library().li_logit_cap(_p(logits), _l(logits.numel()), _f(cap), _stream(logits)), "logit_cap")
 
 
-EPILOGUES = {None: 0, "swiglu": 1, "glu_clamped": 2}
-GATED = ("swiglu", "glu_clamped")
+EPILOGUES = {None: 0, "swiglu": 1, "glu_clamped": 2, "geglu": 3}
+GATED = ("swiglu", "glu_clamped", "geglu")
 
 
 def _linear_args(a, weight, bias, out, epilogue):
@@ -271,7 +271,8 @@ def linear(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], 
     ``epilogue="swiglu"`` (bfloat16 only): ``weight`` holds gate and up rows interleaved in
     groups of 8 (see :func:`interleave_gate_up`) and out[M, N / 2] = up * gate / (1 + exp(-gate)).
     ``epilogue="glu_clamped"`` with ``epilogue_params`` = float32 ``[limit, alpha]`` on the device: the same layout, and
-    out = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    out = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+    ``epilogue="geglu"``: the same layout, out = up * gelu(gate) with the tanh form of gelu."""
     M, N, Kd = _linear_args(a, weight, bias, out, epilogue)
     bias = _gated_params(epilogue, bias, epilogue_params)
     if M == 0:
@@ -443,7 +444,7 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                     old_lens: Optional[torch.Tensor] = None, singles: int = 0,
                     units: Optional[torch.Tensor] = None, unit_slots: Tuple[int, int] = (0, 0),
                     softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                    keep_first: int = 0, sinks: Optional[torch.Tensor] = None) -> None:
+                    keep_first: int = 0, sinks: Optional[torch.Tensor] = None, maps: int = 1) -> None:
     """Causal grouped-query attention of the step's tokens over the paged cache.
 
     Queries are the first ``num_heads * head_dim`` columns of ``qkv`` (already
@@ -462,10 +463,16 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     ``gate`` (run dtype ``[T, num_heads]``): head h's output is multiplied by ``sigmoid(gate[t, h])``.
     ``keep_first`` (with a window): the keys ``0 .. keep_first - 1`` stay visible behind the window, at their own positions.
     ``sinks`` (float32 ``[num_heads]``): ``exp(sinks[h])`` joins the denominator of head h's softmax once; it has no key
-    and no value and is not scaled."""
+    and no value and is not scaled.
+    ``maps`` > 1: a query row of ``head_dim`` elements stands for that many of the ``num_heads`` heads: ``qkv`` holds
+    ``num_heads / maps`` query rows, head h is part ``h % maps`` of row ``h // maps``; its scores take that part of the query
+    and the same part of the key, its values are the whole value row (several maps of attention over the same values)."""
     T = qkv.shape[0]
     S = ctx_lens.shape[0]
-    _need(qkv, "qkv", None, (T, (num_heads + 2 * num_kv_heads) * head_dim))
+    maps = int(maps)
+    if maps < 1 or num_heads % (maps * num_kv_heads) or head_dim % maps:
+        raise KernelError(f"{maps} maps of {num_heads} heads on {num_kv_heads} key/value heads of {head_dim} elements")
+    _need(qkv, "qkv", None, (T, (num_heads // maps + 2 * num_kv_heads) * head_dim))
     _need(out, "attention output", qkv.dtype, (T, num_heads * head_dim))
     _need(k_cache, "key cache", qkv.dtype)
     _need(v_cache, "value cache", qkv.dtype, (k_cache.shape[0], k_cache.shape[1], k_cache.shape[3], k_cache.shape[2]))
@@ -491,7 +498,8 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
             _p(q_start), _p(ctx_lens), _p(seq_of_token), _p(positions), _i(T), _i(S),
             _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(page_size), _i(pages), _f(scale),
             _i(0 if window is None else int(window)), _i(max_q_len), _i(max_ctx_len), _p(old_lens), _i(int(singles)),
-            _p(units), _i(int(unit_slots[0])), _i(int(unit_slots[1])), _f(float(softcap or 0.0)), _p(slopes), _p(gate), _i(int(keep_first or 0)), _p(sinks), _stream(out))
+            _p(units), _i(int(unit_slots[0])), _i(int(unit_slots[1])), _f(float(softcap or 0.0)), _p(slopes), _p(gate), _i(int(keep_first or 0)), _p(sinks), _i(maps),
+            _stream(out))
     if sinks is not None:
         _need(sinks, "softmax sinks", torch.float32, (num_heads,))
     if slopes is not None:
@@ -520,6 +528,14 @@ def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: f
     _need(gate_up, "gate_up")
     _need(out, "glu output", gate_up.dtype, (T, I2 // 2))
     _check(library().li_glu_clamped(_p(gate_up), _p(out), _i(_dt(out)), _i(T), _i(I2 // 2), _f(limit), _f(alpha), _stream(out)), "glu_clamped")
+
+
+def geglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
+    """out = up * gelu(gate), the tanh form of gelu, with gate_up = [gate | up] along the last axis."""
+    T, I2 = gate_up.shape
+    _need(gate_up, "gate_up")
+    _need(out, "geglu output", gate_up.dtype, (T, I2 // 2))
+    _check(library().li_geglu(_p(gate_up), _p(out), _i(_dt(out)), _i(T), _i(I2 // 2), _stream(out)), "geglu")
 
 
 def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor) -> None:
@@ -932,16 +948,18 @@ def gated_rmsnorm(y32: torch.Tensor, gate: torch.Tensor, gate_col: int, weight: 
 class RowSum:
     """An activation [T, H] that stands for ``sum_k rows[place_of[t * top + k]]`` (times ``weights[t, k]`` if given): what a
     mixture of experts leaves, until a kernel that consumes the sum takes it in (:func:`norm_add_norm`);
-    :meth:`materialize` adds the rows up with a kernel of its own (:func:`moe_combine`)."""
+    :meth:`materialize` adds the rows up with a kernel of its own (:func:`moe_combine`).  ``extra`` [T, H]: one more row per
+    token that joins the sum (a shared expert's output)."""
 
-    def __init__(self, rows: torch.Tensor, place_of: torch.Tensor, top: int, weights: Optional[torch.Tensor] = None) -> None:
-        self.rows, self.place_of, self.top, self.weights = rows, place_of, int(top), weights
+    def __init__(self, rows: torch.Tensor, place_of: torch.Tensor, top: int, weights: Optional[torch.Tensor] = None,
+                 extra: Optional[torch.Tensor] = None) -> None:
+        self.rows, self.place_of, self.top, self.weights, self.extra = rows, place_of, int(top), weights, extra
         self.shape = (place_of.numel() // self.top, rows.shape[1])
         self.dtype = rows.dtype
 
     def materialize(self) -> torch.Tensor:
         y = torch.empty(self.shape, dtype=self.rows.dtype, device=self.rows.device)
-        moe_combine(self.rows, self.place_of, self.weights, self.top, y)
+        moe_combine(self.rows, self.place_of, self.weights, self.top, y, extra=self.extra)
         return y
 
 
@@ -959,12 +977,14 @@ def norm_add_norm(x32: torch.Tensor, y, post: Optional[tuple], nxt: Optional[tup
     n_src, H = x32.shape
     _need(x32, "residual stream", torch.float32)
     R = n_src if rows is None else rows.shape[0]
-    places, top, y_weights = None, 0, None
+    places, top, y_weights, y_extra = None, 0, None, None
     if isinstance(y, RowSum):
         if H > 8192:
             y = y.materialize()
         else:
-            places, top, y_weights, y = y.place_of, y.top, y.weights, y.rows
+            places, top, y_weights, y_extra, y = y.place_of, y.top, y.weights, y.extra, y.rows
+            if y_extra is not None:
+                _need(y_extra, "a token's further row", y.dtype, (n_src, H))
             _need(y, "rows of the sublayer's output", None, (y.shape[0], H))
             _need(places, "places of a token's rows", torch.int32, (n_src * top,))
             if y_weights is not None:
@@ -987,7 +1007,18 @@ def norm_add_norm(x32: torch.Tensor, y, post: Optional[tuple], nxt: Optional[tup
     dt = _dt(y) if y is not None else _dt(out)
     _check(library().li_norm_add_norm(_p(x32), _p(y), _i(dt), _p(wp), _i(int(cp)), _f(ep), _p(wn), _i(int(cn)), _f(en),
                                       _p(out if nxt is not None else None), _p(rows), _i(R), _i(n_src), _i(H), _p(places), _i(top), _p(y_weights),
-                                      _stream(x32)), "norm_add_norm")
+                                      _p(y_extra), _stream(x32)), "norm_add_norm")
+
+
+def join_rows(x32: torch.Tensor, delta: Optional[torch.Tensor], x0: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[t] = [x32[t] (+ delta[t]) | x0[t]]`` in the run dtype: what a map of the stream beside the embedding output reads."""
+    T, H = x32.shape
+    _need(x32, "residual stream", torch.float32)
+    _need(x0, "embedding output", torch.float32, (T, H))
+    _need(out, "joined rows", None, (T, 2 * H))
+    if delta is not None:
+        _need(delta, "output to be added", out.dtype, (T, H))
+    _check(library().li_join_rows(_p(x32), _p(delta), _p(x0), _p(out), _i(_dt(out)), _i(T), _i(H), _stream(out)), "join_rows")
 
 
 def add_row(x32: torch.Tensor, row: torch.Tensor) -> None:
@@ -1069,6 +1100,57 @@ def conv_norm_rope_kv(proj: torch.Tensor, out: torch.Tensor, conv_w: Optional[to
         _p(q_norm), _p(k_norm), _f(eps), _i(int(norm_width)), _p(row_rinv), _p(positions), _p(denominators if rotary_dim else None), _i(rotary_dim),
         _p(slot_mapping), _p(k_cache), _p(v_cache), _i(T), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(page_size), _i(pages),
         _i(1 if write else 0), _i(1 if shift else 0), _i(1 if to_cache else 0), _i(out.shape[1]), _stream(out)), "conv_norm_rope_kv")
+
+
+def rope_norm_kv(proj: torch.Tensor, out: torch.Tensor, positions: torch.Tensor, denominators: Optional[torch.Tensor], rotary_dim: int,
+                 magnitude: float, interleaved: bool, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], norm: bool, eps: float,
+                 norm_width: int, slot_mapping: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, num_heads: int, num_kv_heads: int,
+                 head_dim: int, write: bool = True, to_cache: bool = True, keys_are_values: bool = False) -> None:
+    """What stands between a q|k|v product and attention when the norm comes behind the rotation: the first ``rotary_dim``
+    elements of every query and key head are rotated (pair i by ``position / denominators[i]``; ``interleaved``: the pair is
+    (2i, 2i + 1), else (i, i + rotary_dim / 2); cosines and sines times ``magnitude``), then (``norm``) the head is divided by
+    ``sqrt(sum x^2 / norm_width + eps)`` and multiplied by ``q_norm`` / ``k_norm`` [head_dim] if given.  Queries to ``out``
+    [T, (heads + 2 kv_heads) head_dim], keys and values into the paged cache.  ``keys_are_values``: ``proj`` holds q|k only and
+    a key head as projected, before rotation and norm, is the value.  ``to_cache`` false: keys and values go to their columns
+    of ``out`` instead (:func:`rope_kv_write` with ``rotary_dim`` 0 stores them from there)."""
+    T = proj.shape[0]
+    heads_in = num_heads + (1 if keys_are_values else 2) * num_kv_heads
+    _need(proj, "q|k|v projection", None, (T, proj.shape[1]))
+    if proj.shape[1] < heads_in * head_dim:
+        raise KernelError(f"rope_norm_kv: rows of {proj.shape[1]} elements for {heads_in} heads of {head_dim}")
+    _need(out, "q|k|v output", proj.dtype, (T, (num_heads + 2 * num_kv_heads) * head_dim))
+    for t, n in ((q_norm, "query norm weight"), (k_norm, "key norm weight")):
+        if t is not None:
+            _need(t, n, torch.float32, (head_dim,))
+    _need(positions, "positions", torch.int32, (T,))
+    if rotary_dim:
+        _need(denominators, "rope denominators", torch.float32, (rotary_dim // 2,))
+    _need(slot_mapping, "slot mapping", torch.int32, (T,))
+    _need(k_cache, "key cache", proj.dtype)
+    pages, nkv, page_size, dh = k_cache.shape
+    _need(v_cache, "value cache", proj.dtype, (pages, nkv, dh, page_size))
+    if nkv != num_kv_heads or dh != head_dim:
+        raise KernelError(f"cache of {nkv} heads x {dh} does not match {num_kv_heads} x {head_dim}")
+    _check(library().li_rope_norm_kv(
+        _p(proj), _i(proj.shape[1]), _p(out), _i(_dt(proj)), _p(positions), _p(denominators if rotary_dim else None), _f(float(magnitude)),
+        _i(1 if interleaved else 0), _i(rotary_dim), _p(q_norm), _p(k_norm), _i(1 if norm else 0), _f(eps), _i(int(norm_width)), _p(slot_mapping),
+        _p(k_cache), _p(v_cache), _i(T), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(page_size), _i(pages), _i(1 if write else 0),
+        _i(1 if to_cache else 0), _i(1 if keys_are_values else 0), _stream(out)), "rope_norm_kv")
+
+
+def map_difference(att: torch.Tensor, head_dim: int, gate: Optional[torch.Tensor], gate_col: int, mix: float, eps: float, gain: float,
+                   out: torch.Tensor, num_heads: int, value_dim: int) -> None:
+    """Two maps of attention over the same values: ``o = a1 - mix * a2`` per head, ``a1`` and ``a2`` the first ``value_dim`` of the
+    ``head_dim`` columns of heads 2h and 2h + 1 of ``att`` [T, 2 num_heads head_dim]; ``out[t, h] = o / sqrt(mean(o^2) + eps) *
+    gain``, times ``sigmoid`` of the gate's elements (columns of ``gate`` from ``gate_col``; None: no gate), all in float32."""
+    T = att.shape[0]
+    _need(att, "attention output of both maps", None, (T, 2 * num_heads * head_dim))
+    _need(out, "difference of the maps", att.dtype, (T, num_heads * value_dim))
+    if gate is not None:
+        _need(gate, "gate", att.dtype, (T, gate.shape[1]))
+    _check(library().li_map_difference(_p(att), _i(_dt(att)), _i(int(head_dim)), _p(gate), _i(gate.shape[1] if gate is not None else 0), _i(int(gate_col)),
+                                       _f(float(mix)), _f(float(eps)), _f(float(gain)), _p(out), _i(T), _i(num_heads), _i(int(value_dim)),
+                                       _stream(out)), "map_difference")
 
 
 def latent_rope_post(low: torch.Tensor, col_c: int, col_r: int, q: torch.Tensor, dim: int, weight: torch.Tensor, eps: float,
@@ -1230,15 +1312,19 @@ def moe_gather(h: torch.Tensor, pair_at: torch.Tensor, weights: Optional[torch.T
     _check(library().li_moe_gather(_p(h), _i(_dt(h)), _p(pair_at), _p(weights), _i(n), _i(top), _i(H), _p(out), _stream(out)), "moe_gather")
 
 
-def moe_combine(rows: torch.Tensor, place_of: torch.Tensor, weights: Optional[torch.Tensor], top: int, y: torch.Tensor) -> None:
-    """``y[t] = sum_k rows[place_of[t * top + k]]`` (times ``weights[t, k]`` if given), summed in float32 in the order of k."""
+def moe_combine(rows: torch.Tensor, place_of: torch.Tensor, weights: Optional[torch.Tensor], top: int, y: torch.Tensor,
+                extra: Optional[torch.Tensor] = None) -> None:
+    """``y[t] = sum_k rows[place_of[t * top + k]]`` (times ``weights[t, k]`` if given), summed in float32 in the order of k, plus
+    ``extra[t]`` if given."""
     T, H = y.shape
     _need(rows, "sorted rows", None, (rows.shape[0], H))
     _need(place_of, "place of pair", torch.int32, (T * top,))
     if weights is not None:
         _need(weights, "expert weights", torch.float32, (T, top))
     _need(y, "feed-forward output", rows.dtype)
-    _check(library().li_moe_combine(_p(rows), _i(_dt(rows)), _p(place_of), _p(weights), _i(T), _i(top), _i(H), _p(y), _stream(y)), "moe_combine")
+    if extra is not None:
+        _need(extra, "a token's further row", rows.dtype, (T, H))
+    _check(library().li_moe_combine(_p(rows), _i(_dt(rows)), _p(place_of), _p(weights), _p(extra), _i(T), _i(top), _i(H), _p(y), _stream(y)), "moe_combine")
 
 
 def argmax(logits: torch.Tensor, out: torch.Tensor) -> None:
@@ -1343,7 +1429,7 @@ _TIMED = ("embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add
           "rope_kv_write", "linear_rope_kv", "rope_table", "paged_attention", "swiglu", "argmax", "sample", "gather_rows", "scale_inplace",
           "logit_cap", "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift",
           "ssm_scan", "decay_scan", "gated_rmsnorm", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route",
-          "moe_sort", "moe_gather", "moe_combine")
+          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference")
 if profile.enabled:
     for _name in _TIMED:
         globals()[_name] = profile.wrap(_name, globals()[_name])

@@ -56,6 +56,7 @@ class DecoderModel:
         # what else joins the stream after the embedding (an embedding of token pairs); their caches come behind the schedule's
         self.stream_inputs = [STREAM_INPUTS.build(p, prefix, self.dtype, self.device) for p, prefix in spec.stream_inputs]
         self.stream_tables: Dict[str, torch.Tensor] = {}      # vectors that schedule entries add to the stream (ScheduleEntry.add)
+        self.stream_maps: Dict[str, torch.Tensor] = {}        # maps of the stream beside the embedding output (ScheduleEntry.join)
         self.embedding: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
         self.head_is_tied = False
@@ -73,6 +74,8 @@ class DecoderModel:
             out.extend(part.all_params())
         for name, rows in s.stream_tables.items():
             out.append(ParamSpec(name, (int(rows), s.hidden_size), role="vector", std=0.02))
+        for name in s.stream_maps:
+            out.append(ParamSpec(name, (s.hidden_size, 2 * s.hidden_size), role="matrix"))
         for b in self.blocks:
             out.extend(b.all_params())
         out.extend(self.final_norm.all_params())
@@ -91,6 +94,7 @@ class DecoderModel:
         for part in self.stream_inputs:
             part.bind_all(tensors)
         self.stream_tables = {name: tensors.pop(name) for name in s.stream_tables}
+        self.stream_maps = {name: tensors.pop(name) for name in s.stream_maps}
         for b in self.blocks:
             b.bind_all(tensors)
         self.final_norm.bind_all(tensors)
@@ -153,8 +157,17 @@ class DecoderModel:
             x32 = xs
         carry = None
         last = len(s.schedule) - 1
+        # (the blocks change the stream in place: entries that read the embedding output anew get a copy of it)
+        x0 = x32.clone() if any(e.join is not None for e in s.schedule) else None
         for i, e in enumerate(s.schedule):
-            if e.add is not None:
+            if e.join is not None:
+                # the stream beside the embedding output through a map, and the entry's vector as that product's bias; what the
+                # block before still holds goes in on the way
+                both = torch.empty((ctx.num_tokens, 2 * s.hidden_size), dtype=self.dtype, device=self.device)
+                K.join_rows(x32, carry.delta if carry is not None else None, x0, both)
+                carry = None
+                K.linear(both, self.stream_maps[e.join], self.stream_tables[e.add[0]][int(e.add[1])] if e.add is not None else None, x32)
+            elif e.add is not None:
                 # a vector joins the stream before this block: whatever the block before still holds goes in first
                 if carry is not None and carry.delta is not None:
                     K.residual_add(x32, carry.delta)
@@ -162,7 +175,8 @@ class DecoderModel:
                 K.add_row(x32.view(-1, s.hidden_size), self.stream_tables[e.add[0]][int(e.add[1])])
             # a block is told the first norm of the block that runs next, so that it can apply it in its own tail (not
             # when something else is added to the stream in between)
-            next_entry = self.blocks[s.schedule[i + 1].block].entry() if i < last and s.schedule[i + 1].add is None else None
+            follows = s.schedule[i + 1] if i < last else None
+            next_entry = self.blocks[follows.block].entry() if follows is not None and follows.add is None and follows.join is None else None
             x32, carry = self.blocks[e.block].forward(x32, ctx, caches[i], carry, next_entry)
             if self.observer is not None:
                 self.observer(i, x32, carry)

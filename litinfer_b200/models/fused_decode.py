@@ -71,7 +71,8 @@ def describe(model) -> Optional[List[dict]]:
     spec = model.spec
     if model.dtype != torch.bfloat16 or model.device.type != "cuda":
         return None
-    if spec.position is not None or spec.embedding_scale is not None or spec.logit_cap is not None:
+    if spec.position is not None or spec.embedding_scale is not None or spec.logit_cap is not None or spec.stream_inputs \
+            or any(e.add is not None or e.join is not None for e in spec.schedule):
         return None
     final = model.final_norm.fused_decode()
     if final is None or model.lm_head is None or model.lm_head.dtype != torch.bfloat16:

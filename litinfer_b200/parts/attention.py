@@ -34,7 +34,14 @@ Further options of the spec, all off by default:
 * ``keep_first`` (with a window): the first keys of a sequence stay visible behind the window, at their own positions;
 * ``shared_kv`` true: the layer has no keys and values of its own (no such tensors): it projects queries only and reads
   the cache that another layer's entry wrote (the schedule entry names it with ``cache_from``), keys as that layer
-  normalised and rotated them.  Head counts and sizes are that layer's.
+  normalised and rotated them.  Head counts and sizes are that layer's;
+* ``norm_after`` (a mapping with ``eps``): queries and keys are divided by their root mean square per head behind the rotation,
+  without a weight;
+* ``keys_are_values`` true: the layer has no value map; a key as projected, before rotation and norm, is its value too;
+* ``sink`` (a tensor's name below the prefix): a learned number per head whose exponential joins the softmax's denominator.
+
+A position part that pairs neighbours or carries a magnitude (:class:`~litinfer_b200.parts.base.Rotary`) goes with the last
+three: rotation, norm, values and the cache write are then one kernel behind the product (``kernels.rope_norm_kv``).
 """
 
 from __future__ import annotations
@@ -86,6 +93,15 @@ class PagedAttention(Mixer):
         stems = [names.get("q", "q_proj"), names.get("k", "k_proj"), names.get("v", "v_proj")]
         self.real_outs = (self.num_heads * self.qk_dim, self.num_kv_heads * self.qk_dim, self.num_kv_heads * self.value_dim)
         self.head_shapes = ((self.num_heads, self.qk_dim), (self.num_kv_heads, self.qk_dim), (self.num_kv_heads, self.value_dim))
+        norm_after = spec.get("norm_after")
+        self.norm_after_eps = float(norm_after["eps"]) if norm_after else None
+        self.keys_are_values = bool(spec.get("keys_are_values", False))
+        self.sink_name = prefix + str(spec["sink"]) if spec.get("sink") else None
+        self.sinks = None
+        if self.keys_are_values:
+            if self.value_dim != self.qk_dim:
+                raise ValueError(f"values that are the keys have the keys' size {self.qk_dim}, not {self.value_dim}")
+            stems, self.real_outs, self.head_shapes = stems[:2], self.real_outs[:2], self.head_shapes[:2]
         if self.norm_whole and self.taps >= 1:
             raise ValueError("a norm over the whole projection together with a convolution is not supported")
         if self.shared_kv:
@@ -99,8 +115,12 @@ class PagedAttention(Mixer):
         self.gate = FusedLinear(prefix, [gate], self.hidden, [self.num_heads], False, dtype, suffixes=suffixes) if gate else None
         position = spec.get("position")
         self.position = POSITIONS.build(position, prefix, dtype, device, head_dim=self.head_dim) if position is not None else None
-        if getattr(self.position, "interleaved", False) or getattr(self.position, "magnitude", 1.0) != 1.0:
-            raise ValueError(f"attention at {prefix!r}: its kernels rotate halves of a head with plain cosines and sines")
+        # rotation first, a norm behind it, keys that are values: a kernel of its own behind the product
+        self.rotate_apart = (self.keys_are_values or self.norm_after_eps is not None or getattr(self.position, "interleaved", False)
+                             or getattr(self.position, "magnitude", 1.0) != 1.0)
+        if self.rotate_apart and (self.taps >= 1 or qk_norm or self.shared_kv or self.value_dim != self.qk_dim):
+            raise ValueError(f"attention at {prefix!r}: pairs of neighbours, a magnitude, a norm behind the rotation and keys as values do not go "
+                             "with a convolution, a norm before the rotation, shared keys or values of another size")
         self.conv_names = [prefix + n + str(spec.get("conv_suffix", ".conv")) for n in stems] if self.taps >= 1 else []
         self.norm_names = [prefix + str(qk_norm[n]) for n in (("q",) if self.shared_kv else ("q", "k"))] if qk_norm else []
         self.conv_weight = self.q_norm = self.k_norm = None
@@ -116,6 +136,8 @@ class PagedAttention(Mixer):
             out += [ParamSpec(n, (o,), role="vector", init="ones_normal") for n, o in zip(self.norm_names, self.real_outs)]
         else:
             out += [ParamSpec(n, (self.qk_dim,), role="vector", init="ones_normal") for n in self.norm_names]
+        if self.sink_name:
+            out.append(ParamSpec(self.sink_name, (self.num_heads,), role="vector", std=0.5))
         return out
 
     def parts(self):
@@ -126,6 +148,8 @@ class PagedAttention(Mixer):
         self.out.bind(tensors)
         if self.gate is not None:
             self.gate.bind(tensors)
+        if self.sink_name:
+            self.sinks = tensors.pop(self.sink_name)
         conv = [tensors.pop(n) for n in self.conv_names]
         norms = [tensors.pop(n) for n in self.norm_names]
         if self.head_dim != self.qk_dim or self.head_dim != self.value_dim:
@@ -188,7 +212,8 @@ class PagedAttention(Mixer):
         rope = self.position.fused_decode() if self.position is not None else None
         if type(self) is not PagedAttention or rope is None or rope["rotary_dim"] != self.head_dim or self.out.bias is not None:
             return None
-        if self.softcap or self.slopes is not None or self.gate is not None or self.value_dim != self.qk_dim or self.post or self.keep_first or self.shared_kv:
+        if self.softcap or self.slopes is not None or self.gate is not None or self.value_dim != self.qk_dim or self.post or self.keep_first or self.shared_kv \
+                or self.rotate_apart or self.sink_name:
             return None
         return {"w_qkv": self.qkv.weight, "b_qkv": self.qkv.bias, "w_o": self.out.weight, "hidden": self.hidden, "heads": self.num_heads,
                 "kv_heads": self.num_kv_heads, "head_dim": self.head_dim, "scale": self.scale, "window": self.window,
@@ -210,7 +235,20 @@ class PagedAttention(Mixer):
         rot = self.position.rotary(ctx) if self.position is not None else None
         if self.shared_kv and (cache is None or cache.kind != "paged" or cache.writes):
             raise ValueError(f"attention at {self.prefix!r} shares another layer's keys and values: its schedule entry must name that layer's entry (cache_from)")
-        if self.post and (self.norm_whole or self.shared_kv):
+        if self.rotate_apart:
+            # projection; then rotation, norm, values and the cache write as one kernel (in a long step the page-wise writer
+            # stores keys and values)
+            proj = self.qkv(h)
+            T = proj.shape[0]
+            qkv = torch.empty((T, self.qkv_width), dtype=self.dtype, device=proj.device)
+            long_step = T >= self.CACHE_WRITE_APART
+            K.rope_norm_kv(proj, qkv, ctx.positions, rot.denominators if rot else None, rot.rotary_dim if rot else 0, rot.magnitude if rot else 1.0,
+                           bool(rot and rot.interleaved), None, None, self.norm_after_eps is not None, self.norm_after_eps or 0.0, self.qk_dim,
+                           view.slot_mapping, cache.k, cache.v, self.num_heads, self.num_kv_heads, self.head_dim, cache.writes,
+                           to_cache=not long_step, keys_are_values=self.keys_are_values)
+            if long_step and cache.writes:
+                K.rope_kv_write(qkv, ctx.positions, None, 0, view.slot_mapping, cache.k, cache.v, self.num_heads, self.num_kv_heads, self.head_dim, True)
+        elif self.post and (self.norm_whole or self.shared_kv):
             # projection; the factors of the norms over the whole of q and of k; then norm, rotation and the cache write as one
             # kernel.  A layer without keys and values of its own projects queries only, into rows that attention reads as q|k|v.
             proj = self.qkv(h)
@@ -261,5 +299,6 @@ class PagedAttention(Mixer):
             qkv, o, cache.k, cache.v, view.block_table, ctx.q_start, ctx.ctx_lens, ctx.seq_of_token, ctx.positions,
             self.num_heads, self.num_kv_heads, self.head_dim, self.scale, self.window,
             ctx.max_q_len, ctx.max_ctx_len, old_lens=ctx.old_lens, singles=ctx.num_single,
-            units=ctx.attn_units, unit_slots=ctx.attn_unit_slots, softcap=self.softcap, slopes=self.slopes, gate=gate, keep_first=self.keep_first)
+            units=ctx.attn_units, unit_slots=ctx.attn_unit_slots, softcap=self.softcap, slopes=self.slopes, gate=gate, keep_first=self.keep_first,
+            sinks=self.sinks)
         return o

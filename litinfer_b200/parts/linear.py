@@ -84,7 +84,7 @@ class GateUpLinear(FusedLinear):
 
     def __init__(self, prefix, gate_name, up_name, in_features, intermediate, dtype, std=0.02, suffixes=(".weight", ".bias"),
                  epilogue="swiglu", epilogue_params=None):
-        """``epilogue``: the gated activation, "swiglu" or "glu_clamped" (with ``epilogue_params`` = (limit, alpha))."""
+        """``epilogue``: the gated activation, "swiglu", "geglu" or "glu_clamped" (with ``epilogue_params`` = (limit, alpha))."""
         super().__init__(prefix, [gate_name, up_name], in_features, [intermediate, intermediate], False, dtype, std, suffixes)
         self.intermediate = int(intermediate)
         self.epilogue = epilogue
@@ -112,6 +112,8 @@ class GateUpLinear(FusedLinear):
             act = torch.empty((both.shape[0], self.intermediate), dtype=self.dtype, device=both.device)
             if self.epilogue == "swiglu":
                 K.swiglu(both, act)
+            elif self.epilogue == "geglu":
+                K.geglu(both, act)
             else:
                 K.glu_clamped(both, act, *self.epilogue_values)
         return act

@@ -47,6 +47,38 @@ class SwiGLU(FeedForward):
         return tail.apply_linear(self.down, self.gate_up.activation(h))
 
 
+@FEED_FORWARDS.register("geglu")
+class GEGLU(FeedForward):
+    """Dense gated feed-forward with gelu in place of silu: down(gelu(gate(h)) * up(h)), the tanh form of gelu,
+    ``0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))``; no biases.  gate and up are one product; the activation is computed in
+    float32 and rounded once; in bfloat16 it is the epilogue of that product."""
+
+    takes_deferred = True            # the gate|up product applies the factor
+
+    def __init__(self, spec, prefix, dtype, device):
+        super().__init__(spec, prefix, dtype, device)
+        self.hidden = int(spec["hidden_size"])
+        self.intermediate = int(spec["intermediate_size"])
+        names = spec.get("names", {})
+        suffixes = tuple(spec.get("suffixes", (".weight", ".bias")))
+        self.gate_up = GateUpLinear(prefix, names.get("gate", "gate_proj"), names.get("up", "up_proj"), self.hidden, self.intermediate, dtype,
+                                    suffixes=suffixes, epilogue="geglu")
+        self.down = FusedLinear(prefix, [names.get("down", "down_proj")], self.intermediate, [self.hidden], False, dtype, suffixes=suffixes)
+
+    def params(self) -> List[ParamSpec]:
+        return self.gate_up.params() + self.down.params()
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.gate_up.bind(tensors)
+        self.down.bind(tensors)
+
+    def forward(self, h, ctx):
+        return self.down(self.gate_up.activation(h))
+
+    def forward_into(self, h, ctx, tail):
+        return tail.apply_linear(self.down, self.gate_up.activation(h))
+
+
 @FEED_FORWARDS.register("clamped_glu")
 class ClampedGLU(FeedForward):
     """A gated feed-forward with bounded operands: g = min(gate(h), limit), u = clamp(up(h), -limit, limit),

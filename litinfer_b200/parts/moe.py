@@ -14,6 +14,10 @@ choice scores are ``s + correction`` (a stored vector); the outputs form ``group
 score is its largest choice score, and only outputs of the ``keep_groups`` best groups can be chosen; the ``top`` largest
 choice scores choose; the weights are the chosen outputs' s divided by their sum (+ 1e-20), times ``route_scale``.  The last
 ``identity`` outputs are identity experts: they have no tensors and their output is the input h itself (times the weight).
+``scoring`` "softmax" (with ``renormalize``): the same without correction, groups and identity experts: ``s = softmax(z)`` over all
+experts, the ``top`` largest choose, the weights are the chosen experts' s divided by their sum (+ 1e-20).
+``shared`` (the spec of a dense feed-forward, of another kind and size if it likes; its tensors below ``names["shared"]``): one more
+feed-forward that every token takes; its output joins the sum of the chosen experts' as one more row.
 ``activation`` "glu_clamped" (with ``limit``, ``alpha``): ``g = min(W_gate u, limit)``, ``up = clamp(W_up u, -limit, limit)``,
 the expert's inner activation is ``g sigmoid(alpha g) (up + 1)`` instead of ``silu(gate) up``.
 
@@ -53,11 +57,13 @@ class RoutedExperts(FeedForward):
         if not 0 < self.top <= self.experts + int(spec.get("identity") or 0):
             raise ValueError(f"{self.top} of {self.experts} experts")
         self.scoring = str(spec.get("scoring", "sigmoid"))
-        if self.scoring not in ("sigmoid", "softmax_chosen", "softmax_grouped"):
-            raise ValueError(f"routing by '{spec.get('scoring')}' is not supported (sigmoid, softmax_chosen, softmax_grouped)")
+        if self.scoring not in ("sigmoid", "softmax_chosen", "softmax_grouped", "softmax"):
+            raise ValueError(f"routing by '{spec.get('scoring')}' is not supported (sigmoid, softmax_chosen, softmax_grouped, softmax)")
         self.renormalize = bool(spec.get("renormalize", False))
-        if self.renormalize and self.scoring != "softmax_grouped":
-            raise ValueError("renormalised routing weights are not supported")
+        if self.renormalize and self.scoring not in ("softmax_grouped", "softmax"):
+            raise ValueError(f"renormalised routing weights go with softmax scores over all experts, not with '{self.scoring}'")
+        if self.scoring == "softmax" and not self.renormalize:
+            raise ValueError("scoring 'softmax' renormalises the chosen scores (renormalize)")
         self.weight_on = str(spec.get("weight_on", "output"))
         if self.weight_on not in ("input", "output"):
             raise ValueError(f"weight_on must be 'input' or 'output', got {self.weight_on!r}")
@@ -94,6 +100,11 @@ class RoutedExperts(FeedForward):
         # the gated activation is the epilogue of the grouped product (the [rows, 2 F] product never goes to memory)
         self.fused_activation = dtype == torch.bfloat16 and self.intermediate % 8 == 0 and self.hidden % 8 == 0
         self.activation_params = None                        # (limit, alpha) on the device, for the epilogue
+        shared = spec.get("shared")
+        self.shared = FEED_FORWARDS.build(shared, prefix + n.get("shared", "shared."), dtype, device) if shared is not None else None
+
+    def parts(self):
+        return [self.shared] if self.shared is not None else []
 
     def params(self) -> List[ParamSpec]:
         out = self.router.params()
@@ -125,8 +136,14 @@ class RoutedExperts(FeedForward):
     def forward(self, h, ctx):
         return self.forward_rows(h, ctx).materialize()
 
+    def forward_into(self, h, ctx, tail):
+        rows = self.forward_rows(h, ctx)
+        # (a norm that says what it is takes the sum in with its pass over the stream)
+        return tail.apply(rows if hasattr(tail.norm, "statistics") else rows.materialize())
+
     def forward_rows(self, h, ctx) -> "K.RowSum":
         T = h.shape[0]
+        shared = self.shared.forward(h, ctx) if self.shared is not None else None
         E, top, F = self.experts, self.top, self.intermediate
         n_out = self.outputs                                   # experts and identity experts: what the router chooses among
         dev = h.device
@@ -135,6 +152,8 @@ class RoutedExperts(FeedForward):
         weights = torch.empty((T, top), dtype=torch.float32, device=dev)
         if self.scoring == "softmax_grouped":
             K.moe_route_grouped(logits, self.correction, top, self.groups, self.keep_groups, self.route_scale, ids, weights)
+        elif self.scoring == "softmax":
+            K.moe_route_grouped(logits, None, top, 1, 1, 1.0, ids, weights)
         else:
             K.moe_route(logits, top, ids, weights, scoring=self.scoring)
         # a step of many tokens: every expert's run of rows starts at a multiple of 128, so that the products run on
@@ -163,4 +182,4 @@ class RoutedExperts(FeedForward):
             else:
                 K.glu_clamped(both, act, self.limit, self.alpha)
         K.grouped_linear(act, self.down, rows, expert_offsets, tile_group=tiles)
-        return K.RowSum(rows, place_of, top, None if on_input else weights)
+        return K.RowSum(rows, place_of, top, None if on_input else weights, extra=shared)

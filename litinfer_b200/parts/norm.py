@@ -69,6 +69,10 @@ class RMSNorm(Norm):
 
     def add_forward(self, x32, delta):
         out = torch.empty(x32.shape, dtype=self.dtype, device=x32.device)
+        if isinstance(delta, K.RowSum):
+            # a token's experts' rows: summed inside the pass over the stream
+            K.norm_add_norm(x32, delta, None, self.statistics(), out)
+            return out
         K.add_rmsnorm(x32, delta, self.weight, self.eps, out)
         return out
 

@@ -65,7 +65,20 @@ def linear(a, weight, bias, out, epilogue=None, row_scale=None, epilogue_params=
         y = y.view(M, N // 16, 2, 8)
         g, u = torch.clamp(y[:, :, 0, :], max=limit), torch.clamp(y[:, :, 1, :], min=-limit, max=limit)
         y = (g * torch.sigmoid(alpha * g) * (u + 1.0)).reshape(M, N // 2)
+    elif epilogue == "geglu":
+        M, N = y.shape
+        y = y.view(M, N // 16, 2, 8)
+        y = (_gelu(y[:, :, 0, :]) * y[:, :, 1, :]).reshape(M, N // 2)
     _store(out, y)
+
+
+def _gelu(z):
+    return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def geglu(gate_up, out):
+    g, u = gate_up.float().chunk(2, dim=-1)
+    _store(out, _gelu(g) * u)
 
 
 def _factor(row_scale):
@@ -144,15 +157,25 @@ def rope_table(positions, denominators, out):
     out[..., 1] = torch.sin(phi)
 
 
+def _query_heads(qkv, num_heads, head_dim, maps):
+    """[T, num_heads, head_dim]: with maps > 1 a query row stands for that many heads, each with a part of it (zeros elsewhere)."""
+    T, part = qkv.shape[0], head_dim // maps
+    rows = qkv[:, :num_heads // maps * head_dim].reshape(T, num_heads // maps, head_dim).float()
+    q = torch.zeros(T, num_heads // maps, maps, head_dim, dtype=torch.float32, device=qkv.device)
+    for m in range(maps):
+        q[:, :, m, m * part:(m + 1) * part] = rows[..., m * part:(m + 1) * part]
+    return q.reshape(T, num_heads, head_dim)
+
+
 def paged_attention(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, seq_of_token, positions,
                     num_heads, num_kv_heads, head_dim, scale, window, max_q_len, max_ctx_len, implementation=None, old_lens=None, singles=0,
-                    units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None):
+                    units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None, maps=1):
     # old_lens only tells a kernel which keys it may read early, singles which kernel takes which sequence, units how a
     # kernel shares its work out; the result does not depend on them
     T = qkv.shape[0]
     page_size = k_cache.shape[2]
     group = num_heads // num_kv_heads
-    q = qkv[:, :num_heads * head_dim].reshape(T, num_heads, head_dim).float()
+    q = _query_heads(qkv, num_heads, head_dim, maps)
     res = torch.zeros(T, num_heads, head_dim, dtype=torch.float32, device=qkv.device)
     seqs = seq_of_token.tolist()
     poss = positions.tolist()
@@ -184,14 +207,14 @@ def paged_attention(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, 
 
 def paged_attention_dense(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, seq_of_token, positions,
                           num_heads, num_kv_heads, head_dim, scale, window, max_q_len, max_ctx_len, implementation=None, old_lens=None,
-                          singles=0, units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None):
+                          singles=0, units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None, maps=1):
     """The same formula as :func:`paged_attention`, a sequence at a time instead of a token and a head at a time (for
     contexts of thousands of keys): scores of all the sequence's tokens against all its keys in float32, keys outside
     [p - window + 1, p] masked, softmax, weighted sum."""
     T = qkv.shape[0]
     page_size = k_cache.shape[2]
     group = num_heads // num_kv_heads
-    q = qkv[:, :num_heads * head_dim].reshape(T, num_heads, head_dim).float()
+    q = _query_heads(qkv, num_heads, head_dim, maps)
     res = torch.zeros(T, num_heads, head_dim, dtype=torch.float32, device=qkv.device)
     starts, lens = q_start.tolist(), ctx_lens.tolist()
     for s, c in enumerate(lens):
@@ -243,11 +266,18 @@ def norm_add_norm(x32, y, post, nxt, out, rows=None):
     if hasattr(y, "place_of"):                           # a sum of rows (kernels.RowSum), taken in float32
         T, H = x32.shape
         r = y.rows[y.place_of.long()].float().view(T, y.top, H)
+        extra = y.extra
         y = (r * y.weights[:, :, None] if y.weights is not None else r).sum(1)
+        if extra is not None:
+            y = y + extra.float()
     if y is not None:
         x32.add_(_norm_of(y, post) if post is not None else y.float())
     if nxt is not None:
         _store(out, _norm_of(x32 if rows is None else x32[rows.long()], nxt))
+
+
+def join_rows(x32, delta, x0, out):
+    _store(out, torch.cat([x32 + delta.float() if delta is not None else x32, x0], dim=-1))
 
 
 def add_row(x32, row):
@@ -321,6 +351,55 @@ def conv_norm_rope_kv(proj, out, conv_w, state, state_off, q_start, seq_of_token
     v_cache[page, :, :, off] = v
 
 
+def rope_norm_kv(proj, out, positions, denominators, rotary_dim, magnitude, interleaved, q_norm, k_norm, norm, eps, norm_width, slot_mapping,
+                 k_cache, v_cache, num_heads, num_kv_heads, head_dim, write=True, to_cache=True, keys_are_values=False):
+    T = proj.shape[0]
+    q_dim, kv_dim = num_heads * head_dim, num_kv_heads * head_dim
+
+    def shape(x, weight):
+        x = x.clone()
+        if rotary_dim:
+            phi = positions.float()[:, None] / denominators[None, :]
+            cos, sin = (torch.cos(phi) * magnitude)[:, None, :], (torch.sin(phi) * magnitude)[:, None, :]
+            half = rotary_dim // 2
+            first = slice(0, rotary_dim, 2) if interleaved else slice(0, half)
+            second = slice(1, rotary_dim, 2) if interleaved else slice(half, rotary_dim)
+            a, b = x[..., first].clone(), x[..., second].clone()
+            x[..., first] = a * cos - b * sin
+            x[..., second] = b * cos + a * sin
+        if norm:
+            x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / norm_width + eps)
+            if weight is not None:
+                x = x * weight
+        return x
+
+    u = proj.float()
+    out[:, :q_dim] = shape(u[:, :q_dim].reshape(T, num_heads, head_dim), q_norm).reshape(T, q_dim).to(out.dtype)
+    if not write:
+        return
+    raw = u[:, q_dim:q_dim + kv_dim].reshape(T, num_kv_heads, head_dim)
+    k = shape(raw, k_norm).to(out.dtype)
+    v = (raw if keys_are_values else u[:, q_dim + kv_dim:q_dim + 2 * kv_dim].reshape(T, num_kv_heads, head_dim)).to(out.dtype)
+    if not to_cache:
+        out[:, q_dim:q_dim + kv_dim] = k.reshape(T, kv_dim)
+        out[:, q_dim + kv_dim:] = v.reshape(T, kv_dim)
+        return
+    page_size = k_cache.shape[2]
+    page, off = (slot_mapping // page_size).long(), (slot_mapping % page_size).long()
+    k_cache[page, :, off] = k
+    v_cache[page, :, :, off] = v
+
+
+def map_difference(att, head_dim, gate, gate_col, mix, eps, gain, out, num_heads, value_dim):
+    T = att.shape[0]
+    a = att.float().view(T, num_heads, 2, head_dim)[..., :value_dim]
+    o = a[:, :, 0] - mix * a[:, :, 1]
+    o = (o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * gain).reshape(T, num_heads * value_dim)
+    if gate is not None:
+        o = o * torch.sigmoid(gate[:, gate_col:gate_col + num_heads * value_dim].float())
+    _store(out, o)
+
+
 def row_rinv(x, ranges, eps, out):
     out.zero_()
     for j, (col, n, width) in enumerate(ranges):
@@ -361,6 +440,9 @@ def grouped_linear(a, weight, out, row_offsets=None, a_group_cols=0, out_group_c
                     y = y.view(hi - lo, N // 16, 2, 8)
                     gate, up = torch.clamp(y[:, :, 0, :], max=limit), torch.clamp(y[:, :, 1, :], min=-limit, max=limit)
                     y = (gate / (1.0 + torch.exp(-alpha * gate)) * (up + 1.0)).reshape(hi - lo, N // 2)
+                elif epilogue == "geglu":
+                    y = y.view(hi - lo, N // 16, 2, 8)
+                    y = (_gelu(y[:, :, 0, :]) * y[:, :, 1, :]).reshape(hi - lo, N // 2)
                 out[lo:hi] = y.to(out.dtype)
         return
     for g in range(G):
@@ -412,12 +494,12 @@ def moe_gather(h, pair_at, weights, top, out):
     _store(out, src * (pair_at >= 0).float()[:, None])
 
 
-def moe_combine(rows, place_of, weights, top, y):
+def moe_combine(rows, place_of, weights, top, y, extra=None):
     T, H = y.shape
     r = rows[place_of.long()].float().view(T, top, H)
     if weights is not None:
         r = r * weights[:, :, None]
-    _store(y, r.sum(1))
+    _store(y, r.sum(1) + extra.float() if extra is not None else r.sum(1))
 
 
 def gather_rows(src, rows, out):
@@ -789,7 +871,7 @@ def table_gather(resident, updates, slots, out, trash_page):
             out[s, b] = resident[slot, b] if b < cols else trash_page
 
 
-ALL = ["moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
+ALL = ["geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
        "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift", "ssm_scan",
        "decay_scan", "gated_rmsnorm", "table_gather", "gather_rows", "scale_inplace", "logit_cap", "rope_table", "linear_scaled_accepts", "linear_add_scaled_parts", "linear_add_scaled", "apply_row_scale", "linear_rope_kv", "interleave_gate_up", "embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add", "linear", "rope_kv_write",
        "paged_attention", "swiglu", "argmax", "sample"]
