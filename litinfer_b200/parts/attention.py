@@ -294,7 +294,7 @@ class PagedAttention(Mixer):
                 h, self.qkv.weight, self.qkv.bias, qkv, ctx.positions, rot.denominators if rot else None, rot.rotary_dim if rot else 0,
                 view.slot_mapping, cache.k, cache.v, self.num_heads, self.num_kv_heads, self.head_dim, cache.writes, row_scale=row_scale,
                 cos_sin=rot.table if rot else None)
-        o = torch.empty((h.shape[0], self.q_dim), dtype=self.dtype, device=h.device)
+        o = torch.empty((qkv.shape[0], self.q_dim), dtype=self.dtype, device=qkv.device)
         K.paged_attention(
             qkv, o, cache.k, cache.v, view.block_table, ctx.q_start, ctx.ctx_lens, ctx.seq_of_token, ctx.positions,
             self.num_heads, self.num_kv_heads, self.head_dim, self.scale, self.window,
