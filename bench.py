@@ -25,8 +25,8 @@ Weights (3 GB) are larger than L2, so nothing stays cached between steps.
 profiling runs and the summaries under ``profiles/``); ``mixed`` is a step of ``--batch`` requests decoding at
 ``--context`` beside a portion of ``--prefill-tokens`` prompt tokens.
 
-``--only design`` runs a design (``--design filasun|gorulorn|demavik|pifazen``, default filasun) beside the Qwen2 model of equal layer sizes and layer count (``--design-shapes``,
-``--layers``, default 6): prefill of ``--prefill-tokens`` tokens and decode at batch 1, 8 and 32; ``--arch filasun|gorulorn|demavik|pifazen`` puts
+``--only design`` runs a design (``--design filasun|gorulorn|demavik|pifazen|zigolix``, default filasun) beside the Qwen2 model of equal layer sizes and layer count (``--design-shapes``,
+``--layers``, default 6): prefill of ``--prefill-tokens`` tokens and decode at batch 1, 8 and 32; ``--arch filasun|gorulorn|demavik|pifazen|zigolix`` puts
 that design behind ``--only decode|prefill|kernels-decode|kernels-prefill`` (the kernel tables of ``profiles/``).
 
 ``--shape 1.5b|7b|14b`` chooses the layer sizes (default 1.5b, the headline; the other two are the larger workloads of
@@ -185,13 +185,37 @@ def pifazen_config(shape: str, layers: int):
             "max_positions": d["max_position_embeddings"]}
 
 
+def zigolix_config(shape: str, layers: int, window: int = 1024):
+    """A Zigolix model with the layer sizes of a shape of the benchmark description: the same width, heads, key/value heads,
+    head size and vocabulary as the Qwen2 model of that shape.  Layers alternate between differential attention (two maps of
+    half the head size a head over values of head size, scores capped at 50) and attention whose values are its keys (half of
+    each head rotated with blended frequencies, a norm behind the rotation, sinks), both in a window of ``window``.  The first
+    layer has the dense feed-forward of the shape's width, the others 8 experts of half that width, 2 per token, and a shared
+    expert of a quarter of it.  The two layers in the middle run twice (``layers`` + 2 layer runs)."""
+    d = SHAPES[shape]
+    H, nh, nkv, dh, ff = d["hidden_size"], d["num_attention_heads"], d["num_key_value_heads"], d["head_dim"], d["intermediate_size"]
+    moe = {"kind": "moe", "expert": {"ff": ff // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2}, "shared": {"ff": ff // 4, "limit": 7.0}}
+    dif = {"heads": nh, "kv_heads": nkv, "dim": dh // 2, "vdim": dh, "mask": {"size": window}, "scale": (dh // 2) ** -0.5, "softcap": 50.0, "diff": 0.4}
+    att = {"heads": nh, "kv_heads": nkv, "dim": dh, "vdim": dh, "mask": {"size": window}, "scale": dh ** -0.5,
+           "rot": {"dims": dh // 2, "base": d["rope_theta"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mid = max(0, layers // 2 - 1)
+    return {"architecture": "Zigolix", "norm": {"eps": 1e-5}, "logit_scale": 0.5, "vocab": d["vocab_size"], "width": H,
+            "layers": [{"type": "attention_2" if i % 2 == 0 else "attention", "mlp": {"kind": "dense", "ff": ff} if i == 0 else moe,
+                        "mixer": dif if i % 2 == 0 else att} for i in range(layers)],
+            "loop": {"start": mid, "stop": min(layers, mid + 2), "times": 2}, "max_positions": d["max_position_embeddings"]}
+
+
+# the designs that run beside Qwen2: config.json with the layer sizes of a shape, for a count of layers
+DESIGNS = {"filasun": filasun_config, "gorulorn": gorulorn_config, "demavik": demavik_config, "pifazen": pifazen_config, "zigolix": zigolix_config}
+
+
 def design_layer_runs(cfg) -> int:
     loop = cfg.get("loop")
     return len(cfg["layers"]) + ((loop["stop"] - loop["start"]) * (loop["times"] - 1) if loop else 0)
 
 
 def time_design(args, peaks):
-    """Prefill and decode of a design (``--design filasun|gorulorn|demavik|pifazen``) beside the Qwen2 model of the same layer sizes and as
+    """Prefill and decode of a design (``--design filasun|gorulorn|demavik|pifazen|zigolix``) beside the Qwen2 model of the same layer sizes and as
     many layers as the design runs (random weights), through the same step function: tokens per second, and the
     milliseconds behind them."""
     import torch
@@ -205,15 +229,9 @@ def time_design(args, peaks):
     for shape in args.design_shapes.split(","):
         runs = layers
         for arch in (design, "qwen2"):
-            if arch == "filasun":
-                cfg = filasun_config(shape, layers)
-            elif arch == "gorulorn":
-                cfg = gorulorn_config(shape, layers)
+            if arch in DESIGNS:
+                cfg = DESIGNS[arch](shape, layers)
                 runs = design_layer_runs(cfg)
-            elif arch == "demavik":
-                cfg = demavik_config(shape, layers)
-            elif arch == "pifazen":
-                cfg = pifazen_config(shape, layers)
             else:
                 cfg = bench_config(shape)
                 cfg["num_hidden_layers"] = runs
@@ -811,8 +829,8 @@ def main() -> int:
     ap.add_argument("--kernel-rows", type=int, default=16, help="--only kernels-*: how many kernels the table lists")
     ap.add_argument("--no-graphs", action="store_true", help="launch every kernel from the host (so that a profiler lists them)")
     ap.add_argument("--prefill-tokens", type=int, default=2048)
-    ap.add_argument("--design", default="filasun", choices=["filasun", "gorulorn", "demavik", "pifazen"], help="--only design: the design that runs beside Qwen2")
-    ap.add_argument("--arch", default="qwen2", choices=["qwen2", "filasun", "gorulorn", "demavik", "pifazen"],
+    ap.add_argument("--design", default="filasun", choices=list(DESIGNS), help="--only design: the design that runs beside Qwen2")
+    ap.add_argument("--arch", default="qwen2", choices=["qwen2"] + list(DESIGNS),
                     help="which design the parts behind --only are measured on, with the layer sizes of --shape (default: the headline's Qwen2)")
     ap.add_argument("--design-shapes", default="1.5b,7b", help="--only design: the shapes whose layer sizes are run, with commas")
     args = ap.parse_args()
@@ -841,33 +859,12 @@ def main() -> int:
         return 0
     if args.layers:
         cfg["num_hidden_layers"] = args.layers
-    if args.arch == "filasun":
+    if args.arch in DESIGNS:
         if args.only == "all":
-            print("bench.py: --arch filasun goes with --only decode|prefill|kernels-decode|kernels-prefill|design")
+            print(f"bench.py: --arch {args.arch} goes with --only decode|prefill|kernels-decode|kernels-prefill|design")
             return 2
-        cfg = filasun_config(args.shape, args.layers or 6)
-        cfg["num_hidden_layers"], cfg["max_position_embeddings"] = len(cfg["layers"]), cfg["max_positions"]
-        cfg.update(num_key_value_heads=0, head_dim=0, hidden_size=cfg["width"])
-    if args.arch == "gorulorn":
-        if args.only == "all":
-            print("bench.py: --arch gorulorn goes with --only decode|prefill|kernels-decode|kernels-prefill|design")
-            return 2
-        cfg = gorulorn_config(args.shape, args.layers or 6)
+        cfg = DESIGNS[args.arch](args.shape, args.layers or 6)
         cfg["num_hidden_layers"], cfg["max_position_embeddings"] = design_layer_runs(cfg), cfg["max_positions"]
-        cfg.update(num_key_value_heads=0, head_dim=0, hidden_size=cfg["width"])
-    if args.arch == "demavik":
-        if args.only == "all":
-            print("bench.py: --arch demavik goes with --only decode|prefill|kernels-decode|kernels-prefill|design")
-            return 2
-        cfg = demavik_config(args.shape, args.layers or 6)
-        cfg["num_hidden_layers"], cfg["max_position_embeddings"] = len(cfg["layers"]), cfg["max_positions"]
-        cfg.update(num_key_value_heads=0, head_dim=0, hidden_size=cfg["width"])
-    if args.arch == "pifazen":
-        if args.only == "all":
-            print("bench.py: --arch pifazen goes with --only decode|prefill|kernels-decode|kernels-prefill|design")
-            return 2
-        cfg = pifazen_config(args.shape, args.layers or 6)
-        cfg["num_hidden_layers"], cfg["max_position_embeddings"] = len(cfg["layers"]), cfg["max_positions"]
         cfg.update(num_key_value_heads=0, head_dim=0, hidden_size=cfg["width"])
     if args.only in ("decode", "kernels-decode") and args.context + 4096 > cfg["max_position_embeddings"]:
         # a longer context than the shape's own limit, on request: the measurement's model allows it
