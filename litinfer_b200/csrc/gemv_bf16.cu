@@ -336,12 +336,12 @@ bool li_gemv_rope_accepts(const void* a, const void* w, int M, int N, int K, int
 
 int li_linear_gemv_rope(const void* a, const void* w, const float* bias, void* out, int M, int N, int K, const int* positions,
                         const float* denom, const int* slot_mapping, void* kcache, void* vcache, int nh, int nkv, int dh,
-                        int page_size, int num_pages, int write, const RowScale& rs, cudaStream_t stream) {
-    RopeArgs ra{positions, denom, slot_mapping, (bf16*)kcache, (bf16*)vcache, nh, nkv, dh, page_size, num_pages, write};
-    if (M <= 8) return launch_rope<1>(a, w, bias, out, M, N, K, ra, rs, stream);
-    if (M <= 16) return launch_rope<2>(a, w, bias, out, M, N, K, ra, rs, stream);
-    if (M <= 32) return launch_rope<4>(a, w, bias, out, M, N, K, ra, rs, stream);
-    return launch_rope<8>(a, w, bias, out, M, N, K, ra, rs, stream);
+                        int page_size, int num_pages, int write, const RowScale& rs, void* extra_out, int extra, cudaStream_t stream) {
+    RopeArgs ra{positions, denom, slot_mapping, (bf16*)kcache, (bf16*)vcache, nh, nkv, dh, page_size, num_pages, write, (bf16*)extra_out, extra};
+    if (M <= 8) return launch_rope<1>(a, w, bias, out, M, N + extra * dh, K, ra, rs, stream);
+    if (M <= 16) return launch_rope<2>(a, w, bias, out, M, N + extra * dh, K, ra, rs, stream);
+    if (M <= 32) return launch_rope<4>(a, w, bias, out, M, N + extra * dh, K, ra, rs, stream);
+    return launch_rope<8>(a, w, bias, out, M, N + extra * dh, K, ra, rs, stream);
 }
 
 bool li_gemv_bf16_accepts(int M, int N, int K) { return M >= 1 && M <= kMaxM && K % 8 == 0 && N >= 1; }

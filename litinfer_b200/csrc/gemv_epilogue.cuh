@@ -19,6 +19,9 @@ struct RopeArgs {
     bf16* kcache;
     bf16* vcache;
     int nh, nkv, dh, page_size, num_pages, write;
+    // heads behind q|k|v: a further map of the same input, to rows of its own (neither rotated nor cached)
+    bf16* extra_out = nullptr;
+    int extra = 0;
 };
 
 template <int NT, typename Get>
@@ -52,9 +55,14 @@ __device__ __forceinline__ void store_rope(Get get, const float* __restrict__ bi
             y0 = x0 * cs - x1 * sn;
             y1 = x1 * cs + x0 * sn;
         }
-        if (head < ra.nh) {
-            out[(size_t)tok * N + r0] = __float2bfloat16_rn(y0);
-            out[(size_t)tok * N + r1] = __float2bfloat16_rn(y1);
+        if (head >= ra.nh + 2 * ra.nkv) {
+            bf16* dst = ra.extra_out + (size_t)tok * ra.extra * ra.dh + (size_t)(head - ra.nh - 2 * ra.nkv) * ra.dh;
+            dst[jj] = __float2bfloat16_rn(y0);
+            dst[jj + half] = __float2bfloat16_rn(y1);
+        } else if (head < ra.nh) {
+            const size_t ld = (size_t)(ra.nh + 2 * ra.nkv) * ra.dh;
+            out[tok * ld + r0] = __float2bfloat16_rn(y0);
+            out[tok * ld + r1] = __float2bfloat16_rn(y1);
         } else if (ra.write) {
             const int slot = ra.slot_mapping[tok];
             const int page = slot / ra.page_size, off = slot - page * ra.page_size;

@@ -132,8 +132,10 @@ __device__ __forceinline__ void mma16816(float (&c)[4], unsigned a0, unsigned a1
 template <int TM, int TK, int ST, int kSwiglu>
 __global__ void __launch_bounds__(128)
 grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* __restrict__ W, bf16* __restrict__ C, int ldc, int c_gcol,
-                   const int* __restrict__ row_offsets, int M, int N, int K, int G, const float* __restrict__ glu_params) {
+                   const int* __restrict__ row_offsets, int M, int N, int K, int G, const float* __restrict__ glu_params,
+                   const int* __restrict__ row_map, int row_div) {
     __shared__ __align__(16) bf16 As[ST][TM][TK + MPAD];
+    __shared__ int src_row[TM];
     __shared__ __align__(16) bf16 Ws[ST][BN][TK + MPAD];
     pdl_launch_dependents();
     pdl_wait();
@@ -163,12 +165,15 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int gq = lane >> 2, t = lane & 3;
     constexpr int CH = TK / 8;                                      // 16-byte chunks of a row of a stage
+    // row_map: row r of the sorted order is row row_map[r] / row_div of A (the rows of a mixture's tokens, read in place)
+    if (tid < TM) src_row[tid] = (row_map && m0 + tid < m_end) ? row_map[m0 + tid] / row_div : m0 + tid;
+    __syncthreads();
     auto load = [&](int stage, int k0) {
         for (int idx = tid; idx < TM * CH; idx += 128) {
             const int r = idx / CH, ch = idx - r * CH;
             const int k = k0 + ch * 8;
             const bool v = k < K && m0 + r < m_end;
-            cp16(&As[stage][r][ch * 8], v ? a + (size_t)(m0 + r) * lda + k : a, v);
+            cp16(&As[stage][r][ch * 8], v ? a + (size_t)src_row[r] * lda + k : a, v);
         }
         for (int idx = tid; idx < BN * CH; idx += 128) {
             const int r = idx / CH, ch = idx - r * CH;
@@ -240,18 +245,14 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
 
 constexpr int kMaxExpertsPerLane = 8;       // experts <= 256
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, int T, int E, int top, int* __restrict__ ids,
-                                 float* __restrict__ weights) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int lane = threadIdx.x & 31;
-    if (t >= T) return;
+// The choice of one token by a warp: scoring 0 the largest sigmoid scores, which are the weights; 1 the largest logits, the
+// weights their softmax among the chosen.
+__device__ __forceinline__ void route_token(const float* logits, int scoring, int E, int top, int* ids, float* weights, int lane) {
     float s[kMaxExpertsPerLane];
 #pragma unroll
     for (int i = 0; i < kMaxExpertsPerLane; ++i) {
         const int e = lane + 32 * i;
-        const float z = e < E ? logits[(size_t)t * E + e] : 0.0f;
+        const float z = e < E ? logits[e] : 0.0f;
         // sigmoid scores lie in (0, 1): -1 never wins; logits taken as they are: the lowest float never wins
         if (scoring == 0) s[i] = e < E ? 1.0f / (1.0f + expf(-z)) : -1.0f;
         else s[i] = e < E ? fmaxf(z, -3.0e38f) : -3.4e38f;
@@ -272,8 +273,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, 
             if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa;
         }
         if (lane == 0) {
-            ids[(size_t)t * top + k] = arg;
-            weights[(size_t)t * top + k] = best;
+            ids[k] = arg;
+            weights[k] = best;
         }
 #pragma unroll
         for (int i = 0; i < kMaxExpertsPerLane; ++i)
@@ -281,12 +282,20 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, 
     }
     if (scoring == 1 && lane == 0) {
         // the weights are the softmax over the chosen logits alone (the first chosen is the largest)
-        float* wt = weights + (size_t)t * top;
-        const float m = wt[0];
+        const float m = weights[0];
         float sum = 0.0f;
-        for (int k = 0; k < top; ++k) sum += expf(wt[k] - m);
-        for (int k = 0; k < top; ++k) wt[k] = expf(wt[k] - m) / sum;
+        for (int k = 0; k < top; ++k) sum += expf(weights[k] - m);
+        for (int k = 0; k < top; ++k) weights[k] = expf(weights[k] - m) / sum;
     }
+}
+
+__global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, int T, int E, int top, int* __restrict__ ids,
+                                 float* __restrict__ weights) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (t >= T) return;
+    route_token(logits + (size_t)t * E, scoring, E, top, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
 }
 
 // Routing over all experts at once with groups: scores s = softmax(logits) over the E outputs; the choice scores are
@@ -294,19 +303,14 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, 
 // experts of the `keep` best groups can be chosen (the lower index wins a tie, among groups and among experts); the `top`
 // largest choice scores choose; the weights are the chosen experts' s (without the correction), divided by their sum + 1e-20,
 // times `scale`.  One warp a token, everything in float.
-__global__ void moe_route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int T, int E, int top, int groups,
-                                         int keep, float scale, int* __restrict__ ids, float* __restrict__ weights) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int lane = threadIdx.x & 31;
-    if (t >= T) return;
+__device__ __forceinline__ void route_token_grouped(const float* logits, const float* __restrict__ correction, int E, int top, int groups, int keep,
+                                                    float scale, int* ids, float* weights, int lane) {
     float s[kMaxExpertsPerLane], c[kMaxExpertsPerLane];
     float m = -INFINITY;
 #pragma unroll
     for (int i = 0; i < kMaxExpertsPerLane; ++i) {
         const int e = lane + 32 * i;
-        s[i] = e < E ? logits[(size_t)t * E + e] : -INFINITY;
+        s[i] = e < E ? logits[e] : -INFINITY;
         m = fmaxf(m, s[i]);
     }
     m = warp_max(m);
@@ -373,8 +377,8 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, const
             if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa, score = os;
         }
         if (lane == 0) {
-            ids[(size_t)t * top + k] = arg;
-            weights[(size_t)t * top + k] = score;
+            ids[k] = arg;
+            weights[k] = score;
         }
         wsum += score;
 #pragma unroll
@@ -382,8 +386,82 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, const
             if (lane + 32 * i == arg) c[i] = -INFINITY, s[i] = 0.0f;
     }
     if (lane == 0) {
-        float* wt = weights + (size_t)t * top;
-        for (int k = 0; k < top; ++k) wt[k] = wt[k] / (wsum + 1e-20f) * scale;
+        for (int k = 0; k < top; ++k) weights[k] = weights[k] / (wsum + 1e-20f) * scale;
+    }
+}
+
+__global__ void moe_route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int T, int E, int top, int groups,
+                                         int keep, float scale, int* __restrict__ ids, float* __restrict__ weights) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (t >= T) return;
+    route_token_grouped(logits + (size_t)t * E, correction, E, top, groups, keep, scale, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
+}
+
+// The front of a mixture for a small step as one block: the router's product (a warp per token and four experts, float sums),
+// the choice (a warp per token) and the stable sort of the (token, choice) pairs by expert (runs without padding).
+constexpr int kSmallPairs = 256, kSmallLogits = 1024;
+
+template <typename T>
+__global__ void __launch_bounds__(1024)
+moe_small_step_kernel(const T* __restrict__ h, const T* __restrict__ w, const float* __restrict__ bias, int tokens, int H, int E, int top, int scoring,
+                      const float* __restrict__ correction, int groups, int keep, float scale, float* __restrict__ weights, int* __restrict__ offsets,
+                      int* __restrict__ pair_at, int* __restrict__ place_of) {
+    constexpr int V = 16 / (int)sizeof(T);
+    __shared__ float logits[kSmallLogits];
+    __shared__ int ids[kSmallPairs];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int quads = (E + 3) / 4;
+    for (int job = warp; job < tokens * quads; job += 32) {
+        const int t = job / quads, e0 = (job - t * quads) * 4;
+        const T* hr = h + (size_t)t * H;
+        float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int k = V * lane; k < H; k += 32 * V) {
+            const uint4 hv = *reinterpret_cast<const uint4*>(hr + k);
+            uint4 wv[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) wv[j] = __ldg(reinterpret_cast<const uint4*>(w + (size_t)min(e0 + j, E - 1) * H + k));
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const unsigned a[4] = {hv.x, hv.y, hv.z, hv.w}, b[4] = {wv[j].x, wv[j].y, wv[j].z, wv[j].w};
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    if constexpr (sizeof(T) == 2) {
+                        acc[j] = fmaf(__uint_as_float(a[q] << 16), __uint_as_float(b[q] << 16), acc[j]);
+                        acc[j] = fmaf(__uint_as_float(a[q] & 0xffff0000u), __uint_as_float(b[q] & 0xffff0000u), acc[j]);
+                    } else {
+                        acc[j] = fmaf(__uint_as_float(a[q]), __uint_as_float(b[q]), acc[j]);
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float z = warp_sum(acc[j]);
+            if (lane == 0 && e0 + j < E) logits[t * E + e0 + j] = bias ? z + bias[e0 + j] : z;
+        }
+    }
+    __syncthreads();
+    for (int t = warp; t < tokens; t += 32) {
+        if (scoring == 2) route_token_grouped(logits + t * E, correction, E, top, groups, keep, scale, ids + t * top, weights + (size_t)t * top, lane);
+        else route_token(logits + t * E, scoring, E, top, ids + t * top, weights + (size_t)t * top, lane);
+    }
+    __syncthreads();
+    const int n = tokens * top;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const int e = ids[i];
+        int place = 0;
+        for (int j = 0; j < n; ++j) place += (ids[j] < e || (ids[j] == e && j < i)) ? 1 : 0;
+        pair_at[place] = i;
+        place_of[i] = place;
+    }
+    for (int e = threadIdx.x; e <= E; e += blockDim.x) {
+        int before = 0;
+        for (int j = 0; j < n; ++j) before += ids[j] < e ? 1 : 0;
+        offsets[e] = before;
     }
 }
 
@@ -498,10 +576,11 @@ constexpr int kTensorRows = 256;
 
 // epilogue: LI_EPILOGUE_NONE, or a gated one (bfloat16, K a multiple of 8, N a multiple of 16): gate and up rows of
 // every group's matrix interleaved in eights, out rows of N / 2 activations; LI_EPILOGUE_GLU_CLAMPED reads its {limit, alpha}
-// from glu_params on the device.
+// from glu_params on the device.  row_map (may be NULL; bfloat16, rows in groups): row r is row row_map[r] / row_div of a.
 LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* w, void* out, int ldc, int c_gcol, const int* row_offsets,
                                 const int* tile_group, int dtype, int M, int N, int K, int G, int epilogue, const float* glu_params,
-                                cudaStream_t stream) {
+                                const int* row_map, int row_div, cudaStream_t stream) {
+    LI_REQUIRE(row_map == nullptr || (row_offsets != nullptr && tile_group == nullptr && row_div >= 1), "grouped_linear: a map of the rows goes with rows in groups, without padded runs");
     LI_REQUIRE(M >= 0 && N > 0 && K > 0 && G > 0, "grouped_linear: bad sizes M=%d N=%d K=%d G=%d", M, N, K, G);
     LI_REQUIRE(epilogue == LI_EPILOGUE_NONE || li_epilogue_is_gated(epilogue), "grouped_linear: unknown epilogue %d", epilogue);
     LI_REQUIRE(li_epilogue_bias_ok(epilogue, glu_params) || epilogue == LI_EPILOGUE_NONE, "grouped_linear: the bounded unit needs its parameters, the others take none");
@@ -522,6 +601,7 @@ LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* 
     // 16-byte copies: every row and every group's first column on a 16-byte boundary
     const bool aligned = K % 8 == 0 && lda % 8 == 0 && a_gcol % 8 == 0 && ((uintptr_t)a % 16) == 0 && ((uintptr_t)w % 16) == 0;
     LI_REQUIRE(!swiglu || (dtype == LI_BF16 && aligned && N % 16 == 0), "grouped_linear: the swiglu epilogue takes bfloat16, K a multiple of 8 and N a multiple of 16");
+    LI_REQUIRE(row_map == nullptr || (dtype == LI_BF16 && aligned), "grouped_linear: a map of the rows takes bfloat16 with K and rows of multiples of 8");
     // few rows a group (single tokens): tiles of 16 rows, more of the weights in flight
     const bool few = row_offsets ? M <= 32 * G : M <= 32;
     if (dtype == LI_BF16 && aligned && few) {
@@ -529,7 +609,7 @@ LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* 
         const dim3 grid16(ceil_div(N, BN), row_offsets ? tiles16 + G : tiles16, row_offsets ? 1 : G);
 #define LI_GROUPED_MMA(TM_, TK_, ST_, EPI_, GRID_)                                                                                          \
     li_launch_pdl(grouped_mma_kernel<TM_, TK_, ST_, EPI_>, GRID_, dim3(128), 0, stream, (const bf16*)a, lda, a_gcol, (const bf16*)w, (bf16*)out, ldc, \
-                  c_gcol, row_offsets, M, N, K, G, glu_params)
+                  c_gcol, row_offsets, M, N, K, G, glu_params, row_map, row_div)
         e = clamped ? LI_GROUPED_MMA(16, 64, 4, 2, grid16) : geglu ? LI_GROUPED_MMA(16, 64, 4, 3, grid16) : swiglu ? LI_GROUPED_MMA(16, 64, 4, 1, grid16) : LI_GROUPED_MMA(16, 64, 4, 0, grid16);
     } else if (dtype == LI_BF16 && aligned)
         e = clamped ? LI_GROUPED_MMA(64, 32, 3, 2, grid) : geglu ? LI_GROUPED_MMA(64, 32, 3, 3, grid) : swiglu ? LI_GROUPED_MMA(64, 32, 3, 1, grid) : LI_GROUPED_MMA(64, 32, 3, 0, grid);
@@ -612,4 +692,32 @@ LI_EXPORT int li_moe_combine(const void* rows, int dtype, const int* place_of, c
         e = li_launch_pdl(moe_combine_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16*)rows, place_of, weights, top, H, (const bf16*)extra, (bf16*)y);
     if (e != cudaSuccess) return li_fail("moe_combine: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("moe_combine");
+}
+
+// The front of a mixture for a step of few tokens as one launch: router logits h [T, H] w [E, H]^T (+ bias), the choice
+// (scoring 0, 1 as in li_moe_route; 2 as in li_moe_route_grouped) and the stable sort without padding: weights [T, top], offsets
+// [E + 1], pair_at and place_of [T top].  li_moe_small_step_accepts says for which sizes.
+LI_EXPORT int li_moe_small_step_accepts(int dtype, int T, int H, int E, int top) {
+    const int vec = dtype == LI_BF16 ? 8 : 4;
+    return (T >= 1 && E >= 1 && E <= 32 * kMaxExpertsPerLane && top >= 1 && top <= E && T * top <= kSmallPairs && T * E <= kSmallLogits &&
+            T * ((E + 3) / 4) <= 128 && H % vec == 0) ? 1 : 0;
+}
+
+LI_EXPORT int li_moe_small_step(const void* h, const void* w, const float* bias, int dtype, int T, int H, int E, int top, int scoring,
+                                const float* correction, int groups, int keep, float scale, float* weights, int* offsets, int* pair_at,
+                                int* place_of, cudaStream_t stream) {
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "moe_small_step: unknown dtype %d", dtype);
+    LI_REQUIRE(li_moe_small_step_accepts(dtype, T, H, E, top), "moe_small_step: refuses T=%d H=%d, %d of %d experts", T, H, top, E);
+    LI_REQUIRE(scoring >= 0 && scoring <= 2, "moe_small_step: unknown scoring %d", scoring);
+    LI_REQUIRE(scoring != 2 || (groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top),
+               "moe_small_step: %d of %d groups of %d experts cannot give %d choices", keep, groups, E, top);
+    LI_REQUIRE(((uintptr_t)h % 16) == 0 && ((uintptr_t)w % 16) == 0, "moe_small_step: operands must be 16-byte aligned");
+    const int threads = 1024;
+    const cudaError_t e = dtype == LI_F32
+        ? li_launch_pdl(moe_small_step_kernel<float>, dim3(1), dim3(threads), 0, stream, (const float*)h, (const float*)w, bias, T, H, E, top, scoring, correction,
+                        groups, keep, scale, weights, offsets, pair_at, place_of)
+        : li_launch_pdl(moe_small_step_kernel<bf16>, dim3(1), dim3(threads), 0, stream, (const bf16*)h, (const bf16*)w, bias, T, H, E, top, scoring, correction,
+                        groups, keep, scale, weights, offsets, pair_at, place_of);
+    if (e != cudaSuccess) return li_fail("moe_small_step: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("moe_small_step");
 }

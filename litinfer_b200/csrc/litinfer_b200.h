@@ -261,11 +261,12 @@ int li_rope_kv_write(void* qkv, int dtype, const int* positions, const float* de
     slot_mapping, void* kcache, void* vcache, int T, int nh, int nkv, int dh, int page_size, int num_pages, int write,
     cudaStream_t stream);
 
-/* The q|k|v product followed by li_rope_kv_write, as one kernel where the shape allows. */
+/* The q|k|v product followed by li_rope_kv_write, as one kernel where the shape allows.  extra: heads' worth of rows behind q|k|v
+ * in w (and bias), a further map of the same input, to extra_out [T, extra dh]. */
 int li_linear_rope_kv(const void* a, const void* w, const float* bias, void* qkv, int dtype, const int* positions,
     const float* denom, int rotary_dim, const int* slot_mapping, void* kcache, void* vcache, int T, int K, int nh, int
     nkv, int dh, int page_size, int num_pages, int write, int allow_fused, const float* ssq, int nparts, int width,
-    float eps, const float* cos_sin, cudaStream_t stream);
+    float eps, const float* cos_sin, void* extra_out, int extra, cudaStream_t stream);
 
 /* ---- norm_pair.cu: norms before and after a sublayer in one pass over the residual stream ---- */
 /* Per row: x += post(y) (post: a norm of y [R, H] with the weight w_post; NULL: x += y; y NULL: nothing is added), then
@@ -277,8 +278,10 @@ int li_norm_add_norm(float* x, const void* y, int dtype, const float* w_post, in
     int next_centered, float eps_next, void* out, const int* rows, int R, int n_src, int H, const int* y_places,
     int y_top, const float* y_weights, const void* y_extra, cudaStream_t stream);
 
-/* out [T, 2 H] in the run dtype: x [T, H] (plus delta [T, H] if given) beside x0 [T, H], both float. */
-int li_join_rows(const float* x, const void* delta, const float* x0, void* out, int dtype, int T, int H, cudaStream_t stream);
+/* out [T, 2 H] in the run dtype: x [T, H] (plus delta [T, H] if given) beside x0 [T, H], both float.  places (may be NULL): delta
+ * is a sum of rows as in li_norm_add_norm. */
+int li_join_rows(const float* x, const void* delta, const float* x0, void* out, int dtype, int T, int H, const int* places, int top,
+    const float* weights, const void* extra, cudaStream_t stream);
 
 /* x[t] += row for every token. */
 int li_add_row(float* x, const float* row, int T, int H, cudaStream_t stream);
@@ -337,10 +340,11 @@ int li_map_difference(const void* att, int dtype, int dl, const void* gate, int 
  * row_offsets NULL: every group takes all M rows, inputs at column g * a_gcol, outputs at column g * c_gcol.
  * tile_group (may be NULL): with runs of rows that start at multiples of 128, the group of every tile of 128 rows (-1: none);
  * large bfloat16 products then run on tcgen05 tiles.  epilogue 1 (bfloat16): gate and up rows of every matrix interleaved in
- * eights, out rows of N / 2 activations up * gate / (1 + exp(-gate)). */
+ * eights, out rows of N / 2 activations up * gate / (1 + exp(-gate)).  row_map (may be NULL; bfloat16, rows in groups, runs without
+ * padding): row r of the groups is row row_map[r] / row_div of a. */
 int li_grouped_linear(const void* a, int lda, int a_gcol, const void* w, void* out, int ldc, int c_gcol, const int* row_offsets,
     const int* tile_group, int dtype, int M, int N, int K, int G, int epilogue, const float* glu_params,
-    cudaStream_t stream);
+    const int* row_map, int row_div, cudaStream_t stream);
 
 /* ids, weights [T, top]: the experts with the largest sigmoid(logits [T, E]) and those scores (scoring 0), or the experts
  * with the largest logits and the softmax over the chosen logits alone (scoring 1). */
@@ -365,6 +369,13 @@ int li_moe_gather(const void* h, int dtype, const int* pair_at, const float* wei
 /* y [T, H]: y[t] = sum_k rows[place_of[t * top + k]] (times weights[t * top + k] if weights is given), plus extra[t] if given. */
 int li_moe_combine(const void* rows, int dtype, const int* place_of, const float* weights, const void* extra, int T, int top, int H,
     void* y, cudaStream_t stream);
+
+/* The front of a mixture for a step of few tokens as one launch: logits h [T, H] w [E, H]^T (+ bias), the choice (scoring 0, 1 as in
+ * li_moe_route, 2 as in li_moe_route_grouped), the stable sort without padding.  accepts: 1 if the sizes fit. */
+int li_moe_small_step_accepts(int dtype, int T, int H, int E, int top);
+int li_moe_small_step(const void* h, const void* w, const float* bias, int dtype, int T, int H, int E, int top, int scoring,
+    const float* correction, int groups, int keep, float scale, float* weights, int* offsets, int* pair_at,
+    int* place_of, cudaStream_t stream);
 
 /* ---- sampling.cu ---- */
 /* out[r] = the first maximum of logits[r]. */

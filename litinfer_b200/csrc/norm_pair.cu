@@ -275,9 +275,11 @@ __global__ void add_row_kernel(float* __restrict__ x, const float* __restrict__ 
     if (i < n) x[i] += row[i % H];
 }
 
-// out[t] = (x[t] + delta[t] | x0[t]), four elements a thread where rows are multiples of four, else one
+// out[t] = (x[t] + delta[t] | x0[t]), four elements a thread where rows are multiples of four, else one.  places: delta[t] is
+// the sum over j < top of delta[places[t top + j]] (times weights[t top + j]) and extra[t] instead.
 template <typename T, int V>
-__global__ void join_rows_kernel(const float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ x0, T* __restrict__ out, long long n, int H) {
+__global__ void join_rows_kernel(const float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ x0, T* __restrict__ out, long long n, int H,
+                                 const int* __restrict__ places, int top, const float* __restrict__ weights, const T* __restrict__ extra) {
     pdl_launch_dependents();
     pdl_wait();
     const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
@@ -293,9 +295,26 @@ __global__ void join_rows_kernel(const float* __restrict__ x, const T* __restric
     } else {
         v[0] = (first ? x : x0)[src];
     }
-    if (first && delta) {
+    auto add = [&](const T* p, float f) {
+        if constexpr (V == 4 && sizeof(T) == 2) {
+            const uint2 u = *reinterpret_cast<const uint2*>(p);
+            v[0] = fmaf(f, __uint_as_float(u.x << 16), v[0]), v[1] = fmaf(f, __uint_as_float(u.x & 0xffff0000u), v[1]);
+            v[2] = fmaf(f, __uint_as_float(u.y << 16), v[2]), v[3] = fmaf(f, __uint_as_float(u.y & 0xffff0000u), v[3]);
+        } else {
 #pragma unroll
-        for (int k = 0; k < V; ++k) v[k] += to_float(delta[src + k]);
+            for (int k = 0; k < V; ++k) v[k] = fmaf(f, to_float(p[k]), v[k]);
+        }
+    };
+    if (first && places) {
+        float keep[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) keep[k] = v[k], v[k] = 0.0f;
+        for (int j = 0; j < top; ++j) add(delta + (size_t)places[t * top + j] * H + c, weights ? weights[t * top + j] : 1.0f);
+        if (extra) add(extra + src, 1.0f);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] += keep[k];
+    } else if (first && delta) {
+        add(delta + src, 1.0f);
     }
     if constexpr (V == 4 && sizeof(T) == 2) {
         __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3])};
@@ -389,21 +408,25 @@ LI_EXPORT int li_add_row(float* x, const float* row, int T, int H, cudaStream_t 
 }
 
 // out [T, 2 H] in the run dtype: x [T, H] (plus delta [T, H] if given: an output still to be added to the stream) beside x0
-// [T, H], both float.
-LI_EXPORT int li_join_rows(const float* x, const void* delta, const float* x0, void* out, int dtype, int T, int H, cudaStream_t stream) {
+// [T, H], both float.  places (may be NULL): delta is a sum of rows as in li_norm_add_norm (places [T top], weights [T top] and
+// extra [T, H] may be NULL).
+LI_EXPORT int li_join_rows(const float* x, const void* delta, const float* x0, void* out, int dtype, int T, int H, const int* places, int top,
+                           const float* weights, const void* extra, cudaStream_t stream) {
     LI_REQUIRE(T >= 0 && H > 0, "join_rows: bad sizes");
+    LI_REQUIRE(places == nullptr || (delta != nullptr && top > 0), "join_rows: a sum of rows needs the rows and a count");
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "join_rows: unknown dtype %d", dtype);
     if (T == 0) return 0;
     const long long n = 2LL * T * H;
-    const bool vec = H % 4 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)x0 % 16) == 0 && ((uintptr_t)out % 16) == 0;
+    const bool vec = H % 4 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)x0 % 16) == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)delta % 16) == 0 &&
+                     ((uintptr_t)extra % 16) == 0;
     const dim3 grid((unsigned)ceil_div_ll(vec ? n / 4 : n, 256));
     cudaError_t e;
     if (dtype == LI_F32)
-        e = vec ? li_launch_pdl(join_rows_kernel<float, 4>, grid, dim3(256), 0, stream, x, (const float*)delta, x0, (float*)out, n, H)
-                : li_launch_pdl(join_rows_kernel<float, 1>, grid, dim3(256), 0, stream, x, (const float*)delta, x0, (float*)out, n, H);
+        e = vec ? li_launch_pdl(join_rows_kernel<float, 4>, grid, dim3(256), 0, stream, x, (const float*)delta, x0, (float*)out, n, H, places, top, weights, (const float*)extra)
+                : li_launch_pdl(join_rows_kernel<float, 1>, grid, dim3(256), 0, stream, x, (const float*)delta, x0, (float*)out, n, H, places, top, weights, (const float*)extra);
     else
-        e = vec ? li_launch_pdl(join_rows_kernel<bf16, 4>, grid, dim3(256), 0, stream, x, (const bf16*)delta, x0, (bf16*)out, n, H)
-                : li_launch_pdl(join_rows_kernel<bf16, 1>, grid, dim3(256), 0, stream, x, (const bf16*)delta, x0, (bf16*)out, n, H);
+        e = vec ? li_launch_pdl(join_rows_kernel<bf16, 4>, grid, dim3(256), 0, stream, x, (const bf16*)delta, x0, (bf16*)out, n, H, places, top, weights, (const bf16*)extra)
+                : li_launch_pdl(join_rows_kernel<bf16, 1>, grid, dim3(256), 0, stream, x, (const bf16*)delta, x0, (bf16*)out, n, H, places, top, weights, (const bf16*)extra);
     if (e != cudaSuccess) return li_fail("join_rows: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("join_rows");
 }

@@ -75,6 +75,63 @@ __global__ void rope_kv_write_kernel(T* __restrict__ qkv, const int* __restrict_
     }
 }
 
+// Keys and values of many tokens into the cache as they are (rotated before, or not at all), 16 tokens and one key/value head per
+// block, everything in 16-byte pieces: key rows are copied, the values go through shared memory, so that each output column's
+// 16 slots are written as whole pieces when the 16 tokens sit in consecutive slots of one page (the usual case); tokens whose
+// slots are not such a run are written one by one.  head_dim a multiple of 16 bytes.
+template <typename T>
+__global__ void __launch_bounds__(128)
+kv_cache_store_kernel(const T* __restrict__ qkv, const int* __restrict__ slot_mapping, T* __restrict__ kcache, T* __restrict__ vcache, int total, int nh, int nkv,
+                      int dh, int page_size, int num_pages) {
+    extern __shared__ __align__(16) unsigned char vt_raw[];
+    T* vt = reinterpret_cast<T*>(vt_raw);              // [16][dh + V]: the value rows
+    __shared__ int slots[16];
+    constexpr int V = 16 / (int)sizeof(T);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t0 = blockIdx.x * 16, h = blockIdx.y;
+    const int n = min(16, total - t0), pieces = dh / V, ld = dh + V;
+    const size_t row = (size_t)(nh + 2 * nkv) * dh;
+    const T* krow = qkv + (size_t)t0 * row + (size_t)(nh + h) * dh;
+    const T* vrow = krow + (size_t)nkv * dh;
+    if (threadIdx.x < 16) slots[threadIdx.x] = threadIdx.x < n ? slot_mapping[t0 + threadIdx.x] : -1;
+    for (int i = threadIdx.x; i < n * pieces; i += blockDim.x) {
+        const int tk = i / pieces, c = i - tk * pieces;
+        *reinterpret_cast<uint4*>(vt + tk * ld + c * V) = *reinterpret_cast<const uint4*>(vrow + tk * row + c * V);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < n * pieces; i += blockDim.x) {
+        const int tk = i / pieces, c = i - tk * pieces;
+        const int slot = slots[tk];
+        const int page = slot / page_size, off = slot - page * page_size;
+        if (slot < 0 || page >= num_pages) continue;           // validated on the host; never write outside the cache
+        *reinterpret_cast<uint4*>(kcache + (((size_t)page * nkv + h) * page_size + off) * dh + c * V) = *reinterpret_cast<const uint4*>(krow + tk * row + c * V);
+    }
+    const int s0 = slots[0];
+    bool run = n == 16 && s0 >= 0 && (s0 % 16) == 0 && (s0 / page_size) < num_pages && (s0 % page_size) + 16 <= page_size && page_size % 16 == 0;
+    if (run)
+        for (int i = 1; i < 16; ++i) run = run && slots[i] == s0 + i;
+    if (run) {
+        const int page = s0 / page_size, off = s0 - page * page_size;
+        T* dst = vcache + ((size_t)page * nkv + h) * dh * page_size + off;
+        for (int i = threadIdx.x; i < dh * (16 / V); i += blockDim.x) {
+            const int piece = i / dh, d = i - piece * dh;          // neighbouring threads read neighbouring columns
+            __align__(16) T o[V];
+#pragma unroll
+            for (int k = 0; k < V; ++k) o[k] = vt[(piece * V + k) * ld + d];
+            *reinterpret_cast<uint4*>(dst + (size_t)d * page_size + piece * V) = *reinterpret_cast<const uint4*>(o);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n * dh; i += blockDim.x) {
+            const int tk = i / dh, d = i - tk * dh;
+            const int slot = slots[tk];
+            const int page = slot / page_size, off = slot - page * page_size;
+            if (slot < 0 || page >= num_pages) continue;
+            vcache[(((size_t)page * nkv + h) * dh + d) * page_size + off] = vt[tk * ld + d];
+        }
+    }
+}
+
 // The values of many tokens (prefill) into the transposed cache, 16 tokens and one key/value head per block:
 // the tile goes through shared memory, so that each output column's 16 slots are written as one 32-byte
 // piece when the 16 tokens sit in consecutive slots of one page (the usual case), instead of 16 scattered
@@ -153,6 +210,20 @@ LI_EXPORT int li_rope_kv_write(void* qkv, int dtype, const int* positions, const
                rotary_dim, dh);
     LI_REQUIRE(rotary_dim == 0 || denom != nullptr, "rope_kv_write: rotary_dim %d without denominators", rotary_dim);
     if (T == 0) return 0;
+    if (rotary_dim == 0 && !write) return 0;                     // nothing to rotate and nothing to store
+    const int vec = dtype == LI_F32 ? 4 : 8;
+    if (rotary_dim == 0 && T >= 64 && dh % vec == 0 && nkv <= 65535 && ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)kcache % 16) == 0 &&
+        ((uintptr_t)vcache % 16) == 0 && (size_t)16 * (dh + vec) * (16 / vec) <= 48 * 1024) {
+        const dim3 sgrid(ceil_div(T, 16), nkv);
+        const size_t ssmem = (size_t)16 * (dh + vec) * (16 / vec);
+        const cudaError_t e = dtype == LI_F32
+            ? li_launch_pdl(kv_cache_store_kernel<float>, sgrid, dim3(128), ssmem, stream, (const float*)qkv, slot_mapping, (float*)kcache, (float*)vcache, T, nh, nkv,
+                            dh, page_size, num_pages)
+            : li_launch_pdl(kv_cache_store_kernel<bf16>, sgrid, dim3(128), ssmem, stream, (const bf16*)qkv, slot_mapping, (bf16*)kcache, (bf16*)vcache, T, nh, nkv,
+                            dh, page_size, num_pages);
+        if (e != cudaSuccess) return li_fail("rope_kv_write: launch failed: %s", cudaGetErrorString(e));
+        return li_check_launch("rope_kv_write (keys and values)");
+    }
     LI_REQUIRE(T <= 2147483647 && nh + nkv <= 65535, "rope_kv_write: too many heads for one launch");
     const int heads_per_block = T >= 64 ? nh + nkv : 1;
     const int threads = T >= 64 ? 256 : (dh >= 128 ? 64 : 32);
@@ -189,7 +260,7 @@ LI_EXPORT int li_rope_kv_write(void* qkv, int dtype, const int* positions, const
 // Otherwise: the product, then the kernel above.
 int li_linear_gemv_rope(const void* a, const void* w, const float* bias, void* out, int M, int N, int K, const int* positions,
                         const float* denom, const int* slot_mapping, void* kcache, void* vcache, int nh, int nkv, int dh,
-                        int page_size, int num_pages, int write, const RowScale& rs, cudaStream_t stream);
+                        int page_size, int num_pages, int write, const RowScale& rs, void* extra_out, int extra, cudaStream_t stream);
 bool li_gemv_rope_accepts(const void* a, const void* w, int M, int N, int K, int nh, int nkv, int dh, int rotary_dim);
 bool li_tcgen05_rope_wanted(const void* a, const void* w, const void* out, int M, int N, int K);
 int li_linear_tcgen05_rope(const void* a, const void* w, const float* bias, void* out, int M, int N, int K, const RopeEpilogue& rope,
@@ -202,13 +273,17 @@ extern "C" int li_linear_scaled(const void* a, const void* w, const float* bias,
 LI_EXPORT int li_linear_rope_kv(const void* a, const void* w, const float* bias, void* qkv, int dtype, const int* positions,
                                 const float* denom, int rotary_dim, const int* slot_mapping, void* kcache, void* vcache, int T,
                                 int K, int nh, int nkv, int dh, int page_size, int num_pages, int write, int allow_fused,
-                                const float* ssq, int nparts, int width, float eps, const float* cos_sin, cudaStream_t stream) {
+                                const float* ssq, int nparts, int width, float eps, const float* cos_sin, void* extra_out, int extra,
+                                cudaStream_t stream) {
+    // extra heads' worth of rows behind q|k|v in w (and bias): a further map of the same input (an output gate), to extra_out
+    // [T, extra dh]; for few tokens part of the same kernel
     // ssq (or nullptr): partial sums of squares for a factor per token on the product, as in li_linear_scaled
     // cos_sin (or nullptr): the step's table from li_rope_table; with it a long bfloat16 step rotates and writes the cache
     // in the epilogue of the tensor-memory product (head_dim 128)
     const int N = (nh + 2 * nkv) * dh;
     if (T == 0) return 0;
-    if (allow_fused && cos_sin && !ssq && dtype == LI_BF16 && T > 64 && dh == 128 && rotary_dim == 128 && page_size % 16 == 0 &&
+    LI_REQUIRE(extra >= 0 && (extra == 0 || extra_out != nullptr), "linear_rope_kv: %d further heads without an output", extra);
+    if (allow_fused && cos_sin && extra == 0 && !ssq && dtype == LI_BF16 && T > 64 && dh == 128 && rotary_dim == 128 && page_size % 16 == 0 &&
         li_tcgen05_rope_wanted(a, w, qkv, T, N, K)) {
         RopeEpilogue re;
         re.cos_sin = cos_sin;
@@ -232,7 +307,14 @@ LI_EXPORT int li_linear_rope_kv(const void* a, const void* w, const float* bias,
     }
     if (allow_fused && dtype == LI_BF16 && li_gemv_rope_accepts(a, w, T, N, K, nh, nkv, dh, rotary_dim))
         return li_linear_gemv_rope(a, w, bias, qkv, T, N, K, positions, denom, slot_mapping, kcache, vcache, nh, nkv, dh, page_size,
-                                   num_pages, write, rs, stream);
+                                   num_pages, write, rs, extra_out, extra, stream);
+    if (extra) {
+        const size_t esize = dtype == LI_F32 ? 4 : 2;
+        const void* we = (const char*)w + (size_t)N * K * esize;
+        const float* be = bias ? bias + N : nullptr;
+        if (int rc = ssq ? li_linear_scaled(a, we, be, extra_out, dtype, dtype, T, extra * dh, K, LI_EPILOGUE_NONE, ssq, nparts, width, eps, stream)
+                         : li_linear(a, we, be, extra_out, dtype, dtype, T, extra * dh, K, LI_EPILOGUE_NONE, stream)) return rc;
+    }
     if (ssq) {
         if (int rc = li_linear_scaled(a, w, bias, qkv, dtype, dtype, T, N, K, LI_EPILOGUE_NONE, ssq, nparts, width, eps, stream)) return rc;
     } else if (int rc = li_linear(a, w, bias, qkv, dtype, dtype, T, N, K, LI_EPILOGUE_NONE, stream)) return rc;

@@ -162,7 +162,10 @@ def gather_rmsnorm(x32: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, 
            "gather_rmsnorm")
 
 
-def residual_add(x32: torch.Tensor, delta: torch.Tensor) -> None:
+def residual_add(x32: torch.Tensor, delta) -> None:
+    """x32 += delta (float32 sum); ``delta`` may be a :class:`RowSum`."""
+    if isinstance(delta, RowSum):
+        return norm_add_norm(x32, delta, None, None, None)
     _need(x32, "residual", torch.float32)
     _need(delta, "delta", None, x32.shape)
     _check(library().li_residual_add(_p(x32), _p(delta), _i(_dt(delta)), _l(x32.numel()), _stream(x32)), "residual_add")
@@ -388,20 +391,29 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, denominators: torc
 def linear_rope_kv(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], qkv: torch.Tensor,
                    positions: torch.Tensor, denominators: torch.Tensor, rotary_dim: int, slot_mapping: torch.Tensor,
                    k_cache: torch.Tensor, v_cache: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
-                   write: bool = True, fused: bool = True, row_scale=None, cos_sin: Optional[torch.Tensor] = None) -> None:
+                   write: bool = True, fused: bool = True, row_scale=None, cos_sin: Optional[torch.Tensor] = None,
+                   extra: Optional[torch.Tensor] = None) -> None:
     """The fused q|k|v projection followed by :func:`rope_kv_write`: ``qkv = a weight^T + bias``, q rotated in
     place, k rotated and v stored into the caches.  Keys and values are only guaranteed to be in the caches
     afterwards, not in ``qkv``.  For a few bfloat16 tokens both steps run as one kernel (the rotation is the
     product's epilogue); ``fused=False`` forces two kernels, for tests.  ``row_scale`` as in :func:`linear`.
     ``cos_sin``: the step's table from :func:`rope_table`; with it a long bfloat16 step (head_dim 128) rotates and
     writes the cache in the epilogue of the tensor-memory product too.  ``rotary_dim`` 0 (``denominators`` may be
-    None): no rotation, as in :func:`rope_kv_write`."""
+    None): no rotation, as in :func:`rope_kv_write`.
+    ``extra`` [T, n head_dim]: ``weight`` (and ``bias``) hold n heads' worth of further rows behind q|k|v, a map of the same input
+    whose result goes there (an output gate); for few tokens it is part of the same kernel."""
     T, Kd = a.shape
     N = (num_heads + 2 * num_kv_heads) * head_dim
+    more = 0
+    if extra is not None:
+        _need(extra, "output of the further heads", a.dtype, (T, extra.shape[1]))
+        if extra.shape[1] % head_dim:
+            raise KernelError(f"linear_rope_kv: {extra.shape[1]} further columns are no whole heads of {head_dim}")
+        more = extra.shape[1] // head_dim
     _need(a, "linear input")
-    _need(weight, "qkv weight", a.dtype, (N, Kd))
+    _need(weight, "qkv weight", a.dtype, (N + more * head_dim, Kd))
     if bias is not None:
-        _need(bias, "qkv bias", torch.float32, (N,))
+        _need(bias, "qkv bias", torch.float32, (N + more * head_dim,))
     _need(qkv, "qkv", a.dtype, (T, N))
     _need(positions, "positions", torch.int32, (T,))
     if rotary_dim:
@@ -418,7 +430,7 @@ def linear_rope_kv(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.T
         _p(a), _p(weight), _p(bias), _p(qkv), _i(_dt(a)), _p(positions), _p(denominators if rotary_dim else None), _i(rotary_dim), _p(slot_mapping),
         _p(k_cache), _p(v_cache), _i(T), _i(Kd), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(page_size), _i(pages),
         _i(1 if write else 0), _i(1 if fused else 0),
-        *(_row_scale_args(row_scale, T) if row_scale is not None else (_p(None), _i(0), _i(0), _f(0.0))), _p(cos_sin), _stream(qkv)),
+        *(_row_scale_args(row_scale, T) if row_scale is not None else (_p(None), _i(0), _i(0), _f(0.0))), _p(cos_sin), _p(extra), _i(more), _stream(qkv)),
         "linear_rope_kv")
 
 
@@ -1010,15 +1022,26 @@ def norm_add_norm(x32: torch.Tensor, y, post: Optional[tuple], nxt: Optional[tup
                                       _p(y_extra), _stream(x32)), "norm_add_norm")
 
 
-def join_rows(x32: torch.Tensor, delta: Optional[torch.Tensor], x0: torch.Tensor, out: torch.Tensor) -> None:
-    """``out[t] = [x32[t] (+ delta[t]) | x0[t]]`` in the run dtype: what a map of the stream beside the embedding output reads."""
+def join_rows(x32: torch.Tensor, delta, x0: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[t] = [x32[t] (+ delta[t]) | x0[t]]`` in the run dtype: what a map of the stream beside the embedding output reads.
+    ``delta`` may be a :class:`RowSum`: the sum is then taken inside this kernel, in float32."""
     T, H = x32.shape
     _need(x32, "residual stream", torch.float32)
     _need(x0, "embedding output", torch.float32, (T, H))
     _need(out, "joined rows", None, (T, 2 * H))
-    if delta is not None:
+    places, top, weights, extra = None, 0, None, None
+    if isinstance(delta, RowSum):
+        places, top, weights, extra, delta = delta.place_of, delta.top, delta.weights, delta.extra, delta.rows
+        _need(delta, "rows to be added", out.dtype, (delta.shape[0], H))
+        _need(places, "places of a token's rows", torch.int32, (T * top,))
+        if weights is not None:
+            _need(weights, "weights of a token's rows", torch.float32, (T, top))
+        if extra is not None:
+            _need(extra, "a token's further row", out.dtype, (T, H))
+    elif delta is not None:
         _need(delta, "output to be added", out.dtype, (T, H))
-    _check(library().li_join_rows(_p(x32), _p(delta), _p(x0), _p(out), _i(_dt(out)), _i(T), _i(H), _stream(out)), "join_rows")
+    _check(library().li_join_rows(_p(x32), _p(delta), _p(x0), _p(out), _i(_dt(out)), _i(T), _i(H), _p(places), _i(top), _p(weights), _p(extra),
+                                  _stream(out)), "join_rows")
 
 
 def add_row(x32: torch.Tensor, row: torch.Tensor) -> None:
@@ -1198,7 +1221,8 @@ def row_rinv(x: torch.Tensor, ranges, eps: float, out: torch.Tensor) -> None:
 
 def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_offsets: Optional[torch.Tensor] = None,
                    a_group_cols: int = 0, out_group_cols: int = 0, tile_group: Optional[torch.Tensor] = None,
-                   epilogue: Optional[str] = None, epilogue_params: Optional[torch.Tensor] = None) -> None:
+                   epilogue: Optional[str] = None, epilogue_params: Optional[torch.Tensor] = None,
+                   row_source: Optional[Tuple[torch.Tensor, int]] = None) -> None:
     """``weight`` [G, N, K]: a product per group.  With ``row_offsets`` (int32 [G + 1] on the device) group g owns the rows
     ``row_offsets[g] .. row_offsets[g + 1] - 1`` of ``a`` [M, K] and ``out`` [M, N].  Without, every group takes all rows, its
     inputs at column ``g * a_group_cols`` of ``a`` and its outputs at column ``g * out_group_cols`` of ``out`` (a map per head).
@@ -1207,7 +1231,9 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row
     ``epilogue="swiglu"`` (bfloat16, rows in groups): every group's matrix holds gate and up rows interleaved in eights
     (:func:`interleave_gate_up` per group) and ``out`` [M, N / 2] takes ``up * gate / (1 + exp(-gate))``.
     ``epilogue="glu_clamped"``: the same layout, the gated unit with bounded operands; ``epilogue_params`` holds its (limit,
-    alpha), float32 on the device.  Rows that belong to no group (behind ``row_offsets[G]``) are left as they are."""
+    alpha), float32 on the device.  Rows that belong to no group (behind ``row_offsets[G]``) are left as they are.
+    ``row_source`` (int32 [M] on the device, a divisor; bfloat16, rows in groups without padded runs): row r of the groups is row
+    ``row_source[0][r] // row_source[1]`` of ``a``, so that a mixture's rows need not be gathered first."""
     G, N, Kd = weight.shape
     if epilogue not in (None,) + GATED:
         raise KernelError(f"grouped_linear: unknown epilogue {epilogue!r}")
@@ -1221,7 +1247,11 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row
         N_out = N // 2
     else:
         N_out = N
-    M = a.shape[0]
+    M = a.shape[0] if row_source is None else row_source[0].shape[0]
+    if row_source is not None:
+        _need(row_source[0], "source of the rows", torch.int32, (M,))
+        if a.dtype != torch.bfloat16 or row_offsets is None or tile_group is not None or Kd % 8:
+            raise KernelError("grouped_linear: a source of the rows goes with bfloat16 rows in groups, without padded runs, K a multiple of 8")
     _need(a, "grouped input")
     _need(weight, "grouped weights", a.dtype)
     _need(out, "grouped output", a.dtype)
@@ -1239,7 +1269,7 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row
             raise KernelError("grouped_linear: a table of the tiles' groups goes with row offsets and covers every tile of 128 rows")
     _check(library().li_grouped_linear(_p(a), _i(a.shape[1]), _i(a_group_cols), _p(weight), _p(out), _i(out.shape[1]), _i(out_group_cols),
                                        _p(row_offsets), _p(tile_group), _i(_dt(a)), _i(M), _i(N), _i(Kd), _i(G), _i(EPILOGUES[epilogue]), _p(epilogue_params),
-                                       _stream(out)),
+                                       _p(row_source[0] if row_source is not None else None), _i(int(row_source[1]) if row_source is not None else 1), _stream(out)),
            "grouped_linear")
 
 
@@ -1271,6 +1301,37 @@ def moe_route_grouped(logits: torch.Tensor, correction: Optional[torch.Tensor], 
     _need(weights, "expert weights", torch.float32, (T, top))
     _check(library().li_moe_route_grouped(_p(logits), _p(correction), _i(T), _i(E), _i(top), _i(int(groups)), _i(int(keep)), _f(float(scale)),
                                           _p(ids), _p(weights), _stream(ids)), "moe_route_grouped")
+
+
+MOE_SCORINGS = {"sigmoid": 0, "softmax_chosen": 1, "softmax_grouped": 2}
+
+
+def moe_small_step_accepts(h: torch.Tensor, experts: int, top: int) -> bool:
+    """Whether :func:`moe_small_step` takes a step of these tokens (few enough for one block)."""
+    return bool(library().li_moe_small_step_accepts(_i(_dt(h)), _i(h.shape[0]), _i(h.shape[1]), _i(int(experts)), _i(int(top))))
+
+
+def moe_small_step(h: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], top: int, scoring: str, correction: Optional[torch.Tensor],
+                   groups: int, keep: int, scale: float, weights: torch.Tensor, offsets: torch.Tensor, pair_at: torch.Tensor,
+                   place_of: torch.Tensor) -> None:
+    """The front of a mixture for a step of few tokens as one launch: the router's product ``h router^T (+ bias)`` with float32
+    sums, the choice (``scoring`` as in :func:`moe_route`, or "softmax_grouped" as :func:`moe_route_grouped`) and the sort of
+    :func:`moe_sort` without padding: ``weights`` [T, top], ``offsets`` [E + 1], ``pair_at`` and ``place_of`` [T top]."""
+    T, H = h.shape
+    E = router.shape[0]
+    _need(h, "feed-forward input")
+    _need(router, "router weight", h.dtype, (E, H))
+    if bias is not None:
+        _need(bias, "router bias", torch.float32, (E,))
+    if correction is not None:
+        _need(correction, "correction of the choice scores", torch.float32, (E,))
+    _need(weights, "expert weights", torch.float32, (T, top))
+    _need(offsets, "row offsets", torch.int32, (E + 1,))
+    _need(pair_at, "pair at place", torch.int32, (T * top,))
+    _need(place_of, "place of pair", torch.int32, (T * top,))
+    _check(library().li_moe_small_step(_p(h), _p(router), _p(bias), _i(_dt(h)), _i(T), _i(H), _i(E), _i(int(top)), _i(MOE_SCORINGS[scoring]), _p(correction),
+                                       _i(int(groups)), _i(int(keep)), _f(float(scale)), _p(weights), _p(offsets), _p(pair_at), _p(place_of), _stream(h)),
+           "moe_small_step")
 
 
 def sorted_rows(pairs: int, experts: int, pad: int = 1) -> int:
@@ -1429,7 +1490,7 @@ _TIMED = ("embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add
           "rope_kv_write", "linear_rope_kv", "rope_table", "paged_attention", "swiglu", "argmax", "sample", "gather_rows", "scale_inplace",
           "logit_cap", "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift",
           "ssm_scan", "decay_scan", "gated_rmsnorm", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route",
-          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference")
+          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step")
 if profile.enabled:
     for _name in _TIMED:
         globals()[_name] = profile.wrap(_name, globals()[_name])

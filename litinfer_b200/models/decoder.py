@@ -178,6 +178,8 @@ class DecoderModel:
             follows = s.schedule[i + 1] if i < last else None
             next_entry = self.blocks[follows.block].entry() if follows is not None and follows.add is None and follows.join is None else None
             x32, carry = self.blocks[e.block].forward(x32, ctx, caches[i], carry, next_entry)
+            if carry is not None and isinstance(carry.delta, K.RowSum) and follows is not None and follows.add is None and follows.join is None:
+                carry.delta = carry.delta.materialize()              # (a block that was not told of this one's end takes tensors)
             if self.observer is not None:
                 self.observer(i, x32, carry)
         if carry is not None and carry.delta is not None:

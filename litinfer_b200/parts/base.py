@@ -174,8 +174,8 @@ class Tail:
 
 @dataclass
 class Carry:
-    """From one block to the next: ``delta`` is still to be added to the residual stream;
-    ``normed`` is the next block's first norm of the stream, which already holds everything."""
+    """From one block to the next: ``delta`` is still to be added to the residual stream (a tensor; to the model itself also a
+    ``kernels.RowSum``, which it resolves before it hands the carry to another block); ``normed`` is the next block's first norm of the stream, which already holds everything."""
 
     delta: Optional[torch.Tensor] = None
     normed: Optional[torch.Tensor] = None

@@ -64,7 +64,9 @@ class PreNormBlock(Block):
             return x32, Carry(normed=self.mixer.forward_into(h, ctx, cache, Tail(x32, next_entry.norm, next_entry.defer)))
         h = self.mixer.forward_into(h, ctx, cache, Tail(x32, self.feed_forward_norm, self.feed_forward.takes_deferred))
         if next_entry is None:
-            return x32, Carry(delta=self.feed_forward.forward(h, ctx))
+            # (a mixture of experts hands its rows over as they are: whatever adds them to the stream sums a token's rows itself)
+            rows = getattr(self.feed_forward, "produces_row_sums", False)
+            return x32, Carry(delta=self.feed_forward.forward_rows(h, ctx) if rows else self.feed_forward.forward(h, ctx))
         return x32, Carry(normed=self.feed_forward.forward_into(h, ctx, Tail(x32, next_entry.norm, next_entry.defer)))
 
 

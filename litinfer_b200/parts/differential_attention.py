@@ -64,6 +64,8 @@ class DifferentialAttention(Mixer):
         self.out = FusedLinear(prefix, [n.get("o", "o_proj")], H * self.value_dim, [self.hidden], False, dtype, suffixes=suffixes)
         self.mix_names = [prefix + n.get(k, k) for k in ("lq1", "lk1", "lq2", "lk2")]
         self.mix = 0.0
+        self.weight = self.bias = None                   # what the first product reads, made when the weights are bound
+        self.joined = False
 
     def params(self) -> List[ParamSpec]:
         return (self.qkv.params() + (self.gate.params() if self.gate is not None else []) + self.out.params()
@@ -78,6 +80,14 @@ class DifferentialAttention(Mixer):
         self.mix = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + self.diff
         if self.head_dim != MAPS * self.qk_dim or self.head_dim != self.value_dim:
             self._pad_heads()
+        # a gate whose heads are as wide as the cache's joins the q|k|v product (its rows behind them, with a bias of zeros)
+        self.joined = self.gate is not None and self.value_dim == self.head_dim
+        self.weight, self.bias = self.qkv.weight, self.qkv.bias
+        if self.joined:
+            self.weight = torch.cat([self.qkv.weight, self.gate.weight], dim=0).contiguous()
+            if self.bias is not None:
+                self.bias = torch.cat([self.bias, torch.zeros(self.gate.out_features, dtype=self.bias.dtype, device=self.bias.device)]).contiguous()
+            self.qkv.weight = self.gate.weight = None
 
     def _pad_heads(self) -> None:
         """Zero rows of q, k and v (with their biases) up to the cache's head size, behind each map's queries and keys."""
@@ -111,13 +121,15 @@ class DifferentialAttention(Mixer):
         """Everything before the output projection: [tokens, heads * value_dim]."""
         H, G, D = self.num_heads, self.num_kv_heads, self.head_dim
         view = ctx.group(cache.group)
-        gate = self.gate(h) if self.gate is not None else None
-        h, row_scale = undefer(h, self.qkv.weight)
+        gate = self.gate(h) if self.gate is not None and not self.joined else None
+        h, row_scale = undefer(h, self.weight)
         T = h.shape[0]
-        qkv = torch.empty((T, self.qkv.out_features), dtype=self.dtype, device=h.device)
-        # projection and keys and values into the cache: one call (and for few tokens one kernel)
-        K.linear_rope_kv(h, self.qkv.weight, self.qkv.bias, qkv, ctx.positions, None, 0, view.slot_mapping, cache.k, cache.v, H, G, D, cache.writes,
-                         row_scale=row_scale)
+        if self.joined:
+            gate = torch.empty((T, H * D), dtype=self.dtype, device=h.device)
+        qkv = torch.empty((T, (H + 2 * G) * D), dtype=self.dtype, device=h.device)
+        # projection (with the gate's) and keys and values into the cache: one call (and for few tokens one kernel)
+        K.linear_rope_kv(h, self.weight, self.bias, qkv, ctx.positions, None, 0, view.slot_mapping, cache.k, cache.v, H, G, D, cache.writes,
+                         row_scale=row_scale, extra=gate if self.joined else None)
         both = torch.empty((T, MAPS * H * D), dtype=self.dtype, device=h.device)
         K.paged_attention(
             qkv, both, cache.k, cache.v, view.block_table, ctx.q_start, ctx.ctx_lens, ctx.seq_of_token, ctx.positions,

@@ -21,7 +21,8 @@ feed-forward that every token takes; its output joins the sum of the chosen expe
 ``activation`` "glu_clamped" (with ``limit``, ``alpha``): ``g = min(W_gate u, limit)``, ``up = clamp(W_up u, -limit, limit)``,
 the expert's inner activation is ``g sigmoid(alpha g) (up + 1)`` instead of ``silu(gate) up``.
 
-How a step runs it: the router's product with a float32 result, the choice per token (one warp a token), a stable
+How a step runs it (a step of few tokens: router, choice and sort in one launch, and no gather: the first product reads the
+tokens' rows in place): the router's product with a float32 result, the choice per token (one warp a token), a stable
 counting sort of the (token, choice) pairs by expert on the device (in a step of many tokens every expert's run starts
 at a multiple of 128 rows), one gather that builds the experts' input rows in sorted order (with the weight on them), a product per expert over its run of rows for gate|up and for down
 (``kernels.grouped_linear`` with the row offsets the sort left on the device), and a combine that sums a token's rows in
@@ -147,33 +148,40 @@ class RoutedExperts(FeedForward):
         E, top, F = self.experts, self.top, self.intermediate
         n_out = self.outputs                                   # experts and identity experts: what the router chooses among
         dev = h.device
-        logits = self.router(h, out_dtype=torch.float32)
-        ids = torch.empty((T, top), dtype=torch.int32, device=dev)
         weights = torch.empty((T, top), dtype=torch.float32, device=dev)
-        if self.scoring == "softmax_grouped":
-            K.moe_route_grouped(logits, self.correction, top, self.groups, self.keep_groups, self.route_scale, ids, weights)
-        elif self.scoring == "softmax":
-            K.moe_route_grouped(logits, None, top, 1, 1, 1.0, ids, weights)
-        else:
-            K.moe_route(logits, top, ids, weights, scoring=self.scoring)
+        offsets = torch.empty(n_out + 1, dtype=torch.int32, device=dev)
+        place_of = torch.empty(T * top, dtype=torch.int32, device=dev)
         # a step of many tokens: every expert's run of rows starts at a multiple of 128, so that the products run on
         # tensor-core tiles of 128 rows, each of one expert
         pad = self.PAD if (self.dtype == torch.bfloat16 and T * top >= self.PAD_FROM_ROWS) else 1
         R = K.sorted_rows(T * top, n_out, pad)
-        offsets = torch.empty(n_out + 1, dtype=torch.int32, device=dev)
         pair_at = torch.empty(R, dtype=torch.int32, device=dev)
-        place_of = torch.empty(T * top, dtype=torch.int32, device=dev)
         tiles = torch.empty(R // pad, dtype=torch.int32, device=dev) if pad > 1 else None
-        K.moe_sort(ids, n_out, offsets, pair_at, place_of, pad, tiles, matrices=E)
+        grouped = self.scoring in ("softmax_grouped", "softmax")
+        if pad == 1 and K.moe_small_step_accepts(h, n_out, top):
+            # few tokens: the router's product, the choice and the sort are one launch
+            K.moe_small_step(h, self.router.weight, self.router.bias, top, "softmax_grouped" if grouped else self.scoring, self.correction, self.groups,
+                             self.keep_groups, self.route_scale, weights, offsets, pair_at, place_of)
+        else:
+            logits = self.router(h, out_dtype=torch.float32)
+            ids = torch.empty((T, top), dtype=torch.int32, device=dev)
+            if grouped:
+                K.moe_route_grouped(logits, self.correction, top, self.groups, self.keep_groups, self.route_scale, ids, weights)
+            else:
+                K.moe_route(logits, top, ids, weights, scoring=self.scoring)
+            K.moe_sort(ids, n_out, offsets, pair_at, place_of, pad, tiles, matrices=E)
         # (the products see the experts' runs only: the identity experts' rows, behind them, stay as the gather made them)
         expert_offsets = offsets[:E + 1] if n_out != E else offsets
         on_input = self.weight_on == "input"
         rows = torch.empty((R, self.hidden), dtype=self.dtype, device=dev)
-        K.moe_gather(h, pair_at, weights if on_input else None, top, rows)
+        # the first product reads the tokens' rows where they are when it can; else they are gathered in sorted order
+        in_place = self.fused_activation and pad == 1 and not on_input and not self.identity
+        if not in_place:
+            K.moe_gather(h, pair_at, weights if on_input else None, top, rows)
         act = torch.empty((R, F), dtype=self.dtype, device=dev)
         if self.fused_activation:
-            K.grouped_linear(rows, self.gate_up, act, expert_offsets, tile_group=tiles, epilogue=self.activation,
-                             epilogue_params=self.activation_params)
+            K.grouped_linear(h if in_place else rows, self.gate_up, act, expert_offsets, tile_group=tiles, epilogue=self.activation,
+                             epilogue_params=self.activation_params, row_source=(pair_at, top) if in_place else None)
         else:
             both = torch.empty((R, 2 * F), dtype=self.dtype, device=dev)
             K.grouped_linear(rows, self.gate_up, both, expert_offsets, tile_group=tiles)

@@ -18,7 +18,7 @@ dims - 1)`` and ``ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` the fre
 f_i (1 - ramp_i)``, and cosines and sines carry the magnitude ``0.1 ln(factor) + 1`` (:attr:`Rotary.magnitude`).
 
 ``pairing`` "interleaved": element 2j turns with element 2j + 1.  Only mixers whose kernels take that pairing accept it
-(:attr:`Rotary.interleaved`); the paged attention part rotates halves.
+(:attr:`Rotary.interleaved`).
 """
 
 from __future__ import annotations

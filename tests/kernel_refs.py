@@ -44,7 +44,7 @@ def gather_rmsnorm(x32, rows, weight, eps, out):
 
 
 def residual_add(x32, delta):
-    x32.add_(delta.float())
+    x32.add_(_row_sum(delta) if hasattr(delta, "place_of") else delta.float())
 
 
 def linear(a, weight, bias, out, epilogue=None, row_scale=None, epilogue_params=None):
@@ -146,7 +146,11 @@ def rope_kv_write(qkv, positions, denominators, rotary_dim, slot_mapping, k_cach
 
 
 def linear_rope_kv(a, weight, bias, qkv, positions, denominators, rotary_dim, slot_mapping, k_cache, v_cache,
-                   num_heads, num_kv_heads, head_dim, write=True, fused=True, row_scale=None, cos_sin=None):
+                   num_heads, num_kv_heads, head_dim, write=True, fused=True, row_scale=None, cos_sin=None, extra=None):
+    N = (num_heads + 2 * num_kv_heads) * head_dim
+    if extra is not None:
+        linear(a, weight[N:], bias[N:] if bias is not None else None, extra, row_scale=row_scale)
+        weight, bias = weight[:N], bias[:N] if bias is not None else None
     linear(a, weight, bias, qkv, row_scale=row_scale)
     rope_kv_write(qkv, positions, denominators, rotary_dim, slot_mapping, k_cache, v_cache, num_heads, num_kv_heads, head_dim, write)
 
@@ -262,14 +266,15 @@ def _norm_of(v, spec):
     return v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * weight
 
 
+def _row_sum(y):
+    r = y.rows[y.place_of.long()].float().view(y.shape[0], y.top, y.shape[1])
+    r = (r * y.weights[:, :, None] if y.weights is not None else r).sum(1)
+    return r + y.extra.float() if y.extra is not None else r
+
+
 def norm_add_norm(x32, y, post, nxt, out, rows=None):
     if hasattr(y, "place_of"):                           # a sum of rows (kernels.RowSum), taken in float32
-        T, H = x32.shape
-        r = y.rows[y.place_of.long()].float().view(T, y.top, H)
-        extra = y.extra
-        y = (r * y.weights[:, :, None] if y.weights is not None else r).sum(1)
-        if extra is not None:
-            y = y + extra.float()
+        y = _row_sum(y)
     if y is not None:
         x32.add_(_norm_of(y, post) if post is not None else y.float())
     if nxt is not None:
@@ -277,7 +282,10 @@ def norm_add_norm(x32, y, post, nxt, out, rows=None):
 
 
 def join_rows(x32, delta, x0, out):
-    _store(out, torch.cat([x32 + delta.float() if delta is not None else x32, x0], dim=-1))
+    x = x32
+    if delta is not None:
+        x = x32 + (_row_sum(delta) if hasattr(delta, "place_of") else delta.float())
+    _store(out, torch.cat([x, x0], dim=-1))
 
 
 def add_row(x32, row):
@@ -423,8 +431,11 @@ def add_pair_rows(x32, pairs, ids, positions, q_start, seq_of_token, slots, stat
         state[sl[s], 0] = prev
 
 
-def grouped_linear(a, weight, out, row_offsets=None, a_group_cols=0, out_group_cols=0, tile_group=None, epilogue=None, epilogue_params=None):
+def grouped_linear(a, weight, out, row_offsets=None, a_group_cols=0, out_group_cols=0, tile_group=None, epilogue=None, epilogue_params=None,
+                   row_source=None):
     G, N, Kd = weight.shape
+    if row_source is not None:
+        a = a[(row_source[0] // row_source[1]).long()]
     if row_offsets is not None:
         offs = row_offsets.tolist()
         for g in range(G):
@@ -461,6 +472,22 @@ def moe_route(logits, top, ids, weights, scoring="sigmoid"):
     order = torch.sort(s - torch.arange(E, device=s.device) * 0.0, dim=-1, descending=True, stable=True)
     ids.copy_(order.indices[:, :top].to(torch.int32))
     weights.copy_(order.values[:, :top])
+
+
+def moe_small_step_accepts(h, experts, top):
+    return h.shape[0] * top < 64
+
+
+def moe_small_step(h, router, bias, top, scoring, correction, groups, keep, scale, weights, offsets, pair_at, place_of):
+    logits = h.float() @ router.float().t()
+    if bias is not None:
+        logits = logits + bias
+    ids = torch.empty((h.shape[0], top), dtype=torch.int32, device=h.device)
+    if scoring == "softmax_grouped":
+        moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights)
+    else:
+        moe_route(logits, top, ids, weights, scoring)
+    moe_sort(ids, router.shape[0], offsets, pair_at, place_of)
 
 
 def sorted_rows(pairs, experts, pad=1):
@@ -871,7 +898,7 @@ def table_gather(resident, updates, slots, out, trash_page):
             out[s, b] = resident[slot, b] if b < cols else trash_page
 
 
-ALL = ["geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
+ALL = ["moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
        "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift", "ssm_scan",
        "decay_scan", "gated_rmsnorm", "table_gather", "gather_rows", "scale_inplace", "logit_cap", "rope_table", "linear_scaled_accepts", "linear_add_scaled_parts", "linear_add_scaled", "apply_row_scale", "linear_rope_kv", "interleave_gate_up", "embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add", "linear", "rope_kv_write",
        "paged_attention", "swiglu", "argmax", "sample"]

@@ -771,6 +771,14 @@ def test_stream_beside_the_embedding_and_sums_with_a_further_row_kernels(dtype):
         K.moe_combine(rows, places, wts, top, y, extra=delta)
         R.moe_combine(rows, places, wts, top, want, extra=delta)
         _close(y, want, dtype, "combined")
+        both, ref2 = (torch.empty(T, 2 * H, dtype=dt, device=dev) for _ in range(2))
+        K.join_rows(x, K.RowSum(rows, places, top, wts, extra=delta), x0, both)
+        R.join_rows(x, K.RowSum(rows, places, top, wts, extra=delta), x0, ref2)
+        _close(both, ref2, dtype, "joined with a sum of rows")
+        rx = x.clone()
+        K.residual_add(x, K.RowSum(rows, places, top, None, extra=None))
+        R.residual_add(rx, K.RowSum(rows, places, top, None, extra=None))
+        _close(x, rx, "float32", "a sum of rows added to the stream", 1e-5)
 
 
 @pytest.mark.gpu
@@ -806,3 +814,94 @@ def test_gelu_unit_as_a_kernel_and_as_an_epilogue_of_every_product():
         K.grouped_linear(a, w, out, offsets, tile_group=tiles, epilogue="geglu")
         R.grouped_linear(a, w, ref, offsets, tile_group=tiles, epilogue="geglu")
         _close(out, ref, "bfloat16", f"groups of {per} rows")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_front_of_a_mixture_in_one_launch_and_rows_read_in_place(dtype):
+    """Router, choice and sort of a small step against the kernels they stand for; the first product of the experts with the
+    tokens' rows read where they are against the gathered rows."""
+    import kernel_refs as R
+    from litinfer_b200 import kernels as K
+
+    dev, dt = torch.device("cuda:0"), _dt(dtype)
+    torch.manual_seed(12)
+    for T, E, top, H, scoring, groups, keep in ((1, 8, 2, 64, "softmax_grouped", 1, 1), (9, 5, 3, 48, "softmax_grouped", 5, 4), (32, 12, 4, 96, "sigmoid", 1, 1),
+                                                (40, 3, 1, 1536, "softmax_chosen", 1, 1), (64, 8, 3, 256, "softmax_grouped", 4, 2), (4, 100, 6, 128, "softmax_grouped", 1, 1)):
+        h = torch.randn(T, H).to(dev, dt)
+        w = (2.0 * torch.randn(E, H) / math.sqrt(H)).to(dev, dt)
+        bias = (0.3 * torch.randn(E)).to(dev) if scoring == "softmax_chosen" else None
+        corr = (0.05 * torch.randn(E)).to(dev) if groups > 1 else None
+        assert K.moe_small_step_accepts(h, E, top)
+        res = []
+        for F in (K, R):
+            wt = torch.empty(T, top, device=dev)
+            off, at, place = (torch.empty(n, dtype=torch.int32, device=dev) for n in (E + 1, T * top, T * top))
+            F.moe_small_step(h, w, bias, top, scoring, corr, groups, keep, 1.3, wt, off, at, place)
+            res.append((wt, off, at, place))
+        assert torch.equal(res[0][1], res[1][1]) and torch.equal(res[0][2], res[1][2]) and torch.equal(res[0][3], res[1][3]), f"{T} tokens, {E} experts"
+        assert (res[0][0] - res[1][0]).abs().max() < 1e-4
+        if dtype == "bfloat16":
+            _, off, at, _ = res[0]
+            gu = (torch.randn(E, 96, H) / math.sqrt(H)).to(dev, dt)
+            params = torch.tensor([1.2, 1.702], device=dev)
+            rows = torch.empty(T * top, H, dtype=dt, device=dev)
+            K.moe_gather(h, at, None, top, rows)
+            out, want = (torch.empty(T * top, 48, dtype=dt, device=dev) for _ in range(2))
+            K.grouped_linear(h, gu, out, off, epilogue="glu_clamped", epilogue_params=params, row_source=(at, top))
+            K.grouped_linear(rows, gu, want, off, epilogue="glu_clamped", epilogue_params=params)
+            assert torch.equal(out, want)
+    assert not K.moe_small_step_accepts(torch.empty(300, 64, dtype=dt, device=dev), 8, 2)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T", [3, 20, 70])
+def test_projection_with_a_gate_behind_it_kernel(T, dtype):
+    """q|k|v and a further map of the same input in one call: one kernel for few tokens, separate products otherwise."""
+    import kernel_refs as R
+    from litinfer_b200 import kernels as K
+
+    dev, dt = torch.device("cuda:0"), _dt(dtype)
+    torch.manual_seed(T)
+    nh, nkv, dh, more, W, page = 3, 2, 32, 3, 64, 16
+    w = (torch.randn((nh + 2 * nkv + more) * dh, W) / 8).to(dev, dt)
+    b = (0.2 * torch.randn((nh + 2 * nkv + more) * dh)).to(dev)
+    a = torch.randn(T, W).to(dev, dt)
+    pos = torch.arange(T, dtype=torch.int32, device=dev)
+    slots = (torch.arange(T, dtype=torch.int32) + 16).to(dev)
+    ssq = (torch.rand(T, 4, device=dev) + 0.5).contiguous()
+    for scale in (None, (ssq, W, 1e-5)):
+        if scale is not None and (dtype == "float32" or T > 64):
+            continue
+        res = []
+        for F in (K, R):
+            qkv, gate = torch.zeros(T, (nh + 2 * nkv) * dh, dtype=dt, device=dev), torch.zeros(T, more * dh, dtype=dt, device=dev)
+            kc, vc = torch.zeros(8, nkv, page, dh, dtype=dt, device=dev), torch.zeros(8, nkv, dh, page, dtype=dt, device=dev)
+            F.linear_rope_kv(a, w, b, qkv, pos, None, 0, slots, kc, vc, nh, nkv, dh, row_scale=scale, extra=gate)
+            res.append((qkv[:, :nh * dh], gate, kc, vc))
+        for x, y, what in zip(res[0], res[1], ("queries", "gate", "keys", "values")):
+            _close(x, y, dtype, f"{what}, {T} tokens")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("dh,page", [(24, 16), (128, 32), (20, 16), (9, 16)])
+def test_keys_and_values_of_a_long_step_into_pages_kernel(dh, page, dtype):
+    """Runs of consecutive slots (whole pieces of pages), a ragged end, and slots in any order."""
+    import kernel_refs as R
+    from litinfer_b200 import kernels as K
+
+    dev, dt = torch.device("cuda:0"), _dt(dtype)
+    torch.manual_seed(dh)
+    nh, nkv = 2, 3
+    for T, order in ((96, "run"), (101, "run"), (75, "any"), (80, "late")):
+        qkv = torch.randn(T, (nh + 2 * nkv) * dh).to(dev, dt)
+        slots = torch.randperm(12 * page)[:T] if order == "any" else torch.arange(T) + (page if order == "run" else 5)
+        slots = slots.to(torch.int32).to(dev)
+        res = []
+        for F in (K, R):
+            kc, vc = torch.zeros(13, nkv, page, dh, dtype=dt, device=dev), torch.zeros(13, nkv, dh, page, dtype=dt, device=dev)
+            F.rope_kv_write(qkv.clone(), torch.zeros(T, dtype=torch.int32, device=dev), None, 0, slots, kc, vc, nh, nkv, dh)
+            res.append((kc, vc))
+        assert torch.equal(res[0][0], res[1][0]) and torch.equal(res[0][1], res[1][1]), f"{T} tokens, {order}"
