@@ -8,6 +8,9 @@
 // stages) and keeps the accumulator of its rows, 256 columns of tensor memory.  The other 256 columns hold the tile before:
 // the four epilogue warps of each CTA read it, apply bias or SwiGLU and store, while the first CTA's issuer already
 // multiplies the next tile; the producers run ahead through the ring of stages without regard to tile boundaries.
+// Products in groups (a mixture's experts): every 256 rows of a belong to one group, which a table on the device names; the
+// groups' matrices lie one below the other in the tensor map of w, a tile adds group * N to its row there, and tiles of no group
+// are passed over by every role alike.
 // Tiles are taken in the order (row pair fastest, then columns), so that the pairs at work at one time share few tiles of w.
 //
 // Barriers: full / empty per stage as in gemm_tcgen05.cu (both CTAs' loads are counted on the first CTA's full barrier; the
@@ -43,7 +46,8 @@ struct __align__(1024) Smem {
 template <typename Tout, int kSwiglu>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-                               const float* __restrict__ bias, Tout* __restrict__ out, int M, int N, int K, int* __restrict__ error_flag) {
+                               const float* __restrict__ bias, Tout* __restrict__ out, int M, int N, int K, int* __restrict__ error_flag,
+                               const int* __restrict__ tile_group) {
     extern __shared__ unsigned char smem_raw[];
     Smem& sm = *reinterpret_cast<Smem*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -84,6 +88,8 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
             bool ok = true;
             int it = 0;                               // k-blocks loaded so far, over all tiles
             for (int t = pair; t < total && ok; t += npairs) {
+                const int group = tile_group ? tile_group[t % row_pairs] : 0;
+                if (group < 0) continue;
                 const int m0 = ((t % row_pairs) * 2 + (int)rank) * kRows, n0 = (t / row_pairs) * BN;
                 for (int kb = 0; kb < nkb; ++kb, ++it) {
                     const int s = it % kStages;
@@ -91,7 +97,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
                     if (!ok) break;
                     if (rank == 0) mbar_expect_tx(&sm.full[s], 2 * (kBytesA + kBytesB));
                     tma_load_2d_pair(sm.a[s], &map_a, kb * BK, m0, &sm.full[s]);
-                    tma_load_2d_pair(sm.b[s], &map_w, kb * BK, n0 + (int)rank * (BN / 2), &sm.full[s]);
+                    tma_load_2d_pair(sm.b[s], &map_w, kb * BK, group * N + n0 + (int)rank * (BN / 2), &sm.full[s]);
                 }
             }
             if (!ok) atomicExch(error_flag, 21);
@@ -101,7 +107,8 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
             constexpr unsigned idesc = umma_idesc(2 * kRows, BN);
             bool ok = true;
             int it = 0, ti = 0;
-            for (int t = pair; t < total && ok; t += npairs, ++ti) {
+            for (int t = pair; t < total && ok; t += npairs) {
+                if (tile_group && tile_group[t % row_pairs] < 0) continue;
                 const unsigned acc = tmem_acc + (unsigned)((ti & 1) * BN);
                 ok = mbar_wait(&sm.acc_empty[ti & 1], ((ti >> 1) & 1) ^ 1);     // both epilogues are done with this accumulator
                 if (!ok) break;
@@ -118,6 +125,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
                     umma_commit_pair(&sm.empty[s]);
                 }
                 if (ok) umma_commit_pair(&sm.acc_full[ti & 1]);
+                ++ti;
             }
             if (!ok) atomicExch(error_flag, 22);
         }
@@ -126,7 +134,8 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
         const int quarter = warp & 3;
         bool ok = true;
         int ti = 0;
-        for (int t = pair; t < total && ok; t += npairs, ++ti) {
+        for (int t = pair; t < total && ok; t += npairs) {
+            if (tile_group && tile_group[t % row_pairs] < 0) continue;
             const int m0 = ((t % row_pairs) * 2 + (int)rank) * kRows, n0 = (t / row_pairs) * BN;
             ok = mbar_wait(&sm.acc_full[ti & 1], (ti >> 1) & 1);
             if (!ok) break;
@@ -142,6 +151,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
             if (lane == 0) mbar_arrive_remote(&sm.acc_empty[ti & 1], 0);
+            ++ti;
         }
         if (!ok && lane == 0) atomicExch(error_flag, 23);
     }
@@ -156,7 +166,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
 }
 
 template <typename Tout, int kSwiglu>
-int launch(const void* a, const void* w, const float* bias, void* out, int M, int N, int K, cudaStream_t stream) {
+int launch(const void* a, const void* w, const float* bias, void* out, int M, int N, int K, cudaStream_t stream, const int* tile_group = nullptr, int G = 1) {
     EncodeTiledFn encode = nullptr;
     int *err_host = nullptr, *err_dev = nullptr;
     if (int rc = setup(&encode, &err_host, &err_dev)) return rc;
@@ -164,7 +174,7 @@ int launch(const void* a, const void* w, const float* bias, void* out, int M, in
         return li_fail("linear (tcgen05, persistent): an earlier launch gave up waiting on a barrier (status %d); the results since then are invalid", *err_host);
     CUtensorMap map_a, map_w;
     if (int rc = make_map(&map_a, a, M, K, kRows)) return rc;
-    if (int rc = make_map(&map_w, w, N, K, BN / 2)) return rc;
+    if (int rc = make_map(&map_w, w, G * N, K, BN / 2)) return rc;
     const size_t smem = sizeof(Smem) + 1024;
     static bool raised = false;
     if (!raised) {
@@ -183,7 +193,7 @@ int launch(const void* a, const void* w, const float* bias, void* out, int M, in
     int pairs = sms / 2;
     if (pairs > total) pairs = total;
     li_launch_pdl(gemm_tcgen05_persistent_kernel<Tout, kSwiglu>, dim3(2 * pairs), dim3(kThreads), smem, stream, dim3(2, 1, 1), map_a, map_w, bias,
-                  (Tout*)out, M, N, K, err_dev);
+                  (Tout*)out, M, N, K, err_dev, tile_group);
     return li_check_launch("linear (tcgen05, persistent)");
 }
 
@@ -208,4 +218,19 @@ int li_linear_tcgen05_persistent(const void* a, const void* w, const float* bias
     if (dtype_out == LI_BF16) return launch<bf16, 0>(a, w, bias, out, M, N, K, stream);
     if (dtype_out == LI_F32) return launch<float, 0>(a, w, bias, out, M, N, K, stream);
     return li_fail("linear (tcgen05, persistent): unsupported output dtype %d", dtype_out);
+}
+
+// Products in groups on pairs of CTAs: a [M, K] with M a multiple of 256, every 256 rows of one group (tile_group[M / 256], -1:
+// none); w [G, N, K]; out [M, N] bfloat16, or [M, N / 2] with a gated epilogue.
+int li_linear_tcgen05_grouped_pairs(const void* a, const void* w, void* out, int M, int N, int K, int G, const int* tile_group, int epilogue,
+                                    const float* glu_params, cudaStream_t stream) {
+    LI_REQUIRE(M % (2 * kRows) == 0 && G >= 1 && tile_group != nullptr, "grouped linear (tcgen05, pairs): rows %d must be whole tiles of 256 with a table of their groups", M);
+    LI_REQUIRE(K >= 8 && K % 8 == 0 && ((uintptr_t)a % 16 == 0) && ((uintptr_t)w % 16 == 0), "grouped linear (tcgen05, pairs): refuses K=%d or unaligned operands", K);
+    LI_REQUIRE((long long)G * N < (1LL << 31), "grouped linear (tcgen05, pairs): %d matrices of %d rows are too many", G, N);
+    const bool gated = li_epilogue_is_gated(epilogue);
+    LI_REQUIRE(!gated || N % 16 == 0, "grouped linear (tcgen05, pairs): a gated epilogue needs N a multiple of 16, got %d", N);
+    if (epilogue == LI_EPILOGUE_GLU_CLAMPED) return launch<bf16, 2>(a, w, glu_params, out, M, N, K, stream, tile_group, G);
+    if (epilogue == LI_EPILOGUE_GEGLU) return launch<bf16, 3>(a, w, nullptr, out, M, N, K, stream, tile_group, G);
+    if (gated) return launch<bf16, 1>(a, w, nullptr, out, M, N, K, stream, tile_group, G);
+    return launch<bf16, 0>(a, w, nullptr, out, M, N, K, stream, tile_group, G);
 }

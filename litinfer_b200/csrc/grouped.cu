@@ -129,14 +129,15 @@ __device__ __forceinline__ void mma16816(float (&c)[4], unsigned a0, unsigned a1
 // kSwiglu (1, 3: GEGLU, or 2: the gated unit with bounded operands, glu_params = {limit, alpha} on the device): the columns come as 8 gate,
 // 8 up, 8 gate, 8 up, ... (the rows of every group's matrix interleaved in eights), and out [M, N / 2] takes
 // up * gate / (1 + exp(-gate)) (or the bounded unit): a thread holds a gate column and its up column in neighbouring tiles of 8.
-template <int TM, int TK, int ST, int kSwiglu>
+// TN columns a CTA: 64, or 32 for few rows and a product of few columns (more CTAs, six stages: more of the weights on their way).
+template <int TM, int TK, int ST, int kSwiglu, int TN = 64>
 __global__ void __launch_bounds__(128)
 grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* __restrict__ W, bf16* __restrict__ C, int ldc, int c_gcol,
                    const int* __restrict__ row_offsets, int M, int N, int K, int G, const float* __restrict__ glu_params,
                    const int* __restrict__ row_map, int row_div) {
     __shared__ __align__(16) bf16 As[ST][TM][TK + MPAD];
     __shared__ int src_row[TM];
-    __shared__ __align__(16) bf16 Ws[ST][BN][TK + MPAD];
+    __shared__ __align__(16) bf16 Ws[ST][TN][TK + MPAD];
     pdl_launch_dependents();
     pdl_wait();
     int g, m0, m_end;
@@ -161,7 +162,7 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
     const bf16* a = A + (size_t)g * a_gcol;
     const bf16* w = W + (size_t)g * N * K;
     bf16* c = C + (size_t)g * c_gcol;
-    const int n0 = blockIdx.x * BN;
+    const int n0 = blockIdx.x * TN;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int gq = lane >> 2, t = lane & 3;
     constexpr int CH = TK / 8;                                      // 16-byte chunks of a row of a stage
@@ -175,15 +176,16 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
             const bool v = k < K && m0 + r < m_end;
             cp16(&As[stage][r][ch * 8], v ? a + (size_t)src_row[r] * lda + k : a, v);
         }
-        for (int idx = tid; idx < BN * CH; idx += 128) {
+        for (int idx = tid; idx < TN * CH; idx += 128) {
             const int r = idx / CH, ch = idx - r * CH;
             const int k = k0 + ch * 8;
             const bool v = k < K && n0 + r < N;
             cp16(&Ws[stage][r][ch * 8], v ? w + (size_t)(n0 + r) * K + k : w, v);
         }
     };
-    constexpr int NT = TM == 64 ? 8 : 2;                            // tiles of 8 columns a warp
-    const int row0 = TM == 64 ? warp * 16 : 0, col0 = TM == 64 ? 0 : warp * 16;
+    constexpr int NT = TM == 64 ? TN / 8 : TN / 32;                 // tiles of 8 columns a warp
+    static_assert(TN == 64 || (TM == 16 && kSwiglu == 0), "narrow tiles are for few rows without a gated epilogue");
+    const int row0 = TM == 64 ? warp * 16 : 0, col0 = TM == 64 ? 0 : warp * (TN / 4);
     float acc[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
@@ -212,7 +214,7 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
         }
     }
     const int r_lo = m0 + row0 + gq, r_hi = r_lo + 8;
-    if constexpr (kSwiglu) {
+    if constexpr (kSwiglu != 0) {
 #pragma unroll
         for (int j = 0; j < NT; j += 2) {
             const int gate_col = n0 + col0 + j * 8 + 2 * t;           // its up column stands 8 further on
@@ -245,12 +247,13 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
 
 constexpr int kMaxExpertsPerLane = 8;       // experts <= 256
 
-// The choice of one token by a warp: scoring 0 the largest sigmoid scores, which are the weights; 1 the largest logits, the
+// The choice of one token by a warp (PER experts a lane: 32 PER are at least E): scoring 0 the largest sigmoid scores, which are the weights; 1 the largest logits, the
 // weights their softmax among the chosen.
+template <int PER>
 __device__ __forceinline__ void route_token(const float* logits, int scoring, int E, int top, int* ids, float* weights, int lane) {
-    float s[kMaxExpertsPerLane];
+    float s[PER];
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
         const int e = lane + 32 * i;
         const float z = e < E ? logits[e] : 0.0f;
         // sigmoid scores lie in (0, 1): -1 never wins; logits taken as they are: the lowest float never wins
@@ -262,7 +265,7 @@ __device__ __forceinline__ void route_token(const float* logits, int scoring, in
         float best = scoring == 0 ? -2.0f : -INFINITY;
         int arg = 0x7fffffff;
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+        for (int i = 0; i < PER; ++i) {
             const int e = lane + 32 * i;
             if (s[i] > best) best = s[i], arg = e;                 // ascending e within a lane: the lower index keeps a tie
         }
@@ -277,7 +280,7 @@ __device__ __forceinline__ void route_token(const float* logits, int scoring, in
             weights[k] = best;
         }
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i)
+        for (int i = 0; i < PER; ++i)
             if (lane + 32 * i == arg) s[i] = gone;
     }
     if (scoring == 1 && lane == 0) {
@@ -289,13 +292,14 @@ __device__ __forceinline__ void route_token(const float* logits, int scoring, in
     }
 }
 
+template <int PER>
 __global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, int T, int E, int top, int* __restrict__ ids,
                                  float* __restrict__ weights) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (t >= T) return;
-    route_token(logits + (size_t)t * E, scoring, E, top, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
+    route_token<PER>(logits + (size_t)t * E, scoring, E, top, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
 }
 
 // Routing over all experts at once with groups: scores s = softmax(logits) over the E outputs; the choice scores are
@@ -303,12 +307,13 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int scoring, 
 // experts of the `keep` best groups can be chosen (the lower index wins a tie, among groups and among experts); the `top`
 // largest choice scores choose; the weights are the chosen experts' s (without the correction), divided by their sum + 1e-20,
 // times `scale`.  One warp a token, everything in float.
+template <int PER>
 __device__ __forceinline__ void route_token_grouped(const float* logits, const float* __restrict__ correction, int E, int top, int groups, int keep,
                                                     float scale, int* ids, float* weights, int lane) {
-    float s[kMaxExpertsPerLane], c[kMaxExpertsPerLane];
+    float s[PER], c[PER];
     float m = -INFINITY;
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
         const int e = lane + 32 * i;
         s[i] = e < E ? logits[e] : -INFINITY;
         m = fmaxf(m, s[i]);
@@ -316,13 +321,13 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
     m = warp_max(m);
     float sum = 0.0f;
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
         s[i] = lane + 32 * i < E ? expf(s[i] - m) : 0.0f;
         sum += s[i];
     }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
         const int e = lane + 32 * i;
         s[i] = s[i] / sum;
         c[i] = e < E ? s[i] + (correction ? correction[e] : 0.0f) : -INFINITY;
@@ -330,14 +335,14 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
     const int per = E / groups;
     if (keep < groups) {
         // the groups' scores, then `keep` rounds that each take the best group left; an expert stays if its group was taken
-        unsigned taken[kMaxExpertsPerLane];                     // per expert of this lane: its group is among the kept ones
+        unsigned taken[PER];                     // per expert of this lane: its group is among the kept ones
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i) taken[i] = 0u;
+        for (int i = 0; i < PER; ++i) taken[i] = 0u;
         for (int round = 0; round < keep; ++round) {
             float best = -INFINITY;
             int arg = 0x7fffffff;
 #pragma unroll
-            for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+            for (int i = 0; i < PER; ++i) {
                 const int e = lane + 32 * i;
                 if (e < E && !taken[i]) {
                     const int g = e / per;
@@ -351,13 +356,13 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
                 if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa;
             }
 #pragma unroll
-            for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+            for (int i = 0; i < PER; ++i) {
                 const int e = lane + 32 * i;
                 if (e < E && e / per == arg) taken[i] = 1u;
             }
         }
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i)
+        for (int i = 0; i < PER; ++i)
             if (!taken[i]) c[i] = -INFINITY;
     }
     float wsum = 0.0f;
@@ -365,7 +370,7 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
         float best = -INFINITY, score = 0.0f;
         int arg = 0x7fffffff;
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+        for (int i = 0; i < PER; ++i) {
             const int e = lane + 32 * i;
             if (e < E && (c[i] > best || (arg == 0x7fffffff && c[i] == best))) best = c[i], arg = e, score = s[i];
         }
@@ -382,7 +387,7 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
         }
         wsum += score;
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i)
+        for (int i = 0; i < PER; ++i)
             if (lane + 32 * i == arg) c[i] = -INFINITY, s[i] = 0.0f;
     }
     if (lane == 0) {
@@ -390,20 +395,21 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
     }
 }
 
+template <int PER>
 __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int T, int E, int top, int groups,
                                          int keep, float scale, int* __restrict__ ids, float* __restrict__ weights) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (t >= T) return;
-    route_token_grouped(logits + (size_t)t * E, correction, E, top, groups, keep, scale, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
+    route_token_grouped<PER>(logits + (size_t)t * E, correction, E, top, groups, keep, scale, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
 }
 
-// The front of a mixture for a small step as one block: the router's product (a warp per token and four experts, float sums),
+// The front of a mixture for a small step as one block: the router's product (a warp per token and two experts, float sums),
 // the choice (a warp per token) and the stable sort of the (token, choice) pairs by expert (runs without padding).
 constexpr int kSmallPairs = 256, kSmallLogits = 1024;
 
-template <typename T>
+template <typename T, int PER>
 __global__ void __launch_bounds__(1024)
 moe_small_step_kernel(const T* __restrict__ h, const T* __restrict__ w, const float* __restrict__ bias, int tokens, int H, int E, int top, int scoring,
                       const float* __restrict__ correction, int groups, int keep, float scale, float* __restrict__ weights, int* __restrict__ offsets,
@@ -413,41 +419,53 @@ moe_small_step_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
     __shared__ int ids[kSmallPairs];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_launch_dependents();
+    // the router's weights do not depend on the kernel before this one: asked for while that still runs
+    for (size_t i = (size_t)threadIdx.x * 128; i < (size_t)E * H * sizeof(T); i += 1024 * 128)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"((const char*)w + i));
     pdl_wait();
-    const int quads = (E + 3) / 4;
-    for (int job = warp; job < tokens * quads; job += 32) {
-        const int t = job / quads, e0 = (job - t * quads) * 4;
+    // two experts a job, three rounds of loads in flight
+    constexpr int EJ = 2, U = 3;
+    const int pairs = (E + EJ - 1) / EJ;
+    for (int job = warp; job < tokens * pairs; job += 32) {
+        const int t = job / pairs, e0 = (job - t * pairs) * EJ;
         const T* hr = h + (size_t)t * H;
-        float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        for (int k = V * lane; k < H; k += 32 * V) {
-            const uint4 hv = *reinterpret_cast<const uint4*>(hr + k);
-            uint4 wv[4];
+        float acc[EJ] = {0.0f, 0.0f};
+        for (int k0 = V * lane; k0 < H; k0 += 32 * V * U) {
+            uint4 hv[U], wv[U][EJ];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) wv[j] = __ldg(reinterpret_cast<const uint4*>(w + (size_t)min(e0 + j, E - 1) * H + k));
+            for (int u = 0; u < U; ++u) {
+                const int k = k0 + 32 * V * u;
+                const bool in = k < H;
+                hv[u] = in ? *reinterpret_cast<const uint4*>(hr + k) : make_uint4(0, 0, 0, 0);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const unsigned a[4] = {hv.x, hv.y, hv.z, hv.w}, b[4] = {wv[j].x, wv[j].y, wv[j].z, wv[j].w};
+                for (int j = 0; j < EJ; ++j) wv[u][j] = in ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)min(e0 + j, E - 1) * H + k)) : make_uint4(0, 0, 0, 0);
+            }
 #pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    if constexpr (sizeof(T) == 2) {
-                        acc[j] = fmaf(__uint_as_float(a[q] << 16), __uint_as_float(b[q] << 16), acc[j]);
-                        acc[j] = fmaf(__uint_as_float(a[q] & 0xffff0000u), __uint_as_float(b[q] & 0xffff0000u), acc[j]);
-                    } else {
-                        acc[j] = fmaf(__uint_as_float(a[q]), __uint_as_float(b[q]), acc[j]);
+            for (int u = 0; u < U; ++u)
+#pragma unroll
+                for (int j = 0; j < EJ; ++j) {
+                    const unsigned a[4] = {hv[u].x, hv[u].y, hv[u].z, hv[u].w}, b[4] = {wv[u][j].x, wv[u][j].y, wv[u][j].z, wv[u][j].w};
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        if constexpr (sizeof(T) == 2) {
+                            acc[j] = fmaf(__uint_as_float(a[q] << 16), __uint_as_float(b[q] << 16), acc[j]);
+                            acc[j] = fmaf(__uint_as_float(a[q] & 0xffff0000u), __uint_as_float(b[q] & 0xffff0000u), acc[j]);
+                        } else {
+                            acc[j] = fmaf(__uint_as_float(a[q]), __uint_as_float(b[q]), acc[j]);
+                        }
                     }
                 }
-            }
         }
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < EJ; ++j) {
             const float z = warp_sum(acc[j]);
             if (lane == 0 && e0 + j < E) logits[t * E + e0 + j] = bias ? z + bias[e0 + j] : z;
         }
     }
     __syncthreads();
     for (int t = warp; t < tokens; t += 32) {
-        if (scoring == 2) route_token_grouped(logits + t * E, correction, E, top, groups, keep, scale, ids + t * top, weights + (size_t)t * top, lane);
-        else route_token(logits + t * E, scoring, E, top, ids + t * top, weights + (size_t)t * top, lane);
+        if (scoring == 2) route_token_grouped<PER>(logits + t * E, correction, E, top, groups, keep, scale, ids + t * top, weights + (size_t)t * top, lane);
+        else route_token<PER>(logits + t * E, scoring, E, top, ids + t * top, weights + (size_t)t * top, lane);
     }
     __syncthreads();
     const int n = tokens * top;
@@ -570,15 +588,22 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
 int li_linear_tcgen05_grouped(const void* a, const void* w, void* out, int M, int N, int K, int G, const int* tile_group, int epilogue,
                               const float* glu_params, cudaStream_t stream);
 
-// tile_group (may be NULL; rows in groups whose runs start at multiples of 128, li_moe_sort with pad 128): the group of
-// every tile of 128 rows; bfloat16 products of at least kTensorRows rows then run on tcgen05 tiles.
+int li_linear_tcgen05_grouped_pairs(const void* a, const void* w, void* out, int M, int N, int K, int G, const int* tile_group, int epilogue,
+                                    const float* glu_params, cudaStream_t stream);
+
+// tile_group (may be NULL; rows in groups whose runs start at multiples of tile_rows, 128 or 256, li_moe_sort with that pad): the group
+// of every tile of tile_rows rows (256: pairs of CTAs, a persistent kernel); bfloat16 products of at least kTensorRows rows then run on tcgen05 tiles.
 constexpr int kTensorRows = 256;
+int g_narrow_below = 296;         // CTAs of 64 columns below which few rows take tiles of 32 columns: two a multiprocessor
+
+// Measurements: another bound (0: never).
+LI_EXPORT void li_grouped_narrow_below(int ctas) { g_narrow_below = ctas; }
 
 // epilogue: LI_EPILOGUE_NONE, or a gated one (bfloat16, K a multiple of 8, N a multiple of 16): gate and up rows of
 // every group's matrix interleaved in eights, out rows of N / 2 activations; LI_EPILOGUE_GLU_CLAMPED reads its {limit, alpha}
 // from glu_params on the device.  row_map (may be NULL; bfloat16, rows in groups): row r is row row_map[r] / row_div of a.
 LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* w, void* out, int ldc, int c_gcol, const int* row_offsets,
-                                const int* tile_group, int dtype, int M, int N, int K, int G, int epilogue, const float* glu_params,
+                                const int* tile_group, int tile_rows, int dtype, int M, int N, int K, int G, int epilogue, const float* glu_params,
                                 const int* row_map, int row_div, cudaStream_t stream) {
     LI_REQUIRE(row_map == nullptr || (row_offsets != nullptr && tile_group == nullptr && row_div >= 1), "grouped_linear: a map of the rows goes with rows in groups, without padded runs");
     LI_REQUIRE(M >= 0 && N > 0 && K > 0 && G > 0, "grouped_linear: bad sizes M=%d N=%d K=%d G=%d", M, N, K, G);
@@ -591,9 +616,11 @@ LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* 
     LI_REQUIRE(row_offsets == nullptr || (a_gcol == 0 && c_gcol == 0), "grouped_linear: groups are rows or columns, not both");
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "grouped_linear: unknown dtype %d", dtype);
     if (M == 0) return 0;
-    if (dtype == LI_BF16 && row_offsets != nullptr && tile_group != nullptr && M >= kTensorRows && M % 128 == 0 && lda == K && ldc == out_cols &&
+    LI_REQUIRE(tile_group == nullptr || tile_rows == 128 || tile_rows == 256, "grouped_linear: tiles of %d rows", tile_rows);
+    if (dtype == LI_BF16 && row_offsets != nullptr && tile_group != nullptr && M >= kTensorRows && M % tile_rows == 0 && lda == K && ldc == out_cols &&
         K % 8 == 0 && ((uintptr_t)a % 16) == 0 && ((uintptr_t)w % 16) == 0 && (!swiglu || N % 16 == 0))
-        return li_linear_tcgen05_grouped(a, w, out, M, N, K, G, tile_group, epilogue, glu_params, stream);
+        return tile_rows == 256 ? li_linear_tcgen05_grouped_pairs(a, w, out, M, N, K, G, tile_group, epilogue, glu_params, stream)
+                                : li_linear_tcgen05_grouped(a, w, out, M, N, K, G, tile_group, epilogue, glu_params, stream);
     const int row_tiles = ceil_div(M, BM);
     const dim3 grid(ceil_div(N, BN), row_offsets ? row_tiles + G : row_tiles, row_offsets ? 1 : G);
     LI_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "grouped_linear: too many tiles for one launch");
@@ -607,10 +634,13 @@ LI_EXPORT int li_grouped_linear(const void* a, int lda, int a_gcol, const void* 
     if (dtype == LI_BF16 && aligned && few) {
         const int tiles16 = ceil_div(M, 16);
         const dim3 grid16(ceil_div(N, BN), row_offsets ? tiles16 + G : tiles16, row_offsets ? 1 : G);
-#define LI_GROUPED_MMA(TM_, TK_, ST_, EPI_, GRID_)                                                                                          \
-    li_launch_pdl(grouped_mma_kernel<TM_, TK_, ST_, EPI_>, GRID_, dim3(128), 0, stream, (const bf16*)a, lda, a_gcol, (const bf16*)w, (bf16*)out, ldc, \
+        // so few columns that the CTAs of all groups do not fill the multiprocessors twice over: half as wide tiles
+        const bool narrow = !swiglu && (long long)ceil_div(N, BN) * (row_offsets ? (M < G ? M : G) : G * tiles16) < g_narrow_below;
+        const dim3 grid32(ceil_div(N, 32), grid16.y, grid16.z);
+#define LI_GROUPED_MMA(TM_, TK_, ST_, EPI_, GRID_, ...)                                                                                          \
+    li_launch_pdl(grouped_mma_kernel<TM_, TK_, ST_, EPI_ __VA_OPT__(,) __VA_ARGS__>, GRID_, dim3(128), 0, stream, (const bf16*)a, lda, a_gcol, (const bf16*)w, (bf16*)out, ldc, \
                   c_gcol, row_offsets, M, N, K, G, glu_params, row_map, row_div)
-        e = clamped ? LI_GROUPED_MMA(16, 64, 4, 2, grid16) : geglu ? LI_GROUPED_MMA(16, 64, 4, 3, grid16) : swiglu ? LI_GROUPED_MMA(16, 64, 4, 1, grid16) : LI_GROUPED_MMA(16, 64, 4, 0, grid16);
+        e = narrow ? LI_GROUPED_MMA(16, 64, 6, 0, grid32, 32) : clamped ? LI_GROUPED_MMA(16, 64, 4, 2, grid16) : geglu ? LI_GROUPED_MMA(16, 64, 4, 3, grid16) : swiglu ? LI_GROUPED_MMA(16, 64, 4, 1, grid16) : LI_GROUPED_MMA(16, 64, 4, 0, grid16);
     } else if (dtype == LI_BF16 && aligned)
         e = clamped ? LI_GROUPED_MMA(64, 32, 3, 2, grid) : geglu ? LI_GROUPED_MMA(64, 32, 3, 3, grid) : swiglu ? LI_GROUPED_MMA(64, 32, 3, 1, grid) : LI_GROUPED_MMA(64, 32, 3, 0, grid);
 #undef LI_GROUPED_MMA
@@ -631,7 +661,7 @@ LI_EXPORT int li_moe_route(const float* logits, int scoring, int T, int E, int t
     LI_REQUIRE(scoring == 0 || scoring == 1, "moe_route: unknown scoring %d", scoring);
     LI_REQUIRE(E <= 32 * kMaxExpertsPerLane, "moe_route: %d experts are more than %d", E, 32 * kMaxExpertsPerLane);
     if (T == 0) return 0;
-    const cudaError_t e = li_launch_pdl(moe_route_kernel, dim3(ceil_div(T, 4)), dim3(128), 0, stream, logits, scoring, T, E, top, ids, weights);
+    const cudaError_t e = li_launch_pdl(E <= 32 ? moe_route_kernel<1> : moe_route_kernel<kMaxExpertsPerLane>, dim3(ceil_div(T, 4)), dim3(128), 0, stream, logits, scoring, T, E, top, ids, weights);
     if (e != cudaSuccess) return li_fail("moe_route: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("moe_route");
 }
@@ -645,7 +675,7 @@ LI_EXPORT int li_moe_route_grouped(const float* logits, const float* correction,
                "moe_route_grouped: %d of %d groups of %d experts cannot give %d choices", keep, groups, groups >= 1 ? E / groups : 0, top);
     LI_REQUIRE(E <= 32 * kMaxExpertsPerLane, "moe_route_grouped: %d experts are more than %d", E, 32 * kMaxExpertsPerLane);
     if (T == 0) return 0;
-    const cudaError_t e = li_launch_pdl(moe_route_grouped_kernel, dim3(ceil_div(T, 4)), dim3(128), 0, stream, logits, correction, T, E, top, groups, keep,
+    const cudaError_t e = li_launch_pdl(E <= 32 ? moe_route_grouped_kernel<1> : moe_route_grouped_kernel<kMaxExpertsPerLane>, dim3(ceil_div(T, 4)), dim3(128), 0, stream, logits, correction, T, E, top, groups, keep,
                                         scale, ids, weights);
     if (e != cudaSuccess) return li_fail("moe_route_grouped: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("moe_route_grouped");
@@ -700,7 +730,7 @@ LI_EXPORT int li_moe_combine(const void* rows, int dtype, const int* place_of, c
 LI_EXPORT int li_moe_small_step_accepts(int dtype, int T, int H, int E, int top) {
     const int vec = dtype == LI_BF16 ? 8 : 4;
     return (T >= 1 && E >= 1 && E <= 32 * kMaxExpertsPerLane && top >= 1 && top <= E && T * top <= kSmallPairs && T * E <= kSmallLogits &&
-            T * ((E + 3) / 4) <= 128 && H % vec == 0) ? 1 : 0;
+            T * ((E + 1) / 2) <= 64 && H % vec == 0) ? 1 : 0;
 }
 
 LI_EXPORT int li_moe_small_step(const void* h, const void* w, const float* bias, int dtype, int T, int H, int E, int top, int scoring,
@@ -714,9 +744,9 @@ LI_EXPORT int li_moe_small_step(const void* h, const void* w, const float* bias,
     LI_REQUIRE(((uintptr_t)h % 16) == 0 && ((uintptr_t)w % 16) == 0, "moe_small_step: operands must be 16-byte aligned");
     const int threads = 1024;
     const cudaError_t e = dtype == LI_F32
-        ? li_launch_pdl(moe_small_step_kernel<float>, dim3(1), dim3(threads), 0, stream, (const float*)h, (const float*)w, bias, T, H, E, top, scoring, correction,
+        ? li_launch_pdl(E <= 32 ? moe_small_step_kernel<float, 1> : moe_small_step_kernel<float, kMaxExpertsPerLane>, dim3(1), dim3(threads), 0, stream, (const float*)h, (const float*)w, bias, T, H, E, top, scoring, correction,
                         groups, keep, scale, weights, offsets, pair_at, place_of)
-        : li_launch_pdl(moe_small_step_kernel<bf16>, dim3(1), dim3(threads), 0, stream, (const bf16*)h, (const bf16*)w, bias, T, H, E, top, scoring, correction,
+        : li_launch_pdl(E <= 32 ? moe_small_step_kernel<bf16, 1> : moe_small_step_kernel<bf16, kMaxExpertsPerLane>, dim3(1), dim3(threads), 0, stream, (const bf16*)h, (const bf16*)w, bias, T, H, E, top, scoring, correction,
                         groups, keep, scale, weights, offsets, pair_at, place_of);
     if (e != cudaSuccess) return li_fail("moe_small_step: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("moe_small_step");

@@ -338,13 +338,16 @@ int li_map_difference(const void* att, int dtype, int dl, const void* gate, int 
 /* ---- grouped.cu: products in groups, routing of a mixture of experts ---- */
 /* out_g = a_g w_g^T, w [G, N, K].  row_offsets [G + 1] (device): group g owns those rows of a [M, lda] and out [M, ldc].
  * row_offsets NULL: every group takes all M rows, inputs at column g * a_gcol, outputs at column g * c_gcol.
- * tile_group (may be NULL): with runs of rows that start at multiples of 128, the group of every tile of 128 rows (-1: none);
+ * tile_group (may be NULL): with runs of rows that start at multiples of tile_rows (128 or 256), the group of every such tile (-1: none);
  * large bfloat16 products then run on tcgen05 tiles.  epilogue 1 (bfloat16): gate and up rows of every matrix interleaved in
  * eights, out rows of N / 2 activations up * gate / (1 + exp(-gate)).  row_map (may be NULL; bfloat16, rows in groups, runs without
  * padding): row r of the groups is row row_map[r] / row_div of a. */
 int li_grouped_linear(const void* a, int lda, int a_gcol, const void* w, void* out, int ldc, int c_gcol, const int* row_offsets,
-    const int* tile_group, int dtype, int M, int N, int K, int G, int epilogue, const float* glu_params,
+    const int* tile_group, int tile_rows, int dtype, int M, int N, int K, int G, int epilogue, const float* glu_params,
     const int* row_map, int row_div, cudaStream_t stream);
+
+/* Measurements: CTAs of 64 columns below which a product of few rows takes tiles of 32 columns (0: never). */
+void li_grouped_narrow_below(int ctas);
 
 /* ids, weights [T, top]: the experts with the largest sigmoid(logits [T, E]) and those scores (scoring 0), or the experts
  * with the largest logits and the softmax over the chosen logits alone (scoring 1). */

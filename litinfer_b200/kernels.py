@@ -1222,12 +1222,13 @@ def row_rinv(x: torch.Tensor, ranges, eps: float, out: torch.Tensor) -> None:
 def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row_offsets: Optional[torch.Tensor] = None,
                    a_group_cols: int = 0, out_group_cols: int = 0, tile_group: Optional[torch.Tensor] = None,
                    epilogue: Optional[str] = None, epilogue_params: Optional[torch.Tensor] = None,
-                   row_source: Optional[Tuple[torch.Tensor, int]] = None) -> None:
+                   row_source: Optional[Tuple[torch.Tensor, int]] = None, tile_rows: int = 128) -> None:
     """``weight`` [G, N, K]: a product per group.  With ``row_offsets`` (int32 [G + 1] on the device) group g owns the rows
     ``row_offsets[g] .. row_offsets[g + 1] - 1`` of ``a`` [M, K] and ``out`` [M, N].  Without, every group takes all rows, its
     inputs at column ``g * a_group_cols`` of ``a`` and its outputs at column ``g * out_group_cols`` of ``out`` (a map per head).
-    ``tile_group`` (int32 on the device; from :func:`moe_sort` with ``pad`` 128): the group of every tile of 128 rows when
-    the groups' runs start at multiples of 128; large bfloat16 products then run on the tcgen05 tiles.
+    ``tile_group`` (int32 on the device; from :func:`moe_sort` with ``pad`` = ``tile_rows``, 128 or 256): the group of every tile
+    of that many rows when the groups' runs start at multiples of it; large bfloat16 products then run on the tcgen05 tiles
+    (256: on pairs of CTAs, in a persistent kernel).
     ``epilogue="swiglu"`` (bfloat16, rows in groups): every group's matrix holds gate and up rows interleaved in eights
     (:func:`interleave_gate_up` per group) and ``out`` [M, N / 2] takes ``up * gate / (1 + exp(-gate))``.
     ``epilogue="glu_clamped"``: the same layout, the gated unit with bounded operands; ``epilogue_params`` holds its (limit,
@@ -1265,10 +1266,10 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, row
         raise KernelError("grouped_linear: the groups' columns do not fit the rows")
     if tile_group is not None:
         _need(tile_group, "groups of the row tiles", torch.int32)
-        if row_offsets is None or tile_group.numel() * 128 < M:
-            raise KernelError("grouped_linear: a table of the tiles' groups goes with row offsets and covers every tile of 128 rows")
+        if row_offsets is None or tile_rows not in (128, 256) or tile_group.numel() * tile_rows < M:
+            raise KernelError(f"grouped_linear: a table of the tiles' groups goes with row offsets and covers every tile of {tile_rows} rows (128 or 256)")
     _check(library().li_grouped_linear(_p(a), _i(a.shape[1]), _i(a_group_cols), _p(weight), _p(out), _i(out.shape[1]), _i(out_group_cols),
-                                       _p(row_offsets), _p(tile_group), _i(_dt(a)), _i(M), _i(N), _i(Kd), _i(G), _i(EPILOGUES[epilogue]), _p(epilogue_params),
+                                       _p(row_offsets), _p(tile_group), _i(int(tile_rows)), _i(_dt(a)), _i(M), _i(N), _i(Kd), _i(G), _i(EPILOGUES[epilogue]), _p(epilogue_params),
                                        _p(row_source[0] if row_source is not None else None), _i(int(row_source[1]) if row_source is not None else 1), _stream(out)),
            "grouped_linear")
 

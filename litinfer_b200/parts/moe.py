@@ -48,6 +48,7 @@ from .linear import FusedLinear
 class RoutedExperts(FeedForward):
     PAD = 128                      # rows of a tensor-core tile
     PAD_FROM_ROWS = 256            # (token, choice) pairs of a step from which the runs are padded
+    PAIR_PAD = 256                 # rows of a tile on a pair of CTAs; taken when an expert has that many rows on average
 
     def __init__(self, spec, prefix, dtype, device):
         super().__init__(spec, prefix, dtype, device)
@@ -151,12 +152,15 @@ class RoutedExperts(FeedForward):
         weights = torch.empty((T, top), dtype=torch.float32, device=dev)
         offsets = torch.empty(n_out + 1, dtype=torch.int32, device=dev)
         place_of = torch.empty(T * top, dtype=torch.int32, device=dev)
-        # a step of many tokens: every expert's run of rows starts at a multiple of 128, so that the products run on
-        # tensor-core tiles of 128 rows, each of one expert
+        # a step of many tokens: every expert's run of rows starts at a multiple of 128 (or 256), so that the products run on
+        # tensor-core tiles of that many rows, each of one expert
         pad = self.PAD if (self.dtype == torch.bfloat16 and T * top >= self.PAD_FROM_ROWS) else 1
+        if pad > 1 and T * top >= self.PAIR_PAD * n_out:
+            pad = self.PAIR_PAD
         R = K.sorted_rows(T * top, n_out, pad)
         pair_at = torch.empty(R, dtype=torch.int32, device=dev)
         tiles = torch.empty(R // pad, dtype=torch.int32, device=dev) if pad > 1 else None
+        tile_rows = pad if pad > 1 else self.PAD
         grouped = self.scoring in ("softmax_grouped", "softmax")
         if pad == 1 and K.moe_small_step_accepts(h, n_out, top):
             # few tokens: the router's product, the choice and the sort are one launch
@@ -180,14 +184,14 @@ class RoutedExperts(FeedForward):
             K.moe_gather(h, pair_at, weights if on_input else None, top, rows)
         act = torch.empty((R, F), dtype=self.dtype, device=dev)
         if self.fused_activation:
-            K.grouped_linear(h if in_place else rows, self.gate_up, act, expert_offsets, tile_group=tiles, epilogue=self.activation,
+            K.grouped_linear(h if in_place else rows, self.gate_up, act, expert_offsets, tile_group=tiles, tile_rows=tile_rows, epilogue=self.activation,
                              epilogue_params=self.activation_params, row_source=(pair_at, top) if in_place else None)
         else:
             both = torch.empty((R, 2 * F), dtype=self.dtype, device=dev)
-            K.grouped_linear(rows, self.gate_up, both, expert_offsets, tile_group=tiles)
+            K.grouped_linear(rows, self.gate_up, both, expert_offsets, tile_group=tiles, tile_rows=tile_rows)
             if self.activation == "swiglu":
                 K.swiglu(both, act)
             else:
                 K.glu_clamped(both, act, self.limit, self.alpha)
-        K.grouped_linear(act, self.down, rows, expert_offsets, tile_group=tiles)
+        K.grouped_linear(act, self.down, rows, expert_offsets, tile_group=tiles, tile_rows=tile_rows)
         return K.RowSum(rows, place_of, top, None if on_input else weights, extra=shared)

@@ -432,7 +432,7 @@ def add_pair_rows(x32, pairs, ids, positions, q_start, seq_of_token, slots, stat
 
 
 def grouped_linear(a, weight, out, row_offsets=None, a_group_cols=0, out_group_cols=0, tile_group=None, epilogue=None, epilogue_params=None,
-                   row_source=None):
+                   row_source=None, tile_rows=128):
     G, N, Kd = weight.shape
     if row_source is not None:
         a = a[(row_source[0] // row_source[1]).long()]

@@ -826,8 +826,8 @@ def test_front_of_a_mixture_in_one_launch_and_rows_read_in_place(dtype):
 
     dev, dt = torch.device("cuda:0"), _dt(dtype)
     torch.manual_seed(12)
-    for T, E, top, H, scoring, groups, keep in ((1, 8, 2, 64, "softmax_grouped", 1, 1), (9, 5, 3, 48, "softmax_grouped", 5, 4), (32, 12, 4, 96, "sigmoid", 1, 1),
-                                                (40, 3, 1, 1536, "softmax_chosen", 1, 1), (64, 8, 3, 256, "softmax_grouped", 4, 2), (4, 100, 6, 128, "softmax_grouped", 1, 1)):
+    for T, E, top, H, scoring, groups, keep in ((1, 8, 2, 64, "softmax_grouped", 1, 1), (9, 5, 3, 48, "softmax_grouped", 5, 4), (10, 12, 4, 96, "sigmoid", 1, 1),
+                                                (30, 3, 1, 1536, "softmax_chosen", 1, 1), (16, 8, 3, 256, "softmax_grouped", 4, 2), (1, 100, 6, 128, "softmax_grouped", 1, 1)):
         h = torch.randn(T, H).to(dev, dt)
         w = (2.0 * torch.randn(E, H) / math.sqrt(H)).to(dev, dt)
         bias = (0.3 * torch.randn(E)).to(dev) if scoring == "softmax_chosen" else None
@@ -905,3 +905,36 @@ def test_keys_and_values_of_a_long_step_into_pages_kernel(dh, page, dtype):
             F.rope_kv_write(qkv.clone(), torch.zeros(T, dtype=torch.int32, device=dev), None, 0, slots, kc, vc, nh, nkv, dh)
             res.append((kc, vc))
         assert torch.equal(res[0][0], res[1][0]) and torch.equal(res[0][1], res[1][1]), f"{T} tokens, {order}"
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("epilogue", [None, "swiglu", "glu_clamped", "geglu"])
+def test_products_of_experts_on_pairs_of_ctas(epilogue):
+    """Runs padded to 256 rows in the persistent kernel: uneven runs, an expert that nobody chose, tiles of no group among and
+    behind the others, columns that are no whole tile, more tiles than pairs of multiprocessors and fewer; against the
+    reference and, bit for bit, against a second run."""
+    import kernel_refs as R
+    from litinfer_b200 import kernels as K
+
+    dev, dt = torch.device("cuda:0"), torch.bfloat16
+    params = torch.tensor([1.1, 1.702], device=dev) if epilogue == "glu_clamped" else None
+    for T, E, top, W, F, extra in ((700, 3, 2, 64, 80, 1), (2048, 5, 2, 128, 2000, 0), (1500, 4, 1, 264, 304, 0), (512, 2, 1, 1024, 64, 2)):
+        torch.manual_seed(T)
+        ids = torch.randint(0, E + extra, (T, top), dtype=torch.int32, device=dev)
+        if E == 5:
+            ids[ids == 1] = 4
+        n_rows = K.sorted_rows(T * top, E + extra, 256)
+        offsets, pair_at, place_of = (torch.empty(n, dtype=torch.int32, device=dev) for n in (E + extra + 1, n_rows, T * top))
+        tiles = torch.empty(n_rows // 256, dtype=torch.int32, device=dev)
+        K.moe_sort(ids, E + extra, offsets, pair_at, place_of, 256, tiles, matrices=E)
+        a = torch.randn(n_rows, W, device=dev).to(dt)
+        w = (2.0 * torch.randn(E, F, W, device=dev) / math.sqrt(W)).to(dt)
+        cols = F if epilogue is None else F // 2
+        outs = [torch.full((n_rows, cols), 3.0, dtype=dt, device=dev) for _ in range(3)]
+        for out, fn in zip(outs, (K, R, K)):
+            fn.grouped_linear(a, w, out, offsets[:E + 1], tile_group=tiles, tile_rows=256, epilogue=epilogue, epilogue_params=params)
+        lo = int(offsets[E])
+        live = pair_at[:lo] >= 0
+        _close(outs[0][:lo][live], outs[1][:lo][live], "bfloat16", f"{T} tokens, {E} experts")
+        assert torch.equal(outs[0], outs[2])
+        assert (outs[0][lo:] == 3.0).all(), "rows of no expert were written"
