@@ -407,7 +407,7 @@ LI_EXPORT int li_latent_rope_post(const void* low, int dtype, int ld_low, int co
 // A block takes one token and some of its heads, a warp a head at a time; a lane holds V neighbouring elements of every 32 V,
 // so that the pairs of neighbours never leave a lane.  All arithmetic in float from run-dtype inputs, one rounding.
 namespace {
-constexpr int kRopeNormWarps = 4;
+constexpr int kRopeNormWarps = 8;
 
 template <typename T, int V>
 __device__ __forceinline__ void load_elements(float (&v)[V], const T* __restrict__ p, int left) {
@@ -615,7 +615,12 @@ map_difference_kernel(const T* __restrict__ att, int dl, const T* __restrict__ g
         const int d = V * (lane + 32 * i);
         if (d < dv) {
 #pragma unroll
-            for (int k = 0; k < V; ++k) v[i][k] = g ? v[i][k] * f / (1.0f + expf(-gv[i][k])) : v[i][k] * f;
+            for (int k = 0; k < V; ++k) {
+                // (an output that is rounded to 16 bits takes the fast exponential and quotient)
+                if (!g) v[i][k] *= f;
+                else if constexpr (sizeof(T) == 2) v[i][k] = __fdividef(v[i][k] * f, 1.0f + fast_exp2(-1.4426950408889634f * gv[i][k]));
+                else v[i][k] = v[i][k] * f / (1.0f + expf(-gv[i][k]));
+            }
             store_elements_of<T, V>(o + d, v[i], dv - d);
         }
     }
@@ -636,8 +641,8 @@ LI_EXPORT int li_rope_norm_kv(const void* proj, int ld, void* out, int dtype, co
     LI_REQUIRE(proj != out, "rope_norm_kv: the output needs rows of its own");
     if (T == 0) return 0;
     const int heads = nh + (keys_are_values ? 1 : 2) * nkv;
-    // many tokens: four heads a warp (fewer, fuller blocks); few: one
-    const int per_block = T >= 64 ? 4 * kRopeNormWarps : kRopeNormWarps;
+    // many tokens: two heads a warp (fewer, fuller blocks); few: one
+    const int per_block = T >= 64 ? 2 * kRopeNormWarps : kRopeNormWarps;
     const dim3 grid(T, ceil_div(heads, per_block));
     LI_REQUIRE(grid.y <= 65535, "rope_norm_kv: too many heads for one launch");
     const size_t smem = ((size_t)rotary_dim + (interleaved ? 0 : (size_t)kRopeNormWarps * dh)) * sizeof(float);
