@@ -167,14 +167,16 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, int a_gcol, const bf16* 
     const int gq = lane >> 2, t = lane & 3;
     constexpr int CH = TK / 8;                                      // 16-byte chunks of a row of a stage
     // row_map: row r of the sorted order is row row_map[r] / row_div of A (the rows of a mixture's tokens, read in place)
-    if (tid < TM) src_row[tid] = (row_map && m0 + tid < m_end) ? row_map[m0 + tid] / row_div : m0 + tid;
-    __syncthreads();
+    if (row_map) {
+        if (tid < TM) src_row[tid] = m0 + tid < m_end ? row_map[m0 + tid] / row_div : 0;
+        __syncthreads();
+    }
     auto load = [&](int stage, int k0) {
         for (int idx = tid; idx < TM * CH; idx += 128) {
             const int r = idx / CH, ch = idx - r * CH;
             const int k = k0 + ch * 8;
             const bool v = k < K && m0 + r < m_end;
-            cp16(&As[stage][r][ch * 8], v ? a + (size_t)src_row[r] * lda + k : a, v);
+            cp16(&As[stage][r][ch * 8], v ? a + (size_t)(row_map ? src_row[r] : m0 + r) * lda + k : a, v);
         }
         for (int idx = tid; idx < TN * CH; idx += 128) {
             const int r = idx / CH, ch = idx - r * CH;
