@@ -11,7 +11,7 @@ LitInfer has one pool, free list and block table per layer
 
 Pages are allocated when a request grows (``extend``), given back when it ends
 (``release``) and, in a group with a window, as soon as every key on them lies
-behind the window of all further queries (``commit``); the pages that hold the
+behind the window of all further queries (``commit``; in a group with chunks, as soon as the chunk is over); the pages that hold the
 first ``keep_first`` keys of such a group stay.  The extra last page of
 each tensor is a sink for padded tokens of captured decode batches; it is
 never handed out.
@@ -128,6 +128,9 @@ class CacheManager:
         for gid, g in enumerate(self.groups):
             if g.key.window and g.key.keep_first:          # the pages of the first keys never go back behind the window
                 native.check(self._lib.li_cm_keep_first(self._h, gid, int(g.key.keep_first)))
+            if g.key.chunks:                               # pages of chunks that are over go back
+                sizes = (ctypes.c_int * len(g.key.chunks))(*[int(c) for c in g.key.chunks])
+                native.check(self._lib.li_cm_chunks(self._h, gid, len(g.key.chunks), sizes))
         self.slots = PoolView(self, -1, self.max_requests)
         for gid, g in enumerate(self.groups):
             g.pool = PoolView(self, gid, self.num_pages)

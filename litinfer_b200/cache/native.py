@@ -36,6 +36,7 @@ _SIGNATURES = {
     "li_cm_create": (P, [I, IP, I, I, I]),
     "li_cm_destroy": (None, [P]),
     "li_cm_keep_first": (I, [P, I, I]),
+    "li_cm_chunks": (I, [P, I, I, IP]),
     "li_cm_num_free": (I, [P, I]),
     "li_cm_owner": (I, [P, I, I]),
     "li_cm_pool_check": (I, [P, I]),

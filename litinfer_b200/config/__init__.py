@@ -1,3 +1,4 @@
+from .bozolorn import BozolornConfig
 from .demavik import DemavikConfig
 from .filasun import FilasunConfig
 from .gorulorn import GorulornConfig
@@ -15,6 +16,7 @@ from .spec import BlockSpec, ModelSpec, PartSpec, ScheduleEntry, default_schedul
 
 __all__ = [
     "BlockSpec",
+    "BozolornConfig",
     "ConfigError",
     "DemavikConfig",
     "FilasunConfig",

@@ -13,6 +13,7 @@ import json
 from pathlib import Path
 from typing import Any, Dict, Mapping, Type
 
+from .bozolorn import BozolornConfig
 from .demavik import DemavikConfig
 from .filasun import FilasunConfig
 from .gorulorn import GorulornConfig
@@ -89,3 +90,4 @@ register_architecture(GorulornConfig.ARCHITECTURE, GorulornConfig)
 register_architecture(DemavikConfig.ARCHITECTURE, DemavikConfig)
 register_architecture(PifazenConfig.ARCHITECTURE, PifazenConfig)
 register_architecture(ZigolixConfig.ARCHITECTURE, ZigolixConfig)
+register_architecture(BozolornConfig.ARCHITECTURE, BozolornConfig)

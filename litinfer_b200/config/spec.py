@@ -142,6 +142,8 @@ class ModelSpec:
     # parts that add something to the residual stream right after the embedding and may keep a state per request for it
     # (an embedding of token pairs): (spec, tensor-name prefix) each, kinds of the registry of stream inputs
     stream_inputs: Tuple[Tuple[PartSpec, str], ...] = ()
+    # tables with a row per token of the vocabulary that layers read by token id (``parts.base.TokenInput``): tensor name -> columns
+    token_tables: Mapping[str, int] = field(default_factory=dict)
     # other names under which a declared tensor may be stored: declared name -> names tried after it
     aliases: Mapping[str, Tuple[str, ...]] = field(default_factory=dict)
 

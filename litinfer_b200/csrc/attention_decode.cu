@@ -29,7 +29,7 @@
 // only, so a sequence's result does not depend on the batch it is in, as long
 // as the contexts are cut the same way (how long a CTA's range is depends on the
 // number of sequences and on the longest context of the step).
-// Window: keys below p - window + 1 are masked, blocks wholly below it skipped.
+// Window: keys below p - window + 1 are masked, blocks wholly below it skipped; chunks: the same for keys below p - p % chunk.
 //
 // Requires head_dim in {16, 32, ..., 128, 256}, at most 16 query heads per
 // key/value head, page_size a multiple of 16.
@@ -83,7 +83,7 @@ decode_attention_whole_kernel(const bf16* __restrict__ qkv, const bf16* __restri
     if (q_start && q_start[s + 1] - tok != 1) return;
     const int ctx = ctx_lens[s];
     const int p = ctx - 1;
-    const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+    const int lo = first_seen_key(p, window, kMod ? mod.chunk : 0);
     const int G = nh / nkv;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
@@ -157,7 +157,7 @@ decode_attention_whole_kernel(const bf16* __restrict__ qkv, const bf16* __restri
         if (sink != -INFINITY) L += expf(sink - M);            // the sink joins the denominator once
         float res = L > 0.0f ? O / L : 0.0f;
         if constexpr (kMod)
-            if (mod.gate) res *= sigmoid_of(mod.gate[(size_t)tok * nh + kvh * G + r]);
+            if (mod.gate) res *= mod.gate_of(tok, kvh * G + r, DH, d);
         out[((size_t)tok * nh + kvh * G + r) * DH + d] = __float2bfloat16_rn(res);
     }
 }
@@ -274,15 +274,8 @@ bool li_attention_decode_accepts(int nh, int nkv, int dh, int page_size) {
 
 int li_attention_decode(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks,
                         const int* ctx_lens, const int* old_lens, const int* q_start, int S, int nh, int nkv, int dh, int page_size, int num_pages,
-                        float scale, int window, int max_ctx_len, int expected, float softcap, const float* slopes, const void* gate,
-                        int keep_first, const float* sinks, int maps, cudaStream_t stream) {
-    ScoreMod mod;
-    mod.softcap = softcap;
-    mod.slopes = slopes;
-    mod.gate = (const bf16*)gate;
-    mod.keep_first = window > 0 ? keep_first : 0;
-    mod.sinks = sinks;
-    mod.maps = maps;
+                        float scale, int window, int max_ctx_len, int expected, const AttentionOptions& opt, cudaStream_t stream) {
+    const ScoreMod mod(opt, window);
 #define LI_CASE(D)                                                                                                             \
     case D:                                                                                                                    \
         return mod.any() ? launch<D, true>(qkv, out, kcache, vcache, block_table, max_blocks, ctx_lens, old_lens, q_start, S, nh, nkv, page_size, \

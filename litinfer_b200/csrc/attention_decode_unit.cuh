@@ -15,9 +15,8 @@ using namespace attn;
 
 constexpr int kWarps = 8;
 
-__host__ __device__ inline void split_range(int ctx, int window, int kSplit, int* first, int* last) {
-    const int p = ctx - 1;
-    const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+__host__ __device__ inline void split_range(int ctx, int window, int chunk, int kSplit, int* first, int* last) {
+    const int lo = first_seen_key(ctx - 1, window, chunk);
     *first = lo / kSplit;
     *last = (ctx - 1) / kSplit;
 }
@@ -29,7 +28,7 @@ __device__ __forceinline__ void load_query_heads(unsigned (&qa)[DH / 16][4], con
                                                  const attn::ScoreMod& mod) {
     const int G = nh / nkv;
     const int maps = kMod ? mod.maps : 1;
-    const bf16* row = qkv + (size_t)tok * (nh / maps + 2 * nkv) * DH;
+    const bf16* row = qkv + (size_t)tok * ((kMod && mod.q_ld > 0) ? mod.q_ld : (nh / maps + 2 * nkv) * DH);
     const int h_lo = kvh * G + g, h_hi = h_lo + 8;
     const bf16* q_lo = g < G ? row + (size_t)(h_lo / maps) * DH : nullptr;
     const bf16* q_hi = g + 8 < G ? row + (size_t)(h_hi / maps) * DH : nullptr;
@@ -105,7 +104,7 @@ __device__ __forceinline__ void decode_attention_unit(int split, int kvh, int s,
     const int rounds = (kCut && want > 0) ? max(1, ((ctx + KB * kWarps - 1) / (KB * kWarps) + want - 1) / want) : 1;
     const int kSplit = KB * kWarps * rounds;
     const int p = ctx - 1;
-    const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+    const int lo = first_seen_key(p, window, kMod ? mod.chunk : 0);
     const int k_begin = split * kSplit;
     const int k_end = min(ctx, k_begin + kSplit);
     // q_start (a step that also holds portions of prompts): the sequence's token is row q_start[s], and only the
@@ -222,7 +221,7 @@ __device__ __forceinline__ void decode_attention_unit(int split, int kvh, int s,
     }
     // the CTA that finishes last for this (sequence, kv head) merges the splits, in split order
     int first, last;
-    split_range(ctx, window, kSplit, &first, &last);
+    split_range(ctx, window, kMod ? mod.chunk : 0, kSplit, &first, &last);
     __threadfence();
     sync();
     if (tid == 0) {
@@ -299,7 +298,7 @@ __device__ __forceinline__ void decode_attention_unit(int split, int kvh, int s,
                 const float L = l_sm[r];
                 float res = L > 0.0f ? O[q] / L : 0.0f;
                 if constexpr (kMod)
-                    if (mod.gate) res *= attn::sigmoid_of(mod.gate[(size_t)tok * nh + kvh * G + r]);
+                    if (mod.gate) res *= mod.gate_of(tok, kvh * G + r, DH, d);
                 out[((size_t)tok * nh + kvh * G + r) * DH + d] = __float2bfloat16_rn(res);
             }
         }

@@ -20,11 +20,13 @@
 // Optional changes of the scores and the output (all off when zero / null):
 //   softcap > 0:  s <- softcap * tanh(s / softcap) after the scale;
 //   slopes [nh]:  s <- s - slopes[h] * (p - key), a penalty linear in the distance;
-//   gate [T, nh]: the head's output is multiplied by 1 / (1 + exp(-gate[t, h])).
+//   gate:         the head's output is multiplied by 1 / (1 + exp(-g)), g one number a head or one an output element.
 // Optional changes of what is seen and of the softmax's denominator:
+//   chunk > 0:    keys below p - p % chunk are not seen (p sees its own chunk only);
 //   keep_first > 0 (with a window): keys 0 .. keep_first - 1 stay visible behind the window, at their own positions;
 //   sinks [nh]:   exp(sinks[h]) joins the denominator of head h once; it has no key and no value and is not scaled.
 // maps > 1: a query row of head_dim elements stands for `maps` heads (attention_mma.cuh: ScoreMod); qkv then holds nh / maps of them.
+#include "attention_options.h"
 #include "common.cuh"
 
 namespace {
@@ -37,8 +39,7 @@ __global__ void __launch_bounds__(kWarpsPerBlock * 32)
 attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T* __restrict__ kcache, const T* __restrict__ vcache,
                          const int* __restrict__ block_table, int max_blocks, const int* __restrict__ seq_of_token,
                          const int* __restrict__ positions, int total, int nh, int nkv, int dh, int page_size, int num_pages,
-                         float scale, int window, float softcap, const float* __restrict__ slopes, const T* __restrict__ gate,
-                         int keep_first, const float* __restrict__ sinks, int maps) {
+                         float scale, int window, AttentionOptions opt) {
     const int warp = blockIdx.x * kWarpsPerBlock + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     if (warp >= total) return;
@@ -46,9 +47,9 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
     const int kvh = h / (nh / nkv);
     const int s = seq_of_token[t];
     const int p = positions[t];
-    const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
-    const int row = (nh / maps + 2 * nkv) * dh;
-    const T* q = qkv + (size_t)t * row + (h / maps) * dh;
+    const int lo = first_seen_key(p, window, opt.chunk), maps = opt.maps;
+    const size_t row = opt.q_ld > 0 ? opt.q_ld : (nh / maps + 2 * nkv) * dh;
+    const T* q = qkv + t * row + (h / maps) * dh;
     const int per = (dh + 31) >> 5;
     const int part = dh / maps, part_lo = (h % maps) * part, part_hi = part_lo + part;
 
@@ -60,7 +61,8 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
         acc[i] = 0.0f;
     }
     float m = -INFINITY, l = 0.0f;
-    const float slope = slopes ? slopes[h] : 0.0f;
+    const float slope = opt.slopes ? opt.slopes[h] : 0.0f, softcap = opt.softcap;
+    const int keep_first = window > 0 ? opt.keep_first : 0;
     const int* bt = block_table + (size_t)s * max_blocks;
     // the kept first keys that lie behind the window come first, then the window: ascending order either way
     const int kept = keep_first < lo ? keep_first : lo;
@@ -93,8 +95,8 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
         m = mn;
     }
     T* o = out + (size_t)t * nh * dh + h * dh;
-    if (sinks) {
-        const float sk = sinks[h];
+    if (opt.sinks) {
+        const float sk = opt.sinks[h];
         const float mn = fmaxf(m, sk);
         const float alpha = expf(m - mn);
         l = l * alpha + expf(sk - mn);
@@ -102,11 +104,16 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
         for (int i = 0; i < kMaxPerLane; ++i) acc[i] *= alpha;
     }
     float inv = l > 0.0f ? 1.0f / l : 0.0f;
-    if (gate) inv *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * nh + h])));
+    const T* gate = opt.gate ? (const T*)opt.gate + (size_t)t * opt.gate_ld : nullptr;
+    if (gate && !opt.gate_elements) inv *= 1.0f / (1.0f + expf(-to_float(gate[h])));
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
         const int d = lane + 32 * i;
-        if (i < per && d < dh) o[d] = from_float<T>(acc[i] * inv);
+        if (i < per && d < dh) {
+            float r = acc[i] * inv;
+            if (gate && opt.gate_elements) r *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)h * dh + d])));
+            o[d] = from_float<T>(r);
+        }
     }
 }
 
@@ -114,8 +121,7 @@ attention_generic_kernel(const T* __restrict__ qkv, T* __restrict__ out, const T
 
 int li_attention_generic(const void* qkv, void* out, const void* kcache, const void* vcache, int dtype, const int* block_table,
                          int max_blocks, const int* seq_of_token, const int* positions, int T, int nh, int nkv, int dh,
-                         int page_size, int num_pages, float scale, int window, float softcap, const float* slopes, const void* gate,
-                         int keep_first, const float* sinks, int maps, cudaStream_t stream) {
+                         int page_size, int num_pages, float scale, int window, const AttentionOptions& opt, cudaStream_t stream) {
     LI_REQUIRE(dh <= 32 * kMaxPerLane, "attention: head_dim %d is larger than %d", dh, 32 * kMaxPerLane);
     const long long total = (long long)T * nh;
     LI_REQUIRE(total < (1LL << 31), "attention: too many (token, head) pairs");
@@ -123,11 +129,11 @@ int li_attention_generic(const void* qkv, void* out, const void* kcache, const v
     if (dtype == LI_F32)
         attention_generic_kernel<float><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
             (const float*)qkv, (float*)out, (const float*)kcache, (const float*)vcache, block_table, max_blocks, seq_of_token, positions,
-            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, softcap, slopes, (const float*)gate, keep_first, sinks, maps);
+            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, opt);
     else if (dtype == LI_BF16)
         attention_generic_kernel<bf16><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
             (const bf16*)qkv, (bf16*)out, (const bf16*)kcache, (const bf16*)vcache, block_table, max_blocks, seq_of_token, positions,
-            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, softcap, slopes, (const bf16*)gate, keep_first, sinks, maps);
+            (int)total, nh, nkv, dh, page_size, num_pages, scale, window, opt);
     else
         return li_fail("attention: unknown dtype %d", dtype);
     return li_check_launch("attention (generic)");

@@ -17,25 +17,43 @@
 // O = O alpha + p V.  Rows whose keys are all masked so far keep m = -inf.
 #pragma once
 
+#include "attention_options.h"
 #include "common.cuh"
 
 namespace attn {
 
 // Optional changes of the scores and of the output (see attention_generic.cu): a cap softcap * tanh(s / softcap) after
-// the scale, slopes[h] * (p - key) taken off, and the head's output times sigmoid(gate[token, h]).  And of what is seen
+// the scale, slopes[h] * (p - key) taken off, and the
+// head's output times the sigmoid of a gate (a number a head or an output element).  And of what is seen
 // and summed: with a window the keys below keep_first stay visible behind it; exp(sinks[h]) joins the denominator of head
 // h once.  And of what a query head is: with maps > 1 every query row of head_dim elements is cut into `maps` parts of equal
 // length and stands for that many heads (head h is part h % maps of row h / maps); a head's scores take its part of the key
 // against its part of the query only, its values are the whole value row (several maps of attention over the same values,
-// differential attention).  All off when zero (maps: when one).
+// differential attention).  chunk: a query sees the keys of its own chunk of so many positions only.  q_ld: elements of a row
+// of the queries' tensor where that is not a q|k|v row.  All off when zero (maps: when one).
 struct ScoreMod {
     float softcap = 0.0f;
     const float* slopes = nullptr;
     const bf16* gate = nullptr;
+    long long gate_ld = 0;
+    int gate_elements = 0;
     int keep_first = 0;
     const float* sinks = nullptr;
     int maps = 1;
-    bool any() const { return softcap > 0.0f || slopes != nullptr || gate != nullptr || keep_first > 0 || sinks != nullptr || maps > 1; }
+    int chunk = 0;
+    int q_ld = 0;
+    ScoreMod() = default;
+    ScoreMod(const AttentionOptions& o, int window)
+        : softcap(o.softcap), slopes(o.slopes), gate((const bf16*)o.gate), gate_ld(o.gate_ld), gate_elements(o.gate_elements),
+          keep_first(window > 0 ? o.keep_first : 0), sinks(o.sinks), maps(o.maps), chunk(o.chunk), q_ld(o.q_ld) {}
+    bool any() const {
+        return softcap > 0.0f || slopes != nullptr || gate != nullptr || keep_first > 0 || sinks != nullptr || maps > 1 || chunk > 0 || q_ld > 0;
+    }
+    // the gate's factor of one output element of a head (the same for all of them if the gate is one number a head)
+    __device__ __forceinline__ float gate_of(size_t tok, int h, int dh, int d) const {
+        const float g = __bfloat162float(gate[tok * gate_ld + (gate_elements ? (size_t)h * dh + d : (size_t)h)]);
+        return 1.0f / (1.0f + expf(-g));
+    }
 };
 
 // The score of a key at `dist` positions behind its query, from the scaled dot product.
@@ -43,8 +61,6 @@ __device__ __forceinline__ float changed_score(float s, float softcap, float slo
     if (softcap > 0.0f) s = softcap * tanh_fast(__fdividef(s, softcap));
     return fmaf(-slope, (float)dist, s);
 }
-
-__device__ __forceinline__ float sigmoid_of(bf16 g) { return 1.0f / (1.0f + expf(-__bfloat162float(g))); }
 
 // The same for the two rows a thread sees in a tile of 16 rows: their slopes and the position of their query.
 struct RowMod {

@@ -22,7 +22,7 @@
 // values of the portion itself are already in the cache (the rope kernel ran
 // before), so history and new tokens are read the same way, through the block
 // table.  Token i of a portion of n tokens in a context of c sits at position
-// p = c - n + i and sees keys max(0, p - window + 1) .. p.
+// p = c - n + i and sees keys max(0, p - window + 1) .. p (of its own chunk, with one).
 //
 // Requires head_dim in {16, 32, ..., 128, 256} and page_size a multiple of 16.
 #include "attention_mma.cuh"
@@ -84,7 +84,7 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
     const int ctx = ctx_lens[s];
     const int kvh = h / (nh / nkv);
     const int maps = kMod ? mod.maps : 1;                  // heads that a query row stands for; this head's part of it
-    const int row_elems = (nh / maps + 2 * nkv) * DH;
+    const int row_elems = (kMod && mod.q_ld > 0) ? mod.q_ld : (nh / maps + 2 * nkv) * DH;
     [[maybe_unused]] const int part_lo = kMod ? (h % maps) * (DH / maps) : 0, part_hi = kMod ? part_lo + DH / maps : DH;
     const int i0 = cta_i0 + warp * 16;                     // first token of this warp within the portion
     const bool warp_active = i0 < n;
@@ -119,16 +119,17 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
     int lo[2], hi[2];
     hi[0] = (warp_active && r_lo < n) ? ctx - n + r_lo : -1;
     hi[1] = (warp_active && r_hi < n) ? ctx - n + r_hi : -1;
-    lo[0] = (window > 0 && hi[0] - window + 1 > 0) ? hi[0] - window + 1 : 0;
-    lo[1] = (window > 0 && hi[1] - window + 1 > 0) ? hi[1] - window + 1 : 0;
+    const int chunk = kMod ? mod.chunk : 0;
+    lo[0] = first_seen_key(hi[0], window, chunk);
+    lo[1] = first_seen_key(hi[1], window, chunk);
     // what the CTA as a whole reads, and this warp's share of it
     const int cta_rows = min(kTile, n - cta_i0);
     const int cta_p_first = ctx - n + cta_i0, cta_p_last = cta_p_first + cta_rows - 1;
-    const int cta_key_lo = (window > 0 && cta_p_first - window + 1 > 0) ? cta_p_first - window + 1 : 0;
+    const int cta_key_lo = first_seen_key(cta_p_first, window, chunk);
     const int warp_p_first = ctx - n + i0;
     const int warp_p_last = warp_p_first + min(16, n - i0) - 1;
-    const int warp_key_lo = (window > 0 && warp_p_first - window + 1 > 0) ? warp_p_first - window + 1 : 0;
-    const int warp_lo_max = (window > 0 && warp_p_last - window + 1 > 0) ? warp_p_last - window + 1 : 0;     // the largest lower bound among the warp's rows
+    const int warp_key_lo = first_seen_key(warp_p_first, window, chunk);
+    const int warp_lo_max = first_seen_key(warp_p_last, window, chunk);     // the largest lower bound among the warp's rows
     // kMod: the scores are changed (cap, distance penalty) before the softmax; they are then brought to base-2 units at
     // once and the factor below is 1
     const float scale_log2 = kMod ? 1.0f : scale * 1.4426950408889634f;
@@ -303,9 +304,9 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
     }
     float inv0 = l0 > 0.0f ? shrink0 / l0 : 0.0f, inv1 = l1 > 0.0f ? shrink1 / l1 : 0.0f;
     if constexpr (kMod) {
-        if (mod.gate) {
-            if (r_lo < n) inv0 *= attn::sigmoid_of(mod.gate[(size_t)(tok0 + r_lo) * nh + h]);
-            if (r_hi < n) inv1 *= attn::sigmoid_of(mod.gate[(size_t)(tok0 + r_hi) * nh + h]);
+        if (mod.gate && !mod.gate_elements) {
+            if (r_lo < n) inv0 *= mod.gate_of(tok0 + r_lo, h, DH, 0);
+            if (r_hi < n) inv1 *= mod.gate_of(tok0 + r_hi, h, DH, 0);
         }
     }
     bf16* o_lo = out + (size_t)(tok0 + r_lo) * nh * DH + (size_t)h * DH;
@@ -313,6 +314,15 @@ prefill_attention_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ out, c
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
         const int col = j * 8 + 2 * t;
+        if constexpr (kMod) {
+            if (mod.gate && mod.gate_elements) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    if (r_lo < n) st.o[j][e] *= mod.gate_of(tok0 + r_lo, h, DH, col + e);
+                    if (r_hi < n) st.o[j][2 + e] *= mod.gate_of(tok0 + r_hi, h, DH, col + e);
+                }
+            }
+        }
         if (r_lo < n) *reinterpret_cast<unsigned*>(o_lo + col) = pack_bf16(st.o[j][0] * inv0, st.o[j][1] * inv0);
         if (r_hi < n) *reinterpret_cast<unsigned*>(o_hi + col) = pack_bf16(st.o[j][2] * inv1, st.o[j][3] * inv1);
     }
@@ -346,16 +356,9 @@ bool li_attention_prefill_accepts(int nh, int nkv, int dh, int page_size) {
 
 int li_attention_prefill(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks,
                          const int* q_start, const int* ctx_lens, int T, int S, int nh, int nkv, int dh, int page_size,
-                         int num_pages, float scale, int window, int max_q_len, int skip_single, float softcap, const float* slopes,
-                         const void* gate, int keep_first, const float* sinks, int maps, cudaStream_t stream) {
+                         int num_pages, float scale, int window, int max_q_len, int skip_single, const AttentionOptions& opt, cudaStream_t stream) {
     (void)T;
-    attn::ScoreMod mod;
-    mod.softcap = softcap;
-    mod.slopes = slopes;
-    mod.gate = (const bf16*)gate;
-    mod.keep_first = window > 0 ? keep_first : 0;
-    mod.sinks = sinks;
-    mod.maps = maps;
+    const attn::ScoreMod mod(opt, window);
     LI_REQUIRE(scale > 0.0f, "attention (prefill): the scale must be positive, got %g", (double)scale);
 #define LI_CASE(D)                                                                                                                  \
     case D:                                                                                                                         \

@@ -20,7 +20,7 @@
 //              than 2^8 (see kLazy).  S of tile j + 1 is issued before P V of tile j.
 // Keys and values of the portion itself are already in the cache (the rope kernel ran before).  Token i of a
 // portion of n tokens in a context of c sits at position p = c - n + i and sees keys max(0, p - window + 1) .. p (and,
-// with a window, the sequence's first keep_first keys behind it).
+// with a window, the sequence's first keep_first keys behind it; with chunks, of its own chunk only).
 // Keys of a tile that lie past the context are read from whatever page the table names (page 0 if none) and get
 // probability zero; the cache holds finite numbers only.
 //
@@ -29,6 +29,7 @@
 //
 // Requires head_dim 64 or 128 and page_size a multiple of 16.
 #define LI_PDL_KIND 4
+#include "attention_options.h"
 #include "tcgen05.cuh"
 
 namespace tc {
@@ -79,17 +80,20 @@ __device__ __forceinline__ float tanh_small(float x) {
     return x * p;
 }
 
-// kCap: scores are capped, cap * tanh(s / cap), before the mask and the softmax (`softcap` > 0).  maps > 1: a query row of DH elements
+// kForm: what becomes of the scores before the mask and the softmax.  kCapped: cap * tanh(s / cap) (`softcap` > 0); kSloped:
+// slopes[h] * (p - key) is taken off.  maps > 1: a query row of DH elements
 // stands for that many heads, each with a part of it (attention_mma.cuh: ScoreMod): a head's product S takes the k-steps of
 // its own part only, and with head_dim 128 and two maps only that part's panel of the keys is brought in.
-template <int DH, bool kCap>
+enum { kAsTheyAre = 0, kCapped = 1, kSloped = 2 };
+
+template <int DH, int kForm>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const int* __restrict__ block_table,
                             int max_blocks, const int* __restrict__ q_start, const int* __restrict__ ctx_lens, int nh, int nkv,
                             int page_size, int num_pages, float scale, int window, int skip_single, int* __restrict__ error_flag, int trace,
                             const int* __restrict__ units, float* __restrict__ partial, unsigned* __restrict__ counters,
-                            const float* __restrict__ sinks, int keep_first, float softcap, int maps) {
+                            const AttentionOptions opt) {
     extern __shared__ unsigned char smem_raw[];
     Smem<DH>& sm = *reinterpret_cast<Smem<DH>*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     // the tiles want 1024-byte alignment; with head_dim 128 there is not a whole kilobyte to spare for it
@@ -98,6 +102,7 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
         return;
     }
     constexpr int kPanels = DH / 64;
+    const int maps = opt.maps, keep_first = opt.keep_first;
     // this head's part of the query row: k-steps of the product S, and the panels of the keys they read
     const int k_lo = ((int)blockIdx.x % maps) * (DH / 16 / maps), k_hi = k_lo + DH / 16 / maps;
     const int panel_lo = k_lo >> 2, panel_hi = (k_hi + 3) >> 2;
@@ -125,7 +130,7 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
     const int kvh = h / (nh / nkv);
     const int cta_rows = min(kRows, n - cta_i0);
     const int p_first = ctx - n + cta_i0, p_last = p_first + cta_rows - 1;
-    const int key_lo = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+    const int key_lo = first_seen_key(p_first, window, opt.chunk);
     // The key tiles of this tile of tokens.  When the step has so few tiles of tokens that multiprocessors would stand idle,
     // the work list shares them out among several CTAs (entries with parts > 1), at least kPartTiles each, and the last
     // CTA to finish adds the partial results up.  The workspace has room for one partial result per multiprocessor.
@@ -288,10 +293,11 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
         constexpr int HK = kKeys / 2, HD = DH / 2;
         const bool valid = cta_i0 + r < n;
         const int p = valid ? p_first + r : -1;                  // its position; no key is visible to an unused row
-        const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
-        // (capped scores are brought to base-2 units as they are capped, and the factor below is 1)
-        const float scale_log2 = kCap ? 1.0f : scale * 1.4426950408889634f;
-        [[maybe_unused]] const float cap_in = kCap ? scale / softcap : 0.0f, cap_out = softcap * 1.4426950408889634f;
+        const int lo = first_seen_key(p, window, opt.chunk);
+        // (changed scores are brought to base-2 units as they are changed, and the factor below is 1)
+        const float scale_log2 = kForm != kAsTheyAre ? 1.0f : scale * 1.4426950408889634f;
+        [[maybe_unused]] const float cap_in = kForm == kCapped ? scale / opt.softcap : 0.0f, cap_out = opt.softcap * 1.4426950408889634f;
+        [[maybe_unused]] const float slope2 = kForm == kSloped ? opt.slopes[h] * 1.4426950408889634f : 0.0f;
         // m: the maximum the exponentials are taken against.  It follows the true maximum lazily: only when that has grown by
         // more than kLazy (in powers of two) is the output so far, which accumulates in tensor memory, scaled down to the
         // new one.  Until then the probabilities may reach 2^kLazy, which costs bfloat16 and the float sums nothing, and
@@ -329,7 +335,12 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
             // this thread's 64 scores of the tile, read once and kept for both passes; a key the row does not see reads -inf
             float v[HK];
             tmem_ld_32x64(tmem_s + 128 * (j & 1) + lane_addr + half * HK, v);
-            if constexpr (kCap) {
+            if constexpr (kForm == kSloped) {
+                const float first = slope2 * (float)(key0 - p), factor = scale * 1.4426950408889634f;
+#pragma unroll
+                for (int i = 0; i < HK; ++i) v[i] = fmaf(v[i], factor, fmaf(slope2, (float)i, first));
+            }
+            if constexpr (kForm == kCapped) {
                 // cap * tanh(s scale / cap) in base-2 units: small arguments by a polynomial on the multiply-add pipe, and if
                 // any of the thread's is larger all of them through the exponential
                 float top = 0.0f;
@@ -485,8 +496,26 @@ prefill_attention_tc_kernel(const bf16* __restrict__ qkv, long long row_elems, c
             if (lane == 0) atomicExch(error_flag, 13);
         } else if (store) {
             // a sink: exp(sinks[h]) joins the denominator once (it has no key and no value); the maxima are in base-2 units
-            if (sinks != nullptr && m_ref != -INFINITY) l += exp2f(sinks[h] * 1.4426950408889634f - m_ref);
-            const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            if (opt.sinks != nullptr && m_ref != -INFINITY) l += exp2f(opt.sinks[h] * 1.4426950408889634f - m_ref);
+            float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            if (opt.gate != nullptr) {
+                const bf16* gate = (const bf16*)opt.gate + (size_t)(tok0 + cta_i0 + r) * opt.gate_ld;
+                if (!opt.gate_elements) {
+                    inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[h])));
+                } else {
+                    gate += (size_t)h * DH + half * HD;
+#pragma unroll
+                    for (int d = 0; d < HD; d += 8) {
+                        const uint4 g4 = *reinterpret_cast<const uint4*>(gate + d);
+                        const unsigned w[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            o[d + 2 * i] = __fdividef(o[d + 2 * i], 1.0f + fast_exp2(-1.4426950408889634f * __uint_as_float(w[i] << 16)));
+                            o[d + 2 * i + 1] = __fdividef(o[d + 2 * i + 1], 1.0f + fast_exp2(-1.4426950408889634f * __uint_as_float(w[i] & 0xffff0000u)));
+                        }
+                    }
+                }
+            }
             bf16* dst = out + ((size_t)(tok0 + cta_i0 + r) * nh + h) * DH + half * HD;
 #pragma unroll
             for (int d = 0; d < HD; d += 8) {
@@ -542,23 +571,23 @@ SplitSpace& split_space() {
     return space;
 }
 
-template <int DH, bool kCap>
+template <int DH, int kForm>
 int launch(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks, const int* q_start,
            const int* ctx_lens, int T, int S, int nh, int nkv, int page_size, int num_pages, float scale, int window, int max_q_len,
-           int skip_single, const int* units, int unit_slots, const float* sinks, int keep_first, float softcap, int maps, cudaStream_t stream) {
+           int skip_single, const int* units, int unit_slots, const AttentionOptions& opt, cudaStream_t stream) {
     EncodeTiledFn encode = nullptr;
     int *err_host = nullptr, *err_dev = nullptr;
     if (int rc = setup(&encode, &err_host, &err_dev)) return rc;
     if (*err_host != 0)
         return li_fail("attention (tcgen05): an earlier launch gave up waiting on a barrier (status %d); the results since then are invalid", *err_host);
     CUtensorMap map_k, map_v;
-    const long long row_elems = (long long)(nh / maps + 2 * nkv) * DH;
+    const long long row_elems = opt.q_ld > 0 ? opt.q_ld : (long long)(nh / opt.maps + 2 * nkv) * DH;
     if (int rc = make_map_ex(&map_k, kcache, (unsigned long long)num_pages * nkv * page_size, DH, 64, 16, 128)) return rc;
     if (int rc = make_map_ex(&map_v, vcache, (unsigned long long)num_pages * nkv * DH, (unsigned long long)page_size, 16, DH, 32)) return rc;
     const size_t smem = sizeof(Smem<DH>) + smem_pad<DH>();
     static bool raised = false;
     if (!raised) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<DH, kCap>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<DH, kForm>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return li_fail("attention (tcgen05): cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
         raised = true;
     }
@@ -578,9 +607,9 @@ int launch(const void* qkv, void* out, const void* kcache, const void* vcache, c
     }
     const dim3 grid = units ? dim3(nh, unit_slots, 1) : dim3(nh, ceil_div(max_q_len, kRows), S);
     static const int trace = getenv("LITINFER_B200_ATTN_TRACE") ? 1 : 0;
-    li_launch_pdl(prefill_attention_tc_kernel<DH, kCap>, grid, dim3(kThreads), smem, stream, (const bf16*)qkv, row_elems, map_k, map_v, (bf16*)out, block_table, max_blocks,
+    li_launch_pdl(prefill_attention_tc_kernel<DH, kForm>, grid, dim3(kThreads), smem, stream, (const bf16*)qkv, row_elems, map_k, map_v, (bf16*)out, block_table, max_blocks,
                   q_start, ctx_lens, nh, nkv, page_size, num_pages, scale, window, skip_single, err_dev, trace, units, partial,
-                  space.counters, sinks, keep_first, softcap, maps);
+                  space.counters, opt);
     return li_check_launch("attention (tcgen05)");
 }
 
@@ -591,18 +620,24 @@ bool li_attention_tcgen05_accepts(const void* qkv, const void* kcache, const voi
     return aligned && (dh == 64 || dh == 128) && nh % nkv == 0 && page_size % 16 == 0 && page_size <= 256;
 }
 
+// which options these tiles take (the others are the mma.sync tiles' business)
+bool li_attention_tcgen05_takes(const AttentionOptions& opt) {
+    return opt.maps <= 2 && !(opt.softcap > 0.0f && opt.slopes != nullptr) && opt.q_ld % 8 == 0 &&
+           (opt.gate == nullptr || opt.gate_elements == 0 || (opt.gate_ld % 8 == 0 && (uintptr_t)opt.gate % 16 == 0));
+}
+
 int li_attention_tcgen05(const void* qkv, void* out, const void* kcache, const void* vcache, const int* block_table, int max_blocks,
                          const int* q_start, const int* ctx_lens, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages,
-                         float scale, int window, int max_q_len, int skip_single, const int* units, int unit_slots, const float* sinks,
-                         int keep_first, float softcap, int maps, cudaStream_t stream) {
-    LI_REQUIRE(maps == 1 || maps == 2, "attention (tcgen05): takes one or two maps a query row, not %d", maps);
+                         float scale, int window, int max_q_len, int skip_single, const int* units, int unit_slots, const AttentionOptions& opt, cudaStream_t stream) {
+    LI_REQUIRE(opt.maps == 1 || opt.maps == 2, "attention (tcgen05): takes one or two maps a query row, not %d", opt.maps);
+    LI_REQUIRE(li_attention_tcgen05_takes(opt), "attention (tcgen05): a cap together with slopes, or rows that are not on 16-byte boundaries");
     LI_REQUIRE(li_attention_tcgen05_accepts(qkv, kcache, vcache, nh, nkv, dh, page_size),
                "attention (tcgen05): refuses heads=%d/%d head_dim=%d page=%d (head_dim 64 or 128, pages a multiple of 16)", nh, nkv, dh, page_size);
     LI_REQUIRE(scale > 0.0f, "attention (tcgen05): the scale must be positive");
-#define LI_CASE(D, CAP)                                                                                                                        \
-    launch<D, CAP>(qkv, out, kcache, vcache, block_table, max_blocks, q_start, ctx_lens, T, S, nh, nkv, page_size, num_pages, scale, window, \
-                   max_q_len, skip_single, units, unit_slots, sinks, keep_first, softcap, maps, stream)
-    if (dh == 64) return softcap > 0.0f ? LI_CASE(64, true) : LI_CASE(64, false);
-    return softcap > 0.0f ? LI_CASE(128, true) : LI_CASE(128, false);
+#define LI_CASE(D, FORM)                                                                                                                       \
+    launch<D, FORM>(qkv, out, kcache, vcache, block_table, max_blocks, q_start, ctx_lens, T, S, nh, nkv, page_size, num_pages, scale, window, \
+                   max_q_len, skip_single, units, unit_slots, opt, stream)
+    if (dh == 64) return opt.softcap > 0.0f ? LI_CASE(64, kCapped) : opt.slopes ? LI_CASE(64, kSloped) : LI_CASE(64, kAsTheyAre);
+    return opt.softcap > 0.0f ? LI_CASE(128, kCapped) : opt.slopes ? LI_CASE(128, kSloped) : LI_CASE(128, kAsTheyAre);
 #undef LI_CASE
 }

@@ -68,6 +68,18 @@ __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floa
     return r;
 }
 
+// The same for two sums at once.
+__device__ __forceinline__ void block_sum2(float& a, float& b, float* scratch /* >= 64 floats */) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int nwarps = (blockDim.x + 31) >> 5;
+    a = warp_sum(a), b = warp_sum(b);
+    __syncthreads();
+    if (lane == 0) scratch[warp] = a, scratch[32 + warp] = b;
+    __syncthreads();
+    a = warp_sum(lane < nwarps ? scratch[lane] : 0.0f);
+    b = warp_sum(lane < nwarps ? scratch[32 + lane] : 0.0f);
+}
+
 // 2^x by the hardware approximation (about two units in the last place): used where the result is rounded to bfloat16
 // right after (attention probabilities) while the running sums stay in float.
 __device__ __forceinline__ float fast_exp2(float x) {

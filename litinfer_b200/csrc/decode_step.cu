@@ -755,7 +755,7 @@ __device__ void consume(const LiDecodeStep& p, Consumer& c) {
 #pragma unroll 1
             for (int s = 0; s < M; ++s) {
                 int first, last;
-                attn_decode::split_range(p.ctx_lens[s], L->window, 256, &first, &last);
+                attn_decode::split_range(p.ctx_lens[s], L->window, 0, 256, &first, &last);
                 const int nsp = last - first + 1;
                 const long long n = (long long)nsp * nkv;
                 long long j = base + (((long long)r - base) % ctas + ctas) % ctas;

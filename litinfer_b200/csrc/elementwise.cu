@@ -431,6 +431,39 @@ LI_EXPORT int li_geglu(const void* gate_up, void* out, int dtype, int T, int I, 
     return li_check_launch("geglu");
 }
 
+// A gate that opens a token's row of a table: out[t, i] = gelu(z[t, i]) * table[ids[t], col + i], the tanh form of gelu.  z float
+// (a product's sums as they are), table and out in the run dtype; float arithmetic, one rounding.
+namespace {
+template <typename T>
+__global__ void gelu_token_rows_kernel(const float* __restrict__ z, const T* __restrict__ table, long long ld, int col, int rows, const int* __restrict__ ids,
+                                       T* __restrict__ out, int n, long long total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const long long t = i / n;
+    int id = ids[t];
+    if (id < 0 || id >= rows) id = 0;                  // validated on the host; keep the read inside the table
+    out[i] = from_float<T>(geglu_of<T>(z[i], to_float(table[id * ld + col + (int)(i - t * n)])));
+}
+}  // namespace
+
+LI_EXPORT int li_gelu_token_rows(const float* z, const void* table, int dtype, long long ld, int col, int rows, const int* ids, void* out, int T, int n,
+                                 cudaStream_t stream) {
+    LI_REQUIRE(T >= 0 && n > 0 && rows > 0 && col >= 0 && col + n <= ld, "gelu_token_rows: columns %d .. %d of rows of %lld", col, col + n, ld);
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "gelu_token_rows: unknown dtype %d", dtype);
+    if (T == 0) return 0;
+    const long long total = (long long)T * n;
+    const dim3 grid((unsigned)ceil_div_ll(total, 128));
+    cudaError_t e;
+    if (dtype == LI_F32)
+        e = li_launch_pdl(gelu_token_rows_kernel<float>, grid, dim3(128), 0, stream, z, (const float*)table, ld, col, rows, ids, (float*)out, n, total);
+    else
+        e = li_launch_pdl(gelu_token_rows_kernel<bf16>, grid, dim3(128), 0, stream, z, (const bf16*)table, ld, col, rows, ids, (bf16*)out, n, total);
+    if (e != cudaSuccess) return li_fail("gelu_token_rows: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("gelu_token_rows");
+}
+
 // PolyNorm and a sigmoid gate.
 //   li_polynorm: per token row z [n]: out = a N(z) + b N(z^2) + c N(z^3) + e with powers element by element and
 //     N(v) = v / sqrt(mean(v^2) + eps); coef = {a, b, c, e} float on the device.  The three means are taken in one pass (the row

@@ -397,14 +397,115 @@ __device__ __forceinline__ void route_token_grouped(const float* logits, const f
     }
 }
 
+// The same with sigmoid scores: the choice scores are sigmoid(logits) + correction, a group's score is the sum of its two
+// largest choice scores (of its only one where a group has one expert), and the weights are the chosen experts' sigmoid scores
+// times `scale`, not renormalised.  choice: E floats of shared memory of this warp's own (may be where the logits lie).
 template <int PER>
-__global__ void moe_route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int T, int E, int top, int groups,
-                                         int keep, float scale, int* __restrict__ ids, float* __restrict__ weights) {
+__device__ __forceinline__ void route_token_sigmoid_groups(const float* logits, const float* __restrict__ correction, int E, int top, int groups, int keep,
+                                                           float scale, int* ids, float* weights, float* choice, int lane) {
+    float s[PER], c[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int e = lane + 32 * i;
+        s[i] = e < E ? 1.0f / (1.0f + expf(-logits[e])) : 0.0f;
+        c[i] = e < E ? s[i] + (correction ? correction[e] : 0.0f) : -INFINITY;
+    }
+    if (keep < groups) {
+        const int per = E / groups;
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (lane + 32 * i < E) choice[lane + 32 * i] = c[i];
+        __syncwarp();
+        // a lane scores the groups lane, lane + 32, ...
+        float gs[PER];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int g = lane + 32 * i;
+            gs[i] = -INFINITY;
+            if (g < groups) {
+                float first = -INFINITY, second = -INFINITY;
+                for (int j = 0; j < per; ++j) {
+                    const float v = choice[g * per + j];
+                    second = fmaxf(second, fminf(first, v));
+                    first = fmaxf(first, v);
+                }
+                gs[i] = per > 1 ? first + second : first;
+            }
+        }
+        // `keep` rounds that each take the best group left, the lower index among equals
+        unsigned mask[PER];                      // bit g of word g / 32: group g was taken
+#pragma unroll
+        for (int i = 0; i < PER; ++i) mask[i] = 0u;
+        for (int round = 0; round < keep; ++round) {
+            float best = -INFINITY;
+            int arg = 0x7fffffff;
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                const int g = lane + 32 * i;
+                if (g < groups && !((mask[i] >> lane) & 1u) && (gs[i] > best || arg == 0x7fffffff)) best = gs[i], arg = g;
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+                if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa;
+            }
+#pragma unroll
+            for (int i = 0; i < PER; ++i)
+                if (arg >> 5 == i) mask[i] |= 1u << (arg & 31);
+        }
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int g = (lane + 32 * i) / per;
+            bool taken = false;
+#pragma unroll
+            for (int j = 0; j < PER; ++j)
+                if (g >> 5 == j) taken = (mask[j] >> (g & 31)) & 1u;
+            if (!taken) c[i] = -INFINITY;
+        }
+    }
+    for (int k = 0; k < top; ++k) {
+        float best = -INFINITY, score = 0.0f;
+        int arg = 0x7fffffff;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int e = lane + 32 * i;
+            if (e < E && c[i] > best) best = c[i], arg = e, score = s[i];
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+            const float os = __shfl_xor_sync(0xffffffffu, score, o);
+            if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa, score = os;
+        }
+        if (arg >= E) arg = 0, score = 0.0f;     // (scores that are no numbers: any expert, with no weight)
+        if (lane == 0) {
+            ids[k] = arg;
+            weights[k] = score * scale;
+        }
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (lane + 32 * i == arg) c[i] = -INFINITY;
+    }
+}
+
+constexpr int kRouteWarps = 4;
+
+template <int PER>
+__global__ void __launch_bounds__(kRouteWarps * 32)
+moe_route_grouped_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int scoring, int T, int E, int top, int groups,
+                         int keep, float scale, int* __restrict__ ids, float* __restrict__ weights) {
+    __shared__ float choice[kRouteWarps][32 * PER];
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int t = blockIdx.x * kRouteWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= T) return;
-    route_token_grouped<PER>(logits + (size_t)t * E, correction, E, top, groups, keep, scale, ids + (size_t)t * top, weights + (size_t)t * top, threadIdx.x & 31);
+    if (scoring == 3)
+        route_token_sigmoid_groups<PER>(logits + (size_t)t * E, correction, E, top, groups, keep, scale, ids + (size_t)t * top, weights + (size_t)t * top,
+                                        choice[threadIdx.x >> 5], lane);
+    else
+        route_token_grouped<PER>(logits + (size_t)t * E, correction, E, top, groups, keep, scale, ids + (size_t)t * top, weights + (size_t)t * top, lane);
 }
 
 // The front of a mixture for a small step as one block: the router's product (a warp per token and two experts, float sums),
@@ -469,7 +570,8 @@ moe_small_step_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
     }
     __syncthreads();
     for (int t = warp; t < tokens; t += 32) {
-        if (scoring == 2) route_token_grouped<PER>(logits + t * E, correction, E, top, groups, keep, scale, ids + t * top, weights + (size_t)t * top, lane);
+        if (scoring == 3) route_token_sigmoid_groups<PER>(logits + t * E, correction, E, top, groups, keep, scale, ids + t * top, weights + (size_t)t * top, logits + t * E, lane);
+        else if (scoring == 2) route_token_grouped<PER>(logits + t * E, correction, E, top, groups, keep, scale, ids + t * top, weights + (size_t)t * top, lane);
         else route_token<PER>(logits + t * E, scoring, E, top, ids + t * top, weights + (size_t)t * top, lane);
     }
     __syncthreads();
@@ -671,16 +773,18 @@ LI_EXPORT int li_moe_route(const float* logits, int scoring, int T, int E, int t
     return li_check_launch("moe_route");
 }
 
-// See moe_route_grouped_kernel.  correction (may be NULL): [E] float; groups divides E; 1 <= keep <= groups; the kept groups
+// scoring 2: softmax scores, a group counts as its best, weights renormalised (route_token_grouped); 3: sigmoid scores, a group
+// counts as its two best, weights as they are (route_token_sigmoid_groups).  correction (may be NULL): [E] float; groups divides E; 1 <= keep <= groups; the kept groups
 // must hold at least `top` experts.
-LI_EXPORT int li_moe_route_grouped(const float* logits, const float* correction, int T, int E, int top, int groups, int keep, float scale, int* ids,
+LI_EXPORT int li_moe_route_grouped(const float* logits, const float* correction, int scoring, int T, int E, int top, int groups, int keep, float scale, int* ids,
                                    float* weights, cudaStream_t stream) {
     LI_REQUIRE(T >= 0 && E > 0 && top > 0 && top <= E, "moe_route_grouped: %d of %d experts", top, E);
+    LI_REQUIRE(scoring == 2 || scoring == 3, "moe_route_grouped: unknown scoring %d", scoring);
     LI_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top,
                "moe_route_grouped: %d of %d groups of %d experts cannot give %d choices", keep, groups, groups >= 1 ? E / groups : 0, top);
     LI_REQUIRE(E <= 32 * kMaxExpertsPerLane, "moe_route_grouped: %d experts are more than %d", E, 32 * kMaxExpertsPerLane);
     if (T == 0) return 0;
-    const cudaError_t e = li_launch_pdl(E <= 32 ? moe_route_grouped_kernel<1> : moe_route_grouped_kernel<kMaxExpertsPerLane>, dim3(ceil_div(T, 4)), dim3(128), 0, stream, logits, correction, T, E, top, groups, keep,
+    const cudaError_t e = li_launch_pdl(E <= 32 ? moe_route_grouped_kernel<1> : moe_route_grouped_kernel<kMaxExpertsPerLane>, dim3(ceil_div(T, kRouteWarps)), dim3(kRouteWarps * 32), 0, stream, logits, correction, scoring, T, E, top, groups, keep,
                                         scale, ids, weights);
     if (e != cudaSuccess) return li_fail("moe_route_grouped: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("moe_route_grouped");
@@ -730,7 +834,7 @@ LI_EXPORT int li_moe_combine(const void* rows, int dtype, const int* place_of, c
 }
 
 // The front of a mixture for a step of few tokens as one launch: router logits h [T, H] w [E, H]^T (+ bias), the choice
-// (scoring 0, 1 as in li_moe_route; 2 as in li_moe_route_grouped) and the stable sort without padding: weights [T, top], offsets
+// (scoring 0, 1 as in li_moe_route; 2, 3 as in li_moe_route_grouped) and the stable sort without padding: weights [T, top], offsets
 // [E + 1], pair_at and place_of [T top].  li_moe_small_step_accepts says for which sizes.
 LI_EXPORT int li_moe_small_step_accepts(int dtype, int T, int H, int E, int top) {
     const int vec = dtype == LI_BF16 ? 8 : 4;
@@ -743,8 +847,8 @@ LI_EXPORT int li_moe_small_step(const void* h, const void* w, const float* bias,
                                 int* place_of, cudaStream_t stream) {
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "moe_small_step: unknown dtype %d", dtype);
     LI_REQUIRE(li_moe_small_step_accepts(dtype, T, H, E, top), "moe_small_step: refuses T=%d H=%d, %d of %d experts", T, H, top, E);
-    LI_REQUIRE(scoring >= 0 && scoring <= 2, "moe_small_step: unknown scoring %d", scoring);
-    LI_REQUIRE(scoring != 2 || (groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top),
+    LI_REQUIRE(scoring >= 0 && scoring <= 3, "moe_small_step: unknown scoring %d", scoring);
+    LI_REQUIRE(scoring < 2 || (groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top),
                "moe_small_step: %d of %d groups of %d experts cannot give %d choices", keep, groups, E, top);
     LI_REQUIRE(((uintptr_t)h % 16) == 0 && ((uintptr_t)w % 16) == 0, "moe_small_step: operands must be 16-byte aligned");
     const int threads = 1024;

@@ -46,6 +46,9 @@ void li_cm_destroy(void* h);
 /* The first `keys` keys of every request stay readable in a windowed group: their pages never go back behind the window.
  * To be set before any request is admitted. */
 int li_cm_keep_first(void* h, int group, int keys);
+/* Queries of this group read the keys of their own chunk of positions only, with chunks of each of n sizes: pages of chunks
+ * that are over go back.  To be set before any request is admitted. */
+int li_cm_chunks(void* h, int group, int n, const int* sizes);
 
 /* Free ids of a pool; which: -1 the state slots, else a group's pages. */
 int li_cm_num_free(void* h, int which);

@@ -62,6 +62,18 @@ LI_HOST_EXPORT int li_cm_keep_first(void* h, int group, int keys) {
     return LI_HOST_OK;
 }
 
+// Queries of this group read the keys of their own chunk of positions only, with chunks of each of `n` sizes (layers that share
+// the group's cache): pages of chunks that are over go back, whatever the window.  To be set before any request is admitted.
+LI_HOST_EXPORT int li_cm_chunks(void* h, int group, int n, const int* sizes) {
+    Manager* m = static_cast<Manager*>(h);
+    if (group < 0 || group >= (int)m->pools.size() || n < 0) return fail(LI_HOST_VALUE, "chunks: group %d, %d sizes", group, n);
+    for (int i = 0; i < n; ++i)
+        if (sizes[i] <= 0) return fail(LI_HOST_VALUE, "chunks: a chunk of %d positions", sizes[i]);
+    if (!m->live.empty()) return fail(LI_HOST_POOL, "chunks: requests are live");
+    m->chunks[(size_t)group].assign(sizes, sizes + n);
+    return LI_HOST_OK;
+}
+
 // which: -1 the state slots, else a group's pages
 static Pool* pool_of(Manager* m, int which) {
     if (which < 0) return &m->slots;
@@ -131,7 +143,7 @@ LI_HOST_EXPORT int li_cm_commit(void* h, int id, int new_length) {
     if (new_length < r->length) return fail(LI_HOST_POOL, "a request's length never shrinks");
     r->length = new_length;
     for (size_t g = 0; g < m->pools.size(); ++g) {
-        if (m->windows[g] <= 0) continue;
+        if (!m->bounded((int)g)) continue;
         std::vector<int>& t = r->tables[g];
         const int upto = std::min(m->first_needed_page((int)g, new_length), (int)t.size());
         for (int lp = m->kept_pages((int)g); lp < upto; ++lp)

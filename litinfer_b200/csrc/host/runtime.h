@@ -78,12 +78,13 @@ struct Manager {
     int page_size, num_pages, max_requests;
     std::vector<int> windows;                      // per group: keys a query still reads, 0 = all of them
     std::vector<int> keeps;                        // per group: the first keys of a request that every later query still reads
+    std::vector<std::vector<int>> chunks;          // per group: sizes of chunks whose keys a query of the same chunk still reads
     std::vector<Pool> pools;
     Pool slots;
     std::unordered_map<int, Request> live;
 
     Manager(int groups, const int* win, int pages, int page, int requests)
-        : page_size(page), num_pages(pages), max_requests(requests), windows(win, win + groups), keeps((size_t)groups, 0), slots(requests, "state slot") {
+        : page_size(page), num_pages(pages), max_requests(requests), windows(win, win + groups), keeps((size_t)groups, 0), chunks((size_t)groups), slots(requests, "state slot") {
         for (int g = 0; g < groups; ++g) pools.emplace_back(pages, "page");
     }
     Request* find(int id) {
@@ -93,10 +94,15 @@ struct Manager {
     int blocks(int tokens) const { return (tokens + page_size - 1) / page_size; }
     // logical pages at the start of a request that a window never gives back (they hold the kept first keys)
     int kept_pages(int g) const { return blocks(keeps[(size_t)g]); }
-    // first logical page that a query at a position >= length can still read
+    // whether a request's oldest keys are given back at all
+    bool bounded(int g) const { return windows[(size_t)g] > 0 || !chunks[(size_t)g].empty(); }
+    // first logical page that a query at a position >= length can still read, through the window or within a chunk of any of
+    // the sizes (layers that share a cache may have chunks of different sizes)
     int first_needed_page(int g, int length) const {
-        if (windows[(size_t)g] <= 0) return 0;
-        const int first_key = length - windows[(size_t)g] + 1;
+        if (!bounded(g)) return 0;
+        int first_key = length;
+        if (windows[(size_t)g] > 0) first_key = std::min(first_key, length - windows[(size_t)g] + 1);
+        for (int c : chunks[(size_t)g]) first_key = std::min(first_key, length - length % c);
         return first_key > 0 ? first_key / page_size : 0;
     }
 };

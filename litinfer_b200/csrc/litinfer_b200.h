@@ -38,22 +38,26 @@ int li_table_gather(int* resident, int rows, int cols, const int* updates, int u
  * two unused words, then per entry: sequence, tile of 128 tokens, part | parts << 8, unused), with the number of entries
  * to launch when the single tokens go to the decode kernel and when they do not.  softcap > 0: scores become
  * softcap * tanh(score / softcap); slopes [nh] (may be NULL): slopes[h] * (p - key) is taken off the score of head h;
- * gate [T, nh] in the run dtype (may be NULL): head h's output is multiplied by 1 / (1 + exp(-gate[t, h])).
+ * gate in the run dtype (may be NULL), rows of gate_ld: head h's output is multiplied by the sigmoid of gate[t, h], or with
+ * gate_elements each output element by that of gate[t, h dh + d].  chunk > 0: position p sees the keys from p - p % chunk on.
+ * q_ld > 0: the queries are the first nh dh columns of rows of q_ld elements instead of q|k|v rows.
  * keep_first > 0 (with a window): keys 0 .. keep_first - 1 stay visible behind the window; sinks [nh] (may be NULL):
  * exp(sinks[h]) joins the softmax's denominator of head h once, with no key and no value. */
 int li_paged_attention(const void* qkv, void* out, const void* kcache, const void* vcache, int dtype, const int*
-    block_table, int max_blocks, const int* q_start, const int* ctx_lens, const int* seq_of_token, const int*
-    positions, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages, float scale, int window, int
-    max_q_len, int max_ctx_len, const int* old_lens, int singles, const int* units, int slots_portions, int slots_all,
-    float softcap, const float* slopes, const void* gate, int keep_first, const float* sinks, int maps, cudaStream_t stream);
+    block_table, int max_blocks, const int* q_start, const int* ctx_lens, const int* seq_of_token, const int* positions,
+    int T, int S, int nh, int nkv, int dh, int page_size, int num_pages, float scale, int window, int max_q_len, int
+    max_ctx_len, const int* old_lens, int singles, const int* units, int slots_portions, int slots_all, float softcap,
+    const float* slopes, const void* gate, long long gate_ld, int gate_elements, int keep_first, const float* sinks, int
+    maps, int chunk, int q_ld, cudaStream_t stream);
 
 /* The same through one implementation: 0 general, 1 decode, 2 mma.sync tiles, 3 tcgen05 tiles (tests and
  * measurements). */
 int li_paged_attention_with(int which, const void* qkv, void* out, const void* kcache, const void* vcache, int dtype,
-    const int* block_table, int max_blocks, const int* q_start, const int* ctx_lens, const int* seq_of_token, const
-    int* positions, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages, float scale, int window, int
+    const int* block_table, int max_blocks, const int* q_start, const int* ctx_lens, const int* seq_of_token, const int*
+    positions, int T, int S, int nh, int nkv, int dh, int page_size, int num_pages, float scale, int window, int
     max_q_len, int max_ctx_len, const int* old_lens, int singles, const int* units, int slots_portions, int slots_all,
-    float softcap, const float* slopes, const void* gate, int keep_first, const float* sinks, int maps, cudaStream_t stream);
+    float softcap, const float* slopes, const void* gate, long long gate_ld, int gate_elements, int keep_first, const
+    float* sinks, int maps, int chunk, int q_ld, cudaStream_t stream);
 
 /* ---- decode_step.cu: a decode step as one persistent kernel (decode_step.h has the structures) ---- */
 struct LiDecodeStep;
@@ -111,6 +115,11 @@ int li_glu_clamped(const void* gate_up, void* out, int dtype, int T, int I, floa
 
 /* out[t, i] = up * gelu(gate), the tanh form of gelu; gate_up [T, 2 I] as gate | up. */
 int li_geglu(const void* gate_up, void* out, int dtype, int T, int I, cudaStream_t stream);
+
+/* out[t, i] = gelu(z[t, i]) * table[ids[t], col + i]: a gate (tanh form of gelu, z [T, n] float) that opens a token's row of a
+ * table [rows, ld] in the run dtype. */
+int li_gelu_token_rows(const float* z, const void* table, int dtype, long long ld, int col, int rows, const int* ids, void* out, int T, int n,
+    cudaStream_t stream);
 
 /* out = a N(z) + b N(z^2) + c N(z^3) + e per row of z [T, n], powers element by element, N(v) = v / sqrt(mean(v^2) + eps),
  * coef = {a, b, c, e} float on the device. */
@@ -183,15 +192,18 @@ int li_gla_scan(const void* qkv, int dtype, int stride, int q_off, int k_off, in
  * q and k as unit vectors (x / sqrt(sum x^2 + unit_eps), q times q_scale) and k . q into prep_qk [T, kv_heads, 2 DP + 4];
  * g = exp(-exp(A_log[h]) softplus(za [T, za_stride] at za_off + h d + i)) and beta = sigmoid(proj[b_off + h]) into prep_g
  * [T, heads, DP + 4]; v [T, heads dv]; all float, DP = 32, 64, 128 or 256 (the first that holds d).  shift: every sequence has
- * one token and the convolution's state moves on here.  li_delta_scan walks; head h uses key head h / (heads / kv_heads); the
+ * one token and the convolution's state moves on here.  za NULL: one decay a head, g = exp(-exp(A_log[h]) softplus(proj[a_off + h] +
+ * dt_bias[h])), prep_g [T, heads, 4] = (g | beta | unused), and per_head for the walk.  li_delta_scan walks; head h uses key head h / (heads / kv_heads); the
  * state is kept as [heads][dv][d]. */
-int li_delta_prepare(const void* proj, int dtype, int stride, int col0, int b_off, const float* conv_w, int taps, float* state,
-    long long state_stride, long long state_off, const int* q_start, const int* seq_of_token, const int* slots,
-    const float* za, int za_stride, int za_off, const float* A_log, float q_scale, float unit_eps, float* prep_qk,
-    float* prep_g, float* v, int T, int heads, int kv_heads, int d, int dv, int shift, cudaStream_t stream);
+int li_delta_prepare(const void* proj, int dtype, int stride, int col0, int b_off, const float* conv_w, int taps,
+    float* state, long long state_stride, long long state_off, const int* q_start, const int* seq_of_token, const int*
+    slots, const float* za, int za_stride, int za_off, int a_off, const float* dt_bias, const float* A_log, float q_scale,
+    float unit_eps, float* prep_qk, float* prep_g, float* v, int T, int heads, int kv_heads, int d, int dv, int shift,
+    cudaStream_t stream);
 void li_delta_force_columns(int columns);   /* 0: columns a warp of the walk by the launch's size; 2, 4 or 8, for tests and measurements */
-int li_delta_scan(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* q_start,
-    const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, cudaStream_t stream);
+int li_delta_scan(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride,
+    const int* q_start, const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, int per_head,
+    cudaStream_t stream);
 
 /* Per channel c a state S [N]: S = exp(dt_c A[c, :]) S + dt_c x_c B, y_c = (S . C + D[c] x_c) silu(z_c), with
  * dt = softplus(dt_raw) (float, [T, dt_stride]), A = -exp(A_log) [inner, N]; x at column x_off of [T, x_stride], B and C
@@ -273,10 +285,12 @@ int li_linear_rope_kv(const void* a, const void* w, const float* bias, void* qkv
  * out = next(x) if w_next is given (without it, out, if given, takes x as it is in the run dtype).  A norm is centered (mean taken off, variance as the mean of squared deviations:
  * layer norm without bias) or not (RMS norm).  rows (may be NULL; only without y): out[r] = next(x[rows[r]]).
  * y_places (may be NULL): token r's y is the sum over j < y_top of y[y_places[r y_top + j]] (times y_weights[...] if given), plus
- * y_extra[r] if that is given. */
-int li_norm_add_norm(float* x, const void* y, int dtype, const float* w_post, int post_centered, float eps_post, const float* w_next,
-    int next_centered, float eps_next, void* out, const int* rows, int R, int n_src, int H, const int* y_places,
-    int y_top, const float* y_weights, const void* y_extra, cudaStream_t stream);
+ * y_extra[r] if that is given.  y2 (may be NULL): the sublayer's output is s1 y + s2 y2, each first divided by its root mean square
+ * (eps_pair) and multiplied by w_first / w_second if those are given. */
+int li_norm_add_norm(float* x, const void* y, int dtype, const float* w_post, int post_centered, float eps_post, const
+    float* w_next, int next_centered, float eps_next, void* out, const int* rows, int R, int n_src, int H, const int*
+    y_places, int y_top, const float* y_weights, const void* y_extra, const void* y2, float s1, float s2, const float*
+    w_first, const float* w_second, float eps_pair, cudaStream_t stream);
 
 /* out [T, 2 H] in the run dtype: x [T, H] (plus delta [T, H] if given) beside x0 [T, H], both float.  places (may be NULL): delta
  * is a sum of rows as in li_norm_add_norm. */
@@ -320,8 +334,8 @@ int li_row_rinv(const void* x, int dtype, int ld, int col0, int n0, int width0, 
     int T, cudaStream_t stream);
 
 /* Rotation of the first rotary_dim elements of the query and key heads of proj [T, ld] (pair i by float(pos) / denom[i];
- * interleaved: pair (2i, 2i + 1), else (i, i + rotary_dim / 2); cosine and sine times magnitude), then (norm != 0) each head
- * divided by sqrt(sum x^2 / norm_width + eps), times q_norm / k_norm [dh] if given; queries to out [T, (nh + 2 nkv) dh], keys
+ * interleaved: pair (2i, 2i + 1), else (i, i + rotary_dim / 2); cosine and sine times magnitude), each head behind (norm 1) or
+ * before it (norm 2) divided by sqrt(sum x^2 / norm_width + eps), times q_norm / k_norm [dh] if given; queries to out [T, (nh + 2 nkv) dh], keys
  * and values into the paged cache, or with to_cache 0 to their columns of out.  keys_are_values: proj holds q | k only, and
  * a key head as projected, before rotation and norm, is the value. */
 int li_rope_norm_kv(const void* proj, int ld, void* out, int dtype, const int* positions, const float* denom, float magnitude, int interleaved,
@@ -356,9 +370,10 @@ int li_moe_route(const float* logits, int scoring, int T, int E, int top, int* i
 /* The same choice for a router over all experts at once with groups: s = softmax(logits [T, E]); choice scores s + correction
  * (may be NULL); the experts form `groups` equal groups of neighbours, a group's score is its largest choice score, only the
  * `keep` best groups' experts can be chosen; the `top` largest choice scores choose; weights = s of the chosen / (their sum +
- * 1e-20) * scale. */
-int li_moe_route_grouped(const float* logits, const float* correction, int T, int E, int top, int groups, int keep, float scale, int* ids,
-    float* weights, cudaStream_t stream);
+ * 1e-20) * scale (scoring 2).  scoring 3: s = sigmoid(logits), a group's score is the sum of its two largest choice scores,
+ * weights = s of the chosen * scale. */
+int li_moe_route_grouped(const float* logits, const float* correction, int scoring, int T, int E, int top, int groups,
+    int keep, float scale, int* ids, float* weights, cudaStream_t stream);
 
 /* Stable sort of n (token, choice) pairs by expert: offsets [E + 1], pair_at (pair at a sorted place, -1: none), place_of [n].
  * Every expert's run starts at a multiple of pad; pair_at has `places` entries; tile_group (may be NULL) [n_tiles]: the expert of
@@ -374,7 +389,7 @@ int li_moe_combine(const void* rows, int dtype, const int* place_of, const float
     void* y, cudaStream_t stream);
 
 /* The front of a mixture for a step of few tokens as one launch: logits h [T, H] w [E, H]^T (+ bias), the choice (scoring 0, 1 as in
- * li_moe_route, 2 as in li_moe_route_grouped), the stable sort without padding.  accepts: 1 if the sizes fit. */
+ * li_moe_route, 2, 3 as in li_moe_route_grouped), the stable sort without padding.  accepts: 1 if the sizes fit. */
 int li_moe_small_step_accepts(int dtype, int T, int H, int E, int top);
 int li_moe_small_step(const void* h, const void* w, const float* bias, int dtype, int T, int H, int E, int top, int scoring,
     const float* correction, int groups, int keep, float scale, float* weights, int* offsets, int* pair_at,

@@ -211,8 +211,9 @@ __global__ void norm_add_norm_regs_kernel(float* __restrict__ x, const T* __rest
                                           float eps_post, const float* __restrict__ w_next, int next_centered, float eps_next,
                                           T* __restrict__ out, const int* __restrict__ rows, int n_src, int H,
                                           const int* __restrict__ y_places, int y_top, const float* __restrict__ y_weights,
-                                          const T* __restrict__ y_extra) {
-    __shared__ float scratch[32];
+                                          const T* __restrict__ y_extra, const T* __restrict__ y2, float s1, float s2,
+                                          const float* __restrict__ w_first, const float* __restrict__ w_second, float eps_pair) {
+    __shared__ float scratch[64];
     pdl_launch_dependents();
     pdl_wait();
     const int r = blockIdx.x;
@@ -247,6 +248,26 @@ __global__ void norm_add_norm_regs_kernel(float* __restrict__ x, const T* __rest
             }
         } else {
             load_row<kVec>(yv, y + (size_t)r * H, H);
+        }
+        if (y2) {
+            // two outputs side by side (two mixers): their weighted sum, each divided by its root mean square first if it has a weight
+            float other[kRegs];
+            load_row<kVec>(other, y2 + (size_t)r * H, H);
+            if (w_first) {
+                float qa = 0.0f, qb = 0.0f, wa[kRegs], wb[kRegs];
+#pragma unroll
+                for (int k = 0; k < kRegs; ++k) qa = fmaf(yv[k], yv[k], qa), qb = fmaf(other[k], other[k], qb);
+                load_row<kVec>(wa, w_first, H);
+                load_row<kVec>(wb, w_second, H);
+                block_sum2(qa, qb, scratch);
+                const float inv_h = 1.0f / (float)H;
+                const float fa = s1 / sqrtf(qa * inv_h + eps_pair), fb = s2 / sqrtf(qb * inv_h + eps_pair);
+#pragma unroll
+                for (int k = 0; k < kRegs; ++k) yv[k] = fmaf(yv[k] * fa, wa[k], other[k] * fb * wb[k]);
+            } else {
+#pragma unroll
+                for (int k = 0; k < kRegs; ++k) yv[k] = fmaf(s1, yv[k], s2 * other[k]);
+            }
         }
         if (w_post) {
             float nv[kRegs];
@@ -354,10 +375,15 @@ __global__ void rmsnorm_cols_kernel(const T* __restrict__ in, int ld_in, int col
 // be NULL; only without y): out[r] = next(x[rows[r]]).  x is [n_src, H] float and is changed in place when y is given.
 // y_places (may be NULL; H up to 8,192): token r's y is the sum over j < y_top of y[y_places[r y_top + j]] (times
 // y_weights[r y_top + j] if given), summed in float in that order: the combine of a mixture of experts, not written out.
+// y2 (may be NULL; H up to 8,192): a second output; the sublayer's output is then s1 y + s2 y2, each divided by its root mean
+// square (eps_pair) and multiplied by w_first / w_second first if those are given.
 // y_extra (may be NULL; with y_places): one more row per token that joins the sum, y_extra [R, H] (a shared expert's output).
 LI_EXPORT int li_norm_add_norm(float* x, const void* y, int dtype, const float* w_post, int post_centered, float eps_post, const float* w_next,
                                int next_centered, float eps_next, void* out, const int* rows, int R, int n_src, int H, const int* y_places,
-                               int y_top, const float* y_weights, const void* y_extra, cudaStream_t stream) {
+                               int y_top, const float* y_weights, const void* y_extra, const void* y2, float s1, float s2, const float* w_first,
+                               const float* w_second, float eps_pair, cudaStream_t stream) {
+    LI_REQUIRE(y2 == nullptr || (y != nullptr && y_places == nullptr && H <= 8 * 1024), "norm_add_norm: a pair of outputs needs both and at most 8192 columns");
+    LI_REQUIRE((w_first == nullptr) == (w_second == nullptr), "norm_add_norm: the outputs of a pair are normalised together or not at all");
     LI_REQUIRE(y_extra == nullptr || y_places != nullptr, "norm_add_norm: a further row goes with a sum of rows");
     LI_REQUIRE(y_places == nullptr || (y != nullptr && y_top > 0 && H <= 8 * 1024), "norm_add_norm: a sum of rows needs the rows, a count and at most 8192 columns");
     LI_REQUIRE(R >= 0 && H > 0 && n_src >= 0, "norm_add_norm: bad sizes R=%d H=%d", R, H);
@@ -371,11 +397,12 @@ LI_EXPORT int li_norm_add_norm(float* x, const void* y, int dtype, const float* 
         int threads = ((ceil_div(H, kRegs) + 31) / 32) * 32;
         if (threads < 64) threads = 64;
         // 16-byte moves where every row starts on such a boundary
-        const bool vec = H % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)y_extra % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
-                         ((uintptr_t)w_post % 16) == 0 && ((uintptr_t)w_next % 16) == 0;
+        const bool vec = H % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)y_extra % 16) == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)y2 % 16) == 0 && ((uintptr_t)w_first % 16) == 0 &&
+                         ((uintptr_t)w_second % 16) == 0 && ((uintptr_t)w_post % 16) == 0 && ((uintptr_t)w_next % 16) == 0;
 #define LI_NORM_LAUNCH(TT, VEC)                                                                                                                  \
     e = li_launch_pdl(norm_add_norm_regs_kernel<TT, VEC>, dim3(R), dim3(threads), 0, stream, x, (const TT*)y, w_post, post_centered, eps_post, w_next, \
-                      next_centered, eps_next, (TT*)out, rows, n_src, H, y_places, y_top, y_weights, (const TT*)y_extra)
+                      next_centered, eps_next, (TT*)out, rows, n_src, H, y_places, y_top, y_weights, (const TT*)y_extra, (const TT*)y2, s1, s2, w_first, \
+                      w_second, eps_pair)
         if (dtype == LI_F32) {
             if (vec) LI_NORM_LAUNCH(float, true);
             else LI_NORM_LAUNCH(float, false);

@@ -396,18 +396,20 @@ LI_EXPORT int li_latent_rope_post(const void* low, int dtype, int ld_low, int co
     return li_check_launch("latent_rope_post");
 }
 
-// Rotation first, norm behind it, and the projected keys as values: what stands between a q|k (or q|k|v) product and attention
-// in a layer whose queries and keys are rotated and then divided by their root mean square, head by head.
+// Rotation (pairs of neighbours or halves, with a magnitude), a norm per head behind or before it, and, if asked for, the
+// projected keys as values: what stands between a q|k|v (or q|k) product and attention.
 //   * `keys_are_values`: the row holds no values; a key head's projection, before rotation and norm, is also its value;
 //   * rotation of the first rotary_dim elements: pair i turns by float(pos) / denom[i]; `interleaved`: the pair is
 //     (2i, 2i + 1), else (i, i + rotary_dim / 2); cosine and sine are multiplied by `magnitude`;
-//   * norm != 0: x / sqrt(sum x^2 / norm_width + eps) per query and key head, times a weight of head size if given;
+//   * norm: x / sqrt(sum x^2 / norm_width + eps) per query and key head, times a weight of head size if given; 1 behind the
+//     rotation, 2 before it;
 //   * queries to `out` [T, (nh + 2 nkv) dh], keys and values into the paged cache (values transposed), or with to_cache 0 to
 //     their columns of `out`.
 // A block takes one token and some of its heads, a warp a head at a time; a lane holds V neighbouring elements of every 32 V,
 // so that the pairs of neighbours never leave a lane.  All arithmetic in float from run-dtype inputs, one rounding.
 namespace {
 constexpr int kRopeNormWarps = 8;
+enum { kNoNorm = 0, kNormBehind = 1, kNormBefore = 2 };          // where the norm of a head stands to the rotation
 
 template <typename T, int V>
 __device__ __forceinline__ void load_elements(float (&v)[V], const T* __restrict__ p, int left) {
@@ -509,6 +511,25 @@ rope_norm_kv_kernel(const T* __restrict__ proj, int ld, T* __restrict__ out, con
             }
             if (is_v) continue;
         }
+        // the head divided by its root mean square, times the weight if there is one
+        auto normalise = [&]() {
+            float q = 0.0f;
+#pragma unroll
+            for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                for (int k = 0; k < V; ++k) q = fmaf(v[i][k], v[i][k], q);
+            q = warp_sum(q);
+            const float rinv = 1.0f / sqrtf(q / (float)norm_width + eps);
+            const float* w = is_q ? q_norm : k_norm;
+#pragma unroll
+            for (int i = 0; i < STEPS; ++i)
+#pragma unroll
+                for (int k = 0; k < V; ++k) {
+                    const int d = V * (lane + 32 * i) + k;
+                    v[i][k] *= (w && d < dh) ? rinv * w[d] : rinv;
+                }
+        };
+        if (norm == kNormBefore) normalise();
         if (rotary_dim > 0) {
             if (interleaved) {
 #pragma unroll
@@ -545,23 +566,7 @@ rope_norm_kv_kernel(const T* __restrict__ proj, int ld, T* __restrict__ out, con
                     }
             }
         }
-        if (norm) {
-            float q = 0.0f;
-#pragma unroll
-            for (int i = 0; i < STEPS; ++i)
-#pragma unroll
-                for (int k = 0; k < V; ++k) q = fmaf(v[i][k], v[i][k], q);
-            q = warp_sum(q);
-            const float rinv = 1.0f / sqrtf(q / (float)norm_width + eps);
-            const float* w = is_q ? q_norm : k_norm;
-#pragma unroll
-            for (int i = 0; i < STEPS; ++i)
-#pragma unroll
-                for (int k = 0; k < V; ++k) {
-                    const int d = V * (lane + 32 * i) + k;
-                    v[i][k] *= (w && d < dh) ? rinv * w[d] : rinv;
-                }
-        }
+        if (norm == kNormBehind) normalise();
         T* dst;
         if (is_q || !to_cache) dst = orow + (size_t)head * dh;
         else if (slot_ok) dst = kcache + (((size_t)page * nkv + kvh) * page_size + off) * dh;
@@ -636,6 +641,7 @@ LI_EXPORT int li_rope_norm_kv(const void* proj, int ld, void* out, int dtype, co
     LI_REQUIRE(dh <= 512, "rope_norm_kv: head_dim %d is larger than 512", dh);
     LI_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= dh, "rope_norm_kv: rotary_dim %d must be even and at most head_dim %d", rotary_dim, dh);
     LI_REQUIRE(rotary_dim == 0 || denom != nullptr, "rope_norm_kv: rotary_dim %d without denominators", rotary_dim);
+    LI_REQUIRE(norm >= kNoNorm && norm <= kNormBefore, "rope_norm_kv: unknown place %d of the norm", norm);
     LI_REQUIRE(!norm || (norm_width > 0 && norm_width <= dh), "rope_norm_kv: bad norm width %d", norm_width);
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "rope_norm_kv: unknown dtype %d", dtype);
     LI_REQUIRE(proj != out, "rope_norm_kv: the output needs rows of its own");

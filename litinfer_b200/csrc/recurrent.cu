@@ -16,7 +16,7 @@
 //   * li_gla_scan: per head a state S [d, dv] with a decay per token and key channel:  S = diag(a_t) S + k v^T,
 //     o = S^T (q / sqrt(d)),  a_t = sigmoid(z_t)^(1 / tau) from float logits z.
 //   * li_delta_prepare / li_delta_scan: per head a state S [d, dv] under the gated delta rule with a decay per token and key
-//     channel:  S = diag(g) S,  u = beta (v - S^T k),  S = S + k u^T,  o = S^T q; the first kernel makes what does not depend on
+//     channel (or one number a token for the whole head):  S = diag(g) S,  u = beta (v - S^T k),  S = S + k u^T,  o = S^T q; the first kernel makes what does not depend on
 //     the state (convolution, unit vectors q and k, decays, beta), the second walks.
 //   * li_channel_scan: a state S [N] per channel c with a decay per token, channel and element:
 //     S = exp(dt_c A[c, :]) S + dt_c x_c B,  y_c = (S . C + D_c x_c) silu(z_c),  dt = softplus(dt_raw), A = -exp(A_log).
@@ -508,18 +508,20 @@ gla_scan_kernel(const T* __restrict__ qkv, int stride, int q_off, int k_off, int
 // scan stages them as they are: prep_qk [T, kv_heads, 2 DP + 4] (q | k | k . q), prep_g [T, heads, DP + 4] (g | beta),
 // v [T, heads dv].  Every channel of the convolution belongs to one warp, which also moves the channel's state on in a step of
 // single tokens (`shift`).
+// Without za the head has one decay a token, g = exp(-exp(A_log[h]) softplus(a + dt_bias[h])) with a the projections' column
+// a_off + h; prep_g is then [T, heads, 4] (g | beta | unused), written by the warps of the values.
 // TAPS: the taps at compile time (their loads are then all in flight at once), or 0: any number, at run time.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 delta_prepare_kernel(const T* __restrict__ proj, int stride, int col0, int b_off, const float* __restrict__ conv_w, int taps_rt,
                      float* __restrict__ state, long long state_stride, long long state_off, const int* __restrict__ q_start,
                      const int* __restrict__ seq_of_token, const int* __restrict__ slots, const float* __restrict__ za, int za_stride, int za_off,
-                     const float* __restrict__ A_log, float q_scale, float unit_eps, float* __restrict__ prep_qk, float* __restrict__ prep_g,
-                     float* __restrict__ v_out, int total, int heads, int kv_heads, int d, int dv, int DP, int shift) {
+                     int a_off, const float* __restrict__ dt_bias, const float* __restrict__ A_log, float q_scale, float unit_eps, float* __restrict__ prep_qk,
+                     float* __restrict__ prep_g, float* __restrict__ v_out, int total, int heads, int kv_heads, int d, int dv, int DP, int shift) {
     pdl_launch_dependents();
     pdl_wait();
     const int taps = TAPS > 0 ? TAPS : taps_rt;
-    const int units = kv_heads + 2 * heads;
+    const int units = kv_heads + (za ? 2 : 1) * heads;
     const long long id = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (id >= (long long)total * units) return;
     const int t = (int)(id / units), u = (int)(id - (long long)t * units);
@@ -564,7 +566,7 @@ delta_prepare_kernel(const T* __restrict__ proj, int stride, int col0, int b_off
             }
         }
         if (lane == 0) row[2 * DP] = qk * fq * fk;
-    } else if (u < kv_heads + heads) {
+    } else if (za && u < kv_heads + heads) {
         const int h = u - kv_heads;
         const float rate = -expf(A_log[h]);
         const float* zrow = za + (size_t)t * za_stride + za_off + h * d;
@@ -572,7 +574,12 @@ delta_prepare_kernel(const T* __restrict__ proj, int stride, int col0, int b_off
         for (int i = lane; i < DP; i += 32) row[i] = i < d ? expf(rate * softplus_f(zrow[i])) : 0.0f;
         if (lane == 0) row[DP] = sigmoid_f(to_float(proj[(size_t)t * stride + b_off + h]));
     } else {
-        const int h = u - kv_heads - heads;
+        const int h = u - kv_heads - (za ? heads : 0);
+        if (!za && lane == 0) {
+            const T* row = proj + (size_t)t * stride;
+            float2* to = reinterpret_cast<float2*>(prep_g + ((size_t)t * heads + h) * 4);
+            *to = make_float2(expf(-expf(A_log[h]) * softplus_f(to_float(row[a_off + h]) + dt_bias[h])), sigmoid_f(to_float(row[b_off + h])));
+        }
         for (int j = lane; j < dv; j += 32) v_out[(size_t)t * heads * dv + h * dv + j] = conv(2 * kv_heads * d + h * dv + j);
     }
 }
@@ -592,7 +599,9 @@ __device__ __forceinline__ void stage16(float* dst, const float* src, bool valid
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(bytes));
 }
 
-template <int E, int WC>
+// kHead: one decay a token for the whole head, staged with beta (prep_g [T, heads, 4]); the sums are then taken of the state as it
+// was and multiplied by the decay.
+template <int E, int WC, bool kHead>
 __global__ void __launch_bounds__(128)
 delta_scan_kernel(const float* __restrict__ prep_qk, const float* __restrict__ prep_g, const float* __restrict__ vin, float* __restrict__ state,
                   long long state_stride, const int* __restrict__ q_start, const int* __restrict__ slots, float* __restrict__ out, int heads,
@@ -603,7 +612,8 @@ delta_scan_kernel(const float* __restrict__ prep_qk, const float* __restrict__ p
     // stage is walked.  A buffer: q [kStage][DP] | k [kStage][DP] | decays [kStage][DP] | v [kStage][cols] | (beta ...) [kStage][4]
     // | (k . q ...) [kStage][4]
     extern __shared__ __align__(16) float smem[];
-    const int buf_floats = 3 * kStage * DP + kStage * cols + 8 * kStage;
+    constexpr int kRows = kHead ? 2 : 3;
+    const int buf_floats = kRows * kStage * DP + kStage * cols + 8 * kStage;
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.y;
@@ -614,13 +624,13 @@ delta_scan_kernel(const float* __restrict__ prep_qk, const float* __restrict__ p
     const int block_col0 = blockIdx.x * cols;
     const int col0 = block_col0 + warp * WC;
     float* st = state + (size_t)slots[blockIdx.z] * state_stride + (size_t)h * dv * d;
-    constexpr int RQ = 2 * DP + 4, RG = DP + 4;
+    constexpr int RQ = 2 * DP + 4, RG = kHead ? 4 : DP + 4;
     const bool v16 = (dv & 3) == 0 && (cols & 3) == 0 && (((uintptr_t)vin) & 15) == 0;          // the values' rows in pieces of 16 bytes
     auto stage = [&](int b, int t0) {
         float* qs = smem + (size_t)b * buf_floats;
         float* ks = qs + kStage * DP;
         float* as = ks + kStage * DP;
-        float* vs = as + kStage * DP;
+        float* vs = qs + kRows * kStage * DP;
         float* sb = vs + kStage * cols;
         float* sq = sb + 4 * kStage;
         const int nt = min(kStage, q1 - t0);
@@ -630,10 +640,10 @@ delta_scan_kernel(const float* __restrict__ prep_qk, const float* __restrict__ p
             const float* rg = prep_g + ((size_t)(t0 + tk) * heads + h) * RG;
             stage16(qs + tk * DP + 4 * i, rq + 4 * i, true);
             stage16(ks + tk * DP + 4 * i, rq + DP + 4 * i, true);
-            stage16(as + tk * DP + 4 * i, rg + 4 * i, true);
+            if (!kHead) stage16(as + tk * DP + 4 * i, rg + 4 * i, true);
         }
         for (int tk = threadIdx.x; tk < nt; tk += blockDim.x) {
-            stage16(sb + 4 * tk, prep_g + ((size_t)(t0 + tk) * heads + h) * RG + DP, true);
+            stage16(sb + 4 * tk, prep_g + ((size_t)(t0 + tk) * heads + h) * RG + (kHead ? 0 : DP), true);
             stage16(sq + 4 * tk, prep_qk + ((size_t)(t0 + tk) * kv_heads + hk) * RQ + 2 * DP, true);
         }
         if (v16) {
@@ -666,28 +676,28 @@ delta_scan_kernel(const float* __restrict__ prep_qk, const float* __restrict__ p
         const float* qs = smem + (size_t)b * buf_floats;
         const float* ks = qs + kStage * DP;
         const float* as = ks + kStage * DP;
-        const float* vs = as + kStage * DP;
+        const float* vs = qs + kRows * kStage * DP;
         const float* sb = vs + kStage * cols;
         const float* sq = sb + 4 * kStage;
 #pragma unroll 2
         for (int tk = 0; tk < nt; ++tk) {
             float kk[E], aa[E], qq[E], v[WC], acck[WC], accq[WC];
             load_elements<E>(kk, ks + tk * DP + E * lane);
-            load_elements<E>(aa, as + tk * DP + E * lane);
+            if (!kHead) load_elements<E>(aa, as + tk * DP + E * lane);
             load_elements<E>(qq, qs + tk * DP + E * lane);
             load_elements<WC>(v, vs + tk * cols + warp * WC);
-            const float beta = sb[4 * tk], kq = sq[4 * tk];
+            const float decay = kHead ? sb[4 * tk] : 1.0f, beta = sb[4 * tk + (kHead ? 1 : 0)], kq = sq[4 * tk];
 #pragma unroll
             for (int j = 0; j < WC; ++j) {
                 acck[j] = accq[j] = 0.0f;
 #pragma unroll
                 for (int e = 0; e < E; ++e) {
-                    S[j][e] *= aa[e];
+                    if (!kHead) S[j][e] *= aa[e];
                     acck[j] = fmaf(S[j][e], kk[e], acck[j]);
                     accq[j] = fmaf(S[j][e], qq[e], accq[j]);
                 }
             }
-            const float sk = sum_across_warp<WC>(acck, lane), sqv = sum_across_warp<WC>(accq, lane);
+            const float sk = decay * sum_across_warp<WC>(acck, lane), sqv = decay * sum_across_warp<WC>(accq, lane);
             const int jm = column_after_sum<WC>(lane);                   // the column whose sums this lane holds now
             float vm = v[0];
 #pragma unroll
@@ -698,7 +708,7 @@ delta_scan_kernel(const float* __restrict__ prep_qk, const float* __restrict__ p
             for (int j = 0; j < WC; ++j) {
                 const float u = __shfl_sync(0xffffffffu, um, lane_of_column<WC>(j));
 #pragma unroll
-                for (int e = 0; e < E; ++e) S[j][e] = fmaf(kk[e], u, S[j][e]);
+                for (int e = 0; e < E; ++e) S[j][e] = fmaf(kk[e], u, kHead ? decay * S[j][e] : S[j][e]);
             }
         }
     }
@@ -1238,15 +1248,15 @@ static int delta_elements(int d) { return d <= 32 ? 1 : d <= 64 ? 2 : d <= 128 ?
 constexpr int kDeltaWarps = 4;          // warps of a block of the walk at most
 static int g_delta_cols = 0;            // 0: columns a warp by the size of the launch; 2, 4 or 8: that many, for tests and measurements
 
-template <int E, int WC>
+template <int E, int WC, bool kHead>
 static int launch_delta(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* q_start,
                         const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
     int warps = ceil_div(dv, WC);
     warps = warps >= kDeltaWarps ? kDeltaWarps : warps >= 2 ? 2 : 1;
     const int cols = warps * WC;
-    const size_t smem = 2 * ((size_t)3 * kStage * 32 * E + kStage * cols + 8 * kStage) * sizeof(float);          // two buffers
-    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<E, WC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaError_t e = li_launch_pdl(delta_scan_kernel<E, WC>, dim3(ceil_div(dv, cols), heads, S), dim3(warps * 32), smem, stream, prep_qk, prep_g, v, state,
+    const size_t smem = 2 * ((size_t)(kHead ? 2 : 3) * kStage * 32 * E + kStage * cols + 8 * kStage) * sizeof(float);          // two buffers
+    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<E, WC, kHead>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = li_launch_pdl(delta_scan_kernel<E, WC, kHead>, dim3(ceil_div(dv, cols), heads, S), dim3(warps * 32), smem, stream, prep_qk, prep_g, v, state,
                                   state_stride, q_start, slots, out, heads, kv_heads, d, dv);
     if (e != cudaSuccess) return li_fail("delta_scan: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("delta_scan");
@@ -1261,13 +1271,13 @@ static int delta_cols(int S, int heads, int dv) {
     return columns / 8 >= 1184 ? 8 : 4;
 }
 
-template <int E>
+template <int E, bool kHead>
 static int launch_delta_cols(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* q_start,
                              const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
     switch (delta_cols(S, heads, dv)) {
-        case 8: return launch_delta<E, 8>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
-        case 4: return launch_delta<E, 4>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
-        default: return launch_delta<E, 2>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
+        case 8: return launch_delta<E, 8, kHead>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
+        case 4: return launch_delta<E, 4, kHead>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
+        default: return launch_delta<E, 2, kHead>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
     }
 }
 
@@ -1275,26 +1285,27 @@ static int launch_delta_cols(const float* prep_qk, const float* prep_g, const fl
 // holds the convolution's channels q | k | v (kv_heads d, kv_heads d, heads dv) from column col0 and beta's input at b_off + h;
 // conv_w [channels, taps]; the state holds the last taps - 1 inputs at state_off ([taps - 1, channels], oldest first);
 // za [T, za_stride] float: the decays' input at za_off + h d + i.  Outputs: prep_qk [T, kv_heads, 2 DP + 4], prep_g
-// [T, heads, DP + 4], v [T, heads dv], float, with DP = 32, 64, 128 or 256 (the first that holds d).
+// [T, heads, DP + 4] ([T, heads, 4] without za: one decay a head, from column a_off + h and dt_bias), v [T, heads dv], float, with DP = 32, 64, 128 or 256 (the first that holds d).
 LI_EXPORT int li_delta_prepare(const void* proj, int dtype, int stride, int col0, int b_off, const float* conv_w, int taps, float* state,
                                long long state_stride, long long state_off, const int* q_start, const int* seq_of_token, const int* slots,
-                               const float* za, int za_stride, int za_off, const float* A_log, float q_scale, float unit_eps, float* prep_qk,
-                               float* prep_g, float* v, int T, int heads, int kv_heads, int d, int dv, int shift, cudaStream_t stream) {
+                               const float* za, int za_stride, int za_off, int a_off, const float* dt_bias, const float* A_log, float q_scale, float unit_eps,
+                               float* prep_qk, float* prep_g, float* v, int T, int heads, int kv_heads, int d, int dv, int shift, cudaStream_t stream) {
     LI_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && d > 0 && d <= 256 && dv > 0,
                "delta rule: %d heads on %d key heads of %d x %d (keys of at most 256)", heads, kv_heads, d, dv);
     LI_REQUIRE(taps >= 1 && taps <= kMaxTaps && conv_w != nullptr, "delta rule: a convolution of %d taps (at most %d)", taps, kMaxTaps);
-    LI_REQUIRE(za != nullptr && za_off >= 0 && za_off + heads * d <= za_stride, "delta rule: decays at column %d of %d", za_off, za_stride);
+    LI_REQUIRE(za != nullptr || (dt_bias != nullptr && a_off >= 0 && a_off + heads <= stride), "delta rule: no input of the decays");
+    LI_REQUIRE(za == nullptr || (za_off >= 0 && za_off + heads * d <= za_stride), "delta rule: decays at column %d of %d", za_off, za_stride);
     LI_REQUIRE(col0 >= 0 && col0 + 2 * kv_heads * d + heads * dv <= stride && b_off >= 0 && b_off + heads <= stride && A_log != nullptr,
                "delta rule: the projections' columns do not fit rows of %d", stride);
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "delta rule: unknown dtype %d", dtype);
     if (T == 0) return 0;
     const int DP = 32 * delta_elements(d);
-    const long long warps = (long long)T * (kv_heads + 2 * heads);
+    const long long warps = (long long)T * (kv_heads + (za ? 2 : 1) * heads);
     const dim3 grid((unsigned)ceil_div_ll(warps, 4));
     cudaError_t e;
 #define LI_PREPARE(TT, TAPS_)                                                                                                                  \
     e = li_launch_pdl(delta_prepare_kernel<TT, TAPS_>, grid, dim3(128), 0, stream, (const TT*)proj, stride, col0, b_off, conv_w, taps, state,     \
-                      state_stride, state_off, q_start, seq_of_token, slots, za, za_stride, za_off, A_log, q_scale, unit_eps, prep_qk, prep_g, v, T, \
+                      state_stride, state_off, q_start, seq_of_token, slots, za, za_stride, za_off, a_off, dt_bias, A_log, q_scale, unit_eps, prep_qk, prep_g, v, T, \
                       heads, kv_heads, d, dv, DP, shift)
     if (dtype == LI_F32) {
         if (taps == 4) LI_PREPARE(float, 4);
@@ -1315,21 +1326,25 @@ LI_EXPORT int li_delta_prepare(const void* proj, int dtype, int stride, int col0
 // 0: columns a warp of the walk by the size of the launch; 2, 4 or 8: that many.  For tests and measurements.
 LI_EXPORT void li_delta_force_columns(int columns) { g_delta_cols = (columns == 2 || columns == 4 || columns == 8) ? columns : 0; }
 
-// The walk over what li_delta_prepare made.  The state of a slot: [heads][dv][d] (a column of the head's d x dv matrix at a time).
+// The walk over what li_delta_prepare made.  per_head: one decay a token for the whole head (prep_g [T, heads, 4]).  The state of a slot: [heads][dv][d] (a column of the head's d x dv matrix at a time).
 LI_EXPORT int li_delta_scan(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* q_start,
-                            const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
+                            const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, int per_head, cudaStream_t stream) {
     LI_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && d > 0 && d <= 256 && dv > 0,
                "delta rule: %d heads on %d key heads of %d x %d (keys of at most 256)", heads, kv_heads, d, dv);
     LI_REQUIRE(prep_qk != nullptr && prep_g != nullptr && v != nullptr && (uintptr_t)prep_qk % 16 == 0 && (uintptr_t)prep_g % 16 == 0,
                "delta rule: the prepared rows are missing or not on a 16-byte boundary");
     if (S == 0) return 0;
     LI_REQUIRE(S <= 65535 && heads <= 65535, "delta rule: %d sequences or %d heads in one launch", S, heads);
+#define LI_DELTA(E_)                                                                                                                                \
+    return per_head ? launch_delta_cols<E_, true>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream) \
+                    : launch_delta_cols<E_, false>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream)
     switch (delta_elements(d)) {
-        case 1: return launch_delta_cols<1>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
-        case 2: return launch_delta_cols<2>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
-        case 4: return launch_delta_cols<4>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
-        default: return launch_delta_cols<8>(prep_qk, prep_g, v, state, state_stride, q_start, slots, out, S, heads, kv_heads, d, dv, stream);
+        case 1: LI_DELTA(1);
+        case 2: LI_DELTA(2);
+        case 4: LI_DELTA(4);
+        default: LI_DELTA(8);
     }
+#undef LI_DELTA
 }
 
 template <typename T, int E>

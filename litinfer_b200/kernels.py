@@ -456,7 +456,8 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                     old_lens: Optional[torch.Tensor] = None, singles: int = 0,
                     units: Optional[torch.Tensor] = None, unit_slots: Tuple[int, int] = (0, 0),
                     softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                    keep_first: int = 0, sinks: Optional[torch.Tensor] = None, maps: int = 1) -> None:
+                    keep_first: int = 0, sinks: Optional[torch.Tensor] = None, maps: int = 1, chunk: int = 0,
+                    gate_elements: bool = False, gate_col: int = 0) -> None:
     """Causal grouped-query attention of the step's tokens over the paged cache.
 
     Queries are the first ``num_heads * head_dim`` columns of ``qkv`` (already
@@ -472,7 +473,10 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     ``unit_slots`` = how many entries to launch when the single tokens are the decode kernel's, and when not.
     ``softcap`` > 0: a score s becomes ``softcap * tanh(s / softcap)`` (after the scale).  ``slopes`` (float32
     ``[num_heads]``): ``slopes[h] * (p - key)`` is taken off the scores of head h, a penalty linear in the distance.
-    ``gate`` (run dtype ``[T, num_heads]``): head h's output is multiplied by ``sigmoid(gate[t, h])``.
+    ``gate`` (run dtype ``[T, num_heads]``): head h's output is multiplied by ``sigmoid(gate[t, h])``; with ``gate_elements``
+    the gate has a column per output element (``num_heads * head_dim``).  ``gate_col``: its first column in a wider tensor.
+    ``chunk`` > 0: the token at position p sees the keys of its own chunk only, ``p - p % chunk .. p``.
+    ``qkv`` may have rows of another width than q|k|v (queries alone, or beside a gate): its first columns are the queries.
     ``keep_first`` (with a window): the keys ``0 .. keep_first - 1`` stay visible behind the window, at their own positions.
     ``sinks`` (float32 ``[num_heads]``): ``exp(sinks[h])`` joins the denominator of head h's softmax once; it has no key
     and no value and is not scaled.
@@ -484,7 +488,10 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     maps = int(maps)
     if maps < 1 or num_heads % (maps * num_kv_heads) or head_dim % maps:
         raise KernelError(f"{maps} maps of {num_heads} heads on {num_kv_heads} key/value heads of {head_dim} elements")
-    _need(qkv, "qkv", None, (T, (num_heads // maps + 2 * num_kv_heads) * head_dim))
+    _need(qkv, "qkv")
+    q_ld = 0 if qkv.shape[1] == (num_heads // maps + 2 * num_kv_heads) * head_dim else qkv.shape[1]
+    if q_ld and q_ld < num_heads // maps * head_dim:
+        raise KernelError(f"rows of {q_ld} elements cannot hold {num_heads // maps} query heads of {head_dim}")
     _need(out, "attention output", qkv.dtype, (T, num_heads * head_dim))
     _need(k_cache, "key cache", qkv.dtype)
     _need(v_cache, "value cache", qkv.dtype, (k_cache.shape[0], k_cache.shape[1], k_cache.shape[3], k_cache.shape[2]))
@@ -506,18 +513,23 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
         _need(units, "attention work list", torch.int32)
         if units.numel() < 4 + 4 * max(unit_slots) or units.data_ptr() % 16:
             raise KernelError(f"attention work list of {units.numel()} words cannot hold {max(unit_slots)} entries (or is not 16-byte aligned)")
+    gate_ptr, gate_ld = _p(None), 0
+    if gate is not None:
+        gate_ld = gate.shape[1]
+        _need(gate, "gate", qkv.dtype, (T, gate_ld))
+        if gate_col < 0 or gate_col + num_heads * (head_dim if gate_elements else 1) > gate_ld:
+            raise KernelError(f"a gate from column {gate_col} does not fit rows of {gate_ld}")
+        gate_ptr = ctypes.c_void_p(gate.data_ptr() + gate_col * gate.element_size())
     args = (_p(qkv), _p(out), _p(k_cache), _p(v_cache), _i(_dt(qkv)), _p(block_table), _i(block_table.shape[1]),
             _p(q_start), _p(ctx_lens), _p(seq_of_token), _p(positions), _i(T), _i(S),
             _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(page_size), _i(pages), _f(scale),
             _i(0 if window is None else int(window)), _i(max_q_len), _i(max_ctx_len), _p(old_lens), _i(int(singles)),
-            _p(units), _i(int(unit_slots[0])), _i(int(unit_slots[1])), _f(float(softcap or 0.0)), _p(slopes), _p(gate), _i(int(keep_first or 0)), _p(sinks), _i(maps),
-            _stream(out))
+            _p(units), _i(int(unit_slots[0])), _i(int(unit_slots[1])), _f(float(softcap or 0.0)), _p(slopes), gate_ptr, _l(gate_ld), _i(1 if gate_elements else 0),
+            _i(int(keep_first or 0)), _p(sinks), _i(maps), _i(int(chunk or 0)), _i(q_ld), _stream(out))
     if sinks is not None:
         _need(sinks, "softmax sinks", torch.float32, (num_heads,))
     if slopes is not None:
         _need(slopes, "distance slopes", torch.float32, (num_heads,))
-    if gate is not None:
-        _need(gate, "head gate", qkv.dtype, (T, num_heads))
     if implementation is None:
         _check(library().li_paged_attention(*args), "paged_attention")
     else:
@@ -550,6 +562,20 @@ def geglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
     _check(library().li_geglu(_p(gate_up), _p(out), _i(_dt(out)), _i(T), _i(I2 // 2), _stream(out)), "geglu")
 
 
+def gelu_token_rows(z: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[t, i] = gelu(z[t, i]) * table[ids[t], col + i]`` (the tanh form of gelu; ``z`` float32): a gate that opens a token's
+    row of a table."""
+    T, n = z.shape
+    _need(z, "gate", torch.float32)
+    _need(table, "table of token rows")
+    _need(ids, "token ids", torch.int32)
+    _need(out, "opened rows", table.dtype, (T, n))
+    if table.dim() != 2 or col < 0 or col + n > table.shape[1] or ids.shape[0] < T:
+        raise KernelError(f"gelu_token_rows: columns {col} .. {col + n} of a table of shape {tuple(table.shape)} for {T} tokens")
+    _check(library().li_gelu_token_rows(_p(z), _p(table), _i(_dt(table)), _l(table.shape[1]), _i(int(col)), _i(table.shape[0]), _p(ids), _p(out), _i(T),
+                                        _i(n), _stream(out)), "gelu_token_rows")
+
+
 def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor) -> None:
     """``out = a N(z) + b N(z^2) + c N(z^3) + e`` per row of ``z`` [T, n], powers element by element, ``N(v) = v / sqrt(mean(v^2)
     + eps)``; ``coef`` = (a, b, c, e), float32 on the device.  Means and the result in float32, one rounding."""
@@ -574,12 +600,18 @@ def mul_sigmoid(x: torch.Tensor, gate: torch.Tensor, gate_col: int = 0, group: i
 
 class WeightedPair:
     """Two activations that stand for ``sa * a + sb * b`` (two mixers side by side) until a kernel that consumes the sum
-    takes it in (:func:`hc_update`); :meth:`materialize` adds them up with a kernel of its own."""
+    takes it in (:func:`hc_update`, :func:`norm_add_norm`); :meth:`materialize` adds them up with a kernel of its own.
+    ``norms`` (weight of a, weight of b, eps): each is first divided by its root mean square and multiplied by its weight."""
 
-    def __init__(self, a: torch.Tensor, b: torch.Tensor, sa: float, sb: float) -> None:
-        self.a, self.b, self.sa, self.sb = a, b, float(sa), float(sb)
+    def __init__(self, a: torch.Tensor, b: torch.Tensor, sa: float, sb: float, norms: Optional[tuple] = None) -> None:
+        self.a, self.b, self.sa, self.sb, self.norms = a, b, float(sa), float(sb), norms
 
     def materialize(self) -> torch.Tensor:
+        if self.norms is not None:
+            out = torch.empty_like(self.a)
+            x32 = torch.zeros(self.a.shape, dtype=torch.float32, device=self.a.device)
+            norm_add_norm(x32, self, None, (None, False, 0.0), out)          # (the sum onto a stream of zeros, as it is)
+            return out
         out = torch.empty_like(self.a)
         weighted_sum2(self.a, self.b, self.sa, self.sb, out)
         return out
@@ -639,6 +671,8 @@ def hc_update(xs: torch.Tensor, y, mix: torch.Tensor, out_w: torch.Tensor, next_
     ``y`` may be a :class:`WeightedPair` (a, b, sa, sb): the sublayer's output is then sa * a + sb * b, summed in float32."""
     T, s, H = xs.shape
     y2, s1, s2 = None, 1.0, 0.0
+    if isinstance(y, WeightedPair) and y.norms is not None:
+        y = y.materialize()
     if isinstance(y, WeightedPair):
         y, y2, s1, s2 = y.a, y.b, float(y.sa), float(y.sb)
         _need(y2, "sublayer output (second)", y.dtype, (T, H))
@@ -841,9 +875,9 @@ def delta_row_elements(dim: int) -> int:
 
 
 def delta_prepare(proj: torch.Tensor, col: int, b_col: int, conv_w: torch.Tensor, state: torch.Tensor, state_off: int, q_start: torch.Tensor,
-                  seq_of_token: torch.Tensor, slots: torch.Tensor, za: torch.Tensor, za_col: int, A_log: torch.Tensor, prep_qk: torch.Tensor,
+                  seq_of_token: torch.Tensor, slots: torch.Tensor, za: Optional[torch.Tensor], za_col: int, A_log: torch.Tensor, prep_qk: torch.Tensor,
                   prep_g: torch.Tensor, v32: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, unit_eps: float = 1e-6,
-                  shift: bool = False) -> None:
+                  shift: bool = False, a_col: int = 0, dt_bias: Optional[torch.Tensor] = None) -> None:
     """What the gated delta rule needs of every token and does not depend on the state.  ``proj`` [T, *] holds the channels
     q | k | v (``kv_heads * dim``, ``kv_heads * dim``, ``heads * vdim``) from column ``col`` and beta's input at ``b_col + h``.
     Each channel passes a causal convolution (``conv_w`` float32 [channels, taps], the last column the token's own; inputs
@@ -852,7 +886,9 @@ def delta_prepare(proj: torch.Tensor, col: int, b_col: int, conv_w: torch.Tensor
     :func:`delta_row_elements`: ``prep_qk`` [T, kv_heads, 2 DP + 4] = (q | k | k . q), ``prep_g`` [T, heads, DP + 4] = (g | beta)
     with ``g = exp(-exp(A_log[h]) softplus(za[:, za_col + h dim + i]))`` (``za`` float32) and ``beta = sigmoid(.)``, ``v32``
     [T, heads * vdim].  The state is not changed (:func:`conv_state_shift` does that afterwards), unless ``shift``: the caller
-    promises that every sequence of the step has one token."""
+    promises that every sequence of the step has one token.
+    ``za`` None: one decay a head instead of one a key channel, ``g = exp(-exp(A_log[h]) softplus(proj[:, a_col + h] +
+    dt_bias[h]))``, and ``prep_g`` is [T, heads, 4] = (g | beta | unused)."""
     T = proj.shape[0]
     C = 2 * kv_heads * dim + heads * vdim
     DP = delta_row_elements(dim)
@@ -861,20 +897,23 @@ def delta_prepare(proj: torch.Tensor, col: int, b_col: int, conv_w: torch.Tensor
     if conv_w.dim() != 2 or conv_w.shape[0] != C:
         raise KernelError(f"delta_prepare: convolution weight of shape {tuple(conv_w.shape)} for {C} channels")
     taps = conv_w.shape[1]
-    _need(za, "decay inputs", torch.float32)
+    if za is not None:
+        _need(za, "decay inputs", torch.float32)
+    else:
+        _need(dt_bias, "bias of the decays' input", torch.float32, (heads,))
     _need(A_log, "A_log", torch.float32, (heads,))
     _need(prep_qk, "prepared q and k", torch.float32, (T, kv_heads, 2 * DP + 4))
-    _need(prep_g, "prepared decays", torch.float32, (T, heads, DP + 4))
+    _need(prep_g, "prepared decays", torch.float32, (T, heads, DP + 4 if za is not None else 4))
     _need(v32, "prepared values", torch.float32, (T, heads * vdim))
     _need(q_start, "q_start", torch.int32)
     _need(seq_of_token, "seq_of_token", torch.int32, (T,))
     _need(slots, "state slots", torch.int32)
     st, stride, off = _state_args(state, state_off)
-    if state_off + (taps - 1) * C > state.shape[1] or za.shape[0] != T:
+    if state_off + (taps - 1) * C > state.shape[1] or (za is not None and za.shape[0] != T):
         raise KernelError("delta_prepare: the state or the decays are too small")
     _check(library().li_delta_prepare(_p(proj), _i(_dt(proj)), _i(proj.shape[1]), _i(int(col)), _i(int(b_col)), _p(conv_w), _i(taps), st, stride, off,
-                                      _p(q_start), _p(seq_of_token), _p(slots), _p(za), _i(za.shape[1]), _i(int(za_col)), _p(A_log),
-                                      _f(float(dim) ** -0.5), _f(float(unit_eps)), _p(prep_qk), _p(prep_g), _p(v32), _i(T), _i(heads), _i(kv_heads),
+                                      _p(q_start), _p(seq_of_token), _p(slots), _p(za), _i(za.shape[1] if za is not None else 0), _i(int(za_col)), _i(int(a_col)),
+                                      _p(dt_bias), _p(A_log), _f(float(dim) ** -0.5), _f(float(unit_eps)), _p(prep_qk), _p(prep_g), _p(v32), _i(T), _i(heads), _i(kv_heads),
                                       _i(dim), _i(vdim), _i(1 if shift else 0), _stream(v32)), "delta_prepare")
 
 
@@ -883,11 +922,13 @@ def delta_scan(prep_qk: torch.Tensor, prep_g: torch.Tensor, v32: torch.Tensor, s
     """The gated delta rule with a decay per token, head and key channel over what :func:`delta_prepare` made, state
     ``S [dim, vdim]`` per head at the start of ``state[slot]`` (kept column by column, ``[heads, vdim, dim]``):
     ``S = diag(g_t) S``; ``u = beta_t (v_t - S^T k_t)``; ``S = S + k_t u^T``; ``out_t = S^T q_t``; head h uses the q and k of key
-    head ``h // (heads / kv_heads)``.  A sequence's tokens run in order, in one piece."""
+    head ``h // (heads / kv_heads)``.  A sequence's tokens run in order, in one piece.  ``prep_g`` [T, heads, 4]: one decay a
+    head."""
     T = v32.shape[0]
     DP = delta_row_elements(dim)
     _need(prep_qk, "prepared q and k", torch.float32, (T, kv_heads, 2 * DP + 4))
-    _need(prep_g, "prepared decays", torch.float32, (T, heads, DP + 4))
+    per_head = prep_g.shape[-1] == 4
+    _need(prep_g, "prepared decays", torch.float32, (T, heads, 4 if per_head else DP + 4))
     _need(v32, "prepared values", torch.float32, (T, heads * vdim))
     _need(out32, "scan output", torch.float32, (T, heads * vdim))
     S = q_start.shape[0] - 1
@@ -897,7 +938,7 @@ def delta_scan(prep_qk: torch.Tensor, prep_g: torch.Tensor, v32: torch.Tensor, s
     if heads * dim * vdim > state.shape[1]:
         raise KernelError("delta_scan: the state is too small")
     _check(library().li_delta_scan(_p(prep_qk), _p(prep_g), _p(v32), st, stride, _p(q_start), _p(slots), _p(out32), _i(S), _i(heads), _i(kv_heads),
-                                   _i(dim), _i(vdim), _stream(out32)), "delta_scan")
+                                   _i(dim), _i(vdim), _i(1 if per_head else 0), _stream(out32)), "delta_scan")
 
 
 def channel_scan(x: torch.Tensor, x_col: int, bc: torch.Tensor, b_col: int, c_col: int, dt32: torch.Tensor, z: torch.Tensor, z_col: int,
@@ -985,11 +1026,22 @@ def norm_add_norm(x32: torch.Tensor, y, post: Optional[tuple], nxt: Optional[tup
     root of the mean of squares + eps; both multiply by the weight.  ``centered`` 2 (:data:`SCALE_ONLY`): no statistic at
     all, the row times the weight (a learned factor per channel).  ``post`` None: ``x32 += y``; ``y`` None: nothing is
     added; ``nxt`` None: no output; ``nxt`` with a weight of None: ``out`` is ``x32`` as it is, in the run dtype.  ``rows`` (int32, only without ``y``): ``out[r] = nxt(x32[rows[r]])``.  ``y`` may be a
-    :class:`RowSum`: the sum is then taken inside this kernel, in float32."""
+    :class:`RowSum` or a :class:`WeightedPair`: the sum is then taken inside this kernel, in float32."""
     n_src, H = x32.shape
     _need(x32, "residual stream", torch.float32)
     R = n_src if rows is None else rows.shape[0]
     places, top, y_weights, y_extra = None, 0, None, None
+    y2, s1, s2, (w1, w2, eps_pair) = None, 1.0, 0.0, (None, None, 0.0)
+    if isinstance(y, WeightedPair):
+        if H > 8192:
+            raise KernelError(f"norm_add_norm: two outputs side by side of {H} columns (at most 8192)")
+        y2, s1, s2 = y.b, y.sa, y.sb
+        if y.norms is not None:
+            w1, w2, eps_pair = y.norms
+            _need(w1, "norm weight of the first output", torch.float32, (H,))
+            _need(w2, "norm weight of the second output", torch.float32, (H,))
+        y = y.a
+        _need(y2, "sublayer output (second)", y.dtype, (n_src, H))
     if isinstance(y, RowSum):
         if H > 8192:
             y = y.materialize()
@@ -1019,7 +1071,8 @@ def norm_add_norm(x32: torch.Tensor, y, post: Optional[tuple], nxt: Optional[tup
     dt = _dt(y) if y is not None else _dt(out)
     _check(library().li_norm_add_norm(_p(x32), _p(y), _i(dt), _p(wp), _i(int(cp)), _f(ep), _p(wn), _i(int(cn)), _f(en),
                                       _p(out if nxt is not None else None), _p(rows), _i(R), _i(n_src), _i(H), _p(places), _i(top), _p(y_weights),
-                                      _p(y_extra), _stream(x32)), "norm_add_norm")
+                                      _p(y_extra), _p(y2), _f(float(s1)), _f(float(s2)), _p(w1), _p(w2), _f(float(eps_pair)), _stream(x32)),
+           "norm_add_norm")
 
 
 def join_rows(x32: torch.Tensor, delta, x0: torch.Tensor, out: torch.Tensor) -> None:
@@ -1126,12 +1179,12 @@ def conv_norm_rope_kv(proj: torch.Tensor, out: torch.Tensor, conv_w: Optional[to
 
 
 def rope_norm_kv(proj: torch.Tensor, out: torch.Tensor, positions: torch.Tensor, denominators: Optional[torch.Tensor], rotary_dim: int,
-                 magnitude: float, interleaved: bool, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], norm: bool, eps: float,
+                 magnitude: float, interleaved: bool, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], norm, eps: float,
                  norm_width: int, slot_mapping: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, num_heads: int, num_kv_heads: int,
                  head_dim: int, write: bool = True, to_cache: bool = True, keys_are_values: bool = False) -> None:
-    """What stands between a q|k|v product and attention when the norm comes behind the rotation: the first ``rotary_dim``
+    """What stands between a q|k|v product and attention in one kernel: the first ``rotary_dim``
     elements of every query and key head are rotated (pair i by ``position / denominators[i]``; ``interleaved``: the pair is
-    (2i, 2i + 1), else (i, i + rotary_dim / 2); cosines and sines times ``magnitude``), then (``norm``) the head is divided by
+    (2i, 2i + 1), else (i, i + rotary_dim / 2); cosines and sines times ``magnitude``), and behind that (``norm`` true or 1) or before it (``norm`` 2) the head is divided by
     ``sqrt(sum x^2 / norm_width + eps)`` and multiplied by ``q_norm`` / ``k_norm`` [head_dim] if given.  Queries to ``out``
     [T, (heads + 2 kv_heads) head_dim], keys and values into the paged cache.  ``keys_are_values``: ``proj`` holds q|k only and
     a key head as projected, before rotation and norm, is the value.  ``to_cache`` false: keys and values go to their columns
@@ -1156,7 +1209,7 @@ def rope_norm_kv(proj: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,
         raise KernelError(f"cache of {nkv} heads x {dh} does not match {num_kv_heads} x {head_dim}")
     _check(library().li_rope_norm_kv(
         _p(proj), _i(proj.shape[1]), _p(out), _i(_dt(proj)), _p(positions), _p(denominators if rotary_dim else None), _f(float(magnitude)),
-        _i(1 if interleaved else 0), _i(rotary_dim), _p(q_norm), _p(k_norm), _i(1 if norm else 0), _f(eps), _i(int(norm_width)), _p(slot_mapping),
+        _i(1 if interleaved else 0), _i(rotary_dim), _p(q_norm), _p(k_norm), _i(int(norm)), _f(eps), _i(int(norm_width)), _p(slot_mapping),
         _p(k_cache), _p(v_cache), _i(T), _i(num_heads), _i(num_kv_heads), _i(head_dim), _i(page_size), _i(pages), _i(1 if write else 0),
         _i(1 if to_cache else 0), _i(1 if keys_are_values else 0), _stream(out)), "rope_norm_kv")
 
@@ -1289,22 +1342,23 @@ def moe_route(logits: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.
 
 
 def moe_route_grouped(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int, scale: float,
-                      ids: torch.Tensor, weights: torch.Tensor) -> None:
+                      ids: torch.Tensor, weights: torch.Tensor, scoring: str = "softmax_grouped") -> None:
     """Routing over all experts at once: ``s = softmax(logits)``; the choice scores are ``s + correction``; the experts form
     ``groups`` equal groups of neighbours, a group's score is its largest choice score, and only experts of the ``keep`` best
     groups can be chosen; the ``top`` largest choice scores choose (the lower index wins a tie); ``weights`` are the chosen
-    experts' s divided by their sum (+ 1e-20), times ``scale``."""
+    experts' s divided by their sum (+ 1e-20), times ``scale``.  ``scoring`` "sigmoid_grouped": ``s = sigmoid(logits)``, a group's
+    score is the sum of its two largest choice scores, and the weights are the chosen experts' s times ``scale``."""
     T, E = logits.shape
     _need(logits, "router logits", torch.float32)
     if correction is not None:
         _need(correction, "correction of the choice scores", torch.float32, (E,))
     _need(ids, "expert ids", torch.int32, (T, top))
     _need(weights, "expert weights", torch.float32, (T, top))
-    _check(library().li_moe_route_grouped(_p(logits), _p(correction), _i(T), _i(E), _i(top), _i(int(groups)), _i(int(keep)), _f(float(scale)),
+    _check(library().li_moe_route_grouped(_p(logits), _p(correction), _i(MOE_SCORINGS[scoring]), _i(T), _i(E), _i(top), _i(int(groups)), _i(int(keep)), _f(float(scale)),
                                           _p(ids), _p(weights), _stream(ids)), "moe_route_grouped")
 
 
-MOE_SCORINGS = {"sigmoid": 0, "softmax_chosen": 1, "softmax_grouped": 2}
+MOE_SCORINGS = {"sigmoid": 0, "softmax_chosen": 1, "softmax_grouped": 2, "sigmoid_grouped": 3}
 
 
 def moe_small_step_accepts(h: torch.Tensor, experts: int, top: int) -> bool:
@@ -1316,7 +1370,7 @@ def moe_small_step(h: torch.Tensor, router: torch.Tensor, bias: Optional[torch.T
                    groups: int, keep: int, scale: float, weights: torch.Tensor, offsets: torch.Tensor, pair_at: torch.Tensor,
                    place_of: torch.Tensor) -> None:
     """The front of a mixture for a step of few tokens as one launch: the router's product ``h router^T (+ bias)`` with float32
-    sums, the choice (``scoring`` as in :func:`moe_route`, or "softmax_grouped" as :func:`moe_route_grouped`) and the sort of
+    sums, the choice (``scoring`` as in :func:`moe_route`, or "softmax_grouped", "sigmoid_grouped" as :func:`moe_route_grouped`) and the sort of
     :func:`moe_sort` without padding: ``weights`` [T, top], ``offsets`` [E + 1], ``pair_at`` and ``place_of`` [T top]."""
     T, H = h.shape
     E = router.shape[0]
@@ -1491,7 +1545,8 @@ _TIMED = ("embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add
           "rope_kv_write", "linear_rope_kv", "rope_table", "paged_attention", "swiglu", "argmax", "sample", "gather_rows", "scale_inplace",
           "logit_cap", "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift",
           "ssm_scan", "decay_scan", "gated_rmsnorm", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route",
-          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step")
+          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "gelu_token_rows",
+          "mul_sigmoid", "polynorm")
 if profile.enabled:
     for _name in _TIMED:
         globals()[_name] = profile.wrap(_name, globals()[_name])

@@ -56,6 +56,7 @@ class DecoderModel:
         # what else joins the stream after the embedding (an embedding of token pairs); their caches come behind the schedule's
         self.stream_inputs = [STREAM_INPUTS.build(p, prefix, self.dtype, self.device) for p, prefix in spec.stream_inputs]
         self.stream_tables: Dict[str, torch.Tensor] = {}      # vectors that schedule entries add to the stream (ScheduleEntry.add)
+        self.token_tables: Dict[str, torch.Tensor] = {}       # rows per token that layers read (ModelSpec.token_tables)
         self.stream_maps: Dict[str, torch.Tensor] = {}        # maps of the stream beside the embedding output (ScheduleEntry.join)
         self.embedding: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
@@ -76,6 +77,8 @@ class DecoderModel:
             out.append(ParamSpec(name, (int(rows), s.hidden_size), role="vector", std=0.02))
         for name in s.stream_maps:
             out.append(ParamSpec(name, (s.hidden_size, 2 * s.hidden_size), role="matrix"))
+        for name, columns in s.token_tables.items():
+            out.append(ParamSpec(name, (s.vocab_size, int(columns)), role="matrix", std=1.0))
         for b in self.blocks:
             out.extend(b.all_params())
         out.extend(self.final_norm.all_params())
@@ -95,8 +98,10 @@ class DecoderModel:
             part.bind_all(tensors)
         self.stream_tables = {name: tensors.pop(name) for name in s.stream_tables}
         self.stream_maps = {name: tensors.pop(name) for name in s.stream_maps}
+        self.token_tables = {name: tensors.pop(name) for name in s.token_tables}
         for b in self.blocks:
             b.bind_all(tensors)
+            b.take_tables(self.token_tables)
         self.final_norm.bind_all(tensors)
         # a stored head is used; without one the head is the embedding table itself
         # (python/llaisys/models/qwen2.py:196-199: ``if not w.out_embed and w.in_embed``)
@@ -112,6 +117,11 @@ class DecoderModel:
         out = []
         for e in self.spec.schedule:
             out.append(self.blocks[e.block].cache_requirement() if e.cache_from is None else None)
+        # an entry that reads another's cache may see further back than its owner does: the owner keeps what both read
+        for e in self.spec.schedule:
+            reads = self.blocks[e.block].reads_from_cache() if e.cache_from is not None else None
+            if reads is not None and isinstance(out[e.cache_from], PagedKV):
+                out[e.cache_from] = out[e.cache_from].covering(reads)
         out.extend(part.cache_requirement() for part in self.stream_inputs)
         return out
 

@@ -38,10 +38,18 @@ Further options of the spec, all off by default:
 * ``norm_after`` (a mapping with ``eps``): queries and keys are divided by their root mean square per head behind the rotation,
   without a weight;
 * ``keys_are_values`` true: the layer has no value map; a key as projected, before rotation and norm, is its value too;
-* ``sink`` (a tensor's name below the prefix): a learned number per head whose exponential joins the softmax's denominator.
+* ``sink`` (a tensor's name below the prefix): a learned number per head whose exponential joins the softmax's denominator;
+* ``sink_score`` (a number): the same with one constant for every head (0: the denominator is one larger);
+* ``chunk`` (a number of positions): the query at position p sees the keys of its own chunk only, those with
+  ``t // chunk == p // chunk``; chunks are counted from position 0 of the sequence.  The cache gives a chunk's pages back when
+  it is over (a layer that reads another's cache may have chunks of another size; the owner keeps what both read);
+* ``element_gate`` (a tensor's stem): a map from the mixer's input to one number per element of the concatenated heads, which
+  are multiplied by its sigmoid before the output map.
 
-A position part that pairs neighbours or carries a magnitude (:class:`~litinfer_b200.parts.base.Rotary`) goes with the last
-three: rotation, norm, values and the cache write are then one kernel behind the product (``kernels.rope_norm_kv``).
+A position part that pairs neighbours or carries a magnitude (:class:`~litinfer_b200.parts.base.Rotary`) goes with a norm per
+head on either side of the rotation, keys as values, and values of another size than the keys: rotation, norm, values and the
+cache write are then one kernel behind the product (``kernels.rope_norm_kv``).  The gate's rows stand behind q|k|v (or behind the
+queries alone, in a layer that shares another's keys and values) in one product, and attention applies it to its output.
 """
 
 from __future__ import annotations
@@ -78,6 +86,7 @@ class PagedAttention(Mixer):
             raise ValueError(f"{len(slopes)} distance slopes for {self.num_heads} heads")
         self.slopes = torch.tensor([float(x) for x in slopes], dtype=torch.float32, device=self.device) if slopes is not None else None
         self.window = spec.get("window")
+        self.chunk = int(spec.get("chunk") or 0)
         self.keep_first = int(spec.get("keep_first") or 0) if self.window else 0
         self.taps = int(spec.get("conv") or 0)                # 0: no convolution
         qk_norm = spec.get("qk_norm")
@@ -98,6 +107,9 @@ class PagedAttention(Mixer):
         self.keys_are_values = bool(spec.get("keys_are_values", False))
         self.sink_name = prefix + str(spec["sink"]) if spec.get("sink") else None
         self.sinks = None
+        self.sink_score = float(spec["sink_score"]) if spec.get("sink_score") is not None else None
+        if self.sink_score is not None and self.sink_name:
+            raise ValueError("a learned sink and a constant one do not go together")
         if self.keys_are_values:
             if self.value_dim != self.qk_dim:
                 raise ValueError(f"values that are the keys have the keys' size {self.qk_dim}, not {self.value_dim}")
@@ -118,19 +130,27 @@ class PagedAttention(Mixer):
         # rotation first, a norm behind it, keys that are values: a kernel of its own behind the product
         self.rotate_apart = (self.keys_are_values or self.norm_after_eps is not None or getattr(self.position, "interleaved", False)
                              or getattr(self.position, "magnitude", 1.0) != 1.0)
-        if self.rotate_apart and (self.taps >= 1 or qk_norm or self.shared_kv or self.value_dim != self.qk_dim):
+        if self.rotate_apart and (self.taps >= 1 or self.norm_whole or self.shared_kv or (self.norm_after_eps is not None and qk_norm)):
             raise ValueError(f"attention at {prefix!r}: pairs of neighbours, a magnitude, a norm behind the rotation and keys as values do not go "
-                             "with a convolution, a norm before the rotation, shared keys or values of another size")
+                             "with a convolution, a norm over the whole projection, shared keys or two norms")
         self.conv_names = [prefix + n + str(spec.get("conv_suffix", ".conv")) for n in stems] if self.taps >= 1 else []
         self.norm_names = [prefix + str(qk_norm[n]) for n in (("q",) if self.shared_kv else ("q", "k"))] if qk_norm else []
         self.conv_weight = self.q_norm = self.k_norm = None
         # what the q|k|v product's epilogues cannot do goes through a kernel of its own behind a plain product
         self.post = self.taps >= 1 or bool(qk_norm) or self.shared_kv
+        # queries alone, nothing to be done to them: attention reads the product's rows as they are
+        self.plain_queries = self.shared_kv and not qk_norm and position is None
+        element_gate = spec.get("element_gate")
+        self.element_gate = (FusedLinear(prefix, [element_gate], self.hidden, [self.num_heads * self.value_dim], False, dtype, suffixes=suffixes)
+                             if element_gate else None)
+        if self.element_gate is not None and (gate or self.rotate_apart or (self.post and not self.plain_queries)):
+            raise ValueError(f"attention at {prefix!r}: a gate per element goes with plain projections (no norm, convolution, rotation of neighbours or gate per head)")
         # steps of single tokens read the convolution's state through the step's device tensors: they can be captured
         self.decodes_from_device = self.taps > 1
 
     def params(self) -> List[ParamSpec]:
         out = self.qkv.params() + self.out.params() + (self.gate.params() if self.gate is not None else [])
+        out += self.element_gate.params() if self.element_gate is not None else []
         out += [ParamSpec(n, (o, self.taps), role="vector", mean=1.0 / self.taps, std=0.2) for n, o in zip(self.conv_names, self.real_outs)]
         if self.norm_whole:
             out += [ParamSpec(n, (o,), role="vector", init="ones_normal") for n, o in zip(self.norm_names, self.real_outs)]
@@ -148,8 +168,12 @@ class PagedAttention(Mixer):
         self.out.bind(tensors)
         if self.gate is not None:
             self.gate.bind(tensors)
+        if self.element_gate is not None:
+            self.element_gate.bind(tensors)
         if self.sink_name:
             self.sinks = tensors.pop(self.sink_name)
+        elif self.sink_score is not None:
+            self.sinks = torch.full((self.num_heads,), self.sink_score, dtype=torch.float32, device=self.qkv.weight.device)
         conv = [tensors.pop(n) for n in self.conv_names]
         norms = [tensors.pop(n) for n in self.norm_names]
         if self.head_dim != self.qk_dim or self.head_dim != self.value_dim:
@@ -159,6 +183,16 @@ class PagedAttention(Mixer):
                 norms = [self._pad_rows(t, *sh) for t, sh in zip(norms, self.head_shapes)]
             else:
                 norms = [torch.cat([t, torch.zeros(self.head_dim - self.qk_dim, dtype=t.dtype, device=t.device)]) for t in norms]
+        if self.element_gate is not None:
+            # the gate's rows behind q|k|v, as many a head as the cache has
+            w = self.element_gate.weight
+            if self.head_dim != self.value_dim:
+                w = self._pad_rows(w, self.num_heads, self.value_dim)
+            self.qkv.weight = torch.cat([self.qkv.weight, w], dim=0).contiguous()
+            if self.qkv.bias is not None:
+                self.qkv.bias = torch.cat([self.qkv.bias, torch.zeros(w.shape[0], dtype=self.qkv.bias.dtype, device=w.device)]).contiguous()
+            self.qkv.out_features = self.qkv.weight.shape[0]
+            self.element_gate.weight = None
         if conv:
             self.conv_weight = torch.cat(conv, dim=0).contiguous()
         if norms:
@@ -198,11 +232,17 @@ class PagedAttention(Mixer):
     def cache_requirement(self):
         if self.shared_kv:
             return None                        # the schedule entry names the entry whose cache this layer reads
-        paged = PagedKV(self.num_kv_heads, self.head_dim, self.window, self.keep_first)
+        paged = self._reads()
         if self.taps > 1:
             # behind the pages: the last taps - 1 rows of the q|k|v projection, which the convolution of the next step reads
             return (paged, FixedState(((self.taps - 1) * self.qkv_width,), torch.float32))
         return paged
+
+    def _reads(self) -> PagedKV:
+        return PagedKV(self.num_kv_heads, self.head_dim, self.window, self.keep_first, (self.chunk,) if self.chunk else ())
+
+    def reads_from_cache(self):
+        return self._reads() if self.shared_kv else None
 
     @property
     def qkv_width(self) -> int:
@@ -213,7 +253,7 @@ class PagedAttention(Mixer):
         if type(self) is not PagedAttention or rope is None or rope["rotary_dim"] != self.head_dim or self.out.bias is not None:
             return None
         if self.softcap or self.slopes is not None or self.gate is not None or self.value_dim != self.qk_dim or self.post or self.keep_first or self.shared_kv \
-                or self.rotate_apart or self.sink_name:
+                or self.rotate_apart or self.sinks is not None or self.chunk or self.element_gate is not None:
             return None
         return {"w_qkv": self.qkv.weight, "b_qkv": self.qkv.bias, "w_o": self.out.weight, "hidden": self.hidden, "heads": self.num_heads,
                 "kv_heads": self.num_kv_heads, "head_dim": self.head_dim, "scale": self.scale, "window": self.window,
@@ -225,7 +265,17 @@ class PagedAttention(Mixer):
     def forward_into(self, h, ctx, cache, tail):
         return tail.apply_linear(self.out, self._attend(h, ctx, cache))
 
-    def _attend(self, h, ctx, cache):
+    # The first product and what follows it, apart: a mixer of mixers may take the product of several at once
+    # (parts.parallel).  ``projected``: rows that begin with this mixer's q|k|v.
+    def shared_projection(self):
+        return self.qkv if self.rotate_apart and self.gate is None else None
+
+    def forward_projected(self, projected, col, ctx, cache):
+        if col:
+            raise ValueError("attention takes its projections from the first column on")
+        return self.out(self._attend(None, ctx, cache, projected))
+
+    def _attend(self, h, ctx, cache, projected=None):
         """Everything before the output projection: [tokens, heads * head_dim]."""
         state = None
         if self.taps > 1:
@@ -235,19 +285,25 @@ class PagedAttention(Mixer):
         rot = self.position.rotary(ctx) if self.position is not None else None
         if self.shared_kv and (cache is None or cache.kind != "paged" or cache.writes):
             raise ValueError(f"attention at {self.prefix!r} shares another layer's keys and values: its schedule entry must name that layer's entry (cache_from)")
+        gate_col = 0
         if self.rotate_apart:
-            # projection; then rotation, norm, values and the cache write as one kernel (in a long step the page-wise writer
+            # projection; then norm, rotation, values and the cache write as one kernel (in a long step the page-wise writer
             # stores keys and values)
-            proj = self.qkv(h)
+            proj = self.qkv(h) if projected is None else projected
             T = proj.shape[0]
             qkv = torch.empty((T, self.qkv_width), dtype=self.dtype, device=proj.device)
             long_step = T >= self.CACHE_WRITE_APART
             K.rope_norm_kv(proj, qkv, ctx.positions, rot.denominators if rot else None, rot.rotary_dim if rot else 0, rot.magnitude if rot else 1.0,
-                           bool(rot and rot.interleaved), None, None, self.norm_after_eps is not None, self.norm_after_eps or 0.0, self.qk_dim,
+                           bool(rot and rot.interleaved), self.q_norm, self.k_norm, 2 if self.q_norm is not None else self.norm_after_eps is not None,
+                           self.qk_norm_eps if self.q_norm is not None else self.norm_after_eps or 0.0, self.qk_dim,
                            view.slot_mapping, cache.k, cache.v, self.num_heads, self.num_kv_heads, self.head_dim, cache.writes,
                            to_cache=not long_step, keys_are_values=self.keys_are_values)
             if long_step and cache.writes:
                 K.rope_kv_write(qkv, ctx.positions, None, 0, view.slot_mapping, cache.k, cache.v, self.num_heads, self.num_kv_heads, self.head_dim, True)
+        elif self.plain_queries:
+            # queries, and the gate behind them, as the product left them
+            qkv = self.qkv(h)
+            gate, gate_col = (qkv, self.q_dim) if self.element_gate is not None else (gate, 0)
         elif self.post and (self.norm_whole or self.shared_kv):
             # projection; the factors of the norms over the whole of q and of k; then norm, rotation and the cache write as one
             # kernel.  A layer without keys and values of its own projects queries only, into rows that attention reads as q|k|v.
@@ -288,17 +344,19 @@ class PagedAttention(Mixer):
                 K.conv_state_shift(proj, 0, self.qkv_width, self.taps, state.state, 0, ctx.q_start, ctx.state_slots)
         else:
             h, row_scale = undefer(h, self.qkv.weight)
-            qkv = torch.empty((h.shape[0], self.qkv.out_features), dtype=self.dtype, device=h.device)
+            qkv = torch.empty((h.shape[0], self.qkv_width), dtype=self.dtype, device=h.device)
+            if self.element_gate is not None:
+                gate = torch.empty((h.shape[0], self.q_dim), dtype=self.dtype, device=h.device)
             # projection, position encoding of q and k, k and v into the cache: one call (and for few tokens one kernel)
             K.linear_rope_kv(
                 h, self.qkv.weight, self.qkv.bias, qkv, ctx.positions, rot.denominators if rot else None, rot.rotary_dim if rot else 0,
                 view.slot_mapping, cache.k, cache.v, self.num_heads, self.num_kv_heads, self.head_dim, cache.writes, row_scale=row_scale,
-                cos_sin=rot.table if rot else None)
+                cos_sin=rot.table if rot else None, extra=gate if self.element_gate is not None else None)
         o = torch.empty((qkv.shape[0], self.q_dim), dtype=self.dtype, device=qkv.device)
         K.paged_attention(
             qkv, o, cache.k, cache.v, view.block_table, ctx.q_start, ctx.ctx_lens, ctx.seq_of_token, ctx.positions,
             self.num_heads, self.num_kv_heads, self.head_dim, self.scale, self.window,
             ctx.max_q_len, ctx.max_ctx_len, old_lens=ctx.old_lens, singles=ctx.num_single,
             units=ctx.attn_units, unit_slots=ctx.attn_unit_slots, softcap=self.softcap, slopes=self.slopes, gate=gate, keep_first=self.keep_first,
-            sinks=self.sinks)
+            sinks=self.sinks, chunk=self.chunk, gate_elements=self.element_gate is not None, gate_col=gate_col)
         return o

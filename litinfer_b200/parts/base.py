@@ -21,6 +21,7 @@ Interfaces:
 * mixer:         ``forward(h, ctx, cache) -> y``; ``cache_requirement()``;
                  optionally ``forward_into(h, ctx, cache, tail) -> h'``
 * feed-forward:  ``forward(h, ctx) -> y``; optionally ``forward_into(h, ctx, tail) -> h'``
+* token input:   ``forward(x, ctx) -> y``; ``post_norm()``: what a layer adds of the token itself behind its feed-forward
 * block:         ``forward(x32, ctx, cache, carry, next_norm) -> (x32, carry)``; ``first_norm``
 
 A :class:`Tail` says what follows a part's output: it is added to the residual stream and the
@@ -57,12 +58,23 @@ from ..weights.loader import ParamSpec
 
 @dataclass(frozen=True)
 class PagedKV:
-    """Keys and values of every token (or of the last ``window``, and with a window the first ``keep_first`` as well), in pages."""
+    """Keys and values of every token (or of the last ``window``, and with a window the first ``keep_first`` as well; or, with
+    ``chunks``, of the newest token's chunk of each of these sizes, counted from position 0), in pages."""
 
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     keep_first: int = 0
+    chunks: Tuple[int, ...] = ()
+
+    def covering(self, other: "PagedKV") -> "PagedKV":
+        """What keeps the keys that either of the two reads: a layer's own and those of a layer that reads its cache."""
+        if (self.num_kv_heads, self.head_dim) != (other.num_kv_heads, other.head_dim):
+            raise ValueError(f"a cache of {self.num_kv_heads} heads x {self.head_dim} is read as {other.num_kv_heads} x {other.head_dim}")
+        if not all(r.window or r.chunks for r in (self, other)):
+            return PagedKV(self.num_kv_heads, self.head_dim)                  # one of them reads every key
+        return PagedKV(self.num_kv_heads, self.head_dim, max(self.window or 0, other.window or 0) or None,
+                       max(self.keep_first, other.keep_first), tuple(sorted(set(self.chunks) | set(other.chunks))))
 
 
 @dataclass(frozen=True)
@@ -113,6 +125,11 @@ class Part:
         names that file reads, or None: the part is not one the fused kernel is built for, and a model that holds it
         runs part by part.  The default is None, so that parts registered from outside are never fused by accident."""
         return None
+
+    def take_tables(self, tables: Dict[str, torch.Tensor]) -> None:
+        """The model's tables that parts share (``ModelSpec.token_tables``), once they are bound."""
+        for p in self.parts():
+            p.take_tables(tables)
 
     # helpers -----------------------------------------------------------
     def all_params(self) -> List[ParamSpec]:
@@ -197,6 +214,11 @@ class Mixer(Part):
     def cache_requirement(self):
         """PagedKV, FixedState, None, or a tuple of these (one per mixer inside this one: the cache it is handed then
         has ``parts``, in the same order)."""
+        return None
+
+    def reads_from_cache(self):
+        """For a mixer without keys and values of its own: the PagedKV it reads of another entry's cache (the owner then keeps
+        what this mixer still sees as well)."""
         return None
 
     def forward(self, h: torch.Tensor, ctx, cache) -> torch.Tensor:
@@ -292,6 +314,19 @@ class StreamInput(Part):
         raise NotImplementedError
 
 
+class TokenInput(Part):
+    """What a layer adds to the residual stream of the token itself: a part of the arrangement, behind the feed-forward.
+    ``forward(x, ctx) -> y`` reads the stream (in the run dtype) and the step's token ids; y joins the stream through
+    :meth:`post_norm`.  ``tables``: names of the model's token tables it reads (``ModelSpec.token_tables``), which the model hands
+    over with :meth:`take_tables` once its weights are bound."""
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        raise NotImplementedError
+
+    def post_norm(self) -> "Norm":
+        raise NotImplementedError
+
+
 class Block(Part):
     """``spec`` is a :class:`~litinfer_b200.config.spec.BlockSpec`: parts by role."""
 
@@ -310,6 +345,11 @@ class Block(Part):
         """What this block's schedule entry needs from the cache manager: by default its mixer's."""
         mixer = getattr(self, "mixer", None)
         return mixer.cache_requirement() if mixer is not None else None
+
+    def reads_from_cache(self):
+        """What this block reads of another entry's cache, by default its mixer's (:meth:`Mixer.reads_from_cache`)."""
+        mixer = getattr(self, "mixer", None)
+        return mixer.reads_from_cache() if mixer is not None else None
 
     def entry(self) -> Optional[Tail]:
         """The norm this block applies to the residual stream first, and whether its consumer takes a deferred
@@ -355,4 +395,5 @@ FEED_FORWARDS = Registry("feed-forward")
 NORMS = Registry("norm")
 POSITIONS = Registry("position encoding")
 STREAM_INPUTS = Registry("input of the residual stream")
+TOKEN_INPUTS = Registry("input of a layer from the token")
 BLOCKS = Registry("block arrangement")

@@ -23,8 +23,9 @@ from typing import Dict, Optional
 import torch
 
 from .. import kernels as K
+from ..config.spec import PartSpec
 from ..weights.loader import ParamSpec
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, Carry, Tail
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, TOKEN_INPUTS, Block, Carry, Tail
 
 
 @BLOCKS.register("prenorm")
@@ -170,6 +171,8 @@ class SandwichBlock(Block):
     """A norm before and a norm after each sublayer: ``x += post(Mixer(pre(x)))``, then ``x += post'(FeedForward(pre'(x)))``.
     Roles: ``mixer_norm``, ``mixer_post_norm``, and with a feed-forward ``feed_forward_norm``, ``feed_forward_post_norm``;
     any registered norm that says what it is through ``statistics()`` (weight, centered or not, eps) serves in any role.
+    ``token_input`` (optional): a part that adds something of the token itself behind the feed-forward (behind the mixer in a
+    layer without one): ``x += norm(input(x, token))``; it reads the stream itself, which the pass before hands it.
 
     The norm after a sublayer, the addition to the stream and the norm before the next sublayer are one kernel and one
     pass over the stream (``kernels.norm_add_norm``); told the next block's entry, the last sublayer's pass already
@@ -183,13 +186,16 @@ class SandwichBlock(Block):
         self.feed_forward = self.build(FEED_FORWARDS, "feed_forward", required=False)
         self.feed_forward_norm = self.build(NORMS, "feed_forward_norm", required=self.feed_forward is not None)
         self.feed_forward_post_norm = self.build(NORMS, "feed_forward_post_norm", required=self.feed_forward is not None)
+        self.token_input = self.build(TOKEN_INPUTS, "token_input", required=False)
+        # what the pass before a token input leaves for it: the stream as it is
+        self.as_it_is = NORMS.build(PartSpec("identity", {"size": 0}), prefix, dtype, device)
         for n in (self.mixer_norm, self.mixer_post_norm, self.feed_forward_norm, self.feed_forward_post_norm):
             if n is not None and not hasattr(n, "statistics"):
                 raise ValueError(f"block 'sandwich' at {spec.prefix!r}: norm '{n.spec.kind}' does not say what it is (statistics())")
 
     def parts(self) -> List:
         return [p for p in (self.mixer_norm, self.mixer, self.mixer_post_norm, self.feed_forward_norm, self.feed_forward,
-                            self.feed_forward_post_norm) if p is not None]
+                            self.feed_forward_post_norm, self.token_input) if p is not None]
 
     def entry(self):
         return Tail(None, self.mixer_norm, False)
@@ -211,12 +217,22 @@ class SandwichBlock(Block):
         else:
             h = self.mixer_norm.add_forward(x32, carry.delta)
         nxt = next_entry.norm if next_entry is not None and type(next_entry) is Tail else None
-        y = self.mixer.forward(h, ctx, cache)
+        last = self.as_it_is if self.token_input is not None else nxt              # what follows the last sublayer
+        # (a mixer of two side by side hands both outputs over: the pass over the stream adds them up)
+        y = self.mixer.forward_pair(h, ctx, cache) if getattr(self.mixer, "produces_pairs", False) else self.mixer.forward(h, ctx, cache)
         if self.feed_forward is None:
-            h = self._close(x32, y, self.mixer_post_norm, nxt)
+            h = self._close(x32, y, self.mixer_post_norm, last)
+            h = self._token_input(x32, h, ctx, nxt)
             return x32, (Carry(normed=h) if h is not None else None)
         h = self._close(x32, y, self.mixer_post_norm, self.feed_forward_norm)
         # (a mixture of experts hands its rows over as they are: the pass over the stream sums a token's rows itself)
         y = self.feed_forward.forward_rows(h, ctx) if getattr(self.feed_forward, "produces_row_sums", False) else self.feed_forward.forward(h, ctx)
-        h = self._close(x32, y, self.feed_forward_post_norm, nxt)
+        h = self._close(x32, y, self.feed_forward_post_norm, last)
+        h = self._token_input(x32, h, ctx, nxt)
         return x32, (Carry(normed=h) if h is not None else None)
+
+    def _token_input(self, x32, h, ctx, nxt):
+        """What the layer adds of the token itself (``h``: the stream in the run dtype); without such a part ``h`` as it is."""
+        if self.token_input is None:
+            return h
+        return self._close(x32, self.token_input.forward(h, ctx), self.token_input.post_norm(), nxt)

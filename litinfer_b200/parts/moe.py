@@ -14,6 +14,8 @@ choice scores are ``s + correction`` (a stored vector); the outputs form ``group
 score is its largest choice score, and only outputs of the ``keep_groups`` best groups can be chosen; the ``top`` largest
 choice scores choose; the weights are the chosen outputs' s divided by their sum (+ 1e-20), times ``route_scale``.  The last
 ``identity`` outputs are identity experts: they have no tensors and their output is the input h itself (times the weight).
+``scoring`` "sigmoid_grouped" (without ``renormalize``): sigmoid scores with the same correction and groups; a group's score is the
+sum of its two largest choice scores, and the weights are the chosen outputs' s times ``route_scale``.
 ``scoring`` "softmax" (with ``renormalize``): the same without correction, groups and identity experts: ``s = softmax(z)`` over all
 experts, the ``top`` largest choose, the weights are the chosen experts' s divided by their sum (+ 1e-20).
 ``shared`` (the spec of a dense feed-forward, of another kind and size if it likes; its tensors below ``names["shared"]``): one more
@@ -59,8 +61,9 @@ class RoutedExperts(FeedForward):
         if not 0 < self.top <= self.experts + int(spec.get("identity") or 0):
             raise ValueError(f"{self.top} of {self.experts} experts")
         self.scoring = str(spec.get("scoring", "sigmoid"))
-        if self.scoring not in ("sigmoid", "softmax_chosen", "softmax_grouped", "softmax"):
-            raise ValueError(f"routing by '{spec.get('scoring')}' is not supported (sigmoid, softmax_chosen, softmax_grouped, softmax)")
+        if self.scoring not in ("sigmoid", "softmax_chosen", "softmax_grouped", "softmax", "sigmoid_grouped"):
+            raise ValueError(f"routing by '{spec.get('scoring')}' is not supported (sigmoid, softmax_chosen, softmax_grouped, softmax, sigmoid_grouped)")
+        corrected = self.scoring in ("softmax_grouped", "sigmoid_grouped")
         self.renormalize = bool(spec.get("renormalize", False))
         if self.renormalize and self.scoring not in ("softmax_grouped", "softmax"):
             raise ValueError(f"renormalised routing weights go with softmax scores over all experts, not with '{self.scoring}'")
@@ -75,11 +78,11 @@ class RoutedExperts(FeedForward):
         self.groups = int(spec.get("groups") or 1)
         self.keep_groups = int(spec.get("keep_groups") or self.groups)
         self.route_scale = float(spec.get("route_scale", 1.0))
-        if self.scoring != "softmax_grouped" and (self.identity or self.groups != 1):
-            raise ValueError("identity experts and groups of experts go with scoring 'softmax_grouped'")
+        if not corrected and (self.identity or self.groups != 1):
+            raise ValueError("identity experts and groups of experts go with scoring 'softmax_grouped' or 'sigmoid_grouped'")
         if self.identity and self.weight_on != "output":
             raise ValueError("identity experts take their weight on the output")
-        if self.scoring == "softmax_grouped":
+        if corrected:
             if self.top > self.outputs or self.outputs % self.groups or not 1 <= self.keep_groups <= self.groups or \
                     self.keep_groups * (self.outputs // self.groups) < self.top:
                 raise ValueError(f"{self.keep_groups} of {self.groups} groups over {self.outputs} router outputs cannot give {self.top} choices")
@@ -91,7 +94,7 @@ class RoutedExperts(FeedForward):
         suffixes = tuple(spec.get("suffixes", (".weight", ".bias")))
         self.router = FusedLinear(prefix, [n.get("router", "gate")], self.hidden, [self.outputs], bool(spec.get("router_bias", False)), dtype,
                                   suffixes=suffixes)
-        self.correction_name = prefix + n.get("correction", "correction") if self.scoring == "softmax_grouped" else None
+        self.correction_name = prefix + n.get("correction", "correction") if corrected else None
         self.correction = None
         stem = n.get("expert", "experts.{}.")                 # the e-th expert's tensors start with prefix + stem.format(e)
         w = suffixes[0]
@@ -161,16 +164,16 @@ class RoutedExperts(FeedForward):
         pair_at = torch.empty(R, dtype=torch.int32, device=dev)
         tiles = torch.empty(R // pad, dtype=torch.int32, device=dev) if pad > 1 else None
         tile_rows = pad if pad > 1 else self.PAD
-        grouped = self.scoring in ("softmax_grouped", "softmax")
+        grouped = {"softmax": "softmax_grouped"}.get(self.scoring, self.scoring)         # (one group of all, no correction)
         if pad == 1 and K.moe_small_step_accepts(h, n_out, top):
             # few tokens: the router's product, the choice and the sort are one launch
-            K.moe_small_step(h, self.router.weight, self.router.bias, top, "softmax_grouped" if grouped else self.scoring, self.correction, self.groups,
+            K.moe_small_step(h, self.router.weight, self.router.bias, top, grouped, self.correction, self.groups,
                              self.keep_groups, self.route_scale, weights, offsets, pair_at, place_of)
         else:
             logits = self.router(h, out_dtype=torch.float32)
             ids = torch.empty((T, top), dtype=torch.int32, device=dev)
-            if grouped:
-                K.moe_route_grouped(logits, self.correction, top, self.groups, self.keep_groups, self.route_scale, ids, weights)
+            if grouped.endswith("_grouped"):
+                K.moe_route_grouped(logits, self.correction, top, self.groups, self.keep_groups, self.route_scale, ids, weights, scoring=grouped)
             else:
                 K.moe_route(logits, top, ids, weights, scoring=self.scoring)
             K.moe_sort(ids, n_out, offsets, pair_at, place_of, pad, tiles, matrices=E)

@@ -173,7 +173,8 @@ def _query_heads(qkv, num_heads, head_dim, maps):
 
 def paged_attention(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, seq_of_token, positions,
                     num_heads, num_kv_heads, head_dim, scale, window, max_q_len, max_ctx_len, implementation=None, old_lens=None, singles=0,
-                    units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None, maps=1):
+                    units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None, maps=1,
+                    chunk=0, gate_elements=False, gate_col=0):
     # old_lens only tells a kernel which keys it may read early, singles which kernel takes which sequence, units how a
     # kernel shares its work out; the result does not depend on them
     T = qkv.shape[0]
@@ -186,8 +187,9 @@ def paged_attention(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, 
     for t in range(T):
         s, p = seqs[t], poss[t]
         lo = 0 if not window else max(0, p - window + 1)
+        lo = max(lo, p // chunk * chunk) if chunk else lo
         keys = torch.arange(lo, p + 1, device=qkv.device)
-        if keep_first and lo > 0:
+        if window and keep_first and lo > 0:
             keys = torch.cat([torch.arange(0, min(keep_first, lo), device=qkv.device), keys])
         pages = block_table[s].long()[keys // page_size]
         offs = keys % page_size
@@ -205,13 +207,14 @@ def paged_attention(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, 
                 pr = torch.softmax(sc, dim=0)
             res[t, h] = pr @ v[:, h // group]
             if gate is not None:
-                res[t, h] *= torch.sigmoid(gate[t, h].float())
+                res[t, h] *= torch.sigmoid((gate[t, gate_col + h * head_dim:gate_col + (h + 1) * head_dim] if gate_elements else gate[t, gate_col + h]).float())
     _store(out, res.reshape(T, num_heads * head_dim))
 
 
 def paged_attention_dense(qkv, out, k_cache, v_cache, block_table, q_start, ctx_lens, seq_of_token, positions,
                           num_heads, num_kv_heads, head_dim, scale, window, max_q_len, max_ctx_len, implementation=None, old_lens=None,
-                          singles=0, units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None, maps=1):
+                          singles=0, units=None, unit_slots=(0, 0), softcap=0.0, slopes=None, gate=None, keep_first=0, sinks=None, maps=1,
+                          chunk=0, gate_elements=False, gate_col=0):
     """The same formula as :func:`paged_attention`, a sequence at a time instead of a token and a head at a time (for
     contexts of thousands of keys): scores of all the sequence's tokens against all its keys in float32, keys outside
     [p - window + 1, p] masked, softmax, weighted sum."""
@@ -242,6 +245,8 @@ def paged_attention_dense(qkv, out, k_cache, v_cache, block_table, q_start, ctx_
             if keep_first:
                 inside |= keys[None, :] < keep_first
             seen &= inside
+        if chunk:
+            seen &= keys[None, :] // chunk == pos[:, None] // chunk
         sc = sc.masked_fill(~seen[None], float("-inf"))
         if sinks is not None:
             sk = sinks.float()[:, None, None].expand(num_heads, hi - lo, 1)
@@ -250,7 +255,8 @@ def paged_attention_dense(qkv, out, k_cache, v_cache, block_table, q_start, ctx_
             pr = torch.softmax(sc, dim=-1)
         res[lo:hi] = torch.einsum("htc,chd->thd", pr, v)
         if gate is not None:
-            res[lo:hi] *= torch.sigmoid(gate[lo:hi].float())[:, :, None]
+            n = num_heads * head_dim if gate_elements else num_heads
+            res[lo:hi] *= torch.sigmoid(gate[lo:hi, gate_col:gate_col + n].float()).view(hi - lo, num_heads, -1)
     _store(out, res.reshape(T, num_heads * head_dim))
 
 
@@ -272,7 +278,18 @@ def _row_sum(y):
     return r + y.extra.float() if y.extra is not None else r
 
 
+def _pair_sum(y):
+    """sa * a + sb * b, each with its norm first if it has one."""
+    a, b = y.a.float(), y.b.float()
+    if y.norms is not None:
+        wa, wb, eps = y.norms
+        a, b = _norm_of(a, (wa, False, eps)), _norm_of(b, (wb, False, eps))
+    return y.sa * a + y.sb * b
+
+
 def norm_add_norm(x32, y, post, nxt, out, rows=None):
+    if hasattr(y, "sa"):                                 # two outputs side by side (kernels.WeightedPair)
+        y = _pair_sum(y)
     if hasattr(y, "place_of"):                           # a sum of rows (kernels.RowSum), taken in float32
         y = _row_sum(y)
     if y is not None:
@@ -366,6 +383,9 @@ def rope_norm_kv(proj, out, positions, denominators, rotary_dim, magnitude, inte
 
     def shape(x, weight):
         x = x.clone()
+        if int(norm) == 2:                               # the norm before the rotation
+            x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / norm_width + eps)
+            x = x * weight if weight is not None else x
         if rotary_dim:
             phi = positions.float()[:, None] / denominators[None, :]
             cos, sin = (torch.cos(phi) * magnitude)[:, None, :], (torch.sin(phi) * magnitude)[:, None, :]
@@ -375,7 +395,7 @@ def rope_norm_kv(proj, out, positions, denominators, rotary_dim, magnitude, inte
             a, b = x[..., first].clone(), x[..., second].clone()
             x[..., first] = a * cos - b * sin
             x[..., second] = b * cos + a * sin
-        if norm:
+        if int(norm) == 1:
             x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / norm_width + eps)
             if weight is not None:
                 x = x * weight
@@ -483,8 +503,8 @@ def moe_small_step(h, router, bias, top, scoring, correction, groups, keep, scal
     if bias is not None:
         logits = logits + bias
     ids = torch.empty((h.shape[0], top), dtype=torch.int32, device=h.device)
-    if scoring == "softmax_grouped":
-        moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights)
+    if scoring.endswith("_grouped"):
+        moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights, scoring)
     else:
         moe_route(logits, top, ids, weights, scoring)
     moe_sort(ids, router.shape[0], offsets, pair_at, place_of)
@@ -695,12 +715,14 @@ def gated_rmsnorm(y32, gate, gate_col, weight, eps, groups, gate_first, out, gat
 
 
 
-def moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights):
-    s = torch.softmax(logits.float(), dim=-1)
+def moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights, scoring="softmax_grouped"):
+    sigmoid = scoring == "sigmoid_grouped"
+    s = torch.sigmoid(logits.float()) if sigmoid else torch.softmax(logits.float(), dim=-1)
     T, E = s.shape
     choice = s + correction if correction is not None else s.clone()
     if keep < groups:
-        best = choice.view(T, groups, E // groups).max(dim=-1).values
+        each = torch.sort(choice.view(T, groups, E // groups), dim=-1, descending=True).values
+        best = each[..., :2].sum(-1) if sigmoid else each[..., 0]
         order = torch.sort(best, dim=-1, descending=True, stable=True).indices[:, :keep]
         kept = torch.zeros((T, groups), dtype=torch.bool, device=s.device)
         kept.scatter_(1, order, True)
@@ -708,7 +730,11 @@ def moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights
     chosen = torch.sort(choice, dim=-1, descending=True, stable=True).indices[:, :top]
     sc = torch.gather(s, 1, chosen)
     ids.copy_(chosen.to(torch.int32))
-    weights.copy_(sc / (sc.sum(-1, keepdim=True) + 1e-20) * scale)
+    weights.copy_(sc * scale if sigmoid else sc / (sc.sum(-1, keepdim=True) + 1e-20) * scale)
+
+
+def gelu_token_rows(z, table, col, ids, out):
+    _store(out, _gelu(z) * table[ids[:z.shape[0]].long(), col:col + z.shape[1]].float())
 
 
 def polynorm(z, coef, eps, out):
@@ -756,7 +782,7 @@ def delta_row_elements(dim):
 
 
 def delta_prepare(proj, col, b_col, conv_w, state, state_off, q_start, seq_of_token, slots, za, za_col, A_log, prep_qk, prep_g, v32, heads, kv_heads,
-                  dim, vdim, unit_eps=1e-6, shift=False):
+                  dim, vdim, unit_eps=1e-6, shift=False, a_col=0, dt_bias=None):
     T = proj.shape[0]
     C, taps = conv_w.shape
     DP = delta_row_elements(dim)
@@ -783,6 +809,12 @@ def delta_prepare(proj, col, b_col, conv_w, state, state_off, q_start, seq_of_to
     prep_qk[:, :, DP:DP + dim] = k
     prep_qk[:, :, 2 * DP] = (q * k).sum(-1)
     prep_g.zero_()
+    if za is None:                                        # one decay a head
+        a = torch.nn.functional.softplus(proj[:, a_col:a_col + heads].float() + dt_bias, threshold=1e9)
+        prep_g[:, :, 0] = torch.exp(-torch.exp(A_log) * a)
+        prep_g[:, :, 1] = torch.sigmoid(proj[:, b_col:b_col + heads].float())
+        v32.copy_(v)
+        return
     sp = torch.nn.functional.softplus(za[:, za_col:za_col + heads * dim].float(), threshold=1e9).view(T, heads, dim)
     prep_g[:, :, :dim] = torch.exp(-torch.exp(A_log)[None, :, None] * sp)
     prep_g[:, :, DP] = torch.sigmoid(proj[:, b_col:b_col + heads].float())
@@ -801,7 +833,7 @@ def delta_scan(prep_qk, prep_g, v32, state, q_start, slots, out32, heads, kv_hea
         for t in range(lo, hi):
             q = prep_qk[t, :, :dim].repeat_interleave(rep, dim=0)
             k = prep_qk[t, :, DP:DP + dim].repeat_interleave(rep, dim=0)
-            g, beta = prep_g[t, :, :dim], prep_g[t, :, DP]
+            g, beta = (prep_g[t, :, :dim], prep_g[t, :, DP]) if prep_g.shape[-1] > 4 else (prep_g[t, :, :1], prep_g[t, :, 1])
             v = v32[t].view(heads, vdim)
             S.mul_(g[:, :, None])
             u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", S, k))
@@ -898,7 +930,7 @@ def table_gather(resident, updates, slots, out, trash_page):
             out[s, b] = resident[slot, b] if b < cols else trash_page
 
 
-ALL = ["moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
+ALL = ["gelu_token_rows", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
        "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift", "ssm_scan",
        "decay_scan", "gated_rmsnorm", "table_gather", "gather_rows", "scale_inplace", "logit_cap", "rope_table", "linear_scaled_accepts", "linear_add_scaled_parts", "linear_add_scaled", "apply_row_scale", "linear_rope_kv", "interleave_gate_up", "embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add", "linear", "rope_kv_write",
        "paged_attention", "swiglu", "argmax", "sample"]
