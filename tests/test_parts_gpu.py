@@ -78,14 +78,17 @@ def test_rope_part_table_and_refusals():
     with pytest.raises(ValueError, match="pairing"):
         POSITIONS.build(PartSpec("rope", {"theta": 1e4, "rotary_dim": 16, "pairing": "quarters"}), "", torch.float32, DEV, head_dim=16)
     # pairs of neighbours are a pairing of the part; the paged attention part takes them in a kernel of their own behind the
-    # product, and refuses them together with what that kernel does not do (a convolution, a norm before the rotation)
+    # product (with a norm per head, and values of another size, if asked for), and refuses what that kernel does not do
     near = PartSpec("rope", {"theta": 1e4, "rotary_dim": 16, "pairing": "interleaved"})
     assert POSITIONS.build(near, "", torch.float32, DEV, head_dim=16).interleaved
     from litinfer_b200.parts import MIXERS
 
     sizes = {"hidden_size": 32, "num_heads": 2, "num_kv_heads": 1, "head_dim": 16, "scale": 0.25, "position": near}
     assert MIXERS.build(PartSpec("attention", sizes), "", torch.float32, DEV).rotate_apart
-    for more in ({"conv": 3}, {"qk_norm": {"q": "q.norm", "k": "k.norm", "eps": 1e-5}}, {"shared_kv": True}, {"value_dim": 32}):
+    per_head = {"q": "q.norm", "k": "k.norm", "eps": 1e-5}
+    for more in ({"qk_norm": per_head}, {"value_dim": 32}, {"norm_after": {"eps": 1e-5}}):
+        assert MIXERS.build(PartSpec("attention", dict(sizes, **more)), "", torch.float32, DEV).rotate_apart
+    for more in ({"conv": 3}, {"qk_norm": dict(per_head, whole=True)}, {"shared_kv": True}, {"qk_norm": per_head, "norm_after": {"eps": 1e-5}}):
         with pytest.raises(ValueError, match="pairs of neighbours"):
             MIXERS.build(PartSpec("attention", dict(sizes, **more)), "", torch.float32, DEV)
     with pytest.raises(ValueError, match="rotary_dim"):
