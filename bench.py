@@ -25,8 +25,8 @@ Weights (3 GB) are larger than L2, so nothing stays cached between steps.
 profiling runs and the summaries under ``profiles/``); ``mixed`` is a step of ``--batch`` requests decoding at
 ``--context`` beside a portion of ``--prefill-tokens`` prompt tokens.
 
-``--only design`` runs a design (``--design filasun|gorulorn|demavik|pifazen|zigolix``, default filasun) beside the Qwen2 model of equal layer sizes and layer count (``--design-shapes``,
-``--layers``, default 6): prefill of ``--prefill-tokens`` tokens and decode at batch 1, 8 and 32; ``--arch filasun|gorulorn|demavik|pifazen|zigolix`` puts
+``--only design`` runs a design (``--design filasun|gorulorn|demavik|pifazen|zigolix|bozolorn``, default filasun) beside the Qwen2 model of equal layer sizes and layer count (``--design-shapes``,
+``--layers``, default 6): prefill of ``--prefill-tokens`` tokens and decode at batch 1, 8 and 32; ``--arch filasun|gorulorn|demavik|pifazen|zigolix|bozolorn`` puts
 that design behind ``--only decode|prefill|kernels-decode|kernels-prefill`` (the kernel tables of ``profiles/``).
 
 ``--shape 1.5b|7b|14b`` chooses the layer sizes (default 1.5b, the headline; the other two are the larger workloads of
@@ -205,8 +205,33 @@ def zigolix_config(shape: str, layers: int, window: int = 1024):
             "loop": {"start": mid, "stop": min(layers, mid + 2), "times": 2}, "max_positions": d["max_position_embeddings"]}
 
 
+def bozolorn_config(shape: str, layers: int, chunk: int = 1024):
+    """A Bozolorn config.json with the layer sizes of a benchmark shape: every third layer attention in chunks (the last of them on
+    the keys and values of the first), the others rotated attention (blended frequencies, one more in the denominator) beside the
+    gated delta rule; mixtures of 8 experts of half the shape's feed-forward width in 4 groups of which 2 are kept, 2 choices a
+    token; a row of 128 (from a width of 2,048 on 256) elements per layer from the token."""
+    d = SHAPES[shape]
+    W, nh, nkv, dh, ff = d["hidden_size"], d["num_attention_heads"], d["num_key_value_heads"], d["head_dim"], d["intermediate_size"]
+    mlp = {"kind": "moe", "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}, "expert": {"ff": ff // 2, "limit": 7.0}}
+    left = {"heads": nh, "kv_heads": nkv, "dim": dh, "vdim": dh, "scale": dh ** -0.5,
+            "rot": {"base": 1e6, "dims": dh, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": nh, "kv_heads": nh // 2, "dim": dh, "vdim": dh, "conv": 4}
+    out, first = [], None
+    for i in range(layers):
+        if i % 3 != 2:
+            out.append({"type": "parallel", "mlp": mlp, "mixer": {"left": left, "right": right}})
+            continue
+        m = {"heads": nh, "kv_heads": nkv, "dim": dh, "vdim": dh, "scale": dh ** -0.5, "mask": {"size": chunk}}
+        if first is not None and i + 3 >= layers:
+            m["kv_from"] = first
+        first = i if first is None else first
+        out.append({"type": "attention", "mlp": mlp, "mixer": m})
+    return {"architecture": "Bozolorn", "vocab": d["vocab_size"], "width": W, "norm": {"eps": 1e-6}, "embedding": {"scale": W ** 0.5},
+            "token_side": {"dim": 128 if W < 2048 else 256}, "layers": out, "max_positions": 32768}
+
+
 # the designs that run beside Qwen2: config.json with the layer sizes of a shape, for a count of layers
-DESIGNS = {"filasun": filasun_config, "gorulorn": gorulorn_config, "demavik": demavik_config, "pifazen": pifazen_config, "zigolix": zigolix_config}
+DESIGNS = {"filasun": filasun_config, "gorulorn": gorulorn_config, "demavik": demavik_config, "pifazen": pifazen_config, "zigolix": zigolix_config, "bozolorn": bozolorn_config}
 
 
 def design_layer_runs(cfg) -> int:
@@ -215,7 +240,7 @@ def design_layer_runs(cfg) -> int:
 
 
 def time_design(args, peaks):
-    """Prefill and decode of a design (``--design filasun|gorulorn|demavik|pifazen|zigolix``) beside the Qwen2 model of the same layer sizes and as
+    """Prefill and decode of a design (``--design filasun|gorulorn|demavik|pifazen|zigolix|bozolorn``) beside the Qwen2 model of the same layer sizes and as
     many layers as the design runs (random weights), through the same step function: tokens per second, and the
     milliseconds behind them."""
     import torch

@@ -206,8 +206,10 @@ __device__ __forceinline__ void row_norm(float (&dst)[kRegs], const float (&v)[k
     for (int k = 0; k < kRegs; ++k) dst[k] = (v[k] - mean) * rinv * wv[k];
 }
 
-template <typename T, bool kVec>
-__global__ void norm_add_norm_regs_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w_post, int post_centered,
+// kPair: the sublayer's output is a sum of two, each with a norm of its own or as it is.
+template <typename T, bool kVec, bool kPair>
+__global__ void __launch_bounds__(1024)
+norm_add_norm_regs_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w_post, int post_centered,
                                           float eps_post, const float* __restrict__ w_next, int next_centered, float eps_next,
                                           T* __restrict__ out, const int* __restrict__ rows, int n_src, int H,
                                           const int* __restrict__ y_places, int y_top, const float* __restrict__ y_weights,
@@ -249,7 +251,7 @@ __global__ void norm_add_norm_regs_kernel(float* __restrict__ x, const T* __rest
         } else {
             load_row<kVec>(yv, y + (size_t)r * H, H);
         }
-        if (y2) {
+        if constexpr (kPair) {
             // two outputs side by side (two mixers): their weighted sum, each divided by its root mean square first if it has a weight
             float other[kRegs];
             load_row<kVec>(other, y2 + (size_t)r * H, H);
@@ -399,8 +401,8 @@ LI_EXPORT int li_norm_add_norm(float* x, const void* y, int dtype, const float* 
         // 16-byte moves where every row starts on such a boundary
         const bool vec = H % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)y_extra % 16) == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)y2 % 16) == 0 && ((uintptr_t)w_first % 16) == 0 &&
                          ((uintptr_t)w_second % 16) == 0 && ((uintptr_t)w_post % 16) == 0 && ((uintptr_t)w_next % 16) == 0;
-#define LI_NORM_LAUNCH(TT, VEC)                                                                                                                  \
-    e = li_launch_pdl(norm_add_norm_regs_kernel<TT, VEC>, dim3(R), dim3(threads), 0, stream, x, (const TT*)y, w_post, post_centered, eps_post, w_next, \
+#define LI_NORM_LAUNCH(TT, VEC)                                                                                                                \
+    e = li_launch_pdl(y2 ? norm_add_norm_regs_kernel<TT, VEC, true> : norm_add_norm_regs_kernel<TT, VEC, false>, dim3(R), dim3(threads), 0, stream, x, (const TT*)y, w_post, post_centered, eps_post, w_next, \
                       next_centered, eps_next, (TT*)out, rows, n_src, H, y_places, y_top, y_weights, (const TT*)y_extra, (const TT*)y2, s1, s2, w_first, \
                       w_second, eps_pair)
         if (dtype == LI_F32) {
