@@ -1,0 +1,525 @@
+// The gated delta rule with one decay a head, for long portions: chunks of 64 tokens as matrix products in float.
+//
+// Per head, with g_t the token's decay, beta_t its step size, and S [d, dv] the state before the chunk:
+//     S_t = g_t S_(t-1) + k_t u_t^T,   u_t = beta_t (v_t - g_t S_(t-1)^T k_t),   o_t = S_t^T q_t.
+// With c_t = g_1 ... g_t inside the chunk, unrolling S_t gives  u_t = beta_t (v_t - c_t S^T k_t - sum_(s<t) (c_t / c_s) (k_t . k_s) u_s),
+// a triangular system: (I + A) U = diag(beta) V - diag(beta c) K S with A_ts = beta_t (c_t / c_s) (k_t . k_s), s < t.  So
+//     U = X - W S,   X = (I + A)^-1 diag(beta) V,   W = (I + A)^-1 diag(beta c) K      (X, W: nothing of the state),
+//     O = diag(c) Q S + P U,   P_ts = (c_t / c_s) (q_t . k_s), s <= t,
+//     S <- c_C S + K^T diag(c_C / c_t) U.
+// Three kernels over what li_delta_prepare made (recurrent.cu):
+//   * delta_chunk_solve: every chunk and head by itself: A, P, and the two triangular solves, a thread a column;
+//   * delta_chunk_carry: the chunks of a sequence in order, for a head and 16 columns of the values: U, the state before every
+//     chunk, and the sequence's last state back into its slot.  The only part that walks, and it walks chunks;
+//   * delta_chunk_output: every chunk and head by itself: O, with the norm over the head, its weight and the silu gate.
+// Ratios of decays are exponentials of differences of summed logarithms (double), so nothing overflows however fast a head forgets.
+// Everything is float on the multiply-add pipes; the results differ from the walk's by rounding.
+#include "common.cuh"
+
+namespace {
+
+constexpr int kC = 64;              // tokens of a chunk
+constexpr int kLA = kC + 4;         // a row of a [.., tokens] tile in shared memory
+constexpr int kThreads = 256;
+constexpr int kSlice = 16;          // value columns a block of the carry takes
+constexpr int kCols = 128;          // value columns a block of the output takes at a time
+constexpr int kRowsB = 32;          // rows of its second operand that it stages at a time
+
+__device__ __forceinline__ void copy16(float* dst, const float* src, bool valid) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+    const int bytes = valid ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(bytes));
+}
+__device__ __forceinline__ void copies_done() { asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory"); }
+
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float dot4(float4 a, float4 b, float c) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, c)))); }
+
+template <int DP>
+__host__ __device__ constexpr size_t solve_smem() { return ((size_t)2 * kC * (DP + 4) + 2 * kC * kLA + 4 * kC) * sizeof(float); }
+
+// prep_qk [T, kv_heads, 2 DP + 4] (q | k | k . q), prep_g [T, heads, 4] (g | beta | log g), v [T, heads dv]; seg: a chunk's first token,
+// end, number, slot.  Out, per chunk and head: wt [d, 64] and xt [dv, 64] (W and X transposed), pt [64, 64] (P transposed), sums [2, 64] (c_t, and c_64 / c_t).
+template <int DP>
+__global__ void __launch_bounds__(kThreads, DP <= 128 ? 2 : 1)
+delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restrict__ prep_g, const float* __restrict__ v, const int4* __restrict__ seg,
+                         float* __restrict__ wt, float* __restrict__ xt, float* __restrict__ pt, float* __restrict__ sums, int heads, int kv_heads, int d,
+                         int dv) {
+    constexpr int LD = DP + 4, RQ = 2 * DP + 4;
+    extern __shared__ __align__(16) float smem[];
+    float* Ks = smem;                       // [64][LD]
+    float* Qs = Ks + kC * LD;
+    float* At = Qs + kC * LD;               // [s][t]
+    float* Ps = At + kC * kLA;              // [s][t]
+    float* cum = Ps + kC * kLA;             // [64] log(c_t), as a sum of two floats: heads that forget at once reach hundreds, and
+    float* low = cum + kC;                  //      what counts are differences
+    float* beta = low + kC;
+    float* bc = beta + kC;                  // beta_t c_t
+    pdl_wait();
+    const int h = blockIdx.x, hk = h / (heads / kv_heads);
+    const int4 sg = seg[blockIdx.y];
+    const int q0 = sg.x, n = min(sg.y - sg.x, kC);
+    const size_t unit = (size_t)sg.z * heads + h;
+    const int tid = threadIdx.x, lane = tid & 31;
+    for (int idx = tid; idx < kC * (DP / 4); idx += kThreads) {
+        const int t = idx / (DP / 4), i = idx - t * (DP / 4);
+        const float* row = prep_qk + ((size_t)(q0 + (t < n ? t : 0)) * kv_heads + hk) * RQ + 4 * i;
+        copy16(Qs + t * LD + 4 * i, row, t < n);
+        copy16(Ks + t * LD + 4 * i, row + DP, t < n);
+    }
+    if (tid < 32) {
+        double a[2];
+        float b[2];
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int t = lane + 32 * j;
+            const float4 g = t < n ? ld4(prep_g + ((size_t)(q0 + t) * heads + h) * 4) : make_float4(1.0f, 0.0f, 0.0f, 0.0f);
+            a[j] = (double)g.z;
+            b[j] = g.y;
+        }
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double x = __shfl_up_sync(0xffffffffu, a[0], o), y = __shfl_up_sync(0xffffffffu, a[1], o);
+            if (lane >= o) a[0] += x, a[1] += y;
+        }
+        a[1] += __shfl_sync(0xffffffffu, a[0], 31);
+        const double end = __shfl_sync(0xffffffffu, a[1], 31);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int t = lane + 32 * j;
+            const float c = expf((float)a[j]);
+            cum[t] = (float)a[j];
+            low[t] = (float)(a[j] - (double)(float)a[j]);
+            beta[t] = b[j];
+            bc[t] = b[j] * c;
+            sums[(unit * 2) * kC + t] = c;
+            sums[(unit * 2 + 1) * kC + t] = expf((float)(end - a[j]));
+        }
+    }
+    copies_done();
+    __syncthreads();
+    // the products of keys with keys and of queries with keys: a thread takes tokens ty + 16 i against ty's of tx + 16 j, j <= i
+    {
+        const int tx = tid & 15, ty = tid >> 4;
+        const int blocks = (n + 15) >> 4;
+        float kk[4][4], qk[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = 0.0f;
+#pragma unroll 2
+        for (int k = 0; k < DP; k += 4) {
+            float4 col[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) col[j] = ld4(Ks + (tx + 16 * j) * LD + k);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (i < blocks) {
+                    const float4 kr = ld4(Ks + (ty + 16 * i) * LD + k), qr = ld4(Qs + (ty + 16 * i) * LD + k);
+#pragma unroll
+                    for (int j = 0; j <= i; ++j) {
+                        kk[i][j] = dot4(kr, col[j], kk[i][j]);
+                        qk[i][j] = dot4(qr, col[j], qk[i][j]);
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int t = ty + 16 * i, s = tx + 16 * j;
+                const float f = s <= t ? expf((cum[t] - cum[s]) + (low[t] - low[s])) : 0.0f;
+                At[s * kLA + t] = s < t ? beta[t] * f * kk[i][j] : 0.0f;
+                Ps[s * kLA + t] = f * qk[i][j];
+            }
+    }
+    __syncthreads();
+    for (int idx = tid; idx < kC * (kC / 4); idx += kThreads) {
+        const int s = idx / (kC / 4), i = idx - s * (kC / 4);
+        *reinterpret_cast<float4*>(pt + (unit * kC + s) * kC + 4 * i) = ld4(Ps + s * kLA + 4 * i);
+    }
+    // the triangular solves, a column a thread: as soon as x_s is known it is taken off the rows behind it
+    for (int c = tid; c < d + dv; c += kThreads) {
+        float x[kC];
+        if (c < d) {
+#pragma unroll
+            for (int t = 0; t < kC; ++t) x[t] = bc[t] * Ks[t * LD + c];
+        } else {
+            const float* col = v + (size_t)q0 * heads * dv + (size_t)h * dv + (c - d);
+#pragma unroll
+            for (int t = 0; t < kC; ++t) x[t] = t < n ? beta[t] * col[(size_t)t * heads * dv] : 0.0f;
+        }
+#pragma unroll
+        for (int s8 = 0; s8 < kC; s8 += 8) {
+            if (s8 < n) {
+#pragma unroll
+                for (int s = s8; s < s8 + 8; ++s) {
+#pragma unroll
+                    for (int t4 = (s + 1) / 4 * 4; t4 < kC; t4 += 4) {
+                        const float4 a = ld4(At + s * kLA + t4);         // (zeros where t <= s)
+                        x[t4] = fmaf(-a.x, x[s], x[t4]);
+                        x[t4 + 1] = fmaf(-a.y, x[s], x[t4 + 1]);
+                        x[t4 + 2] = fmaf(-a.z, x[s], x[t4 + 2]);
+                        x[t4 + 3] = fmaf(-a.w, x[s], x[t4 + 3]);
+                    }
+                }
+            }
+        }
+        float* out = c < d ? wt + (unit * d + c) * kC : xt + (unit * dv + (c - d)) * kC;
+#pragma unroll
+        for (int t = 0; t < kC; t += 4) *reinterpret_cast<float4*>(out + t) = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
+    }
+    pdl_launch_dependents();
+}
+
+template <int DP>
+__host__ __device__ constexpr int carry_buffers() { return DP <= 128 ? 2 : 1; }
+template <int DP>
+__host__ __device__ constexpr int carry_buffer() { return DP * kC + kC * DP + kSlice * kC + 2 * kC; }
+template <int DP>
+__host__ __device__ constexpr int carry_scratch() { return 4 * kC * kSlice > (kThreads / DP - 1) * DP * kSlice ? 4 * kC * kSlice : (kThreads / DP - 1) * DP * kSlice; }
+template <int DP>
+__host__ __device__ constexpr size_t carry_smem() {
+    return ((size_t)carry_buffers<DP>() * carry_buffer<DP>() + DP * kSlice + carry_scratch<DP>() + kC * kSlice) * sizeof(float);
+}
+
+// runs: triples (first chunk, chunks, slot).  s0 [chunk, head, d, dv]: the state before every chunk; u [chunk, head, 64, dv].
+template <int DP>
+__global__ void __launch_bounds__(kThreads)
+delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restrict__ seg, const int* __restrict__ runs, const float* __restrict__ wt,
+                         const float* __restrict__ xt, const float* __restrict__ sums, float* __restrict__ state, long long state_stride,
+                         float* __restrict__ s0, float* __restrict__ u, int heads, int kv_heads, int d, int dv) {
+    constexpr int RQ = 2 * DP + 4, NB = carry_buffers<DP>(), SPLIT = kThreads / DP;
+    extern __shared__ __align__(16) float smem[];
+    float* S = smem + NB * carry_buffer<DP>();          // [DP][16]
+    float* red = S + DP * kSlice;
+    float* Us = red + carry_scratch<DP>();              // [64][16]: U with the decay to the chunk's end
+    const int tid = threadIdx.x;
+    const int h = blockIdx.y, hk = h / (heads / kv_heads), c0 = blockIdx.x * kSlice;
+    pdl_wait();
+    const int first = runs[3 * blockIdx.z], count = runs[3 * blockIdx.z + 1], slot = runs[3 * blockIdx.z + 2];
+    float* st = state + (size_t)slot * state_stride + (size_t)h * dv * d;
+    auto stage = [&](int b, int chunk) {
+        float* W = smem + b * carry_buffer<DP>();       // [DP][64]
+        float* Kb = W + DP * kC;                        // [64][DP]
+        float* X = Kb + kC * DP;                        // [16][64]
+        float* cm = X + kSlice * kC;                    // [2][64]
+        const int4 sg = seg[chunk];
+        const int n = min(sg.y - sg.x, kC);
+        const size_t unit = (size_t)chunk * heads + h;
+        for (int idx = tid; idx < DP * (kC / 4); idx += kThreads) {
+            const int k = idx / (kC / 4), i = idx - k * (kC / 4);
+            copy16(W + k * kC + 4 * i, wt + (unit * d + (k < d ? k : 0)) * kC + 4 * i, k < d);
+        }
+        for (int idx = tid; idx < kC * (DP / 4); idx += kThreads) {
+            const int t = idx / (DP / 4), i = idx - t * (DP / 4);
+            copy16(Kb + t * DP + 4 * i, prep_qk + ((size_t)(sg.x + (t < n ? t : 0)) * kv_heads + hk) * RQ + DP + 4 * i, t < n);
+        }
+        if (tid < kSlice * (kC / 4)) {
+            const int c = tid / (kC / 4), i = tid - c * (kC / 4);
+            copy16(X + c * kC + 4 * i, xt + (unit * dv + (c0 + c < dv ? c0 + c : 0)) * kC + 4 * i, c0 + c < dv);
+        }
+        if (tid < 2 * kC / 4) copy16(cm + 4 * tid, sums + unit * 2 * kC + 4 * tid, true);
+    };
+    stage(0, first);
+    for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
+        const int c = idx / DP, k = idx - c * DP;
+        S[k * kSlice + c] = (k < d && c0 + c < dv) ? st[(size_t)(c0 + c) * d + k] : 0.0f;
+    }
+    const bool vec = (dv & 3) == 0;
+    for (int j = 0; j < count; ++j) {
+        const int chunk = first + j, b = j % NB;
+        copies_done();
+        __syncthreads();                                 // this chunk's rows are here, and everybody has left the other buffer
+        if (NB > 1 && j + 1 < count) stage(b ^ 1, chunk + 1);
+        const float* W = smem + b * carry_buffer<DP>();
+        const float* Kb = W + DP * kC;
+        const float* X = Kb + kC * DP;
+        const float* cm = X + kSlice * kC;
+        const size_t unit = (size_t)chunk * heads + h;
+        // the state before this chunk, for the outputs
+        for (int idx = tid; idx < d * (kSlice / 4); idx += kThreads) {
+            const int k = idx / (kSlice / 4), c = 4 * (idx - k * (kSlice / 4));
+            const float4 val = ld4(S + k * kSlice + c);
+            float* to = s0 + (unit * d + k) * dv + c0 + c;
+            if (vec) {
+                if (c0 + c < dv) *reinterpret_cast<float4*>(to) = val;
+            } else {
+                const float e[4] = {val.x, val.y, val.z, val.w};
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (c0 + c + q < dv) to[q] = e[q];
+            }
+        }
+        // W S: four tokens by four columns a thread, a quarter of the key channels each
+        {
+            const int part = tid >> 6, ct = tid & 3, tt = (tid & 63) >> 2;
+            float acc[4][4];
+#pragma unroll
+            for (int a = 0; a < 4; ++a)
+#pragma unroll
+                for (int q = 0; q < 4; ++q) acc[a][q] = 0.0f;
+#pragma unroll 8
+            for (int k = part * (DP / 4); k < (part + 1) * (DP / 4); ++k) {
+                const float4 w = ld4(W + k * kC + 4 * tt), s = ld4(S + k * kSlice + 4 * ct);
+                const float wa[4] = {w.x, w.y, w.z, w.w}, sa[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+                for (int a = 0; a < 4; ++a)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) acc[a][q] = fmaf(wa[a], sa[q], acc[a][q]);
+            }
+#pragma unroll
+            for (int a = 0; a < 4; ++a)
+                *reinterpret_cast<float4*>(red + (part * kC + 4 * tt + a) * kSlice + 4 * ct) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+        }
+        __syncthreads();
+        {
+            const int t = tid >> 2, c = 4 * (tid & 3);
+            float4 sum = ld4(red + t * kSlice + c);
+#pragma unroll
+            for (int part = 1; part < 4; ++part) {
+                const float4 p = ld4(red + (part * kC + t) * kSlice + c);
+                sum.x += p.x, sum.y += p.y, sum.z += p.z, sum.w += p.w;
+            }
+            const float4 val = make_float4(X[c * kC + t] - sum.x, X[(c + 1) * kC + t] - sum.y, X[(c + 2) * kC + t] - sum.z, X[(c + 3) * kC + t] - sum.w);
+            float* to = u + (unit * kC + t) * dv + c0 + c;
+            if (vec) {
+                if (c0 + c < dv) *reinterpret_cast<float4*>(to) = val;
+            } else {
+                const float e[4] = {val.x, val.y, val.z, val.w};
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (c0 + c + q < dv) to[q] = e[q];
+            }
+            const float f = cm[kC + t];
+            *reinterpret_cast<float4*>(Us + t * kSlice + c) = make_float4(f * val.x, f * val.y, f * val.z, f * val.w);
+        }
+        __syncthreads();
+        // the state behind the chunk: four key channels by four columns a thread, a part of the tokens each
+        {
+            const int part = tid / DP, tile = tid - part * DP, ct = tile & 3, kt = tile >> 2;
+            float acc[4][4];
+#pragma unroll
+            for (int a = 0; a < 4; ++a)
+#pragma unroll
+                for (int q = 0; q < 4; ++q) acc[a][q] = 0.0f;
+#pragma unroll 8
+            for (int t = part * (kC / SPLIT); t < (part + 1) * (kC / SPLIT); ++t) {
+                const float4 k = ld4(Kb + t * DP + 4 * kt), w = ld4(Us + t * kSlice + 4 * ct);
+                const float ka[4] = {k.x, k.y, k.z, k.w}, ua[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+                for (int a = 0; a < 4; ++a)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) acc[a][q] = fmaf(ka[a], ua[q], acc[a][q]);
+            }
+            if (SPLIT > 1) {
+                if (part > 0) {
+#pragma unroll
+                    for (int a = 0; a < 4; ++a)
+                        *reinterpret_cast<float4*>(red + ((part - 1) * DP + 4 * kt + a) * kSlice + 4 * ct) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+                }
+                __syncthreads();
+            }
+            if (part == 0) {
+                const float f = cm[kC - 1];
+#pragma unroll
+                for (int a = 0; a < 4; ++a) {
+                    float* row = S + (4 * kt + a) * kSlice + 4 * ct;
+                    float4 s = ld4(row);
+                    float4 sum = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+#pragma unroll
+                    for (int p = 0; p < SPLIT - 1; ++p) {
+                        const float4 r = ld4(red + (p * DP + 4 * kt + a) * kSlice + 4 * ct);
+                        sum.x += r.x, sum.y += r.y, sum.z += r.z, sum.w += r.w;
+                    }
+                    s.x = fmaf(f, s.x, sum.x), s.y = fmaf(f, s.y, sum.y), s.z = fmaf(f, s.z, sum.z), s.w = fmaf(f, s.w, sum.w);
+                    *reinterpret_cast<float4*>(row) = s;
+                }
+            }
+        }
+        __syncthreads();
+        if (NB == 1 && j + 1 < count) stage(0, chunk + 1);
+    }
+    pdl_launch_dependents();
+    for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
+        const int c = idx / DP, k = idx - c * DP;
+        if (k < d && c0 + c < dv) st[(size_t)(c0 + c) * d + k] = S[k * kSlice + c];
+    }
+}
+
+template <int DP>
+__host__ __device__ constexpr size_t output_smem() { return ((size_t)(DP + kC) * kLA + 2 * kRowsB * kCols) * sizeof(float); }
+
+// o = diag(c) Q S + P U as one product over d + 64 rows.  norm_w given (dv at most 128): y = o / sqrt(mean(o^2) + eps) * norm_w * silu(gate),
+// in the run dtype; else out takes o as it is.
+template <typename T, int DP>
+__global__ void __launch_bounds__(kThreads, 2)
+delta_chunk_output_kernel(const float* __restrict__ prep_qk, const int4* __restrict__ seg, const float* __restrict__ pt, const float* __restrict__ sums,
+                          const float* __restrict__ s0, const float* __restrict__ u, float* __restrict__ out, const T* __restrict__ gate, int gate_ld,
+                          int gate_off, const float* __restrict__ norm_w, float eps, T* __restrict__ y, int heads, int kv_heads, int d, int dv) {
+    constexpr int RQ = 2 * DP + 4;
+    extern __shared__ __align__(16) float smem[];
+    float* At = smem;                        // [DP + 64][68]: rows of Q^T with the decay, then of P^T
+    float* B = At + (DP + kC) * kLA;         // [2][32][128]
+    pdl_wait();
+    const int h = blockIdx.x, hk = h / (heads / kv_heads);
+    const int4 sg = seg[blockIdx.y];
+    const int q0 = sg.x, n = min(sg.y - sg.x, kC);
+    const size_t unit = (size_t)sg.z * heads + h;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, t0 = 8 * warp;
+    const bool vec = (dv & 3) == 0;
+    constexpr int kBlocks = DP / kRowsB + kC / kRowsB;
+    auto stage = [&](int b, int kb, int cb) {
+        for (int idx = tid; idx < kRowsB * (kCols / 4); idx += kThreads) {
+            const int r = idx / (kCols / 4), c = 4 * (idx - r * (kCols / 4));
+            const int k = kb * kRowsB + r, col = cb + c;
+            const bool from_state = k < DP;
+            const bool row_ok = from_state ? k < d : true;
+            const float* row = from_state ? s0 + (unit * d + (row_ok ? k : 0)) * dv : u + (unit * kC + (k - DP)) * dv;
+            float* dst = B + (b * kRowsB + r) * kCols + c;
+            if (vec) {
+                copy16(dst, row + (col < dv ? col : 0), row_ok && col < dv);
+            } else {
+#pragma unroll
+                for (int q = 0; q < 4; ++q) dst[q] = (row_ok && col + q < dv) ? row[col + q] : 0.0f;
+            }
+        }
+    };
+    stage(0, 0, 0);
+    for (int idx = tid; idx < kC * (DP / 4); idx += kThreads) {
+        const int i = idx / kC, t = idx - i * kC;
+        float4 q = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (t < n) {
+            q = ld4(prep_qk + ((size_t)(q0 + t) * kv_heads + hk) * RQ + 4 * i);
+            const float f = sums[unit * 2 * kC + t];
+            q.x *= f, q.y *= f, q.z *= f, q.w *= f;
+        }
+        float* to = At + 4 * i * kLA + t;
+        to[0] = q.x, to[kLA] = q.y, to[2 * kLA] = q.z, to[3 * kLA] = q.w;
+    }
+    for (int idx = tid; idx < kC * (kC / 4); idx += kThreads) {
+        const int s = idx / (kC / 4), i = idx - s * (kC / 4);
+        copy16(At + (DP + s) * kLA + 4 * i, pt + (unit * kC + s) * kC + 4 * i, true);
+    }
+    for (int cb = 0; cb < dv; cb += kCols) {
+        float acc[8][4];
+#pragma unroll
+        for (int a = 0; a < 8; ++a)
+#pragma unroll
+            for (int q = 0; q < 4; ++q) acc[a][q] = 0.0f;
+        for (int kb = 0; kb < kBlocks; ++kb) {
+            const int b = kb & 1;
+            copies_done();
+            __syncthreads();
+            if (kb + 1 < kBlocks) stage(b ^ 1, kb + 1, cb);
+            // (rows of P^T: a token sees those up to its own; tokens behind the portion's end see nothing)
+            const bool some = t0 < n && (kb * kRowsB < DP || kb * kRowsB - DP <= t0 + 7);
+            if (some) {
+#pragma unroll 4
+                for (int r = 0; r < kRowsB; ++r) {
+                    const float* at = At + (kb * kRowsB + r) * kLA + t0;
+                    const float4 a0 = ld4(at), a1 = ld4(at + 4), bv = ld4(B + (b * kRowsB + r) * kCols + 4 * lane);
+                    const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w}, bb[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+                    for (int a = 0; a < 8; ++a)
+#pragma unroll
+                        for (int q = 0; q < 4; ++q) acc[a][q] = fmaf(av[a], bb[q], acc[a][q]);
+                }
+            }
+        }
+        const int col = cb + 4 * lane;
+#pragma unroll
+        for (int a = 0; a < 8; ++a) {
+            const int t = t0 + a;
+            if (t >= n) break;                                     // (the same for the whole warp)
+            if (norm_w) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int q = 0; q < 4; ++q) ss = fmaf(acc[a][q], acc[a][q], ss);           // (zeros behind the last column)
+                const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
+                const T* gr = gate + (size_t)(q0 + t) * gate_ld + gate_off + (size_t)h * dv + col;
+                T* to = y + (size_t)(q0 + t) * heads * dv + (size_t)h * dv + col;
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (col + q < dv) {
+                        const float g = to_float(gr[q]);
+                        to[q] = from_float<T>(acc[a][q] * rinv * norm_w[h * dv + col + q] * (g / (1.0f + expf(-g))));
+                    }
+            } else {
+                float* to = out + (size_t)(q0 + t) * heads * dv + (size_t)h * dv + col;
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (col + q < dv) to[q] = acc[a][q];
+            }
+        }
+        __syncthreads();                                           // everybody has left the last rows staged
+        if (cb + kCols < dv) stage(0, 0, cb + kCols);
+    }
+    pdl_launch_dependents();
+}
+
+template <typename K>
+int raise_smem(K kernel, size_t bytes, const char* what) {
+    if (bytes <= 48 * 1024) return 0;
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+    return e == cudaSuccess ? 0 : li_fail("%s: cannot raise shared memory to %zu: %s", what, bytes, cudaGetErrorString(e));
+}
+
+template <int DP>
+int launch(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* seg, int chunks, const int* runs,
+           int nruns, float* wt, float* xt, float* pt, float* sums, float* s0, float* u, float* out, const void* gate, int dtype, int gate_ld, int gate_off,
+           const float* norm_w, float eps, void* y, int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
+    static bool raised = false;
+    if (!raised) {
+        if (int rc = raise_smem(delta_chunk_solve_kernel<DP>, solve_smem<DP>(), "delta chunks")) return rc;
+        if (int rc = raise_smem(delta_chunk_carry_kernel<DP>, carry_smem<DP>(), "delta chunks")) return rc;
+        if (int rc = raise_smem(delta_chunk_output_kernel<float, DP>, output_smem<DP>(), "delta chunks")) return rc;
+        if (int rc = raise_smem(delta_chunk_output_kernel<bf16, DP>, output_smem<DP>(), "delta chunks")) return rc;
+        raised = true;
+    }
+    cudaError_t e = li_launch_pdl(delta_chunk_solve_kernel<DP>, dim3(heads, chunks), dim3(kThreads), solve_smem<DP>(), stream, prep_qk, prep_g, v, (const int4*)seg,
+                                  wt, xt, pt, sums, heads, kv_heads, d, dv);
+    if (e == cudaSuccess)
+        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, dim3(ceil_div(dv, kSlice), heads, nruns), dim3(kThreads), carry_smem<DP>(), stream, prep_qk,
+                          (const int4*)seg, runs, wt, xt, sums, state, state_stride, s0, u, heads, kv_heads, d, dv);
+    if (e == cudaSuccess) {
+        if (dtype == LI_F32)
+            e = li_launch_pdl(delta_chunk_output_kernel<float, DP>, dim3(heads, chunks), dim3(kThreads), output_smem<DP>(), stream, prep_qk, (const int4*)seg, pt,
+                              sums, s0, u, out, (const float*)gate, gate_ld, gate_off, norm_w, eps, (float*)y, heads, kv_heads, d, dv);
+        else
+            e = li_launch_pdl(delta_chunk_output_kernel<bf16, DP>, dim3(heads, chunks), dim3(kThreads), output_smem<DP>(), stream, prep_qk, (const int4*)seg, pt,
+                              sums, s0, u, out, (const bf16*)gate, gate_ld, gate_off, norm_w, eps, (bf16*)y, heads, kv_heads, d, dv);
+    }
+    if (e != cudaSuccess) return li_fail("delta chunks: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("delta chunks");
+}
+
+}  // namespace
+
+// seg [chunks] quadruples (first token, end, chunk, slot), at most 64 tokens each; runs [nruns] triples (first chunk, chunks, slot).
+// Workspace, float: wt [chunks, heads, d, 64], xt [chunks, heads, dv, 64], pt [chunks, heads, 64, 64], sums [chunks, heads, 2, 64],
+// s0 [chunks, heads, d, dv], u [chunks, heads, 64, dv].  norm_w [heads dv] (may be NULL; dv at most 128): y [T, heads dv] in the run dtype takes
+// the normed and gated outputs, gate [T, gate_ld] from column gate_off; without it out [T, heads dv] float takes the outputs.
+LI_EXPORT int li_delta_chunks(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* seg, int chunks,
+                              const int* runs, int nruns, float* wt, float* xt, float* pt, float* sums, float* s0, float* u, float* out, const void* gate,
+                              int dtype, int gate_ld, int gate_off, const float* norm_w, float eps, void* y, int heads, int kv_heads, int d, int dv,
+                              cudaStream_t stream) {
+    LI_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && d > 0 && d <= 256 && dv > 0, "delta chunks: %d heads on %d key heads of %d x %d (keys of at most 256)",
+               heads, kv_heads, d, dv);
+    LI_REQUIRE(chunks >= 0 && nruns >= 0 && chunks <= 65535 && nruns <= 65535 && heads <= 65535, "delta chunks: %d chunks of %d sequences in one launch", chunks, nruns);
+    LI_REQUIRE(norm_w != nullptr ? (dv <= kCols && y != nullptr && gate != nullptr && gate_off >= 0 && gate_off + heads * dv <= gate_ld) : out != nullptr,
+               "delta chunks: outputs of %d columns a head, gate at column %d of %d", dv, gate_off, gate_ld);
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "delta chunks: unknown dtype %d", dtype);
+    LI_REQUIRE(((uintptr_t)prep_qk | (uintptr_t)prep_g | (uintptr_t)seg | (uintptr_t)wt | (uintptr_t)xt | (uintptr_t)pt | (uintptr_t)sums | (uintptr_t)s0 | (uintptr_t)u) % 16 == 0,
+               "delta chunks: an operand is not on a 16-byte boundary");
+    if (chunks == 0 || nruns == 0) return 0;
+#define LI_CHUNKS(DP)                                                                                                                                  \
+    return launch<DP>(prep_qk, prep_g, v, state, state_stride, seg, chunks, runs, nruns, wt, xt, pt, sums, s0, u, out, gate, dtype, gate_ld, gate_off, norm_w, eps, \
+                      y, heads, kv_heads, d, dv, stream)
+    if (d <= 32) LI_CHUNKS(32);
+    if (d <= 64) LI_CHUNKS(64);
+    if (d <= 128) LI_CHUNKS(128);
+    LI_CHUNKS(256);
+#undef LI_CHUNKS
+}

@@ -193,7 +193,7 @@ int li_gla_scan(const void* qkv, int dtype, int stride, int q_off, int k_off, in
  * g = exp(-exp(A_log[h]) softplus(za [T, za_stride] at za_off + h d + i)) and beta = sigmoid(proj[b_off + h]) into prep_g
  * [T, heads, DP + 4]; v [T, heads dv]; all float, DP = 32, 64, 128 or 256 (the first that holds d).  shift: every sequence has
  * one token and the convolution's state moves on here.  za NULL: one decay a head, g = exp(-exp(A_log[h]) softplus(proj[a_off + h] +
- * dt_bias[h])), prep_g [T, heads, 4] = (g | beta | unused), and per_head for the walk.  li_delta_scan walks; head h uses key head h / (heads / kv_heads); the
+ * dt_bias[h])), prep_g [T, heads, 4] = (g | beta | log g | 0), and per_head for the walk.  li_delta_scan walks; head h uses key head h / (heads / kv_heads); the
  * state is kept as [heads][dv][d]. */
 int li_delta_prepare(const void* proj, int dtype, int stride, int col0, int b_off, const float* conv_w, int taps,
     float* state, long long state_stride, long long state_off, const int* q_start, const int* seq_of_token, const int*
@@ -204,6 +204,16 @@ void li_delta_force_columns(int columns);   /* 0: columns a warp of the walk by 
 int li_delta_scan(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride,
     const int* q_start, const int* slots, float* out, int S, int heads, int kv_heads, int d, int dv, int per_head,
     cudaStream_t stream);
+
+/* The same rule with one decay a head for long portions, in chunks of at most 64 tokens as matrix products in float (delta_chunks.cu):
+ * seg [chunks] quadruples (first token, end, chunk, slot), runs [nruns] triples (first chunk, chunks, slot).  Workspace, float: wt
+ * [chunks, heads, d, 64], xt [chunks, heads, dv, 64], pt [chunks, heads, 64, 64], sums [chunks, heads, 2, 64], s0 [chunks, heads, d, dv], u
+ * [chunks, heads, 64, dv].  norm_w [heads dv] (may be NULL; dv at most 128): y [T, heads dv] in the run dtype takes each head's output
+ * divided by its root mean square (eps), times norm_w, times silu(gate [T, gate_ld] from column gate_off); else out [T, heads dv] float. */
+int li_delta_chunks(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride,
+    const int* seg, int chunks, const int* runs, int nruns, float* wt, float* xt, float* pt, float* sums, float* s0,
+    float* u, float* out, const void* gate, int dtype, int gate_ld, int gate_off, const float* norm_w, float eps, void* y,
+    int heads, int kv_heads, int d, int dv, cudaStream_t stream);
 
 /* Per channel c a state S [N]: S = exp(dt_c A[c, :]) S + dt_c x_c B, y_c = (S . C + D[c] x_c) silu(z_c), with
  * dt = softplus(dt_raw) (float, [T, dt_stride]), A = -exp(A_log) [inner, N]; x at column x_off of [T, x_stride], B and C

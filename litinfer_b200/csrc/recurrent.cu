@@ -509,7 +509,7 @@ gla_scan_kernel(const T* __restrict__ qkv, int stride, int q_off, int k_off, int
 // v [T, heads dv].  Every channel of the convolution belongs to one warp, which also moves the channel's state on in a step of
 // single tokens (`shift`).
 // Without za the head has one decay a token, g = exp(-exp(A_log[h]) softplus(a + dt_bias[h])) with a the projections' column
-// a_off + h; prep_g is then [T, heads, 4] (g | beta | unused), written by the warps of the values.
+// a_off + h; prep_g is then [T, heads, 4] (g | beta | log g | 0), written by the warps of the values.
 // TAPS: the taps at compile time (their loads are then all in flight at once), or 0: any number, at run time.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
@@ -577,8 +577,8 @@ delta_prepare_kernel(const T* __restrict__ proj, int stride, int col0, int b_off
         const int h = u - kv_heads - (za ? heads : 0);
         if (!za && lane == 0) {
             const T* row = proj + (size_t)t * stride;
-            float2* to = reinterpret_cast<float2*>(prep_g + ((size_t)t * heads + h) * 4);
-            *to = make_float2(expf(-expf(A_log[h]) * softplus_f(to_float(row[a_off + h]) + dt_bias[h])), sigmoid_f(to_float(row[b_off + h])));
+            const float lg = -expf(A_log[h]) * softplus_f(to_float(row[a_off + h]) + dt_bias[h]);
+            *reinterpret_cast<float4*>(prep_g + ((size_t)t * heads + h) * 4) = make_float4(expf(lg), sigmoid_f(to_float(row[b_off + h])), lg, 0.0f);
         }
         for (int j = lane; j < dv; j += 32) v_out[(size_t)t * heads * dv + h * dv + j] = conv(2 * kv_heads * d + h * dv + j);
     }

@@ -888,7 +888,7 @@ def delta_prepare(proj: torch.Tensor, col: int, b_col: int, conv_w: torch.Tensor
     [T, heads * vdim].  The state is not changed (:func:`conv_state_shift` does that afterwards), unless ``shift``: the caller
     promises that every sequence of the step has one token.
     ``za`` None: one decay a head instead of one a key channel, ``g = exp(-exp(A_log[h]) softplus(proj[:, a_col + h] +
-    dt_bias[h]))``, and ``prep_g`` is [T, heads, 4] = (g | beta | unused)."""
+    dt_bias[h]))``, and ``prep_g`` is [T, heads, 4] = (g | beta | log g | 0)."""
     T = proj.shape[0]
     C = 2 * kv_heads * dim + heads * vdim
     DP = delta_row_elements(dim)
@@ -939,6 +939,38 @@ def delta_scan(prep_qk: torch.Tensor, prep_g: torch.Tensor, v32: torch.Tensor, s
         raise KernelError("delta_scan: the state is too small")
     _check(library().li_delta_scan(_p(prep_qk), _p(prep_g), _p(v32), st, stride, _p(q_start), _p(slots), _p(out32), _i(S), _i(heads), _i(kv_heads),
                                    _i(dim), _i(vdim), _i(1 if per_head else 0), _stream(out32)), "delta_scan")
+
+
+def delta_chunks(prep_qk: torch.Tensor, prep_g: torch.Tensor, v32: torch.Tensor, state: torch.Tensor, chunks: "ScanChunks", heads: int, kv_heads: int,
+                 dim: int, vdim: int, gate: torch.Tensor, gate_col: int, weight: torch.Tensor, eps: float, y: torch.Tensor) -> None:
+    """The rule of :func:`delta_scan` with one decay a head and what follows it, for a step with long portions: the sequences in
+    chunks of 64 tokens (``chunks``), each a few matrix products in float32, so that only the states walk from chunk to chunk; then
+    every head's output divided by its root mean square, times ``weight`` [heads * vdim], times silu of the columns of ``gate`` from
+    ``gate_col``, into ``y`` [T, heads * vdim] in the run dtype.  The same results as the walk but for rounding."""
+    T, dev = v32.shape[0], v32.device
+    DP, n, C = delta_row_elements(dim), chunks.count, ScanChunks.LENGTH
+    _need(prep_qk, "prepared q and k", torch.float32, (T, kv_heads, 2 * DP + 4))
+    _need(prep_g, "prepared decays", torch.float32, (T, heads, 4))
+    _need(v32, "prepared values", torch.float32, (T, heads * vdim))
+    _need(gate, "gate", y.dtype, (T, gate.shape[1]))
+    _need(weight, "rmsnorm weight", torch.float32, (heads * vdim,))
+    _need(y, "mixer output", None, (T, heads * vdim))
+    st, stride, _ = _state_args(state, 0)
+    if heads * dim * vdim > state.shape[1]:
+        raise KernelError("delta_chunks: the state is too small")
+    if n == 0:
+        return
+    fused = vdim <= 128
+    wt, xt, pt, sums, s0, u = (torch.empty((n, heads) + s, dtype=torch.float32, device=dev)
+                               for s in ((dim, C), (vdim, C), (C, C), (2, C), (dim, vdim), (C, vdim)))
+    out32 = None if fused else torch.empty((T, heads * vdim), dtype=torch.float32, device=dev)
+    _check(library().li_delta_chunks(_p(prep_qk), _p(prep_g), _p(v32), st, stride, _p(chunks.seg), _i(n), _p(chunks.runs), _i(chunks.nruns), _p(wt), _p(xt), _p(pt),
+                                     _p(sums), _p(s0), _p(u), _p(out32), _p(gate), _i(_dt(y)), _i(gate.shape[1]), _i(int(gate_col)),
+                                     _p(weight if fused else None), _f(eps), _p(y), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream(y)), "delta_chunks")
+    global launches
+    launches += 2                     # (three kernels)
+    if not fused:
+        gated_rmsnorm(out32, gate, gate_col, weight, eps, heads, False, y, gate_act="silu")
 
 
 def channel_scan(x: torch.Tensor, x_col: int, bc: torch.Tensor, b_col: int, c_col: int, dt32: torch.Tensor, z: torch.Tensor, z_col: int,
@@ -1545,7 +1577,7 @@ _TIMED = ("embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add
           "rope_kv_write", "linear_rope_kv", "rope_table", "paged_attention", "swiglu", "argmax", "sample", "gather_rows", "scale_inplace",
           "logit_cap", "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift",
           "ssm_scan", "decay_scan", "gated_rmsnorm", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route",
-          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "gelu_token_rows",
+          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "delta_chunks", "gelu_token_rows",
           "mul_sigmoid", "polynorm")
 if profile.enabled:
     for _name in _TIMED:

@@ -25,8 +25,9 @@ The convolution's results stay float32 on their way into the recurrence.
 One product serves q | k | v | b | a1 | g1 (or q | k | v | b | a | g); the second products of the two low-rank maps read that row's columns through
 matrices with zero columns elsewhere, so nothing is copied.  What does not depend on the state (convolution, unit vectors,
 decays, beta) is made once per token by one kernel, the walk over the state is a second one.  The kernels find the step's sequences and their slots on the
-device, so steps of single tokens are replayed from a captured graph.  A portion runs in one piece, token after token:
-the rule is not elementwise in S (the correction mixes the key channels), so chunks of it do not run side by side.
+device, so steps of single tokens are replayed from a captured graph.  A portion runs in one piece, token after token
+(the rule is not elementwise in S: the correction mixes the key channels); with one decay a head, long portions run in chunks
+whose corrections are solved for at once (``kernels.delta_chunks``).
 """
 
 from __future__ import annotations
@@ -39,6 +40,7 @@ from .. import kernels as K
 from ..weights.loader import ParamSpec
 from .base import MIXERS, FixedState, Mixer
 from .linear import FusedLinear
+from .scan import scan_chunks
 
 UNIT_EPS = 1e-6          # inside the root of the unit norms of q and k: the rule's own constant
 
@@ -148,8 +150,14 @@ class GatedDeltaRule(Mixer):
                         a_col=col + self.a_col, dt_bias=self.dt_bias)
         if not single and self.taps > 1:
             K.conv_state_shift(proj, col, self.channels, self.taps, cache.state, self.scan_elements, ctx.q_start, ctx.state_slots)
+        y = torch.empty((T, self.vv), dtype=self.dtype, device=dev)
+        chunks = scan_chunks(ctx) if self.head_decay and self.full_gate else None
+        if chunks is not None:
+            # a long portion: chunks as matrix products, with the norm and the gate behind them
+            K.delta_chunks(prep_qk, prep_g, v32, cache.state, chunks, self.heads, self.kv_heads, self.dim, self.value_dim, gate, gate_col, self.norm_weight,
+                           self.eps, y)
+            return self.out(y)
         o32 = torch.empty((T, self.vv), dtype=torch.float32, device=dev)
         K.delta_scan(prep_qk, prep_g, v32, cache.state, ctx.q_start, ctx.state_slots, o32, self.heads, self.kv_heads, self.dim, self.value_dim)
-        y = torch.empty((T, self.vv), dtype=self.dtype, device=dev)
         K.gated_rmsnorm(o32, gate, gate_col, self.norm_weight, self.eps, self.heads, False, y, gate_act="silu" if self.full_gate else "sigmoid")
         return self.out(y)

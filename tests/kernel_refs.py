@@ -811,7 +811,8 @@ def delta_prepare(proj, col, b_col, conv_w, state, state_off, q_start, seq_of_to
     prep_g.zero_()
     if za is None:                                        # one decay a head
         a = torch.nn.functional.softplus(proj[:, a_col:a_col + heads].float() + dt_bias, threshold=1e9)
-        prep_g[:, :, 0] = torch.exp(-torch.exp(A_log) * a)
+        prep_g[:, :, 2] = -torch.exp(A_log) * a
+        prep_g[:, :, 0] = torch.exp(prep_g[:, :, 2])
         prep_g[:, :, 1] = torch.sigmoid(proj[:, b_col:b_col + heads].float())
         v32.copy_(v)
         return
@@ -839,6 +840,17 @@ def delta_scan(prep_qk, prep_g, v32, state, q_start, slots, out32, heads, kv_hea
             u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", S, k))
             S.add_(k[:, :, None] * u[:, None, :])
             out32[t] = torch.einsum("hdv,hd->hv", S, q).reshape(heads * vdim)
+
+
+def delta_chunks(prep_qk, prep_g, v32, state, chunks, heads, kv_heads, dim, vdim, gate, gate_col, weight, eps, y):
+    """The walk, token by token, over the chunks' sequences; then the norm and the gate."""
+    out32 = torch.zeros_like(v32)
+    seg, runs = chunks.seg.tolist(), chunks.runs.tolist()
+    starts, slots = [seg[f][0] for f, _, _ in runs], [s for _, _, s in runs]
+    ends = [seg[f + c - 1][1] for f, c, _ in runs]
+    for lo, hi, slot in zip(starts, ends, slots):
+        delta_scan(prep_qk[lo:hi], prep_g[lo:hi], v32[lo:hi], state, torch.tensor([0, hi - lo]), torch.tensor([slot]), out32[lo:hi], heads, kv_heads, dim, vdim)
+    gated_rmsnorm(out32, gate, gate_col, weight, eps, heads, False, y, gate_act="silu")
 
 
 def argmax(logits, out):
@@ -930,7 +942,7 @@ def table_gather(resident, updates, slots, out, trash_page):
             out[s, b] = resident[slot, b] if b < cols else trash_page
 
 
-ALL = ["gelu_token_rows", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
+ALL = ["gelu_token_rows", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_chunks", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
        "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift", "ssm_scan",
        "decay_scan", "gated_rmsnorm", "table_gather", "gather_rows", "scale_inplace", "logit_cap", "rope_table", "linear_scaled_accepts", "linear_add_scaled_parts", "linear_add_scaled", "apply_row_scale", "linear_rope_kv", "interleave_gate_up", "embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add", "linear", "rope_kv_write",
        "paged_attention", "swiglu", "argmax", "sample"]

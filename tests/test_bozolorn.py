@@ -837,6 +837,48 @@ def test_delta_rule_with_one_decay_a_head(heads, kv, d, dv, taps, dtype):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads,kv,d,dv", [(4, 2, 12, 20), (3, 3, 7, 11), (2, 1, 128, 128), (6, 2, 64, 48), (1, 1, 1, 1), (2, 2, 200, 160), (2, 1, 40, 130)])
+@pytest.mark.parametrize("forget", [0.3, 60.0, 0.0])
+def test_delta_rule_in_chunks(heads, kv, d, dv, forget, dtype):
+    """Chunks as matrix products against the walk: portions that end on a chunk's edge, one token before and behind it, single tokens,
+    several sequences, states of their own; heads that forget slowly, at once (decays of nothing), and never."""
+    import kernel_refs as R
+    from litinfer_b200 import kernels as K
+
+    dev, dt = torch.device("cuda:0"), _dt(dtype)
+    torch.manual_seed(d + dv)
+    DP = K.delta_row_elements(d)
+    first = 0.5 * torch.randn(6, heads * d * dv + 8, device=dev)
+    for lens, slots in (([64, 63, 65, 1, 200], [4, 0, 2, 1, 3]), ([129, 0, 128], [1, 0, 2]), ([300], [5])):
+        T = sum(lens)
+        starts = [0]
+        for n in lens:
+            starts.append(starts[-1] + n)
+        q, k = (torch.nn.functional.normalize(torch.randn(T, kv, d, device=dev) + 0.7, dim=-1) for _ in range(2))
+        qk = torch.zeros(T, kv, 2 * DP + 4, device=dev)
+        qk[..., :d], qk[..., DP:DP + d], qk[..., 2 * DP] = q, k, (q * k).sum(-1)
+        g = torch.zeros(T, heads, 4, device=dev)
+        g[..., 2] = -forget * torch.rand(T, heads, device=dev) ** 2
+        g[..., 0], g[..., 1] = torch.exp(g[..., 2]), torch.rand(T, heads, device=dev)
+        v, gate = torch.randn(T, heads * dv, device=dev), torch.randn(T, heads * dv + 7).to(dev, dt)
+        w = 1 + 0.2 * torch.randn(heads * dv, device=dev)
+        chunks = K.ScanChunks(starts, slots, dev)
+        res = []
+        for F in (K, R):
+            state, y = first.clone(), torch.empty(T, heads * dv, dtype=dt, device=dev)
+            F.delta_chunks(qk, g, v, state, chunks, heads, kv, d, dv, gate, 7, w, 1e-5, y)
+            res.append((state, y))
+        _close(res[0][0], res[1][0], "float32", f"states, portions of {lens}", 1e-5)
+        _close(res[0][1], res[1][1], dtype, f"outputs, portions of {lens}", 2e-4 if dtype == "float32" else 2e-2)
+        # and the walk's kernel gives the same states
+        state, o = first.clone(), torch.empty(T, heads * dv, device=dev)
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        K.delta_scan(qk, g, v, state, i32(starts), i32(slots), o, heads, kv, d, dv)
+        _close(res[0][0], state, "float32", "states of the walk", 1e-5)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_routing_by_sigmoid_scores_in_groups(dtype):
     import kernel_refs as R
     from litinfer_b200 import kernels as K
