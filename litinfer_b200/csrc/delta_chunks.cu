@@ -21,9 +21,10 @@ namespace {
 constexpr int kC = 64;              // tokens of a chunk
 constexpr int kLA = kC + 4;         // a row of a [.., tokens] tile in shared memory
 constexpr int kThreads = 256;
+constexpr int kCarryThreads = 512;
 constexpr int kSlice = 16;          // value columns a block of the carry takes
 constexpr int kCols = 128;          // value columns a block of the output takes at a time
-constexpr int kRowsB = 32;          // rows of its second operand that it stages at a time
+constexpr int kRowsB = 16;          // rows of its second operand that it stages at a time
 
 __device__ __forceinline__ void copy16(float* dst, const float* src, bool valid) {
     const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
@@ -33,18 +34,32 @@ __device__ __forceinline__ void copy16(float* dst, const float* src, bool valid)
 __device__ __forceinline__ void copies_done() { asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory"); }
 
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float dot4(float4 a, float4 b, float c) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, c)))); }
+
+// Two multiply-adds in one instruction, each rounded like fmaf.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;"
+        : "=l"(*reinterpret_cast<unsigned long long*>(&d))
+        : "l"(*reinterpret_cast<unsigned long long*>(&a)), "l"(*reinterpret_cast<unsigned long long*>(&b)), "l"(*reinterpret_cast<unsigned long long*>(&c)));
+    return d;
+}
+__device__ __forceinline__ float2 lo2(float4 v) { return make_float2(v.x, v.y); }
+__device__ __forceinline__ float2 hi2(float4 v) { return make_float2(v.z, v.w); }
+__device__ __forceinline__ float2 dot4(float4 a, float4 b, float2 c) { return fma2(lo2(a), lo2(b), fma2(hi2(a), hi2(b), c)); }
+
+// columns of the values in the workspace: rows of whole 16-byte pieces
+__host__ __device__ constexpr int padded(int dv) { return (dv + 3) / 4 * 4; }
 
 template <int DP>
 __host__ __device__ constexpr size_t solve_smem() { return ((size_t)2 * kC * (DP + 4) + 2 * kC * kLA + 4 * kC) * sizeof(float); }
 
 // prep_qk [T, kv_heads, 2 DP + 4] (q | k | k . q), prep_g [T, heads, 4] (g | beta | log g), v [T, heads dv]; seg: a chunk's first token,
-// end, number, slot.  Out, per chunk and head: wt [d, 64] and xt [dv, 64] (W and X transposed), pt [64, 64] (P transposed), sums [2, 64] (c_t, and c_64 / c_t).
+// end, number, slot.  Out, per chunk and head: wm [64, DP] and xm [64, dv] (W and X), pt [64, 64] (P transposed), sums [2, 64] (c_t, and
+// c_64 / c_t).
 template <int DP>
 __global__ void __launch_bounds__(kThreads, DP <= 128 ? 2 : 1)
 delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restrict__ prep_g, const float* __restrict__ v, const int4* __restrict__ seg,
-                         float* __restrict__ wt, float* __restrict__ xt, float* __restrict__ pt, float* __restrict__ sums, int heads, int kv_heads, int d,
-                         int dv) {
+                         float* __restrict__ wm, float* __restrict__ xm, float* __restrict__ pt, float* __restrict__ sums, int heads, int kv_heads, int dv) {
     constexpr int LD = DP + 4, RQ = 2 * DP + 4;
     extern __shared__ __align__(16) float smem[];
     float* Ks = smem;                       // [64][LD]
@@ -98,16 +113,16 @@ delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restr
     }
     copies_done();
     __syncthreads();
-    // the products of keys with keys and of queries with keys: a thread takes tokens ty + 16 i against ty's of tx + 16 j, j <= i
+    // the products of keys with keys and of queries with keys: a thread takes tokens ty + 16 i against those of tx + 16 j, j <= i
     {
         const int tx = tid & 15, ty = tid >> 4;
         const int blocks = (n + 15) >> 4;
-        float kk[4][4], qk[4][4];
+        float2 kk[4][4], qk[4][4];
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = 0.0f;
-#pragma unroll 2
+            for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = make_float2(0.0f, 0.0f);
+#pragma unroll 1
         for (int k = 0; k < DP; k += 4) {
             float4 col[4];
 #pragma unroll
@@ -130,8 +145,8 @@ delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restr
             for (int j = 0; j < 4; ++j) {
                 const int t = ty + 16 * i, s = tx + 16 * j;
                 const float f = s <= t ? expf((cum[t] - cum[s]) + (low[t] - low[s])) : 0.0f;
-                At[s * kLA + t] = s < t ? beta[t] * f * kk[i][j] : 0.0f;
-                Ps[s * kLA + t] = f * qk[i][j];
+                At[s * kLA + t] = s < t ? beta[t] * f * (kk[i][j].x + kk[i][j].y) : 0.0f;
+                Ps[s * kLA + t] = f * (qk[i][j].x + qk[i][j].y);
             }
     }
     __syncthreads();
@@ -140,35 +155,42 @@ delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restr
         *reinterpret_cast<float4*>(pt + (unit * kC + s) * kC + 4 * i) = ld4(Ps + s * kLA + 4 * i);
     }
     // the triangular solves, a column a thread: as soon as x_s is known it is taken off the rows behind it
-    for (int c = tid; c < d + dv; c += kThreads) {
-        float x[kC];
-        if (c < d) {
+    const int dvp = padded(dv);
+    for (int c = tid; c < DP + dvp; c += kThreads) {
+        float2 x[kC / 2];
+        if (c < DP) {
 #pragma unroll
-            for (int t = 0; t < kC; ++t) x[t] = bc[t] * Ks[t * LD + c];
+            for (int t = 0; t < kC; t += 2) x[t / 2] = make_float2(bc[t] * Ks[t * LD + c], bc[t + 1] * Ks[(t + 1) * LD + c]);
         } else {
-            const float* col = v + (size_t)q0 * heads * dv + (size_t)h * dv + (c - d);
+            const bool real = c - DP < dv;
+            const float* col = v + (size_t)q0 * heads * dv + (size_t)h * dv + (real ? c - DP : 0);
 #pragma unroll
-            for (int t = 0; t < kC; ++t) x[t] = t < n ? beta[t] * col[(size_t)t * heads * dv] : 0.0f;
+            for (int t = 0; t < kC; t += 2)
+                x[t / 2] = make_float2(real && t < n ? beta[t] * col[(size_t)t * heads * dv] : 0.0f, real && t + 1 < n ? beta[t + 1] * col[(size_t)(t + 1) * heads * dv] : 0.0f);
         }
 #pragma unroll
         for (int s8 = 0; s8 < kC; s8 += 8) {
             if (s8 < n) {
 #pragma unroll
                 for (int s = s8; s < s8 + 8; ++s) {
+                    const float xs = (s & 1) ? -x[s / 2].y : -x[s / 2].x;
+                    const float2 both = make_float2(xs, xs);
 #pragma unroll
                     for (int t4 = (s + 1) / 4 * 4; t4 < kC; t4 += 4) {
                         const float4 a = ld4(At + s * kLA + t4);         // (zeros where t <= s)
-                        x[t4] = fmaf(-a.x, x[s], x[t4]);
-                        x[t4 + 1] = fmaf(-a.y, x[s], x[t4 + 1]);
-                        x[t4 + 2] = fmaf(-a.z, x[s], x[t4 + 2]);
-                        x[t4 + 3] = fmaf(-a.w, x[s], x[t4 + 3]);
+                        x[t4 / 2] = fma2(lo2(a), both, x[t4 / 2]);
+                        x[t4 / 2 + 1] = fma2(hi2(a), both, x[t4 / 2 + 1]);
                     }
                 }
             }
         }
-        float* out = c < d ? wt + (unit * d + c) * kC : xt + (unit * dv + (c - d)) * kC;
+        float* out = c < DP ? wm + unit * kC * DP + c : xm + unit * kC * dvp + (c - DP);
+        const int ld = c < DP ? DP : dvp;
 #pragma unroll
-        for (int t = 0; t < kC; t += 4) *reinterpret_cast<float4*>(out + t) = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
+        for (int t = 0; t < kC; t += 2) {
+            out[(size_t)t * ld] = x[t / 2].x;
+            out[(size_t)(t + 1) * ld] = x[t / 2].y;
+        }
     }
     pdl_launch_dependents();
 }
@@ -176,214 +198,181 @@ delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restr
 template <int DP>
 __host__ __device__ constexpr int carry_buffers() { return DP <= 128 ? 2 : 1; }
 template <int DP>
-__host__ __device__ constexpr int carry_buffer() { return DP * kC + kC * DP + kSlice * kC + 2 * kC; }
-template <int DP>
-__host__ __device__ constexpr int carry_scratch() { return 4 * kC * kSlice > (kThreads / DP - 1) * DP * kSlice ? 4 * kC * kSlice : (kThreads / DP - 1) * DP * kSlice; }
+__host__ __device__ constexpr int carry_buffer() { return kC * (DP + 4) + kC * DP + kC * kSlice + 2 * kC; }
+constexpr int kCarryScratch = kCarryThreads * 16;
 template <int DP>
 __host__ __device__ constexpr size_t carry_smem() {
-    return ((size_t)carry_buffers<DP>() * carry_buffer<DP>() + DP * kSlice + carry_scratch<DP>() + kC * kSlice) * sizeof(float);
+    return ((size_t)carry_buffers<DP>() * carry_buffer<DP>() + kSlice * (DP + 4) + kCarryScratch + 2 * kC * kSlice) * sizeof(float);
 }
 
-// runs: triples (first chunk, chunks, slot).  s0 [chunk, head, d, dv]: the state before every chunk; u [chunk, head, 64, dv].
+// runs: triples (first chunk, chunks, slot).  s0 [chunk, head, DP, dv]: the state before every chunk; u [chunk, head, 64, dv].
 template <int DP>
-__global__ void __launch_bounds__(kThreads)
-delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restrict__ seg, const int* __restrict__ runs, const float* __restrict__ wt,
-                         const float* __restrict__ xt, const float* __restrict__ sums, float* __restrict__ state, long long state_stride,
+__global__ void __launch_bounds__(kCarryThreads, 1)
+delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restrict__ seg, const int* __restrict__ runs, const float* __restrict__ wm,
+                         const float* __restrict__ xm, const float* __restrict__ sums, float* __restrict__ state, long long state_stride,
                          float* __restrict__ s0, float* __restrict__ u, int heads, int kv_heads, int d, int dv) {
-    constexpr int RQ = 2 * DP + 4, NB = carry_buffers<DP>(), SPLIT = kThreads / DP;
+    constexpr int RQ = 2 * DP + 4, LD = DP + 4, NB = carry_buffers<DP>(), SPLIT = kCarryThreads / DP;
     extern __shared__ __align__(16) float smem[];
-    float* S = smem + NB * carry_buffer<DP>();          // [DP][16]
-    float* red = S + DP * kSlice;
-    float* Us = red + carry_scratch<DP>();              // [64][16]: U with the decay to the chunk's end
+    float* S = smem + NB * carry_buffer<DP>();          // [16][LD]: a column of the state after the other
+    float* red = S + kSlice * LD;
+    float2* Us = reinterpret_cast<float2*>(red + kCarryScratch);        // [64][16]: U with the decay to the chunk's end, every number twice
     const int tid = threadIdx.x;
-    const int h = blockIdx.y, hk = h / (heads / kv_heads), c0 = blockIdx.x * kSlice;
+    const int h = blockIdx.y, hk = h / (heads / kv_heads), c0 = blockIdx.x * kSlice, dvp = padded(dv);
     pdl_wait();
     const int first = runs[3 * blockIdx.z], count = runs[3 * blockIdx.z + 1], slot = runs[3 * blockIdx.z + 2];
     float* st = state + (size_t)slot * state_stride + (size_t)h * dv * d;
     auto stage = [&](int b, int chunk) {
-        float* W = smem + b * carry_buffer<DP>();       // [DP][64]
-        float* Kb = W + DP * kC;                        // [64][DP]
-        float* X = Kb + kC * DP;                        // [16][64]
-        float* cm = X + kSlice * kC;                    // [2][64]
+        float* W = smem + b * carry_buffer<DP>();       // [64][LD]
+        float* Kb = W + kC * LD;                        // [64][DP]
+        float* X = Kb + kC * DP;                        // [64][16]
+        float* cm = X + kC * kSlice;                    // [2][64]
         const int4 sg = seg[chunk];
         const int n = min(sg.y - sg.x, kC);
         const size_t unit = (size_t)chunk * heads + h;
-        for (int idx = tid; idx < DP * (kC / 4); idx += kThreads) {
-            const int k = idx / (kC / 4), i = idx - k * (kC / 4);
-            copy16(W + k * kC + 4 * i, wt + (unit * d + (k < d ? k : 0)) * kC + 4 * i, k < d);
-        }
-        for (int idx = tid; idx < kC * (DP / 4); idx += kThreads) {
+        for (int idx = tid; idx < kC * (DP / 4); idx += kCarryThreads) {
             const int t = idx / (DP / 4), i = idx - t * (DP / 4);
+            copy16(W + t * LD + 4 * i, wm + (unit * kC + t) * DP + 4 * i, true);
             copy16(Kb + t * DP + 4 * i, prep_qk + ((size_t)(sg.x + (t < n ? t : 0)) * kv_heads + hk) * RQ + DP + 4 * i, t < n);
         }
-        if (tid < kSlice * (kC / 4)) {
-            const int c = tid / (kC / 4), i = tid - c * (kC / 4);
-            copy16(X + c * kC + 4 * i, xt + (unit * dv + (c0 + c < dv ? c0 + c : 0)) * kC + 4 * i, c0 + c < dv);
+        if (tid < kC * (kSlice / 4)) {
+            const int t = tid / (kSlice / 4), c = 4 * (tid - t * (kSlice / 4));
+            copy16(X + t * kSlice + c, xm + (unit * kC + t) * dvp + (c0 + c < dvp ? c0 + c : 0), c0 + c < dvp);
         }
         if (tid < 2 * kC / 4) copy16(cm + 4 * tid, sums + unit * 2 * kC + 4 * tid, true);
     };
     stage(0, first);
-    for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
+    for (int idx = tid; idx < DP * kSlice; idx += kCarryThreads) {
         const int c = idx / DP, k = idx - c * DP;
-        S[k * kSlice + c] = (k < d && c0 + c < dv) ? st[(size_t)(c0 + c) * d + k] : 0.0f;
+        S[c * LD + k] = (k < d && c0 + c < dv) ? st[(size_t)(c0 + c) * d + k] : 0.0f;
     }
-    const bool vec = (dv & 3) == 0;
     for (int j = 0; j < count; ++j) {
         const int chunk = first + j, b = j % NB;
         copies_done();
         __syncthreads();                                 // this chunk's rows are here, and everybody has left the other buffer
         if (NB > 1 && j + 1 < count) stage(b ^ 1, chunk + 1);
         const float* W = smem + b * carry_buffer<DP>();
-        const float* Kb = W + DP * kC;
+        const float* Kb = W + kC * LD;
         const float* X = Kb + kC * DP;
-        const float* cm = X + kSlice * kC;
+        const float* cm = X + kC * kSlice;
         const size_t unit = (size_t)chunk * heads + h;
         // the state before this chunk, for the outputs
-        for (int idx = tid; idx < d * (kSlice / 4); idx += kThreads) {
+        for (int idx = tid; idx < DP * (kSlice / 4); idx += kCarryThreads) {
             const int k = idx / (kSlice / 4), c = 4 * (idx - k * (kSlice / 4));
-            const float4 val = ld4(S + k * kSlice + c);
-            float* to = s0 + (unit * d + k) * dv + c0 + c;
-            if (vec) {
-                if (c0 + c < dv) *reinterpret_cast<float4*>(to) = val;
-            } else {
-                const float e[4] = {val.x, val.y, val.z, val.w};
-#pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    if (c0 + c + q < dv) to[q] = e[q];
-            }
+            if (c0 + c < dvp)
+                *reinterpret_cast<float4*>(s0 + (unit * DP + k) * dvp + c0 + c) = make_float4(S[c * LD + k], S[(c + 1) * LD + k], S[(c + 2) * LD + k], S[(c + 3) * LD + k]);
         }
-        // W S: four tokens by four columns a thread, a quarter of the key channels each
+        // W S: tokens tt + 16 i by columns ct + 4 q a thread, an eighth of the key channels each
         {
-            const int part = tid >> 6, ct = tid & 3, tt = (tid & 63) >> 2;
-            float acc[4][4];
+            const int part = tid >> 6, tile = tid & 63, ct = tile & 3, tt = tile >> 2;
+            float2 acc[4][4];
 #pragma unroll
-            for (int a = 0; a < 4; ++a)
+            for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int q = 0; q < 4; ++q) acc[a][q] = 0.0f;
-#pragma unroll 8
-            for (int k = part * (DP / 4); k < (part + 1) * (DP / 4); ++k) {
-                const float4 w = ld4(W + k * kC + 4 * tt), s = ld4(S + k * kSlice + 4 * ct);
-                const float wa[4] = {w.x, w.y, w.z, w.w}, sa[4] = {s.x, s.y, s.z, s.w};
+                for (int q = 0; q < 4; ++q) acc[i][q] = make_float2(0.0f, 0.0f);
 #pragma unroll
-                for (int a = 0; a < 4; ++a)
+            for (int k = part * (DP / 8); k < (part + 1) * (DP / 8); k += 4) {
+                float4 w[4], s[4];
 #pragma unroll
-                    for (int q = 0; q < 4; ++q) acc[a][q] = fmaf(wa[a], sa[q], acc[a][q]);
+                for (int i = 0; i < 4; ++i) w[i] = ld4(W + (tt + 16 * i) * LD + k);
+#pragma unroll
+                for (int q = 0; q < 4; ++q) s[q] = ld4(S + (ct + 4 * q) * LD + k);
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) acc[i][q] = dot4(w[i], s[q], acc[i][q]);
             }
 #pragma unroll
-            for (int a = 0; a < 4; ++a)
-                *reinterpret_cast<float4*>(red + (part * kC + 4 * tt + a) * kSlice + 4 * ct) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int q = 0; q < 4; ++q) red[(part * 16 + i * 4 + q) * 64 + tile] = acc[i][q].x + acc[i][q].y;
         }
         __syncthreads();
-        {
-            const int t = tid >> 2, c = 4 * (tid & 3);
-            float4 sum = ld4(red + t * kSlice + c);
 #pragma unroll
-            for (int part = 1; part < 4; ++part) {
-                const float4 p = ld4(red + (part * kC + t) * kSlice + c);
-                sum.x += p.x, sum.y += p.y, sum.z += p.z, sum.w += p.w;
-            }
-            const float4 val = make_float4(X[c * kC + t] - sum.x, X[(c + 1) * kC + t] - sum.y, X[(c + 2) * kC + t] - sum.z, X[(c + 3) * kC + t] - sum.w);
-            float* to = u + (unit * kC + t) * dv + c0 + c;
-            if (vec) {
-                if (c0 + c < dv) *reinterpret_cast<float4*>(to) = val;
-            } else {
-                const float e[4] = {val.x, val.y, val.z, val.w};
+        for (int o = tid; o < kC * kSlice; o += kCarryThreads) {
+            const int iq = o >> 6, tile = o & 63, t = (tile >> 2) + 16 * (iq >> 2), c = (tile & 3) + 4 * (iq & 3);
+            float sum = 0.0f;
 #pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    if (c0 + c + q < dv) to[q] = e[q];
-            }
-            const float f = cm[kC + t];
-            *reinterpret_cast<float4*>(Us + t * kSlice + c) = make_float4(f * val.x, f * val.y, f * val.z, f * val.w);
+            for (int part = 0; part < 8; ++part) sum += red[part * 1024 + o];
+            const float val = X[t * kSlice + c] - sum;
+            if (c0 + c < dvp) u[(unit * kC + t) * dvp + c0 + c] = val;
+            const float f = cm[kC + t] * val;
+            Us[t * kSlice + c] = make_float2(f, f);
         }
         __syncthreads();
         // the state behind the chunk: four key channels by four columns a thread, a part of the tokens each
         {
             const int part = tid / DP, tile = tid - part * DP, ct = tile & 3, kt = tile >> 2;
-            float acc[4][4];
+            float2 acc[4][2];
 #pragma unroll
-            for (int a = 0; a < 4; ++a)
-#pragma unroll
-                for (int q = 0; q < 4; ++q) acc[a][q] = 0.0f;
+            for (int q = 0; q < 4; ++q) acc[q][0] = acc[q][1] = make_float2(0.0f, 0.0f);
 #pragma unroll 8
             for (int t = part * (kC / SPLIT); t < (part + 1) * (kC / SPLIT); ++t) {
-                const float4 k = ld4(Kb + t * DP + 4 * kt), w = ld4(Us + t * kSlice + 4 * ct);
-                const float ka[4] = {k.x, k.y, k.z, k.w}, ua[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-                for (int a = 0; a < 4; ++a)
-#pragma unroll
-                    for (int q = 0; q < 4; ++q) acc[a][q] = fmaf(ka[a], ua[q], acc[a][q]);
+                const float4 k = ld4(Kb + t * DP + 4 * kt);
+                const float* us = reinterpret_cast<const float*>(Us + t * kSlice + 4 * ct);
+                const float4 u01 = ld4(us), u23 = ld4(us + 4);
+                acc[0][0] = fma2(lo2(k), lo2(u01), acc[0][0]), acc[0][1] = fma2(hi2(k), lo2(u01), acc[0][1]);
+                acc[1][0] = fma2(lo2(k), hi2(u01), acc[1][0]), acc[1][1] = fma2(hi2(k), hi2(u01), acc[1][1]);
+                acc[2][0] = fma2(lo2(k), lo2(u23), acc[2][0]), acc[2][1] = fma2(hi2(k), lo2(u23), acc[2][1]);
+                acc[3][0] = fma2(lo2(k), hi2(u23), acc[3][0]), acc[3][1] = fma2(hi2(k), hi2(u23), acc[3][1]);
             }
-            if (SPLIT > 1) {
-                if (part > 0) {
 #pragma unroll
-                    for (int a = 0; a < 4; ++a)
-                        *reinterpret_cast<float4*>(red + ((part - 1) * DP + 4 * kt + a) * kSlice + 4 * ct) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
-                }
-                __syncthreads();
-            }
-            if (part == 0) {
-                const float f = cm[kC - 1];
-#pragma unroll
-                for (int a = 0; a < 4; ++a) {
-                    float* row = S + (4 * kt + a) * kSlice + 4 * ct;
-                    float4 s = ld4(row);
-                    float4 sum = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
-#pragma unroll
-                    for (int p = 0; p < SPLIT - 1; ++p) {
-                        const float4 r = ld4(red + (p * DP + 4 * kt + a) * kSlice + 4 * ct);
-                        sum.x += r.x, sum.y += r.y, sum.z += r.z, sum.w += r.w;
-                    }
-                    s.x = fmaf(f, s.x, sum.x), s.y = fmaf(f, s.y, sum.y), s.z = fmaf(f, s.z, sum.z), s.w = fmaf(f, s.w, sum.w);
-                    *reinterpret_cast<float4*>(row) = s;
-                }
+            for (int q = 0; q < 4; ++q) {
+                float* to = red + (size_t)(part * 16 + q * 4) * DP + tile;
+                to[0] = acc[q][0].x, to[DP] = acc[q][0].y, to[2 * DP] = acc[q][1].x, to[3 * DP] = acc[q][1].y;
             }
         }
         __syncthreads();
-        if (NB == 1 && j + 1 < count) stage(0, chunk + 1);
+        {
+            const float f = cm[kC - 1];
+            for (int o = tid; o < 16 * DP; o += kCarryThreads) {
+                const int e = o / DP, tile = o - e * DP, c = 4 * (tile & 3) + (e >> 2), k = 4 * (tile >> 2) + (e & 3);
+                float sum = 0.0f;
+#pragma unroll
+                for (int part = 0; part < SPLIT; ++part) sum += red[part * 16 * DP + o];
+                S[c * LD + k] = fmaf(f, S[c * LD + k], sum);
+            }
+        }
+        if (NB == 1 && j + 1 < count) {
+            __syncthreads();
+            stage(0, chunk + 1);
+        }
     }
     pdl_launch_dependents();
-    for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
+    __syncthreads();
+    for (int idx = tid; idx < DP * kSlice; idx += kCarryThreads) {
         const int c = idx / DP, k = idx - c * DP;
-        if (k < d && c0 + c < dv) st[(size_t)(c0 + c) * d + k] = S[k * kSlice + c];
+        if (k < d && c0 + c < dv) st[(size_t)(c0 + c) * d + k] = S[c * LD + k];
     }
 }
 
 template <int DP>
 __host__ __device__ constexpr size_t output_smem() { return ((size_t)(DP + kC) * kLA + 2 * kRowsB * kCols) * sizeof(float); }
 
-// o = diag(c) Q S + P U as one product over d + 64 rows.  norm_w given (dv at most 128): y = o / sqrt(mean(o^2) + eps) * norm_w * silu(gate),
+// o = diag(c) Q S + P U as one product over DP + 64 rows.  norm_w given (dv at most 128): y = o / sqrt(mean(o^2) + eps) * norm_w * silu(gate),
 // in the run dtype; else out takes o as it is.
 template <typename T, int DP>
-__global__ void __launch_bounds__(kThreads, 2)
+__global__ void __launch_bounds__(kThreads, DP <= 128 ? 3 : 2)
 delta_chunk_output_kernel(const float* __restrict__ prep_qk, const int4* __restrict__ seg, const float* __restrict__ pt, const float* __restrict__ sums,
                           const float* __restrict__ s0, const float* __restrict__ u, float* __restrict__ out, const T* __restrict__ gate, int gate_ld,
-                          int gate_off, const float* __restrict__ norm_w, float eps, T* __restrict__ y, int heads, int kv_heads, int d, int dv) {
+                          int gate_off, const float* __restrict__ norm_w, float eps, T* __restrict__ y, int heads, int kv_heads, int dv) {
     constexpr int RQ = 2 * DP + 4;
     extern __shared__ __align__(16) float smem[];
     float* At = smem;                        // [DP + 64][68]: rows of Q^T with the decay, then of P^T
-    float* B = At + (DP + kC) * kLA;         // [2][32][128]
+    float* B = At + (DP + kC) * kLA;         // [2][16][128]
     pdl_wait();
-    const int h = blockIdx.x, hk = h / (heads / kv_heads);
+    const int h = blockIdx.x, hk = h / (heads / kv_heads), dvp = padded(dv);
     const int4 sg = seg[blockIdx.y];
     const int q0 = sg.x, n = min(sg.y - sg.x, kC);
     const size_t unit = (size_t)sg.z * heads + h;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, t0 = 8 * warp;
-    const bool vec = (dv & 3) == 0;
-    constexpr int kBlocks = DP / kRowsB + kC / kRowsB;
+    constexpr int kBlocks = (DP + kC) / kRowsB;
     auto stage = [&](int b, int kb, int cb) {
+#pragma unroll
         for (int idx = tid; idx < kRowsB * (kCols / 4); idx += kThreads) {
             const int r = idx / (kCols / 4), c = 4 * (idx - r * (kCols / 4));
             const int k = kb * kRowsB + r, col = cb + c;
-            const bool from_state = k < DP;
-            const bool row_ok = from_state ? k < d : true;
-            const float* row = from_state ? s0 + (unit * d + (row_ok ? k : 0)) * dv : u + (unit * kC + (k - DP)) * dv;
-            float* dst = B + (b * kRowsB + r) * kCols + c;
-            if (vec) {
-                copy16(dst, row + (col < dv ? col : 0), row_ok && col < dv);
-            } else {
-#pragma unroll
-                for (int q = 0; q < 4; ++q) dst[q] = (row_ok && col + q < dv) ? row[col + q] : 0.0f;
-            }
+            const float* row = k < DP ? s0 + (unit * DP + k) * dvp : u + (unit * kC + (k - DP)) * dvp;
+            copy16(B + (b * kRowsB + r) * kCols + c, row + (col < dvp ? col : 0), col < dvp);
         }
     };
     stage(0, 0, 0);
@@ -403,28 +392,28 @@ delta_chunk_output_kernel(const float* __restrict__ prep_qk, const int4* __restr
         copy16(At + (DP + s) * kLA + 4 * i, pt + (unit * kC + s) * kC + 4 * i, true);
     }
     for (int cb = 0; cb < dv; cb += kCols) {
-        float acc[8][4];
+        float2 acc[4][4];                    // tokens t0 + 2 a and t0 + 2 a + 1 by four columns
 #pragma unroll
-        for (int a = 0; a < 8; ++a)
+        for (int a = 0; a < 4; ++a)
 #pragma unroll
-            for (int q = 0; q < 4; ++q) acc[a][q] = 0.0f;
+            for (int q = 0; q < 4; ++q) acc[a][q] = make_float2(0.0f, 0.0f);
         for (int kb = 0; kb < kBlocks; ++kb) {
             const int b = kb & 1;
             copies_done();
             __syncthreads();
             if (kb + 1 < kBlocks) stage(b ^ 1, kb + 1, cb);
             // (rows of P^T: a token sees those up to its own; tokens behind the portion's end see nothing)
-            const bool some = t0 < n && (kb * kRowsB < DP || kb * kRowsB - DP <= t0 + 7);
-            if (some) {
+            if (t0 < n && kb * kRowsB <= DP + t0 + 7) {
 #pragma unroll 4
                 for (int r = 0; r < kRowsB; ++r) {
                     const float* at = At + (kb * kRowsB + r) * kLA + t0;
                     const float4 a0 = ld4(at), a1 = ld4(at + 4), bv = ld4(B + (b * kRowsB + r) * kCols + 4 * lane);
-                    const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w}, bb[4] = {bv.x, bv.y, bv.z, bv.w};
+                    const float2 av[4] = {lo2(a0), hi2(a0), lo2(a1), hi2(a1)};
+                    const float2 bb[4] = {make_float2(bv.x, bv.x), make_float2(bv.y, bv.y), make_float2(bv.z, bv.z), make_float2(bv.w, bv.w)};
 #pragma unroll
-                    for (int a = 0; a < 8; ++a)
+                    for (int a = 0; a < 4; ++a)
 #pragma unroll
-                        for (int q = 0; q < 4; ++q) acc[a][q] = fmaf(av[a], bb[q], acc[a][q]);
+                        for (int q = 0; q < 4; ++q) acc[a][q] = fma2(av[a], bb[q], acc[a][q]);
                 }
             }
         }
@@ -433,10 +422,13 @@ delta_chunk_output_kernel(const float* __restrict__ prep_qk, const int4* __restr
         for (int a = 0; a < 8; ++a) {
             const int t = t0 + a;
             if (t >= n) break;                                     // (the same for the whole warp)
+            float o[4];
+#pragma unroll
+            for (int q = 0; q < 4; ++q) o[q] = (a & 1) ? acc[a / 2][q].y : acc[a / 2][q].x;
             if (norm_w) {
                 float ss = 0.0f;
 #pragma unroll
-                for (int q = 0; q < 4; ++q) ss = fmaf(acc[a][q], acc[a][q], ss);           // (zeros behind the last column)
+                for (int q = 0; q < 4; ++q) ss = fmaf(o[q], o[q], ss);                     // (zeros behind the last column)
                 const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
                 const T* gr = gate + (size_t)(q0 + t) * gate_ld + gate_off + (size_t)h * dv + col;
                 T* to = y + (size_t)(q0 + t) * heads * dv + (size_t)h * dv + col;
@@ -444,13 +436,13 @@ delta_chunk_output_kernel(const float* __restrict__ prep_qk, const int4* __restr
                 for (int q = 0; q < 4; ++q)
                     if (col + q < dv) {
                         const float g = to_float(gr[q]);
-                        to[q] = from_float<T>(acc[a][q] * rinv * norm_w[h * dv + col + q] * (g / (1.0f + expf(-g))));
+                        to[q] = from_float<T>(o[q] * rinv * norm_w[h * dv + col + q] * (g / (1.0f + expf(-g))));
                     }
             } else {
                 float* to = out + (size_t)(q0 + t) * heads * dv + (size_t)h * dv + col;
 #pragma unroll
                 for (int q = 0; q < 4; ++q)
-                    if (col + q < dv) to[q] = acc[a][q];
+                    if (col + q < dv) to[q] = o[q];
             }
         }
         __syncthreads();                                           // everybody has left the last rows staged
@@ -468,7 +460,7 @@ int raise_smem(K kernel, size_t bytes, const char* what) {
 
 template <int DP>
 int launch(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* seg, int chunks, const int* runs,
-           int nruns, float* wt, float* xt, float* pt, float* sums, float* s0, float* u, float* out, const void* gate, int dtype, int gate_ld, int gate_off,
+           int nruns, float* wm, float* xm, float* pt, float* sums, float* s0, float* u, float* out, const void* gate, int dtype, int gate_ld, int gate_off,
            const float* norm_w, float eps, void* y, int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
     static bool raised = false;
     if (!raised) {
@@ -479,17 +471,17 @@ int launch(const float* prep_qk, const float* prep_g, const float* v, float* sta
         raised = true;
     }
     cudaError_t e = li_launch_pdl(delta_chunk_solve_kernel<DP>, dim3(heads, chunks), dim3(kThreads), solve_smem<DP>(), stream, prep_qk, prep_g, v, (const int4*)seg,
-                                  wt, xt, pt, sums, heads, kv_heads, d, dv);
+                                  wm, xm, pt, sums, heads, kv_heads, dv);
     if (e == cudaSuccess)
-        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, dim3(ceil_div(dv, kSlice), heads, nruns), dim3(kThreads), carry_smem<DP>(), stream, prep_qk,
-                          (const int4*)seg, runs, wt, xt, sums, state, state_stride, s0, u, heads, kv_heads, d, dv);
+        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, dim3(ceil_div(dv, kSlice), heads, nruns), dim3(kCarryThreads), carry_smem<DP>(), stream, prep_qk,
+                          (const int4*)seg, runs, wm, xm, sums, state, state_stride, s0, u, heads, kv_heads, d, dv);
     if (e == cudaSuccess) {
         if (dtype == LI_F32)
             e = li_launch_pdl(delta_chunk_output_kernel<float, DP>, dim3(heads, chunks), dim3(kThreads), output_smem<DP>(), stream, prep_qk, (const int4*)seg, pt,
-                              sums, s0, u, out, (const float*)gate, gate_ld, gate_off, norm_w, eps, (float*)y, heads, kv_heads, d, dv);
+                              sums, s0, u, out, (const float*)gate, gate_ld, gate_off, norm_w, eps, (float*)y, heads, kv_heads, dv);
         else
             e = li_launch_pdl(delta_chunk_output_kernel<bf16, DP>, dim3(heads, chunks), dim3(kThreads), output_smem<DP>(), stream, prep_qk, (const int4*)seg, pt,
-                              sums, s0, u, out, (const bf16*)gate, gate_ld, gate_off, norm_w, eps, (bf16*)y, heads, kv_heads, d, dv);
+                              sums, s0, u, out, (const bf16*)gate, gate_ld, gate_off, norm_w, eps, (bf16*)y, heads, kv_heads, dv);
     }
     if (e != cudaSuccess) return li_fail("delta chunks: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("delta chunks");
@@ -498,11 +490,11 @@ int launch(const float* prep_qk, const float* prep_g, const float* v, float* sta
 }  // namespace
 
 // seg [chunks] quadruples (first token, end, chunk, slot), at most 64 tokens each; runs [nruns] triples (first chunk, chunks, slot).
-// Workspace, float: wt [chunks, heads, d, 64], xt [chunks, heads, dv, 64], pt [chunks, heads, 64, 64], sums [chunks, heads, 2, 64],
-// s0 [chunks, heads, d, dv], u [chunks, heads, 64, dv].  norm_w [heads dv] (may be NULL; dv at most 128): y [T, heads dv] in the run dtype takes
+// Workspace, float, with DP = 32, 64, 128 or 256 (the first that holds d) and dv rounded up to a multiple of 4: wm [chunks, heads, 64, DP],
+// xm [chunks, heads, 64, dv], pt [chunks, heads, 64, 64], sums [chunks, heads, 2, 64], s0 [chunks, heads, DP, dv], u [chunks, heads, 64, dv].  norm_w [heads dv] (may be NULL; dv at most 128): y [T, heads dv] in the run dtype takes
 // the normed and gated outputs, gate [T, gate_ld] from column gate_off; without it out [T, heads dv] float takes the outputs.
 LI_EXPORT int li_delta_chunks(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride, const int* seg, int chunks,
-                              const int* runs, int nruns, float* wt, float* xt, float* pt, float* sums, float* s0, float* u, float* out, const void* gate,
+                              const int* runs, int nruns, float* wm, float* xm, float* pt, float* sums, float* s0, float* u, float* out, const void* gate,
                               int dtype, int gate_ld, int gate_off, const float* norm_w, float eps, void* y, int heads, int kv_heads, int d, int dv,
                               cudaStream_t stream) {
     LI_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && d > 0 && d <= 256 && dv > 0, "delta chunks: %d heads on %d key heads of %d x %d (keys of at most 256)",
@@ -511,11 +503,11 @@ LI_EXPORT int li_delta_chunks(const float* prep_qk, const float* prep_g, const f
     LI_REQUIRE(norm_w != nullptr ? (dv <= kCols && y != nullptr && gate != nullptr && gate_off >= 0 && gate_off + heads * dv <= gate_ld) : out != nullptr,
                "delta chunks: outputs of %d columns a head, gate at column %d of %d", dv, gate_off, gate_ld);
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "delta chunks: unknown dtype %d", dtype);
-    LI_REQUIRE(((uintptr_t)prep_qk | (uintptr_t)prep_g | (uintptr_t)seg | (uintptr_t)wt | (uintptr_t)xt | (uintptr_t)pt | (uintptr_t)sums | (uintptr_t)s0 | (uintptr_t)u) % 16 == 0,
+    LI_REQUIRE(((uintptr_t)prep_qk | (uintptr_t)prep_g | (uintptr_t)seg | (uintptr_t)wm | (uintptr_t)xm | (uintptr_t)pt | (uintptr_t)sums | (uintptr_t)s0 | (uintptr_t)u) % 16 == 0,
                "delta chunks: an operand is not on a 16-byte boundary");
     if (chunks == 0 || nruns == 0) return 0;
 #define LI_CHUNKS(DP)                                                                                                                                  \
-    return launch<DP>(prep_qk, prep_g, v, state, state_stride, seg, chunks, runs, nruns, wt, xt, pt, sums, s0, u, out, gate, dtype, gate_ld, gate_off, norm_w, eps, \
+    return launch<DP>(prep_qk, prep_g, v, state, state_stride, seg, chunks, runs, nruns, wm, xm, pt, sums, s0, u, out, gate, dtype, gate_ld, gate_off, norm_w, eps, \
                       y, heads, kv_heads, d, dv, stream)
     if (d <= 32) LI_CHUNKS(32);
     if (d <= 64) LI_CHUNKS(64);

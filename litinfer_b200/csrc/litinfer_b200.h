@@ -206,14 +206,24 @@ int li_delta_scan(const float* prep_qk, const float* prep_g, const float* v, flo
     cudaStream_t stream);
 
 /* The same rule with one decay a head for long portions, in chunks of at most 64 tokens as matrix products in float (delta_chunks.cu):
- * seg [chunks] quadruples (first token, end, chunk, slot), runs [nruns] triples (first chunk, chunks, slot).  Workspace, float: wt
- * [chunks, heads, d, 64], xt [chunks, heads, dv, 64], pt [chunks, heads, 64, 64], sums [chunks, heads, 2, 64], s0 [chunks, heads, d, dv], u
- * [chunks, heads, 64, dv].  norm_w [heads dv] (may be NULL; dv at most 128): y [T, heads dv] in the run dtype takes each head's output
+ * seg [chunks] quadruples (first token, end, chunk, slot), runs [nruns] triples (first chunk, chunks, slot).  Workspace, float, with
+ * DP = 32, 64, 128 or 256 and dv rounded up to a multiple of 4: wm [chunks, heads, 64, DP], xm [chunks, heads, 64, dv], pt
+ * [chunks, heads, 64, 64], sums [chunks, heads, 2, 64], s0 [chunks, heads, DP, dv], u [chunks, heads, 64, dv].  norm_w [heads dv] (may be NULL; dv at most 128): y [T, heads dv] in the run dtype takes each head's output
  * divided by its root mean square (eps), times norm_w, times silu(gate [T, gate_ld] from column gate_off); else out [T, heads dv] float. */
 int li_delta_chunks(const float* prep_qk, const float* prep_g, const float* v, float* state, long long state_stride,
-    const int* seg, int chunks, const int* runs, int nruns, float* wt, float* xt, float* pt, float* sums, float* s0,
+    const int* seg, int chunks, const int* runs, int nruns, float* wm, float* xm, float* pt, float* sums, float* s0,
     float* u, float* out, const void* gate, int dtype, int gate_ld, int gate_off, const float* norm_w, float eps, void* y,
     int heads, int kv_heads, int d, int dv, cudaStream_t stream);
+
+/* One token a sequence under the rule with one decay a head, from the projections to the gated norm, as one kernel (delta_step.cu): proj
+ * [S, stride] holds the convolution's channels q | k | v from column col0, beta's, the decays' and the gate's inputs from b_off, a_off,
+ * g_off; the states and the convolution's inputs (at state_off) move on; y [S, heads dv] takes o / sqrt(mean(o^2) + eps) * norm_w *
+ * silu(gate).  accepts: 1 if the sizes fit. */
+int li_delta_step_accepts(int heads, int kv_heads, int d, int dv);
+int li_delta_step(const void* proj, int dtype, int stride, int col0, int b_off, int a_off, int g_off, const float*
+    conv_w, int taps, float* state, long long state_stride, long long state_off, const int* slots, const float* dt_bias,
+    const float* A_log, float q_scale, float unit_eps, const float* norm_w, float eps, void* y, int S, int heads, int
+    kv_heads, int d, int dv, cudaStream_t stream);
 
 /* Per channel c a state S [N]: S = exp(dt_c A[c, :]) S + dt_c x_c B, y_c = (S . C + D[c] x_c) silu(z_c), with
  * dt = softplus(dt_raw) (float, [T, dt_stride]), A = -exp(A_log) [inner, N]; x at column x_off of [T, x_stride], B and C

@@ -584,6 +584,125 @@ delta_prepare_kernel(const T* __restrict__ proj, int stride, int col0, int b_off
     }
 }
 
+// The same for many tokens and one decay a head: a warp takes eight consecutive tokens of a unit (a key head, or a head's values), a lane
+// four neighbouring channels, so that the taps are read once and every projected row once (a token's older inputs are the window
+// of the rows before it).  Keys of at most 128, channels in whole groups of four on 8-byte (bfloat16) or 16-byte (float) boundaries.
+constexpr int kRunTokens = 8;
+
+__device__ __forceinline__ void load_four(float (&v)[4], const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(u.x << 16), v[1] = __uint_as_float(u.x & 0xffff0000u), v[2] = __uint_as_float(u.y << 16), v[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+__device__ __forceinline__ void load_four(float (&v)[4], const float* p) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    v[0] = u.x, v[1] = u.y, v[2] = u.z, v[3] = u.w;
+}
+
+// Four channels of the convolution, with silu, for the tokens t0 .. t0 + n - 1 of the step: each(i, values) is called in order.
+template <typename T, int TAPS, typename Each>
+__device__ __forceinline__ void conv_run(const T* __restrict__ proj, int stride, int col, int c, int C, const float* __restrict__ conv_w, const float* __restrict__ state,
+                                         long long state_stride, long long state_off, const int* __restrict__ q_start, const int* __restrict__ seq_of_token,
+                                         const int* __restrict__ slots, int t0, int n, bool real, Each each) {
+    float w[4][TAPS], win[TAPS][4];
+    float rows[kRunTokens][4];
+    if (real) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k) w[j][k] = conv_w[(size_t)(c + j) * TAPS + k];
+#pragma unroll
+        for (int i = 0; i < kRunTokens; ++i)
+            if (i < n) load_four(rows[i], proj + (size_t)(t0 + i) * stride + col + c);
+    }
+#pragma unroll
+    for (int i = 0; i < kRunTokens; ++i) {
+        if (i >= n) break;                                              // (the same for the whole warp)
+        const int t = t0 + i, s = seq_of_token[t], q0 = q_start[s];
+        float out[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        if (real) {
+            if (i == 0 || t == q0) {
+                // the inputs before this token: of its own portion, or from the request's state
+                const float* st = state + (size_t)slots[s] * state_stride + state_off;
+#pragma unroll
+                for (int k = 0; k + 1 < TAPS; ++k) {
+                    const int before = t - q0 - (TAPS - 1) + k;
+                    if (before >= 0) {
+                        load_four(win[k], proj + (size_t)(q0 + before) * stride + col + c);
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) win[k][j] = st[(size_t)(TAPS - 1 + before) * C + c + j];
+                    }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                float acc = 0.0f;
+#pragma unroll
+                for (int k = 0; k + 1 < TAPS; ++k) acc = fmaf(w[j][k], win[k][j], acc);
+                out[j] = silu_f(fmaf(w[j][TAPS - 1], rows[i][j], acc));
+#pragma unroll
+                for (int k = 0; k + 2 < TAPS; ++k) win[k][j] = win[k + 1][j];
+                if (TAPS > 1) win[TAPS - 2][j] = rows[i][j];
+            }
+        }
+        each(i, out);
+    }
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+delta_prepare_run_kernel(const T* __restrict__ proj, int stride, int col0, int b_off, int a_off, const float* __restrict__ conv_w, const float* __restrict__ state,
+                         long long state_stride, long long state_off, const int* __restrict__ q_start, const int* __restrict__ seq_of_token,
+                         const int* __restrict__ slots, const float* __restrict__ dt_bias, const float* __restrict__ A_log, float q_scale, float unit_eps,
+                         float* __restrict__ prep_qk, float* __restrict__ prep_g, float* __restrict__ v_out, int total, int heads, int kv_heads, int d, int dv, int DP) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int units = kv_heads + heads;
+    const int id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int run = id / units, u = id - run * units, t0 = run * kRunTokens;
+    if (t0 >= total) return;
+    const int n = min(kRunTokens, total - t0), lane = threadIdx.x & 31;
+    const int C = 2 * kv_heads * d + heads * dv;
+    if (u < kv_heads) {
+        const int c = 4 * lane;
+        const bool real = c < d;
+        float q[kRunTokens][4];
+        conv_run<T, TAPS>(proj, stride, col0, u * d + c, C, conv_w, state, state_stride, state_off, q_start, seq_of_token, slots, t0, n, real,
+                          [&](int i, const float (&o)[4]) {
+#pragma unroll
+                              for (int j = 0; j < 4; ++j) q[i][j] = o[j];
+                          });
+        conv_run<T, TAPS>(proj, stride, col0, kv_heads * d + u * d + c, C, conv_w, state, state_stride, state_off, q_start, seq_of_token, slots, t0, n, real,
+                          [&](int i, const float (&k)[4]) {
+                              float qq = 0.0f, kk = 0.0f, qk = 0.0f;
+#pragma unroll
+                              for (int j = 0; j < 4; ++j) qq = fmaf(q[i][j], q[i][j], qq), kk = fmaf(k[j], k[j], kk), qk = fmaf(q[i][j], k[j], qk);
+                              qq = warp_sum(qq), kk = warp_sum(kk), qk = warp_sum(qk);
+                              const float fq = q_scale / sqrtf(qq + unit_eps), fk = 1.0f / sqrtf(kk + unit_eps);
+                              float* row = prep_qk + ((size_t)(t0 + i) * kv_heads + u) * (2 * DP + 4);
+                              if (c < DP) {
+                                  *reinterpret_cast<float4*>(row + c) = make_float4(q[i][0] * fq, q[i][1] * fq, q[i][2] * fq, q[i][3] * fq);
+                                  *reinterpret_cast<float4*>(row + DP + c) = make_float4(k[0] * fk, k[1] * fk, k[2] * fk, k[3] * fk);
+                              }
+                              if (lane == 0) row[2 * DP] = qk * fq * fk;
+                          });
+        return;
+    }
+    const int h = u - kv_heads;
+    if (lane < n) {
+        const T* row = proj + (size_t)(t0 + lane) * stride;
+        const float lg = -expf(A_log[h]) * softplus_f(to_float(row[a_off + h]) + dt_bias[h]);
+        *reinterpret_cast<float4*>(prep_g + ((size_t)(t0 + lane) * heads + h) * 4) = make_float4(expf(lg), sigmoid_f(to_float(row[b_off + h])), lg, 0.0f);
+    }
+    for (int c0 = 0; c0 < dv; c0 += 128) {
+        const int c = c0 + 4 * lane;
+        conv_run<T, TAPS>(proj, stride, col0, 2 * kv_heads * d + h * dv + c, C, conv_w, state, state_stride, state_off, q_start, seq_of_token, slots, t0, n, c < dv,
+                          [&](int i, const float (&o)[4]) {
+                              if (c < dv) *reinterpret_cast<float4*>(v_out + (size_t)(t0 + i) * heads * dv + h * dv + c) = make_float4(o[0], o[1], o[2], o[3]);
+                          });
+    }
+}
+
 // The walk itself.  A column of S moves on by itself here too (u[c] depends on column c alone), so it is the walk of
 // gla_scan_kernel: a warp holds WC columns (eight, four or two), each lane E neighbouring key channels of all of them; with few
 // sequences and heads the columns are spread over more warps, since a token's chain of instructions is as long as its warp has
@@ -1300,6 +1419,29 @@ LI_EXPORT int li_delta_prepare(const void* proj, int dtype, int stride, int col0
     LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "delta rule: unknown dtype %d", dtype);
     if (T == 0) return 0;
     const int DP = 32 * delta_elements(d);
+    const int four = dtype == LI_F32 ? 16 : 8;
+    if (za == nullptr && !shift && T >= 4 * kRunTokens && d <= 128 && d % 4 == 0 && dv % 4 == 0 && taps >= 2 && taps <= 4 && stride % 4 == 0 && col0 % 4 == 0 &&
+        (uintptr_t)proj % four == 0 && (uintptr_t)prep_qk % 16 == 0 && (uintptr_t)v % 16 == 0 && (uintptr_t)prep_g % 16 == 0) {
+        const long long jobs = (long long)ceil_div(T, kRunTokens) * (kv_heads + heads);
+        LI_REQUIRE(jobs < (1LL << 31) - 4, "delta rule: too many tokens for one launch");
+        cudaError_t er;
+#define LI_PREPARE_RUN(TT, TAPS_)                                                                                                                          \
+    er = li_launch_pdl(delta_prepare_run_kernel<TT, TAPS_>, dim3((unsigned)ceil_div_ll(jobs, 4)), dim3(128), 0, stream, (const TT*)proj, stride, col0, b_off, a_off, \
+                       conv_w, (const float*)state, state_stride, state_off, q_start, seq_of_token, slots, dt_bias, A_log, q_scale, unit_eps, prep_qk, prep_g, v, T, heads, kv_heads, d, \
+                       dv, DP)
+        if (dtype == LI_F32) {
+            if (taps == 4) LI_PREPARE_RUN(float, 4);
+            else if (taps == 3) LI_PREPARE_RUN(float, 3);
+            else LI_PREPARE_RUN(float, 2);
+        } else {
+            if (taps == 4) LI_PREPARE_RUN(bf16, 4);
+            else if (taps == 3) LI_PREPARE_RUN(bf16, 3);
+            else LI_PREPARE_RUN(bf16, 2);
+        }
+#undef LI_PREPARE_RUN
+        if (er != cudaSuccess) return li_fail("delta_prepare: launch failed: %s", cudaGetErrorString(er));
+        return li_check_launch("delta_prepare (runs of tokens)");
+    }
     const long long warps = (long long)T * (kv_heads + (za ? 2 : 1) * heads);
     const dim3 grid((unsigned)ceil_div_ll(warps, 4));
     cudaError_t e;

@@ -960,17 +960,46 @@ def delta_chunks(prep_qk: torch.Tensor, prep_g: torch.Tensor, v32: torch.Tensor,
         raise KernelError("delta_chunks: the state is too small")
     if n == 0:
         return
-    fused = vdim <= 128
-    wt, xt, pt, sums, s0, u = (torch.empty((n, heads) + s, dtype=torch.float32, device=dev)
-                               for s in ((dim, C), (vdim, C), (C, C), (2, C), (dim, vdim), (C, vdim)))
+    fused, VP = vdim <= 128, -(-vdim // 4) * 4
+    wm, xm, pt, sums, s0, u = (torch.empty((n, heads) + s, dtype=torch.float32, device=dev)
+                               for s in ((C, DP), (C, VP), (C, C), (2, C), (DP, VP), (C, VP)))
     out32 = None if fused else torch.empty((T, heads * vdim), dtype=torch.float32, device=dev)
-    _check(library().li_delta_chunks(_p(prep_qk), _p(prep_g), _p(v32), st, stride, _p(chunks.seg), _i(n), _p(chunks.runs), _i(chunks.nruns), _p(wt), _p(xt), _p(pt),
+    _check(library().li_delta_chunks(_p(prep_qk), _p(prep_g), _p(v32), st, stride, _p(chunks.seg), _i(n), _p(chunks.runs), _i(chunks.nruns), _p(wm), _p(xm), _p(pt),
                                      _p(sums), _p(s0), _p(u), _p(out32), _p(gate), _i(_dt(y)), _i(gate.shape[1]), _i(int(gate_col)),
                                      _p(weight if fused else None), _f(eps), _p(y), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream(y)), "delta_chunks")
     global launches
     launches += 2                     # (three kernels)
     if not fused:
         gated_rmsnorm(out32, gate, gate_col, weight, eps, heads, False, y, gate_act="silu")
+
+
+def delta_step_accepts(heads: int, kv_heads: int, dim: int, vdim: int) -> bool:
+    """Whether :func:`delta_step` takes heads of these sizes."""
+    return bool(library().li_delta_step_accepts(_i(heads), _i(kv_heads), _i(dim), _i(vdim)))
+
+
+def delta_step(proj: torch.Tensor, col: int, b_col: int, a_col: int, g_col: int, conv_w: torch.Tensor, state: torch.Tensor, state_off: int, slots: torch.Tensor,
+               dt_bias: torch.Tensor, A_log: torch.Tensor, weight: torch.Tensor, eps: float, y: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
+               unit_eps: float = 1e-6) -> None:
+    """A step of single tokens under the gated delta rule with one decay a head as one kernel: :func:`delta_prepare` (with ``shift``),
+    :func:`delta_scan` and :func:`gated_rmsnorm` with a silu gate (the columns of ``proj`` from ``g_col``), row s of ``proj`` the token of the
+    sequence in slot ``slots[s]``."""
+    S = proj.shape[0]
+    C = 2 * kv_heads * dim + heads * vdim
+    _need(proj, "projections")
+    _need(conv_w, "convolution weight", torch.float32, (C, conv_w.shape[1]))
+    taps = conv_w.shape[1]
+    _need(slots, "state slots", torch.int32, (S,))
+    for t, n in ((dt_bias, "bias of the decays' input"), (A_log, "A_log")):
+        _need(t, n, torch.float32, (heads,))
+    _need(weight, "rmsnorm weight", torch.float32, (heads * vdim,))
+    _need(y, "mixer output", proj.dtype, (S, heads * vdim))
+    st, stride, off = _state_args(state, state_off)
+    if state_off < heads * dim * vdim or state_off + (taps - 1) * C > state.shape[1]:
+        raise KernelError("delta_step: the state is too small")
+    _check(library().li_delta_step(_p(proj), _i(_dt(proj)), _i(proj.shape[1]), _i(int(col)), _i(int(b_col)), _i(int(a_col)), _i(int(g_col)), _p(conv_w), _i(taps), st,
+                                   stride, off, _p(slots), _p(dt_bias), _p(A_log), _f(float(dim) ** -0.5), _f(float(unit_eps)), _p(weight), _f(float(eps)), _p(y),
+                                   _i(S), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream(y)), "delta_step")
 
 
 def channel_scan(x: torch.Tensor, x_col: int, bc: torch.Tensor, b_col: int, c_col: int, dt32: torch.Tensor, z: torch.Tensor, z_col: int,
@@ -1577,7 +1606,7 @@ _TIMED = ("embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add
           "rope_kv_write", "linear_rope_kv", "rope_table", "paged_attention", "swiglu", "argmax", "sample", "gather_rows", "scale_inplace",
           "logit_cap", "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift",
           "ssm_scan", "decay_scan", "gated_rmsnorm", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route",
-          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "delta_chunks", "gelu_token_rows",
+          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "delta_chunks", "delta_step", "gelu_token_rows",
           "mul_sigmoid", "polynorm")
 if profile.enabled:
     for _name in _TIMED:

@@ -139,12 +139,18 @@ class GatedDeltaRule(Mixer):
         T, dev = proj.shape[0], proj.device
         za = self.decay_out(proj, out_dtype=torch.float32) if self.decay_out is not None else None      # the softplus' input, bias added
         gate, gate_col = (self.gate_out(proj), 0) if self.gate_out is not None else (proj, col + self.g_col)
+        single = ctx.max_q_len == 1                 # a step of single tokens: the convolution moves its state on itself
+        if single and self.head_decay and self.full_gate and K.delta_step_accepts(self.heads, self.kv_heads, self.dim, self.value_dim):
+            # one token a sequence: everything up to the output map is one kernel
+            y = torch.empty((T, self.vv), dtype=self.dtype, device=dev)
+            K.delta_step(proj, col, col + self.b_col, col + self.a_col, gate_col, self.conv_w, cache.state, self.scan_elements, ctx.state_slots, self.dt_bias,
+                         self.A_log, self.norm_weight, self.eps, y, self.heads, self.kv_heads, self.dim, self.value_dim, UNIT_EPS)
+            return self.out(y)
         # what does not depend on the state, once per token: convolution and silu, unit vectors, decays, beta
         DP = K.delta_row_elements(self.dim)
         prep_qk = torch.empty((T, self.kv_heads, 2 * DP + 4), dtype=torch.float32, device=dev)
         prep_g = torch.empty((T, self.heads, 4 if self.head_decay else DP + 4), dtype=torch.float32, device=dev)
         v32 = torch.empty((T, self.vv), dtype=torch.float32, device=dev)
-        single = ctx.max_q_len == 1                 # a step of single tokens: the convolution moves its state on itself
         K.delta_prepare(proj, col, col + self.b_col, self.conv_w, cache.state, self.scan_elements, ctx.q_start, ctx.seq_of_token, ctx.state_slots, za, 0,
                         self.A_log, prep_qk, prep_g, v32, self.heads, self.kv_heads, self.dim, self.value_dim, UNIT_EPS, shift=single,
                         a_col=col + self.a_col, dt_bias=self.dt_bias)

@@ -842,6 +842,21 @@ def delta_scan(prep_qk, prep_g, v32, state, q_start, slots, out32, heads, kv_hea
             out32[t] = torch.einsum("hdv,hd->hv", S, q).reshape(heads * vdim)
 
 
+def delta_step_accepts(heads, kv_heads, dim, vdim):
+    return dim <= 256
+
+
+def delta_step(proj, col, b_col, a_col, g_col, conv_w, state, state_off, slots, dt_bias, A_log, weight, eps, y, heads, kv_heads, dim, vdim, unit_eps=1e-6):
+    """Preparation, walk, norm and gate of a step of single tokens."""
+    S, DP, dev = proj.shape[0], delta_row_elements(dim), proj.device
+    qk, g, v, o = (torch.zeros(s, device=dev) for s in ((S, kv_heads, 2 * DP + 4), (S, heads, 4), (S, heads * vdim), (S, heads * vdim)))
+    starts = torch.arange(S + 1, dtype=torch.int32, device=dev)
+    delta_prepare(proj, col, b_col, conv_w, state, state_off, starts, starts[:S], slots, None, 0, A_log, qk, g, v, heads, kv_heads, dim, vdim, unit_eps, True,
+                  a_col=a_col, dt_bias=dt_bias)
+    delta_scan(qk, g, v, state, starts, slots, o, heads, kv_heads, dim, vdim)
+    gated_rmsnorm(o, proj, g_col, weight, eps, heads, False, y, gate_act="silu")
+
+
 def delta_chunks(prep_qk, prep_g, v32, state, chunks, heads, kv_heads, dim, vdim, gate, gate_col, weight, eps, y):
     """The walk, token by token, over the chunks' sequences; then the norm and the gate."""
     out32 = torch.zeros_like(v32)
@@ -942,7 +957,7 @@ def table_gather(resident, updates, slots, out, trash_page):
             out[s, b] = resident[slot, b] if b < cols else trash_page
 
 
-ALL = ["gelu_token_rows", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_chunks", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
+ALL = ["gelu_token_rows", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_chunks", "delta_step", "delta_step_accepts", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
        "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift", "ssm_scan",
        "decay_scan", "gated_rmsnorm", "table_gather", "gather_rows", "scale_inplace", "logit_cap", "rope_table", "linear_scaled_accepts", "linear_add_scaled_parts", "linear_add_scaled", "apply_row_scale", "linear_rope_kv", "interleave_gate_up", "embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add", "linear", "rope_kv_write",
        "paged_attention", "swiglu", "argmax", "sample"]

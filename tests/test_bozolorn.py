@@ -833,6 +833,19 @@ def test_delta_rule_with_one_decay_a_head(heads, kv, d, dv, taps, dtype):
             res.append((qk[..., :2 * DP + 1], g[..., :2], v, o, state))
         for a, b, what in zip(res[0], res[1], ("q and k", "decay and beta", "values", "outputs", "state")):
             _close(a, b, "float32", f"{what}, portions of {lens}", 1e-4)
+    # one token a sequence, from the projections to the gated norm, as one kernel; twice, so that the second reads what the first left
+    proj = torch.randn(4, width + heads * dv).to(dev, dt)
+    w = 1 + 0.2 * torch.randn(heads * dv, device=dev)
+    assert K.delta_step_accepts(heads, kv, d, dv)
+    res = []
+    for F in (K, R):
+        state, y = first.clone(), torch.empty(4, heads * dv, dtype=dt, device=dev)
+        for again in range(2):
+            F.delta_step(proj if not again else (0.5 * proj), col, col + C, col + C + heads, width, conv_w, state, heads * d * dv, i32([2, 0, 4, 1]), dt_bias, A_log, w,
+                         1e-5, y, heads, kv, d, dv)
+        res.append((y, state))
+    _close(res[0][0], res[1][0], dtype, "outputs of single tokens", 2e-4 if dtype == "float32" else 2e-2)
+    _close(res[0][1], res[1][1], "float32", "state after single tokens", 1e-5)
 
 
 @pytest.mark.gpu
