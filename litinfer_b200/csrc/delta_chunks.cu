@@ -21,7 +21,6 @@ namespace {
 constexpr int kC = 64;              // tokens of a chunk
 constexpr int kLA = kC + 4;         // a row of a [.., tokens] tile in shared memory
 constexpr int kThreads = 256;
-constexpr int kCarryThreads = 512;
 constexpr int kSlice = 16;          // value columns a block of the carry takes
 constexpr int kCols = 128;          // value columns a block of the output takes at a time
 constexpr int kRowsB = 16;          // rows of its second operand that it stages at a time
@@ -195,151 +194,178 @@ delta_chunk_solve_kernel(const float* __restrict__ prep_qk, const float* __restr
     pdl_launch_dependents();
 }
 
-template <int DP>
-__host__ __device__ constexpr int carry_buffers() { return DP <= 128 ? 2 : 1; }
-template <int DP>
-__host__ __device__ constexpr int carry_buffer() { return kC * (DP + 4) + kC * DP + kC * kSlice + 2 * kC; }
-constexpr int kCarryScratch = kCarryThreads * 16;
+constexpr int kCarryScratch = kThreads * 16;
+constexpr int kUs = kSlice + 2;     // numbers (twice each) of a row of U in shared memory
 template <int DP>
 __host__ __device__ constexpr size_t carry_smem() {
-    return ((size_t)carry_buffers<DP>() * carry_buffer<DP>() + kSlice * (DP + 4) + kCarryScratch + 2 * kC * kSlice) * sizeof(float);
+    return ((size_t)kC * (DP + 4) + kC * (DP + 16) + 2 * (kC * kSlice + 2 * kC) + kSlice * (DP + 4) + kCarryScratch + 2 * kC * kUs) * sizeof(float);
 }
 
-// runs: triples (first chunk, chunks, slot).  s0 [chunk, head, DP, dv]: the state before every chunk; u [chunk, head, 64, dv].
+// runs: triples (first chunk, chunks, slot).  s0 [chunk, head, DP, dv]: the state before every chunk; u [chunk, head, 64, dv].  A block
+// takes 16 columns of a head's values.  W of the next chunk is on its way from the moment this chunk's W has been used, K likewise, so
+// that one buffer each is enough and two blocks can share a multiprocessor.  Both products give a thread eight rows by four columns,
+// summed over a part of the third index; lanes 16 apart hold neighbouring parts and add up first, the rest goes through shared memory.
 template <int DP>
-__global__ void __launch_bounds__(kCarryThreads, 1)
+__global__ void __launch_bounds__(kThreads, DP <= 128 ? 2 : 1)
 delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restrict__ seg, const int* __restrict__ runs, const float* __restrict__ wm,
                          const float* __restrict__ xm, const float* __restrict__ sums, float* __restrict__ state, long long state_stride,
                          float* __restrict__ s0, float* __restrict__ u, int heads, int kv_heads, int d, int dv) {
-    constexpr int RQ = 2 * DP + 4, LD = DP + 4, NB = carry_buffers<DP>(), SPLIT = kCarryThreads / DP;
+    constexpr int RQ = 2 * DP + 4, LD = DP + 4, LK = DP + 16;
+    constexpr int NW = DP / 32, PH = 8 / NW, TB = DP / 2;               // K^T U: warps side by side over the key channels, parts, tiles
+    constexpr int kXBuf = kC * kSlice + 2 * kC;
     extern __shared__ __align__(16) float smem[];
-    float* S = smem + NB * carry_buffer<DP>();          // [16][LD]: a column of the state after the other
+    float* W = smem;                                    // [64][LD]
+    float* Kb = W + kC * LD;                            // [64][LK]
+    float* Xs = Kb + kC * LK;                           // [2]: X [64][16], then sums [2][64]
+    float* S = Xs + 2 * kXBuf;                          // [16][LD]: a column of the state after the other
     float* red = S + kSlice * LD;
-    float2* Us = reinterpret_cast<float2*>(red + kCarryScratch);        // [64][16]: U with the decay to the chunk's end, every number twice
-    const int tid = threadIdx.x;
+    float2* Us = reinterpret_cast<float2*>(red + kCarryScratch);        // [64][kUs]: U with the decay to the chunk's end, every number twice
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, ct = lane & 3, quarter = (lane >> 2) & 3, pb = lane >> 4;
     const int h = blockIdx.y, hk = h / (heads / kv_heads), c0 = blockIdx.x * kSlice, dvp = padded(dv);
     pdl_wait();
     const int first = runs[3 * blockIdx.z], count = runs[3 * blockIdx.z + 1], slot = runs[3 * blockIdx.z + 2];
     float* st = state + (size_t)slot * state_stride + (size_t)h * dv * d;
-    auto stage = [&](int b, int chunk) {
-        float* W = smem + b * carry_buffer<DP>();       // [64][LD]
-        float* Kb = W + kC * LD;                        // [64][DP]
-        float* X = Kb + kC * DP;                        // [64][16]
-        float* cm = X + kC * kSlice;                    // [2][64]
-        const int4 sg = seg[chunk];
-        const int n = min(sg.y - sg.x, kC);
-        const size_t unit = (size_t)chunk * heads + h;
-        for (int idx = tid; idx < kC * (DP / 4); idx += kCarryThreads) {
-            const int t = idx / (DP / 4), i = idx - t * (DP / 4);
-            copy16(W + t * LD + 4 * i, wm + (unit * kC + t) * DP + 4 * i, true);
-            copy16(Kb + t * DP + 4 * i, prep_qk + ((size_t)(sg.x + (t < n ? t : 0)) * kv_heads + hk) * RQ + DP + 4 * i, t < n);
+    auto stage_w = [&](int j) {
+        if (j < count) {
+            const size_t unit = (size_t)(first + j) * heads + h;
+            float* X = Xs + (j & 1) * kXBuf;
+#pragma unroll 4
+            for (int idx = tid; idx < kC * (DP / 4); idx += kThreads) {
+                const int t = idx / (DP / 4), i = idx - t * (DP / 4);
+                copy16(W + t * LD + 4 * i, wm + unit * kC * DP + 4 * idx, true);
+            }
+            {
+                const int t = tid >> 2, c = 4 * (tid & 3);
+                copy16(X + t * kSlice + c, xm + (unit * kC + t) * dvp + (c0 + c < dvp ? c0 + c : 0), c0 + c < dvp);
+            }
+            if (tid < 2 * kC / 4) copy16(X + kC * kSlice + 4 * tid, sums + unit * 2 * kC + 4 * tid, true);
         }
-        if (tid < kC * (kSlice / 4)) {
-            const int t = tid / (kSlice / 4), c = 4 * (tid - t * (kSlice / 4));
-            copy16(X + t * kSlice + c, xm + (unit * kC + t) * dvp + (c0 + c < dvp ? c0 + c : 0), c0 + c < dvp);
-        }
-        if (tid < 2 * kC / 4) copy16(cm + 4 * tid, sums + unit * 2 * kC + 4 * tid, true);
+        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    stage(0, first);
-    for (int idx = tid; idx < DP * kSlice; idx += kCarryThreads) {
+    auto stage_k = [&](int j) {
+        if (j < count) {
+            const int4 sg = seg[first + j];
+            const int n = min(sg.y - sg.x, kC);
+            const float* from = prep_qk + ((size_t)sg.x * kv_heads + hk) * RQ + DP;
+#pragma unroll 4
+            for (int idx = tid; idx < kC * (DP / 4); idx += kThreads) {
+                const int t = idx / (DP / 4), i = idx - t * (DP / 4);
+                copy16(Kb + t * LK + 4 * i, from + (size_t)(t < n ? t : 0) * kv_heads * RQ + 4 * i, t < n);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage_w(0);
+    stage_k(0);
+    for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
         const int c = idx / DP, k = idx - c * DP;
         S[c * LD + k] = (k < d && c0 + c < dv) ? st[(size_t)(c0 + c) * d + k] : 0.0f;
     }
     for (int j = 0; j < count; ++j) {
-        const int chunk = first + j, b = j % NB;
-        copies_done();
-        __syncthreads();                                 // this chunk's rows are here, and everybody has left the other buffer
-        if (NB > 1 && j + 1 < count) stage(b ^ 1, chunk + 1);
-        const float* W = smem + b * carry_buffer<DP>();
-        const float* Kb = W + kC * LD;
-        const float* X = Kb + kC * DP;
+        const size_t unit = (size_t)(first + j) * heads + h;
+        const float* X = Xs + (j & 1) * kXBuf;
         const float* cm = X + kC * kSlice;
-        const size_t unit = (size_t)chunk * heads + h;
+        asm volatile("cp.async.wait_group 1;" ::: "memory");        // W and X of this chunk (its K may still be on its way)
+        __syncthreads();
         // the state before this chunk, for the outputs
-        for (int idx = tid; idx < DP * (kSlice / 4); idx += kCarryThreads) {
-            const int k = idx / (kSlice / 4), c = 4 * (idx - k * (kSlice / 4));
+        for (int idx = tid; idx < DP * 4; idx += kThreads) {
+            const int k = idx >> 2, c = 4 * (idx & 3);
             if (c0 + c < dvp)
                 *reinterpret_cast<float4*>(s0 + (unit * DP + k) * dvp + c0 + c) = make_float4(S[c * LD + k], S[(c + 1) * LD + k], S[(c + 2) * LD + k], S[(c + 3) * LD + k]);
         }
-        // W S: tokens tt + 16 i by columns ct + 4 q a thread, an eighth of the key channels each
+        // W S: tokens tt + 8 i by columns ct + 4 q a thread, an eighth of the key channels each
         {
-            const int part = tid >> 6, tile = tid & 63, ct = tile & 3, tt = tile >> 2;
-            float2 acc[4][4];
+            const int tt = quarter + 4 * (warp & 1), ph = warp >> 1, part = 2 * ph + pb;
+            float2 acc[8][4];
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+            for (int i = 0; i < 8; ++i)
 #pragma unroll
                 for (int q = 0; q < 4; ++q) acc[i][q] = make_float2(0.0f, 0.0f);
+            const float* w0 = W + tt * LD + part * (DP / 8);
+            const float* sp = S + ct * LD + part * (DP / 8);
+#pragma unroll 1
+            for (int k = 0; k < DP / 8; k += 4) {
+                float4 s[4];
 #pragma unroll
-            for (int k = part * (DP / 8); k < (part + 1) * (DP / 8); k += 4) {
-                float4 w[4], s[4];
+                for (int q = 0; q < 4; ++q) s[q] = ld4(sp + 4 * q * LD + k);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) w[i] = ld4(W + (tt + 16 * i) * LD + k);
+                for (int i = 0; i < 8; ++i) {
+                    const float4 w = ld4(w0 + 8 * i * LD + k);
 #pragma unroll
-                for (int q = 0; q < 4; ++q) s[q] = ld4(S + (ct + 4 * q) * LD + k);
-#pragma unroll
-                for (int i = 0; i < 4; ++i)
-#pragma unroll
-                    for (int q = 0; q < 4; ++q) acc[i][q] = dot4(w[i], s[q], acc[i][q]);
+                    for (int q = 0; q < 4; ++q) acc[i][q] = dot4(w, s[q], acc[i][q]);
+                }
             }
+            float* to = red + (ph * 32 + 16 * pb) * 32 + ct + 4 * tt;
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int q = 0; q < 4; ++q) red[(part * 16 + i * 4 + q) * 64 + tile] = acc[i][q].x + acc[i][q].y;
+            for (int e = 0; e < 16; ++e) {
+                // this lane keeps rows i = 4 pb .. 4 pb + 3; the other half's go to the lane 16 away
+                const float2 a = acc[e >> 2][e & 3], b = acc[4 + (e >> 2)][e & 3];
+                const float lo = a.x + a.y, hi = b.x + b.y;
+                const float other = __shfl_xor_sync(0xffffffffu, pb ? lo : hi, 16);
+                to[e * 32] = (pb ? hi : lo) + other;
+            }
         }
         __syncthreads();
+        stage_w(j + 1);
 #pragma unroll
-        for (int o = tid; o < kC * kSlice; o += kCarryThreads) {
-            const int iq = o >> 6, tile = o & 63, t = (tile >> 2) + 16 * (iq >> 2), c = (tile & 3) + 4 * (iq & 3);
-            float sum = 0.0f;
-#pragma unroll
-            for (int part = 0; part < 8; ++part) sum += red[part * 1024 + o];
-            const float val = X[t * kSlice + c] - sum;
+        for (int o = tid; o < kC * kSlice; o += kThreads) {
+            const int e = o >> 5, tile = o & 31, t = (tile >> 2) + 8 * (e >> 2), c = (tile & 3) + 4 * (e & 3);
+            const float val = X[t * kSlice + c] - ((red[o] + red[1024 + o]) + (red[2048 + o] + red[3072 + o]));
             if (c0 + c < dvp) u[(unit * kC + t) * dvp + c0 + c] = val;
             const float f = cm[kC + t] * val;
-            Us[t * kSlice + c] = make_float2(f, f);
+            Us[t * kUs + c] = make_float2(f, f);
         }
+        asm volatile("cp.async.wait_group 1;" ::: "memory");        // K of this chunk (the next W may still be on its way)
         __syncthreads();
-        // the state behind the chunk: four key channels by four columns a thread, a part of the tokens each
+        // the state behind the chunk: key channels 4 kt .. and DP / 2 + 4 kt .. by columns 4 ct .. a thread, a part of the tokens each
         {
-            const int part = tid / DP, tile = tid - part * DP, ct = tile & 3, kt = tile >> 2;
-            float2 acc[4][2];
+            const int kt = quarter + 4 * (warp % NW), ph = warp / NW;
+            float2 acc[4][4];                                           // [column][pair of key channels]
 #pragma unroll
-            for (int q = 0; q < 4; ++q) acc[q][0] = acc[q][1] = make_float2(0.0f, 0.0f);
-#pragma unroll 8
-            for (int t = part * (kC / SPLIT); t < (part + 1) * (kC / SPLIT); ++t) {
-                const float4 k = ld4(Kb + t * DP + 4 * kt);
-                const float* us = reinterpret_cast<const float*>(Us + t * kSlice + 4 * ct);
+            for (int q = 0; q < 4; ++q)
+#pragma unroll
+                for (int p = 0; p < 4; ++p) acc[q][p] = make_float2(0.0f, 0.0f);
+            const float* kp = Kb + (ph * (kC / PH) + pb) * LK + 4 * kt;
+            const float2* up = Us + (ph * (kC / PH) + pb) * kUs + 4 * ct;
+#pragma unroll 4
+            for (int i = 0; i < kC / PH / 2; ++i) {
+                const float4 ka = ld4(kp + 2 * i * LK), kb = ld4(kp + 2 * i * LK + DP / 2);
+                const float* us = reinterpret_cast<const float*>(up + 2 * i * kUs);
                 const float4 u01 = ld4(us), u23 = ld4(us + 4);
-                acc[0][0] = fma2(lo2(k), lo2(u01), acc[0][0]), acc[0][1] = fma2(hi2(k), lo2(u01), acc[0][1]);
-                acc[1][0] = fma2(lo2(k), hi2(u01), acc[1][0]), acc[1][1] = fma2(hi2(k), hi2(u01), acc[1][1]);
-                acc[2][0] = fma2(lo2(k), lo2(u23), acc[2][0]), acc[2][1] = fma2(hi2(k), lo2(u23), acc[2][1]);
-                acc[3][0] = fma2(lo2(k), hi2(u23), acc[3][0]), acc[3][1] = fma2(hi2(k), hi2(u23), acc[3][1]);
-            }
+                const float2 uu[4] = {lo2(u01), hi2(u01), lo2(u23), hi2(u23)};
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
-                float* to = red + (size_t)(part * 16 + q * 4) * DP + tile;
-                to[0] = acc[q][0].x, to[DP] = acc[q][0].y, to[2 * DP] = acc[q][1].x, to[3 * DP] = acc[q][1].y;
+                for (int q = 0; q < 4; ++q) {
+                    acc[q][0] = fma2(lo2(ka), uu[q], acc[q][0]);
+                    acc[q][1] = fma2(hi2(ka), uu[q], acc[q][1]);
+                    acc[q][2] = fma2(lo2(kb), uu[q], acc[q][2]);
+                    acc[q][3] = fma2(hi2(kb), uu[q], acc[q][3]);
+                }
+            }
+            float* to = red + (ph * 32 + 16 * pb) * TB + ct + 4 * kt;
+#pragma unroll
+            for (int e = 0; e < 16; ++e) {
+                // columns 2 pb and 2 pb + 1 stay with this lane
+                const float2 a = acc[e >> 3][(e >> 1) & 3], b = acc[2 + (e >> 3)][(e >> 1) & 3];
+                const float lo = (e & 1) ? a.y : a.x, hi = (e & 1) ? b.y : b.x;
+                const float other = __shfl_xor_sync(0xffffffffu, pb ? lo : hi, 16);
+                to[e * TB] = (pb ? hi : lo) + other;
             }
         }
         __syncthreads();
-        {
-            const float f = cm[kC - 1];
-            for (int o = tid; o < 16 * DP; o += kCarryThreads) {
-                const int e = o / DP, tile = o - e * DP, c = 4 * (tile & 3) + (e >> 2), k = 4 * (tile >> 2) + (e & 3);
-                float sum = 0.0f;
+        stage_k(j + 1);
+        const float f = cm[kC - 1];
 #pragma unroll
-                for (int part = 0; part < SPLIT; ++part) sum += red[part * 16 * DP + o];
-                S[c * LD + k] = fmaf(f, S[c * LD + k], sum);
-            }
-        }
-        if (NB == 1 && j + 1 < count) {
-            __syncthreads();
-            stage(0, chunk + 1);
+        for (int o = tid; o < 32 * TB; o += kThreads) {
+            const int e = o / TB, tile = o - e * TB, c = 4 * (tile & 3) + (e >> 3), kk = e & 7, k = 4 * (tile >> 2) + (kk & 3) + (kk >> 2) * (DP / 2);
+            float sum = red[o];
+#pragma unroll
+            for (int ph = 1; ph < PH; ++ph) sum += red[ph * 32 * TB + o];
+            S[c * LD + k] = fmaf(f, S[c * LD + k], sum);
         }
     }
     pdl_launch_dependents();
     __syncthreads();
-    for (int idx = tid; idx < DP * kSlice; idx += kCarryThreads) {
+    for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
         const int c = idx / DP, k = idx - c * DP;
         if (k < d && c0 + c < dv) st[(size_t)(c0 + c) * d + k] = S[c * LD + k];
     }
@@ -473,7 +499,7 @@ int launch(const float* prep_qk, const float* prep_g, const float* v, float* sta
     cudaError_t e = li_launch_pdl(delta_chunk_solve_kernel<DP>, dim3(heads, chunks), dim3(kThreads), solve_smem<DP>(), stream, prep_qk, prep_g, v, (const int4*)seg,
                                   wm, xm, pt, sums, heads, kv_heads, dv);
     if (e == cudaSuccess)
-        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, dim3(ceil_div(dv, kSlice), heads, nruns), dim3(kCarryThreads), carry_smem<DP>(), stream, prep_qk,
+        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, dim3(ceil_div(dv, kSlice), heads, nruns), dim3(kThreads), carry_smem<DP>(), stream, prep_qk,
                           (const int4*)seg, runs, wm, xm, sums, state, state_stride, s0, u, heads, kv_heads, d, dv);
     if (e == cudaSuccess) {
         if (dtype == LI_F32)

@@ -13,7 +13,7 @@
 
 namespace {
 
-constexpr int kThreads = 256, kWarps = kThreads / 32;
+constexpr int kThreads = 512, kWarps = kThreads / 32;
 constexpr int kCols = 8;
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }

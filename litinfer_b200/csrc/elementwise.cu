@@ -13,7 +13,7 @@ namespace {
 constexpr int kRowThreads = 256;
 
 template <typename T>
-__global__ void embedding_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out, int H, int V) {
+__global__ void embedding_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out, int H, int V, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -21,7 +21,7 @@ __global__ void embedding_kernel(const T* __restrict__ table, const int* __restr
     id = id < 0 ? 0 : (id >= V ? V - 1 : id);          // ids are validated on the host; never read outside the table
     const T* row = table + (size_t)id * H;
     float* dst = out + (size_t)t * H;
-    for (int j = threadIdx.x; j < H; j += blockDim.x) dst[j] = to_float(row[j]);
+    for (int j = threadIdx.x; j < H; j += blockDim.x) dst[j] = to_float(row[j]) * scale;
 }
 
 // x[t] += pairs[row of (previous token, token)]; the previous token of a portion's first token is the sequence's state.
@@ -189,13 +189,13 @@ LI_EXPORT int li_add_pair_rows(float* x, const void* pairs, int dtype, const int
     return li_check_launch("add_pair_rows");
 }
 
-LI_EXPORT int li_embedding(const void* table, int dtype, const int* ids, float* out, int T, int H, int V, cudaStream_t stream) {
+LI_EXPORT int li_embedding(const void* table, int dtype, const int* ids, float* out, int T, int H, int V, float scale, cudaStream_t stream) {
     LI_REQUIRE(T >= 0 && H > 0 && V > 0, "embedding: bad sizes T=%d H=%d V=%d", T, H, V);
     if (T == 0) return 0;
     if (dtype == LI_F32)
-        li_launch_pdl(embedding_kernel<float>, dim3(T), dim3(kRowThreads), 0, stream, (const float*)table, ids, out, H, V);
+        li_launch_pdl(embedding_kernel<float>, dim3(T), dim3(kRowThreads), 0, stream, (const float*)table, ids, out, H, V, scale);
     else if (dtype == LI_BF16)
-        li_launch_pdl(embedding_kernel<bf16>, dim3(T), dim3(kRowThreads), 0, stream, (const bf16*)table, ids, out, H, V);
+        li_launch_pdl(embedding_kernel<bf16>, dim3(T), dim3(kRowThreads), 0, stream, (const bf16*)table, ids, out, H, V, scale);
     else
         return li_fail("embedding: unknown dtype %d", dtype);
     return li_check_launch("embedding");
@@ -462,6 +462,87 @@ LI_EXPORT int li_gelu_token_rows(const float* z, const void* table, int dtype, l
         e = li_launch_pdl(gelu_token_rows_kernel<bf16>, grid, dim3(128), 0, stream, z, (const bf16*)table, ld, col, rows, ids, (bf16*)out, n, total);
     if (e != cudaSuccess) return li_fail("gelu_token_rows: launch failed: %s", cudaGetErrorString(e));
     return li_check_launch("gelu_token_rows");
+}
+
+// The gate's product and the opening of the row as one kernel, for few tokens: out[t, i] = gelu(x[t] . w[i]) * table[ids[t], col + i], a
+// block per column i, eight tokens at a time, 16-byte loads, float sums.
+namespace {
+template <typename T>
+__device__ __forceinline__ void unpack16(float (&v)[16 / sizeof(T)], uint4 u) {
+    const unsigned w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        if constexpr (sizeof(T) == 2) v[2 * k] = __uint_as_float(w[k] << 16), v[2 * k + 1] = __uint_as_float(w[k] & 0xffff0000u);
+        else v[k] = __uint_as_float(w[k]);
+    }
+}
+
+constexpr int kGateWarps = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kGateWarps * 32)
+token_gate_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ table, long long ld, int col, int rows, const int* __restrict__ ids,
+                  T* __restrict__ out, int tokens, int H, int n) {
+    constexpr int V = 16 / (int)sizeof(T), TK = 8;
+    __shared__ float part[kGateWarps][TK];
+    const int i = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_launch_dependents();
+    const T* wr = w + (size_t)i * H;
+    // the weights do not depend on the kernel before this one: asked for while that still runs
+    for (int k = threadIdx.x * (128 / (int)sizeof(T)); k < H; k += kGateWarps * 32 * (128 / (int)sizeof(T))) asm volatile("prefetch.global.L2 [%0];" ::"l"(wr + k));
+    pdl_wait();
+    for (int t0 = 0; t0 < tokens; t0 += TK) {
+        float acc[TK];
+#pragma unroll
+        for (int j = 0; j < TK; ++j) acc[j] = 0.0f;
+        for (int k = V * threadIdx.x; k < H; k += kGateWarps * 32 * V) {
+            const uint4 wu = __ldg(reinterpret_cast<const uint4*>(wr + k));
+            uint4 xu[TK];
+#pragma unroll
+            for (int j = 0; j < TK; ++j) xu[j] = *reinterpret_cast<const uint4*>(x + (size_t)min(t0 + j, tokens - 1) * H + k);
+            float wv[V];
+            unpack16<T>(wv, wu);
+#pragma unroll
+            for (int j = 0; j < TK; ++j) {
+                float xv[V];
+                unpack16<T>(xv, xu[j]);
+#pragma unroll
+                for (int q = 0; q < V; ++q) acc[j] = fmaf(xv[q], wv[q], acc[j]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < TK; ++j) {
+            const float z = warp_sum(acc[j]);
+            if (lane == j) part[warp][j] = z;
+        }
+        __syncthreads();
+        if (threadIdx.x < TK && t0 + (int)threadIdx.x < tokens) {
+            const int t = t0 + threadIdx.x;
+            float z = 0.0f;
+#pragma unroll
+            for (int p = 0; p < kGateWarps; ++p) z += part[p][threadIdx.x];
+            int id = ids[t];
+            if (id < 0 || id >= rows) id = 0;
+            out[(size_t)t * n + i] = from_float<T>(geglu_of<T>(z, to_float(table[id * ld + col + i])));
+        }
+        __syncthreads();
+    }
+}
+}  // namespace
+
+LI_EXPORT int li_token_gate_accepts(int dtype, int T, int H) { return (T >= 1 && T <= 16 && H > 0 && H % (dtype == LI_F32 ? 4 : 8) == 0) ? 1 : 0; }
+
+LI_EXPORT int li_token_gate(const void* x, const void* w, const void* table, int dtype, long long ld, int col, int rows, const int* ids, void* out, int T, int H,
+                            int n, cudaStream_t stream) {
+    LI_REQUIRE(dtype == LI_F32 || dtype == LI_BF16, "token_gate: unknown dtype %d", dtype);
+    LI_REQUIRE(li_token_gate_accepts(dtype, T, H) && ((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0, "token_gate: refuses %d tokens of %d", T, H);
+    LI_REQUIRE(n > 0 && rows > 0 && col >= 0 && col + n <= ld, "token_gate: columns %d .. %d of rows of %lld", col, col + n, ld);
+    const dim3 grid(n);
+    const cudaError_t e = dtype == LI_F32
+        ? li_launch_pdl(token_gate_kernel<float>, grid, dim3(kGateWarps * 32), 0, stream, (const float*)x, (const float*)w, (const float*)table, ld, col, rows, ids, (float*)out, T, H, n)
+        : li_launch_pdl(token_gate_kernel<bf16>, grid, dim3(kGateWarps * 32), 0, stream, (const bf16*)x, (const bf16*)w, (const bf16*)table, ld, col, rows, ids, (bf16*)out, T, H, n);
+    if (e != cudaSuccess) return li_fail("token_gate: launch failed: %s", cudaGetErrorString(e));
+    return li_check_launch("token_gate");
 }
 
 // PolyNorm and a sigmoid gate.

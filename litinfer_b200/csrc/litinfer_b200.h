@@ -67,8 +67,9 @@ int li_decode_step_plan(int M, int hidden, int heads, int kv_heads, int head_dim
 int li_decode_step(const LiDecodeStep* step, cudaStream_t stream);
 
 /* ---- elementwise.cu ---- */
-/* out[t] = table[ids[t]] as float. */
-int li_embedding(const void* table, int dtype, const int* ids, float* out, int T, int H, int V, cudaStream_t stream);
+/* out[t] = scale * table[ids[t]] as float. */
+int li_embedding(const void* table, int dtype, const int* ids, float* out, int T, int H, int V, float scale,
+    cudaStream_t stream);
 
 /* x[t] += pairs[row] with row = (prev * mul_prev + ids[t] * mul_cur) mod buckets, prev the token before t in its sequence:
  * ids[t - 1] inside a portion, for a portion's first token the sequence's last token of the step before (state [slots,
@@ -120,6 +121,12 @@ int li_geglu(const void* gate_up, void* out, int dtype, int T, int I, cudaStream
  * table [rows, ld] in the run dtype. */
 int li_gelu_token_rows(const float* z, const void* table, int dtype, long long ld, int col, int rows, const int* ids, void* out, int T, int n,
     cudaStream_t stream);
+
+/* The gate's product with it, for few tokens: out[t, i] = gelu(x[t] . w[i]) * table[ids[t], col + i], x [T, H], w [n, H].  accepts: 1 if the
+ * sizes fit. */
+int li_token_gate_accepts(int dtype, int T, int H);
+int li_token_gate(const void* x, const void* w, const void* table, int dtype, long long ld, int col, int rows, const
+    int* ids, void* out, int T, int H, int n, cudaStream_t stream);
 
 /* out = a N(z) + b N(z^2) + c N(z^3) + e per row of z [T, n], powers element by element, N(v) = v / sqrt(mean(v^2) + eps),
  * coef = {a, b, c, e} float on the device. */

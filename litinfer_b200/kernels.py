@@ -99,14 +99,14 @@ _l = ctypes.c_longlong
 
 
 # --------------------------------------------------------------------------
-def embedding(table: torch.Tensor, ids: torch.Tensor, out32: torch.Tensor) -> None:
-    """out32[t, :] = float(table[ids[t], :])."""
+def embedding(table: torch.Tensor, ids: torch.Tensor, out32: torch.Tensor, scale: float = 1.0) -> None:
+    """out32[t, :] = scale * float(table[ids[t], :])."""
     V, H = table.shape
     T = ids.shape[0]
     _need(table, "embedding table")
     _need(ids, "token ids", torch.int32)
     _need(out32, "embedding output", torch.float32, (T, H))
-    _check(library().li_embedding(_p(table), _i(_dt(table)), _p(ids), _p(out32), _i(T), _i(H), _i(V), _stream(out32)), "embedding")
+    _check(library().li_embedding(_p(table), _i(_dt(table)), _p(ids), _p(out32), _i(T), _i(H), _i(V), _f(float(scale)), _stream(out32)), "embedding")
 
 
 def add_pair_rows(x32: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, q_start: torch.Tensor,
@@ -574,6 +574,27 @@ def gelu_token_rows(z: torch.Tensor, table: torch.Tensor, col: int, ids: torch.T
         raise KernelError(f"gelu_token_rows: columns {col} .. {col + n} of a table of shape {tuple(table.shape)} for {T} tokens")
     _check(library().li_gelu_token_rows(_p(z), _p(table), _i(_dt(table)), _l(table.shape[1]), _i(int(col)), _i(table.shape[0]), _p(ids), _p(out), _i(T),
                                         _i(n), _stream(out)), "gelu_token_rows")
+
+
+def token_gate_accepts(x: torch.Tensor) -> bool:
+    """Whether :func:`token_gate` takes a step of these tokens (few of them)."""
+    return bool(library().li_token_gate_accepts(_i(_dt(x)), _i(x.shape[0]), _i(x.shape[1])))
+
+
+def token_gate(x: torch.Tensor, weight: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor, out: torch.Tensor) -> None:
+    """The product of a gate and what :func:`gelu_token_rows` does with it, for few tokens: ``out[t, i] = gelu(x[t] . weight[i]) *
+    table[ids[t], col + i]``, sums and gelu in float32."""
+    T, H = x.shape
+    n = weight.shape[0]
+    _need(x, "gate input")
+    _need(weight, "gate weight", x.dtype, (n, H))
+    _need(table, "table of token rows", x.dtype)
+    _need(ids, "token ids", torch.int32)
+    _need(out, "opened rows", x.dtype, (T, n))
+    if table.dim() != 2 or col < 0 or col + n > table.shape[1] or ids.shape[0] < T:
+        raise KernelError(f"token_gate: columns {col} .. {col + n} of a table of shape {tuple(table.shape)} for {T} tokens")
+    _check(library().li_token_gate(_p(x), _p(weight), _p(table), _i(_dt(x)), _l(table.shape[1]), _i(int(col)), _i(table.shape[0]), _p(ids), _p(out), _i(T), _i(H),
+                                   _i(n), _stream(out)), "token_gate")
 
 
 def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor) -> None:
@@ -1606,7 +1627,7 @@ _TIMED = ("embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add
           "rope_kv_write", "linear_rope_kv", "rope_table", "paged_attention", "swiglu", "argmax", "sample", "gather_rows", "scale_inplace",
           "logit_cap", "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift",
           "ssm_scan", "decay_scan", "gated_rmsnorm", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route",
-          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "delta_chunks", "delta_step", "gelu_token_rows",
+          "moe_sort", "moe_gather", "moe_combine", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_small_step", "moe_route_grouped", "delta_prepare", "delta_scan", "delta_chunks", "delta_step", "gelu_token_rows", "token_gate",
           "mul_sigmoid", "polynorm")
 if profile.enabled:
     for _name in _TIMED:

@@ -153,9 +153,7 @@ class DecoderModel:
             if logits is not None:
                 return logits
         x32 = torch.empty((ctx.num_tokens, s.hidden_size), dtype=torch.float32, device=self.device)
-        K.embedding(self.embedding, ctx.token_ids, x32)
-        if s.embedding_scale is not None:
-            K.scale_inplace(x32, float(s.embedding_scale))
+        K.embedding(self.embedding, ctx.token_ids, x32, scale=float(s.embedding_scale) if s.embedding_scale is not None else 1.0)
         if self.position is not None:
             self.position.add_to_stream(x32, ctx)
         for k, part in enumerate(self.stream_inputs):

@@ -57,7 +57,11 @@ class GatedTokenRow(TokenInput):
         return self.norm
 
     def forward(self, x, ctx):
+        g = torch.empty((x.shape[0], self.dim), dtype=self.dtype, device=x.device)
+        if K.token_gate_accepts(x):
+            # few tokens: the gate's product opens the row itself
+            K.token_gate(x, self.gate.weight, self.table, self.column, ctx.token_ids, g)
+            return self.proj(g)
         z = self.gate(x, out_dtype=torch.float32)
-        g = torch.empty(z.shape, dtype=self.dtype, device=z.device)
         K.gelu_token_rows(z, self.table, self.column, ctx.token_ids, g)
         return self.proj(g)

@@ -20,8 +20,8 @@ def _store(out, value):
     out.copy_(value.to(out.dtype))
 
 
-def embedding(table, ids, out32):
-    _store(out32, table[ids.long()].float())
+def embedding(table, ids, out32, scale=1.0):
+    _store(out32, table[ids.long()].float() * scale)
 
 
 def _rms(x, weight, eps):
@@ -733,6 +733,14 @@ def moe_route_grouped(logits, correction, top, groups, keep, scale, ids, weights
     weights.copy_(sc * scale if sigmoid else sc / (sc.sum(-1, keepdim=True) + 1e-20) * scale)
 
 
+def token_gate_accepts(x):
+    return x.shape[0] <= 16
+
+
+def token_gate(x, weight, table, col, ids, out):
+    gelu_token_rows(x.float() @ weight.float().t(), table, col, ids, out)
+
+
 def gelu_token_rows(z, table, col, ids, out):
     _store(out, _gelu(z) * table[ids[:z.shape[0]].long(), col:col + z.shape[1]].float())
 
@@ -957,7 +965,7 @@ def table_gather(resident, updates, slots, out, trash_page):
             out[s, b] = resident[slot, b] if b < cols else trash_page
 
 
-ALL = ["gelu_token_rows", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_chunks", "delta_step", "delta_step_accepts", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
+ALL = ["gelu_token_rows", "token_gate", "token_gate_accepts", "moe_small_step_accepts", "moe_small_step", "geglu", "join_rows", "rope_norm_kv", "map_difference", "moe_route_grouped", "polynorm", "mul_sigmoid", "latent_rope_post", "delta_prepare", "delta_scan", "delta_chunks", "delta_step", "delta_step_accepts", "delta_row_elements", "row_rinv", "add_pair_rows", "gla_scan", "channel_scan", "sorted_rows", "norm_add_norm", "add_row", "rmsnorm_cols", "conv_norm_rope_kv", "grouped_linear", "moe_route", "moe_sort", "moe_gather", "moe_combine",
        "glu_clamped", "weighted_sum2", "add_position_rows", "hc_expand", "hc_read_norm", "hc_update", "causal_conv_silu", "conv_state_shift", "ssm_scan",
        "decay_scan", "gated_rmsnorm", "table_gather", "gather_rows", "scale_inplace", "logit_cap", "rope_table", "linear_scaled_accepts", "linear_add_scaled_parts", "linear_add_scaled", "apply_row_scale", "linear_rope_kv", "interleave_gate_up", "embedding", "rmsnorm", "add_rmsnorm", "gather_rmsnorm", "residual_add", "linear", "rope_kv_write",
        "paged_attention", "swiglu", "argmax", "sample"]

@@ -952,3 +952,12 @@ def test_two_outputs_with_norms_into_the_stream_and_an_opened_token_row(dtype):
     _close(out, ref, dtype, "opened rows")
     with pytest.raises(K.KernelError, match="columns"):
         K.gelu_token_rows(z, table, 41, ids, out)
+    for T, H, n in ((1, 64, 20), (9, 1536, 13), (16, 40, 60), (11, 2056, 24)):
+        x, w = torch.randn(T, H).to(dev, dt), (2.0 * torch.randn(n, H) / math.sqrt(H)).to(dev, dt)
+        ids = torch.randint(0, 50, (T,), dtype=torch.int32, device=dev)
+        out, ref = (torch.empty(T, n, dtype=dt, device=dev) for _ in range(2))
+        assert K.token_gate_accepts(x)
+        K.token_gate(x, w, table, 60 - n, ids, out)
+        R.token_gate(x, w, table, 60 - n, ids, ref)
+        _close(out, ref, dtype, f"gate of {T} tokens")
+    assert not K.token_gate_accepts(torch.empty(17, 64, dtype=dt, device=dev)) and not K.token_gate_accepts(torch.empty(3, 50, dtype=dt, device=dev))
