@@ -21,6 +21,8 @@ namespace {
 constexpr int kC = 64;              // tokens of a chunk
 constexpr int kLA = kC + 4;         // a row of a [.., tokens] tile in shared memory
 constexpr int kThreads = 256;
+constexpr int kMultiprocessors = 148;
+constexpr size_t kMoreThanHalf = 120 * 1024;      // of a multiprocessor's shared memory
 constexpr int kSlice = 16;          // value columns a block of the carry takes
 constexpr int kCols = 128;          // value columns a block of the output takes at a time
 constexpr int kRowsB = 16;          // rows of its second operand that it stages at a time
@@ -491,16 +493,22 @@ int launch(const float* prep_qk, const float* prep_g, const float* v, float* sta
     static bool raised = false;
     if (!raised) {
         if (int rc = raise_smem(delta_chunk_solve_kernel<DP>, solve_smem<DP>(), "delta chunks")) return rc;
-        if (int rc = raise_smem(delta_chunk_carry_kernel<DP>, carry_smem<DP>(), "delta chunks")) return rc;
+        if (int rc = raise_smem(delta_chunk_carry_kernel<DP>, carry_smem<DP>() > kMoreThanHalf ? carry_smem<DP>() : kMoreThanHalf, "delta chunks")) return rc;
         if (int rc = raise_smem(delta_chunk_output_kernel<float, DP>, output_smem<DP>(), "delta chunks")) return rc;
         if (int rc = raise_smem(delta_chunk_output_kernel<bf16, DP>, output_smem<DP>(), "delta chunks")) return rc;
         raised = true;
     }
     cudaError_t e = li_launch_pdl(delta_chunk_solve_kernel<DP>, dim3(heads, chunks), dim3(kThreads), solve_smem<DP>(), stream, prep_qk, prep_g, v, (const int4*)seg,
                                   wm, xm, pt, sums, heads, kv_heads, dv);
-    if (e == cudaSuccess)
-        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, dim3(ceil_div(dv, kSlice), heads, nruns), dim3(kThreads), carry_smem<DP>(), stream, prep_qk,
-                          (const int4*)seg, runs, wm, xm, sums, state, state_stride, s0, u, heads, kv_heads, d, dv);
+    if (e == cudaSuccess) {
+        // The walk lasts as long as its slowest block: while there is a multiprocessor for each, none shares one (blocks are placed as the
+        // kernel before drains, two at a time where two fit; more shared memory than half of a multiprocessor's keeps them apart).
+        const dim3 grid(ceil_div(dv, kSlice), heads, nruns);
+        const bool apart = (long long)grid.x * heads * nruns <= kMultiprocessors;
+        const size_t bytes = apart && carry_smem<DP>() < kMoreThanHalf ? kMoreThanHalf : carry_smem<DP>();
+        e = li_launch_pdl(delta_chunk_carry_kernel<DP>, grid, dim3(kThreads), bytes, stream, prep_qk, (const int4*)seg, runs, wm, xm, sums, state, state_stride, s0, u, heads,
+                          kv_heads, d, dv);
+    }
     if (e == cudaSuccess) {
         if (dtype == LI_F32)
             e = li_launch_pdl(delta_chunk_output_kernel<float, DP>, dim3(heads, chunks), dim3(kThreads), output_smem<DP>(), stream, prep_qk, (const int4*)seg, pt,
