@@ -244,9 +244,8 @@ delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restri
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    auto stage_k = [&](int j) {
+    auto stage_k = [&](int j, int4 sg) {
         if (j < count) {
-            const int4 sg = seg[first + j];
             const int n = min(sg.y - sg.x, kC);
             const float* from = prep_qk + ((size_t)sg.x * kv_heads + hk) * RQ + DP;
 #pragma unroll 4
@@ -258,7 +257,7 @@ delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restri
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage_w(0);
-    stage_k(0);
+    stage_k(0, seg[first]);
     for (int idx = tid; idx < DP * kSlice; idx += kThreads) {
         const int c = idx / DP, k = idx - c * DP;
         S[c * LD + k] = (k < d && c0 + c < dv) ? st[(size_t)(c0 + c) * d + k] : 0.0f;
@@ -267,6 +266,7 @@ delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restri
         const size_t unit = (size_t)(first + j) * heads + h;
         const float* X = Xs + (j & 1) * kXBuf;
         const float* cm = X + kC * kSlice;
+        const int4 after = seg[first + min(j + 1, count - 1)];      // the next chunk's tokens: asked for long before they are needed
         asm volatile("cp.async.wait_group 1;" ::: "memory");        // W and X of this chunk (its K may still be on its way)
         __syncthreads();
         // the state before this chunk, for the outputs
@@ -354,7 +354,6 @@ delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restri
             }
         }
         __syncthreads();
-        stage_k(j + 1);
         const float f = cm[kC - 1];
 #pragma unroll
         for (int o = tid; o < 32 * TB; o += kThreads) {
@@ -364,6 +363,7 @@ delta_chunk_carry_kernel(const float* __restrict__ prep_qk, const int4* __restri
             for (int ph = 1; ph < PH; ++ph) sum += red[ph * 32 * TB + o];
             S[c * LD + k] = fmaf(f, S[c * LD + k], sum);
         }
+        stage_k(j + 1, after);
     }
     pdl_launch_dependents();
     __syncthreads();
